@@ -23,7 +23,7 @@ import shutil
 import subprocess
 import sys
 from pathlib import Path
-from typing import List
+from typing import List, Sequence
 
 PKG = Path(__file__).resolve().parent
 OUT = PKG / "_C"
@@ -62,16 +62,21 @@ def _run(cmd: List[str], verbose: bool, log: Path) -> None:
         raise RuntimeError(f"build command failed ({r.returncode}): {' '.join(cmd)}\n{r.stdout[-4000:]}")
 
 
-def build_kernels(force: bool = False, verbose: bool = False) -> Path:
+# kernels of the layer-listed models alone: what a command that serves one of them has to compile in a fresh checkout
+LAYERED_SOURCES = ("residual", "delta_rule", "talking_attn", "gemm_f32", "gemm_tcgen05", "moe_route")
+
+
+def build_kernels(force: bool = False, verbose: bool = False, only: Sequence[str] = (), name: str = "kernels") -> Path:
+    """``libbg_<name>.so`` of every kernel source, or of the sources named in ``only`` (file stems)."""
     OUT.mkdir(exist_ok=True)
-    srcs = [p for d in KERNEL_DIRS if d.exists() for p in sorted(d.glob("*.cu"))]
+    srcs = [p for d in KERNEL_DIRS if d.exists() for p in sorted(d.glob("*.cu")) if not only or p.stem in only]
     hdrs = [p for d in KERNEL_DIRS if d.exists() for p in sorted(list(d.glob("*.cuh")) + list(d.glob("*.h")))]
-    so = OUT / "libbg_kernels.so"
-    stamp = OUT / "libbg_kernels.hash"
+    so = OUT / f"libbg_{name}.so"
+    stamp = OUT / f"libbg_{name}.hash"
     digest = _hash(srcs + hdrs, " ".join(NVCC_FLAGS))
     if so.exists() and stamp.exists() and stamp.read_text() == digest and not force:
         return so
-    log = OUT / "build_kernels.log"
+    log = OUT / f"build_{name}.log"
     log.write_text("")
     nvcc = _nvcc()
     objdir = OUT / "obj"
@@ -94,6 +99,22 @@ def build_kernels(force: bool = False, verbose: bool = False) -> Path:
     _run([nvcc, "-shared", "-o", str(so), *[str(o) for o in objs], "-lcudart"], verbose, log)
     stamp.write_text(digest)
     return so
+
+
+def kernels_current() -> bool:
+    """The whole kernel library is built from the sources as they are now."""
+    srcs = [p for d in KERNEL_DIRS if d.exists() for p in sorted(d.glob("*.cu"))]
+    hdrs = [p for d in KERNEL_DIRS if d.exists() for p in sorted(list(d.glob("*.cuh")) + list(d.glob("*.h")))]
+    so, stamp = OUT / "libbg_kernels.so", OUT / "libbg_kernels.hash"
+    return so.exists() and stamp.exists() and stamp.read_text() == _hash(srcs + hdrs, " ".join(NVCC_FLAGS))
+
+
+def layered_library() -> Path:
+    """A kernel library that serves layer-listed models: the whole one when it is built and current, otherwise one of
+    their kernels only (compiled now if need be)."""
+    if kernels_current():
+        return OUT / "libbg_kernels.so"
+    return build_kernels(only=LAYERED_SOURCES, name="layered")
 
 
 def build_core(force: bool = False, verbose: bool = False) -> Path:

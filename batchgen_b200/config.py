@@ -14,15 +14,74 @@ from __future__ import annotations
 import dataclasses
 import json
 import math
+import os
 import re
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Tuple
 
 
+@dataclass(frozen=True)
+class MixerSpec:
+    """The token mixer of one layer of a layer-listed model."""
+    kind: str                              # "attention" | "general_delta"
+    heads: int
+    dim: int                               # query / key width of a head
+    kv_heads: int = 0                      # attention: key / value heads (query head h reads h // (heads / kv_heads))
+    vdim: int = 0                          # value width of a head
+    scale: float = 1.0                     # attention: factor of the scores
+    chunk: int = 0                         # attention: keys are seen inside the query's own chunk of this many positions (0 = all)
+    talking: bool = False                  # attention: a [heads, heads] matrix mixes the heads' scores before the softmax
+    sink: bool = False                     # attention: one is added to the softmax denominator
+    decay_rank: int = 0                    # general_delta: width of the low-rank decay projection
+
+    @property
+    def recurrent(self) -> bool:
+        return self.kind == "general_delta"
+
+    @property
+    def dim_p(self) -> int:
+        """Head width as stored: padded with zero channels to a multiple of 8 (16-byte bf16 vectors)."""
+        return -(-self.dim // 8) * 8
+
+    @property
+    def vdim_p(self) -> int:
+        return -(-self.vdim // 8) * 8
+
+    @property
+    def kv_row(self) -> int:
+        """Elements of a cached token row: keys of every key head, then values."""
+        return 0 if self.recurrent else self.kv_heads * (self.dim_p + self.vdim_p)
+
+    @property
+    def state_shape(self) -> Tuple[int, int, int]:
+        """fp32 state [head, key channel, value channel]; empty for attention."""
+        return (self.heads, self.dim_p, self.vdim_p) if self.recurrent else (0, 0, 0)
+
+
+@dataclass(frozen=True)
+class MlpSpec:
+    """The feed-forward of one layer of a layer-listed model."""
+    kind: str = "none"                     # none | dense | moe
+    ff: int = 0                            # dense width, or width of one routed expert
+    activation: str = "gelu_tanh"          # gelu_tanh | swiglu_oai (clamped gate and up, sigmoid slope 1.702, up + 1)
+    limit: float = 0.0                     # clamp of swiglu_oai
+    experts: int = 0
+    top: int = 0
+    weight_on_input: bool = False          # the routing weight scales the expert's input instead of its output
+    shared_ff: int = 0                     # shared expert (0 = none), same activation, scaled by a sigmoid gate per token
+    shared_limit: float = 0.0
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: MixerSpec
+    mlp: MlpSpec = MlpSpec()
+
+
 @dataclass
 class ModelConfig:
     name: str = "tiny-deepseek-v3"
-    family: str = "deepseek_v3"  # deepseek_v3 | deepseek_v2 | deepseek_v4 | glm5 | kimi_k3 | kimi_k25 | gpt_oss | minimax | mixtral | qwen2_moe
+    family: str = "deepseek_v3"  # deepseek_v3 | deepseek_v2 | deepseek_v4 | glm5 | kimi_k3 | kimi_k25 | gpt_oss | minimax | mixtral | qwen2_moe | nanurax
     vocab_size: int = 1024
     hidden_size: int = 256
     num_layers: int = 2
@@ -90,6 +149,11 @@ class ModelConfig:
     # ---- quantisation of linear / expert weights
     quant: str = "none"                    # none | fp8_block | mxfp4 | int4
     quant_block: int = 128
+    # ---- layer-listed models: every layer has its own mixer and feed-forward, both reading one norm of the residual
+    # stream (parallel block), with an fp32 residual and scaled embeddings
+    layer_specs: Tuple[LayerSpec, ...] = ()
+    embed_scale: float = 1.0
+    checkpoint_dir: str = ""               # directory the config was read from (its .safetensors files are the weights)
     # ---- misc
     eos_token_id: int = 1
     bos_token_id: int = 0
@@ -103,6 +167,22 @@ class ModelConfig:
     @property
     def is_v4(self) -> bool:
         return len(self.compress_ratios) > 0
+
+    @property
+    def is_layered(self) -> bool:
+        return len(self.layer_specs) > 0
+
+    @property
+    def recurrent_layers(self) -> Tuple[int, ...]:
+        return tuple(l for l, s in enumerate(self.layer_specs) if s.mixer.recurrent)
+
+    @property
+    def has_state(self) -> bool:
+        """A live sequence holds a state slot besides (or instead of) paged KV."""
+        return self.has_kda or self.is_v4 or len(self.recurrent_layers) > 0
+
+    def layered_state_floats_per_seq(self) -> int:
+        return sum(math.prod(self.layer_specs[l].mixer.state_shape) for l in self.recurrent_layers)
 
     def v4_state_floats_per_seq(self) -> int:
         """fp32 words of per-sequence state of a DeepSeek-V4 model: per layer the window ring, the compressor's
@@ -122,13 +202,15 @@ class ModelConfig:
         """Width of one cached latent row (normalised c_kv followed by roped k_pe)."""
         if self.is_v4:
             return self.head_dim
+        if self.is_layered:
+            return sum(s.mixer.kv_row for s in self.layer_specs)
         if self.num_kv_heads > 0:
             return 2 * self.num_kv_heads * self.head_dim
         return self.kv_lora_rank + self.qk_rope_head_dim
 
     @property
     def is_mla(self) -> bool:
-        return self.num_kv_heads == 0
+        return self.num_kv_heads == 0 and not self.is_layered
 
     @property
     def has_dsa(self) -> bool:
@@ -181,6 +263,8 @@ class ModelConfig:
                     if r == 4:
                         b += self.index_head_dim * kv_dtype_bytes / r
             return int(math.ceil(b))
+        if self.is_layered:
+            return max(self.kv_cache_dim * kv_dtype_bytes, 1)
         b = (self.num_layers - len(self.kda_layers)) * self.kv_cache_dim * kv_dtype_bytes
         if self.has_dsa:
             n_idx = len(self.indexer_full_layers) or self.num_layers
@@ -202,6 +286,15 @@ class ModelConfig:
                         n += self.q_lora_rank * self.index_n_heads * Di + h * self.index_n_heads + 4 * h * Di
                 n += 3 * h * self.moe_intermediate_size * (self.n_routed_experts + self.n_shared_experts)
                 n += h * self.n_routed_experts + 2 * (2 + self.hc_mult) * self.hc_mult * self.hc_mult * h
+            return n
+        if self.is_layered:
+            for spec in self.layer_specs:
+                m, f = spec.mixer, spec.mlp
+                if m.recurrent:
+                    n += h * (6 * m.heads * m.dim + m.decay_rank) + m.decay_rank * m.heads * m.dim
+                else:
+                    n += h * (m.heads + m.kv_heads) * (m.dim + m.vdim) + m.heads * m.heads
+                n += 3 * h * f.ff * (f.experts if f.kind == "moe" else 1) + h * f.experts + 3 * h * f.shared_ff
             return n
         for l in range(self.num_layers):
             if self.layer_is_kda(l):
@@ -236,6 +329,10 @@ class ModelConfig:
             kw["indexer_full_layers"] = tuple(kw["indexer_full_layers"])
         if "compress_ratios" in kw:
             kw["compress_ratios"] = tuple(kw["compress_ratios"])
+        if "layer_specs" in kw:
+            kw["layer_specs"] = tuple(
+                x if isinstance(x, LayerSpec) else LayerSpec(MixerSpec(**x["mixer"]), MlpSpec(**x["mlp"]))
+                for x in kw["layer_specs"])
         return cls(**kw)
 
 
@@ -493,7 +590,106 @@ def minimax_m25() -> ModelConfig:
         quant="fp8_block")
 
 
+# ------------------------------------------------------------------ Nanurax: layer-listed config.json
+def _nanurax_layer(d: Dict, index: int) -> LayerSpec:
+    m, kind = d["mixer"], d["type"]
+    if kind == "general_delta":
+        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], vdim=m["dim"])
+    elif kind == "attention":
+        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], kv_heads=m.get("kv_heads", m["heads"]),
+                          vdim=m.get("vdim", m["dim"]), scale=float(m["scale"]),
+                          chunk=int((m.get("mask") or {}).get("size", 0)), talking=True, sink=True)
+        if mixer.heads % mixer.kv_heads:
+            raise ValueError(f"layer {index}: {mixer.heads} heads do not divide over {mixer.kv_heads} key/value heads")
+    else:
+        raise ValueError(f"layer {index}: unknown mixer type {kind!r}")
+    f = d.get("mlp")
+    if not f:
+        return LayerSpec(mixer)
+    if f["kind"] == "dense":
+        return LayerSpec(mixer, MlpSpec("dense", ff=f["ff"]))
+    if f["kind"] != "moe":
+        raise ValueError(f"layer {index}: unknown feed-forward kind {f['kind']!r}")
+    sh = f.get("shared") or {}
+    return LayerSpec(mixer, MlpSpec("moe", ff=f["expert"]["ff"], activation="swiglu_oai", limit=float(f["expert"]["limit"]),
+                                    experts=f["router"]["experts"], top=f["router"]["top"], weight_on_input=True,
+                                    shared_ff=sh.get("ff", 0), shared_limit=float(sh.get("limit", 0.0))))
+
+
+def nanurax_config(d: Dict, name: str = "nanurax", decay_ranks: Optional[Dict[int, int]] = None) -> ModelConfig:
+    """A Nanurax config.json (parsed) as a ``ModelConfig``.  ``decay_ranks``: per recurrent layer the width of its
+    low-rank decay projection, which only the checkpoint's tensor shapes tell (default 64)."""
+    layers = [_nanurax_layer(x, i) for i, x in enumerate(d["layers"])]
+    for i, s in enumerate(layers):
+        if s.mixer.recurrent:
+            rank = (decay_ranks or {}).get(i, 64)
+            layers[i] = dataclasses.replace(s, mixer=dataclasses.replace(s.mixer, decay_rank=rank))
+    moe = [s.mlp for s in layers if s.mlp.kind == "moe"]
+    att = [s.mixer for s in layers if not s.mixer.recurrent]
+    return ModelConfig(
+        name=name, family="nanurax", vocab_size=d["vocab"], hidden_size=d["width"], num_layers=len(layers),
+        layer_specs=tuple(layers), embed_scale=float(d["embedding"]["scale"]), rms_eps=float(d["norm"]["eps"]),
+        # summaries that planners read; the layers themselves are described by ``layer_specs``
+        num_heads=max(s.mixer.heads for s in layers), num_kv_heads=max((m.kv_heads for m in att), default=1),
+        head_dim=max(s.mixer.dim for s in layers), first_k_dense=0,
+        intermediate_size=max((s.mlp.ff for s in layers if s.mlp.kind == "dense"), default=0),
+        moe_intermediate_size=max((f.ff for f in moe), default=0), n_routed_experts=max((f.experts for f in moe), default=0),
+        num_experts_per_tok=max((f.top for f in moe), default=0), n_shared_experts=int(any(f.shared_ff for f in moe)),
+        attention_sinks=bool(att), max_position_embeddings=1 << 30, eos_token_id=-1, bos_token_id=-1)
+
+
+def _nanurax_dir(path: str, d: Dict) -> ModelConfig:
+    from .ckpt.safetensors_dir import tensor_shapes
+    shapes = tensor_shapes(path)
+    ranks = {i: shapes[f"l{i}.mix.w1"][0] for i in range(len(d["layers"])) if f"l{i}.mix.w1" in shapes}
+    cfg = nanurax_config(d, os.path.basename(os.path.normpath(path)) or "nanurax", ranks)
+    cfg.checkpoint_dir = path
+    return cfg
+
+
+_ARCHITECTURES = {"Nanurax": _nanurax_dir}        # config.json "architecture" -> reader of the model directory
+
+
+def load_model_dir(path: str) -> ModelConfig:
+    """Config of a model directory (config.json + .safetensors), chosen by the file's ``architecture``."""
+    with open(os.path.join(path, "config.json")) as f:
+        d = json.load(f)
+    arch = d.get("architecture")
+    if arch not in _ARCHITECTURES:
+        raise KeyError(f"{path}: architecture {arch!r} is not supported from a directory; known: {sorted(_ARCHITECTURES)}")
+    return _ARCHITECTURES[arch](path, d)
+
+
+def tiny_nanurax() -> ModelConfig:
+    """One attention layer between two delta-rule layers; dense, mixture and no feed-forward."""
+    delta = {"type": "general_delta", "mixer": {"heads": 3, "dim": 24}}
+    attn = {"type": "attention", "mixer": {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 32, "scale": 0.25,
+                                           "mask": {"size": 40}}}
+    moe = {"kind": "moe", "expert": {"ff": 40, "limit": 1.25}, "router": {"experts": 6, "top": 2},
+           "shared": {"ff": 56, "limit": 0.8}}
+    return nanurax_config({
+        "vocab": 320, "width": 120, "norm": {"eps": 1e-5}, "embedding": {"scale": 9.0},
+        "layers": [dict(delta, mlp={"kind": "dense", "ff": 200}), dict(attn, mlp=moe), dict(delta, mlp=None)]},
+        "tiny-nanurax", {0: 12, 2: 12})
+
+
+def nanurax_bench() -> ModelConfig:
+    """Layers of a real model's size: three delta-rule layers to one attention layer, dense and mixture feed-forwards."""
+    delta = {"type": "general_delta", "mixer": {"heads": 32, "dim": 128}}
+    attn = {"type": "attention", "mixer": {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                           "mask": {"size": 4096}}}
+    dense = {"kind": "dense", "ff": 9216}
+    moe = {"kind": "moe", "expert": {"ff": 1024, "limit": 7.0}, "router": {"experts": 64, "top": 8},
+           "shared": {"ff": 1024, "limit": 7.0}}
+    return nanurax_config({
+        "vocab": 163840, "width": 2304, "norm": {"eps": 1e-6}, "embedding": {"scale": 48.0},
+        "layers": [dict(delta, mlp=dense), dict(delta, mlp=moe), dict(delta, mlp=moe), dict(attn, mlp=moe)]},
+        "nanurax-bench")
+
+
 _PRESETS = {
+    "tiny-nanurax": tiny_nanurax,
+    "nanurax-bench": nanurax_bench,
     "tiny-deepseek-v3": tiny_deepseek_v3,
     "tiny-glm5": tiny_glm5,
     "tiny-kimi-k3": tiny_kimi_k3,
@@ -544,6 +740,7 @@ _PATTERNS = [
     (r"kimi[-_]?k2", "kimi-k2.5"),
     (r"gpt[-_]?oss", "gpt-oss-120b"),
     (r"minimax", "minimax-m2.5"),
+    (r"nanurax", "nanurax-bench"),
 ]
 
 
@@ -552,7 +749,15 @@ def list_models() -> List[str]:
 
 
 def get_model_config(name: str, **overrides) -> ModelConfig:
+    """Config of a preset, of a Hugging Face style id, or of a model directory (``load_model_dir``)."""
     key = name.lower()
+    if key not in _PRESETS and os.path.isfile(os.path.join(name, "config.json")):
+        cfg = load_model_dir(name)
+        for k, v in overrides.items():
+            if not hasattr(cfg, k):
+                raise AttributeError(f"ModelConfig has no field {k!r}")
+            setattr(cfg, k, v)
+        return cfg
     if key not in _PRESETS:
         for pat, preset in _PATTERNS:
             if re.search(pat, key):

@@ -1,5 +1,5 @@
-"""Model families.  ``build_model`` creates a ``Transformer`` (or, for DeepSeek-V4, a ``DeepSeekV4``) for any
-registered config."""
+"""Model families.  ``build_model`` creates a ``Transformer`` (for DeepSeek-V4 a ``DeepSeekV4``, for layer-listed models
+such as Nanurax a ``LayeredDecoder``) for any registered config."""
 from __future__ import annotations
 
 from typing import Optional
@@ -20,6 +20,9 @@ def build_model(cfg: ModelConfig, device="cpu", dtype="fp32", seed: int = 0, lay
     get_initializer / get_parallel_strategy_manager (batchgen/get_initializer.py:19-46)."""
     dt = _DTYPES[dtype] if isinstance(dtype, str) else dtype
     layout = layout or ParallelLayout()
+    if loader is None and cfg.checkpoint_dir:
+        from ..ckpt.safetensors_dir import SafetensorsDir
+        loader = SafetensorsDir(cfg.checkpoint_dir).loader()
     if loader is not None:
         from .checkpoint_names import aliased_loader
         loader = aliased_loader(cfg, loader)            # published names of the family, when they differ
@@ -27,6 +30,11 @@ def build_model(cfg: ModelConfig, device="cpu", dtype="fp32", seed: int = 0, lay
     if cfg.is_v4:
         from .deepseek_v4 import DeepSeekV4, build_v4_weights
         return DeepSeekV4(cfg, build_v4_weights(cfg, layout, src, dt), layout, comm, max_positions)
+    if cfg.is_layered:
+        from .layered import LayeredDecoder, build_layered_weights
+        if stream_experts:
+            raise NotImplementedError("streamed experts cover the block-quantised expert formats of Transformer models")
+        return LayeredDecoder(cfg, build_layered_weights(cfg, layout, src, dt), layout, comm, max_positions)
     w = build_weights(cfg, layout, src, dt, alias_experts_every=alias_experts_every,
                       experts_on_host=stream_experts)
     model = Transformer(cfg, w, layout, comm, max_positions)

@@ -22,6 +22,14 @@ class KernelError(RuntimeError):
     pass
 
 
+def use_library(path) -> None:
+    """Load kernels from ``path`` (a library of a subset of the sources) instead of the whole library."""
+    global _LIB_PATH
+    if _LIB is not None and Path(path) != _LIB_PATH:
+        raise KernelError("a kernel library is loaded already")
+    _LIB_PATH = Path(path)
+
+
 def available() -> bool:
     return _LIB_PATH.exists()
 

@@ -20,7 +20,7 @@ constexpr int kMaxTopK = 16;
 
 // One warp per token.  E <= 1024, K <= 16, n_group <= 32.
 __global__ void __launch_bounds__(128)
-router_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ idx_out,
+router_topk_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ bias, int* __restrict__ idx_out,
                    float* __restrict__ w_out, int T, int E, int K, int n_group, int topk_group, int norm, float scale,
                    int softmax_mode, const int* __restrict__ num_valid) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
@@ -39,7 +39,7 @@ router_topk_kernel(const float* __restrict__ logits, const float* __restrict__ b
     }
     return;
   }
-  const float* lrow = logits + (size_t)t * E;
+  const float* lrow = logits + (size_t)t * ldl;
   // scoring modes: 0 sigmoid, 1 softmax over the selected logits, 2 softmax over every expert, 3 sqrt(softplus)
   float rmax = -INFINITY, rinv = 0.f;
   if (softmax_mode == 2) {
@@ -285,13 +285,14 @@ moe_combine_kernel(const __nv_bfloat16* __restrict__ y, int ldy, const int* __re
 
 extern "C" {
 
-int bg_router_topk(const float* logits, const float* bias, int* idx, float* w, int T, int E, int K, int n_group,
+// logits: rows of E values, ldl apart
+int bg_router_topk(const float* logits, int ldl, const float* bias, int* idx, float* w, int T, int E, int K, int n_group,
                    int topk_group, int norm, float scale, int softmax_mode, const int* num_valid,
                    cudaStream_t stream) {
   using namespace bg;
   if (T <= 0) return 0;
-  if (E > kMaxExperts || K > kMaxTopK || n_group > 32 || (n_group > 1 && E % n_group != 0)) return -1;
-  bg::launch_pdl(router_topk_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, bias, idx, w, T, E, K, n_group, topk_group, norm, scale,
+  if (E > kMaxExperts || K > kMaxTopK || K > E || ldl < E || n_group > 32 || (n_group > 1 && E % n_group != 0)) return -1;
+  bg::launch_pdl(router_topk_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, ldl, bias, idx, w, T, E, K, n_group, topk_group, norm, scale,
                                                       softmax_mode, num_valid);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }

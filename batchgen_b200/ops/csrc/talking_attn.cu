@@ -1,0 +1,417 @@
+// Grouped-query attention over a paged K/V cache with mixed heads ("talking heads"), chunked visibility and a zero-score
+// sink, one query row per CTA (decode, short pieces of prompts, and the fp32 form).
+//
+//   s[h, j]  = scale * sum_g talk[h, g] (q[g] . k[kv(g), j])        g over all query heads, kv(g) = g / (H / G)
+//   seen     = first <= j <= position, first = position - position % chunk (chunk 0: first = 0)
+//   p[h, j]  = exp(s[h, j]) / (1 + sum exp(s[h, :]))                 (the 1 only with a sink)
+//   o[h]     = sum_j p[h, j] v[kv(h), j]
+//
+// Mixing couples all heads at a key, so a CTA takes all heads of its row.  Keys go in tiles of 32 (a lane per key); a
+// tile's steps are: raw scores (each warp takes key heads, whose K rows it stages through its own shared-memory buffer;
+// the next tile's rows are fetched while the rest of this tile runs), mixing and online softmax (a warp owns blocks of 4
+// heads, all 32 keys in its lanes), P.V (a thread owns 4 value columns of up to 4 heads that share a value head, so V is
+// read once).  With `n_splits` > 1 the key range is split over CTAs and merged by a second kernel.
+//
+// The cache row of a token holds the keys of all G heads (dp each), then the values (dvp each); dp and dvp are the head
+// widths padded to multiples of 8 with zero channels.
+#define BG_FILE_TAG 23     // kernel-trace ids of this file are (tag << 16) | line
+#include "common.cuh"
+
+namespace bg {
+namespace talk {
+
+constexpr int kThreads = 256;
+constexpr int kWarps = kThreads / 32;
+constexpr int NT = 32;          // keys per tile
+
+struct Params {
+  const float* q;               // [T, ldq]: H heads x dp
+  int ldq;
+  const float* talk;            // [H, H] or null (no mixing)
+  const void* cache;            // [pages, page, row]
+  long long page_stride;        // elements between pages
+  int page, row;                // tokens per page, elements per token
+  const int* block_table;       // [*, bt_stride]
+  int bt_stride;
+  const int* row_seq;           // [R] block-table row of each query row, or null (identity)
+  const int* row_ids;           // [R] row of q / out of each query row, or null (identity)
+  const int* lens;              // [T] position + 1 of each row of q; 0 = no query (zero output)
+  void* out;                    // [T, ldo]: H heads x dvp
+  int ldo;
+  float* part_o;                // [R, n_splits, H * dvp]
+  float* part_ml;               // [R, n_splits, H, 2]
+  int H, G, dp, dvp, chunk, sink, n_splits;
+  float scale_log2;
+};
+
+template <typename T> __device__ __forceinline__ float to_f(T v);
+template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+__device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 raw = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat162* v = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) { const float2 a = __bfloat1622float2(v[i]); f[2 * i] = a.x; f[2 * i + 1] = a.y; }
+}
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(__nv_bfloat16* p, float4 v) {
+  __align__(8) __nv_bfloat162 o[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+  *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(o);
+}
+__device__ __forceinline__ void cp16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_wait0() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+// shared memory, in floats: q [H dp] | talk^T [H][Hp] | raw scores [H][NT] | probabilities [Hp][NT] | m, l, a [Hp] each |
+// key offsets [NT] (long long), then the K buffers (one per warp), reused for the last reduction
+__host__ __device__ inline int pad4(int x) { return (x + 3) / 4 * 4; }
+__host__ __device__ inline size_t smem_floats(int H, int dp) {
+  const int Hp = pad4(H);
+  return (size_t)pad4(H * dp) + (size_t)H * Hp + (size_t)H * NT + (size_t)Hp * NT + 3 * (size_t)Hp + 2 * NT;
+}
+template <typename KT>
+__host__ __device__ inline size_t kbuf_bytes(int dp) { return (size_t)NT * (dp * sizeof(KT) + 16); }
+
+template <typename KT, int NI>
+__global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
+  bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
+  extern __shared__ __align__(16) float sm[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int H = p.H, G = p.G, dp = p.dp, dvp = p.dvp, rep = H / G, Hp = pad4(H);
+  float* q_s = sm;
+  float* tt = q_s + pad4(H * dp);
+  float* raw = tt + H * Hp;
+  float* pr = raw + H * NT;
+  float* m_s = pr + Hp * NT;
+  float* l_s = m_s + Hp;
+  float* a_s = l_s + Hp;
+  long long* koff = reinterpret_cast<long long*>(a_s + Hp);     // 16-byte aligned: every part is a multiple of 4 floats
+  char* kb_all = reinterpret_cast<char*>(koff + NT);
+  const int r = blockIdx.x, split = blockIdx.y;
+  const int t = p.row_ids != nullptr ? p.row_ids[r] : r;
+  const int L = p.lens[t];
+  KT* out = reinterpret_cast<KT*>(p.out) + (size_t)t * p.ldo;
+  if (L <= 0) {
+    if (p.n_splits == 1)
+      for (int i = tid; i < H * dvp / 4; i += kThreads) put4(out + 4 * i, make_float4(0.f, 0.f, 0.f, 0.f));
+    return;                                                       // (a split row without a query is zeroed by the merge)
+  }
+  const float* qr = p.q + (size_t)t * p.ldq;
+  for (int i = tid; i < H * dp / 4; i += kThreads) reinterpret_cast<float4*>(q_s)[i] = reinterpret_cast<const float4*>(qr)[i];
+  for (int i = tid; i < H * Hp; i += kThreads) {
+    const int g = i / Hp, h = i % Hp;
+    float v = 0.f;
+    if (h < H) v = p.talk != nullptr ? p.talk[h * H + g] : (h == g ? 1.f : 0.f);
+    tt[i] = v * p.scale_log2;
+  }
+  for (int i = tid; i < Hp; i += kThreads) { m_s[i] = -INFINITY; l_s[i] = 0.f; }
+  const int first = p.chunk > 0 ? (L - 1) - (L - 1) % p.chunk : 0;
+  const int t_lo = first / NT, n_t = (L + NT - 1) / NT - t_lo;
+  const int my_lo = t_lo + (int)(((long long)n_t * split) / p.n_splits);
+  const int my_hi = t_lo + (int)(((long long)n_t * (split + 1)) / p.n_splits);
+  const int* bt = p.block_table + (size_t)(p.row_seq != nullptr ? p.row_seq[r] : r) * p.bt_stride;
+  const KT* cache = reinterpret_cast<const KT*>(p.cache);
+
+  const int hg_n = (rep + 3) / 4;                                 // groups of up to 4 heads per key head
+  const int units = G * hg_n;
+  const int krow = dp * (int)sizeof(KT) + 16;                     // bytes of a staged K row
+  char* kb = kb_all + (size_t)warp * kbuf_bytes<KT>(dp);
+  auto key_offset = [&](int tile) -> long long {                  // element offset of this lane's key, < 0 = not seen
+    const int pos = tile * NT + lane;
+    if (pos < first || pos >= L) return -1;
+    return (long long)bt[pos / p.page] * p.page_stride + (long long)(pos % p.page) * p.row;
+  };
+  auto fetch = [&](int unit, long long off) {                     // K rows of unit's key head -> this warp's buffer
+    const int c = unit / hg_n, vec = dp * (int)sizeof(KT) / 16;
+    for (int i = lane; i < NT * vec; i += 32) {                    // NT * vec is a multiple of 32: the shuffle is warp-wide
+      const int kr = i / vec, cc = i % vec;
+      const long long o = __shfl_sync(0xffffffffu, off, kr);
+      if (o >= 0) cp16(kb + kr * krow + cc * 16, reinterpret_cast<const char*>(cache + o + c * dp) + cc * 16);
+    }
+    cp_commit();
+  };
+  // P.V: item = (value head c, group of 4 heads, 4 columns); KG groups of threads take alternate keys
+  const int cols = dvp / 4, items = G * hg_n * cols;
+  const int KG = items >= kThreads ? 1 : kThreads / items;
+  const int kg = items >= kThreads ? 0 : tid / items, item0 = items >= kThreads ? tid : tid % items;
+  float acc[NI][4][4];
+#pragma unroll
+  for (int n = 0; n < NI; ++n)
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[n][i][j] = 0.f;
+
+  long long off = my_lo < my_hi ? key_offset(my_lo) : -1;
+  if (my_lo < my_hi && warp < units) fetch(warp, off);
+  __syncthreads();                                                 // q_s, tt, m_s, l_s
+  for (int tile = my_lo; tile < my_hi; ++tile) {
+    const long long off_now = off;
+    if (warp == 0) koff[lane] = off_now;
+    off = tile + 1 < my_hi ? key_offset(tile + 1) : -1;
+    for (int u = warp; u < units; u += kWarps) {
+      cp_wait0();
+      __syncwarp();
+      const int c = u / hg_n, h0 = c * rep + (u % hg_n) * 4, nh = min(4, rep - (u % hg_n) * 4);
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
+      const KT* kr = reinterpret_cast<const KT*>(kb + lane * krow);
+      const float* qh[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) qh[i] = q_s + (h0 + min(i, nh - 1)) * dp;
+#pragma unroll 2
+      for (int e = 0; e < dp; e += 8) {
+        float k[8], qv[8];
+        load8(kr + e, k);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          load8(qh[i] + e, qv);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) s[i] = fmaf(qv[j], k[j], s[i]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (i < nh) raw[(h0 + i) * NT + lane] = s[i];
+      __syncwarp();
+      if (u + kWarps < units) fetch(u + kWarps, off_now);
+      else if (tile + 1 < my_hi) fetch(warp, off);                 // next tile's rows fly during the rest of this tile
+    }
+    __syncthreads();
+    // mixing + online softmax
+    for (int hb = warp; hb < Hp / 4; hb += kWarps) {
+      float v[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+      for (int g = 0; g < H; ++g) {
+        const float sg = raw[g * NT + lane];
+        const float4 w = *reinterpret_cast<const float4*>(tt + g * Hp + hb * 4);
+        v[0] = fmaf(w.x, sg, v[0]); v[1] = fmaf(w.y, sg, v[1]); v[2] = fmaf(w.z, sg, v[2]); v[3] = fmaf(w.w, sg, v[3]);
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int h = hb * 4 + i;
+        const float x = off_now >= 0 ? v[i] : -INFINITY;
+        const float mo = m_s[h], mn = fmaxf(mo, warp_max(x));
+        const float e = mn == -INFINITY ? 0.f : exp2f(x - mn);
+        const float sum = warp_sum(e);
+        pr[h * NT + lane] = e;
+        __syncwarp();
+        if (lane == 0) {
+          const float al = mn == -INFINITY ? 1.f : exp2f(mo - mn);
+          a_s[h] = al;
+          m_s[h] = mn;
+          l_s[h] = l_s[h] * al + sum;
+        }
+      }
+    }
+    __syncthreads();
+    // O = O * alpha + P . V
+    const int j_lo = max(first - tile * NT, 0), j_hi = min(L - tile * NT, NT);
+    if (kg < KG) {
+#pragma unroll
+      for (int n = 0; n < NI; ++n) {
+        const int it = item0 + n * kThreads;
+        if (it < items) {
+          const int u = it / cols, cc = it % cols, c = u / hg_n;
+          const int h0 = c * rep + (u % hg_n) * 4, nh = min(4, rep - (u % hg_n) * 4);
+          const KT* vb = cache + (size_t)G * dp + (size_t)c * dvp + cc * 4;
+          const float* ph[4];
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const int h = h0 + min(i, nh - 1);
+            ph[i] = pr + h * NT;
+            const float al = a_s[h];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[n][i][j] *= al;
+          }
+#pragma unroll 8
+          for (int j = j_lo + kg; j < j_hi; j += KG) {
+            const float4 v = load4(vb + koff[j]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const float w = ph[i][j];
+              acc[n][i][0] = fmaf(w, v.x, acc[n][i][0]); acc[n][i][1] = fmaf(w, v.y, acc[n][i][1]);
+              acc[n][i][2] = fmaf(w, v.z, acc[n][i][2]); acc[n][i][3] = fmaf(w, v.w, acc[n][i][3]);
+            }
+          }
+        }
+      }
+    }
+    __syncthreads();                                               // koff, pr and raw are free again
+  }
+  // sum over the key groups (only when all items fit one pass: NI == 1)
+  float* red = reinterpret_cast<float*>(kb_all);
+  if (KG > 1) {
+    cp_wait0();
+    __syncthreads();
+    if (kg > 0 && kg < KG) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(red + ((size_t)i * kThreads + tid) * 4) =
+          make_float4(acc[0][i][0], acc[0][i][1], acc[0][i][2], acc[0][i][3]);
+    }
+    __syncthreads();
+    if (kg == 0) {
+      for (int k = 1; k < KG; ++k) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float4 v = *reinterpret_cast<const float4*>(red + ((size_t)i * kThreads + k * items + tid) * 4);
+          acc[0][i][0] += v.x; acc[0][i][1] += v.y; acc[0][i][2] += v.z; acc[0][i][3] += v.w;
+        }
+      }
+    }
+  }
+  if (kg == 0) {
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int it = item0 + n * kThreads;
+      if (it < items) {
+        const int u = it / cols, cc = it % cols, c = u / hg_n;
+        const int h0 = c * rep + (u % hg_n) * 4, nh = min(4, rep - (u % hg_n) * 4);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          if (i >= nh) break;
+          const int h = h0 + i, col = h * dvp + cc * 4;
+          const float4 v = make_float4(acc[n][i][0], acc[n][i][1], acc[n][i][2], acc[n][i][3]);
+          if (p.n_splits == 1) {
+            const float inv = 1.0f / (l_s[h] + (p.sink ? exp2f(-m_s[h]) : 0.f));
+            put4(out + col, make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv));
+          } else {
+            *reinterpret_cast<float4*>(p.part_o + ((size_t)r * p.n_splits + split) * H * dvp + col) = v;
+          }
+        }
+      }
+    }
+  }
+  if (p.n_splits > 1)
+    for (int h = tid; h < H; h += kThreads) {
+      float* ml = p.part_ml + (((size_t)r * p.n_splits + split) * H + h) * 2;
+      ml[0] = m_s[h];
+      ml[1] = l_s[h];
+    }
+}
+
+// one block per (row, head)
+template <typename KT>
+__global__ void merge_kernel(const Params p) {
+  bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
+  const int r = blockIdx.x, h = blockIdx.y, S = p.n_splits;
+  const int t = p.row_ids != nullptr ? p.row_ids[r] : r;
+  KT* out = reinterpret_cast<KT*>(p.out) + (size_t)t * p.ldo + h * p.dvp;
+  if (p.lens[t] <= 0) {
+    for (int i = threadIdx.x; i < p.dvp / 4; i += blockDim.x) put4(out + 4 * i, make_float4(0.f, 0.f, 0.f, 0.f));
+    return;
+  }
+  const float* ml = p.part_ml + (size_t)r * S * p.H * 2 + h * 2;
+  float m = p.sink ? 0.f : -INFINITY;
+  for (int s = 0; s < S; ++s) m = fmaxf(m, ml[(size_t)s * p.H * 2]);
+  float l = p.sink ? exp2f(-m) : 0.f;
+  for (int s = 0; s < S; ++s) {
+    const float ms = ml[(size_t)s * p.H * 2];
+    if (ms != -INFINITY) l += ml[(size_t)s * p.H * 2 + 1] * exp2f(ms - m);
+  }
+  const float inv = 1.0f / l;
+  for (int i = threadIdx.x; i < p.dvp / 4; i += blockDim.x) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < S; ++s) {
+      const float ms = ml[(size_t)s * p.H * 2];
+      if (ms == -INFINITY) continue;
+      const float f = exp2f(ms - m);
+      const float4 v = *reinterpret_cast<const float4*>(p.part_o + ((size_t)r * S + s) * p.H * p.dvp + h * p.dvp + 4 * i);
+      a.x += f * v.x; a.y += f * v.y; a.z += f * v.z; a.w += f * v.w;
+    }
+    put4(out + 4 * i, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv));
+  }
+}
+
+// cache[slot[t]] = kv[t] (fp32 projection columns: keys of all heads, then values); slot < 0 writes nothing
+template <typename KT>
+__global__ void __launch_bounds__(128)
+kv_write_kernel(const float* __restrict__ kv, int ld, const long long* __restrict__ slots, KT* __restrict__ cache,
+                long long page_stride, int page, int row) {
+  bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
+  const long long slot = slots[blockIdx.x];
+  if (slot < 0) return;
+  KT* dst = cache + (slot / page) * page_stride + (slot % page) * row;
+  const float4* src = reinterpret_cast<const float4*>(kv + (size_t)blockIdx.x * ld);
+  for (int i = threadIdx.x; i < row / 4; i += blockDim.x) put4(dst + 4 * i, src[i]);
+}
+
+template <typename KT, int NI>
+static int launch_rows(const Params& p, int R, cudaStream_t stream) {
+  size_t kb = kWarps * kbuf_bytes<KT>(p.dp);
+  const size_t red = (size_t)kThreads * 16 * sizeof(float);
+  if (kb < red) kb = red;
+  const size_t smem = smem_floats(p.H, p.dp) * sizeof(float) + kb;
+  if (smem > 227 * 1024) return -3;
+  static DeviceOnce once;
+  auto kern = rows_kernel<KT, NI>;
+  if (!ensure_dynamic_smem(kern, 227 * 1024, once)) return -4;
+  bg::launch_pdl(kern, dim3(R, p.n_splits), dim3(kThreads), smem, stream, p);
+  if (p.n_splits > 1) bg::launch_pdl(merge_kernel<KT>, dim3(R, p.H), dim3(64), 0, stream, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
+}  // namespace talk
+}  // namespace bg
+
+extern "C" {
+
+// dt: 0 = bf16 cache and output, 1 = fp32.  -1: sizes out of contract; -3: heads x width need more shared memory than a CTA has.
+int bg_talk_rows(int dt, const float* q, int ldq, const float* talk, const void* cache, long long page_stride, int page,
+                 int row, const int* block_table, int bt_stride, const int* row_seq, const int* row_ids, const int* lens,
+                 void* out, int ldo, float* part_o, float* part_ml, int R, int H, int G, int dp, int dvp, int chunk,
+                 int sink, float scale, int n_splits, cudaStream_t stream) {
+  using namespace bg::talk;
+  if (R <= 0) return 0;
+  if (H <= 0 || G <= 0 || H % G || dp <= 0 || dp % 8 || dvp <= 0 || dvp % 8 || row != G * (dp + dvp) || page <= 0 ||
+      page_stride % 8 || ldq % 4 || ldo % 4 || n_splits < 1 || n_splits > 65535 || H > 65535 ||
+      (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
+    return -1;
+  Params p;
+  p.q = q; p.ldq = ldq; p.talk = talk; p.cache = cache; p.page_stride = page_stride; p.page = page; p.row = row;
+  p.block_table = block_table; p.bt_stride = bt_stride; p.row_seq = row_seq; p.row_ids = row_ids; p.lens = lens;
+  p.out = out; p.ldo = ldo; p.part_o = part_o; p.part_ml = part_ml; p.H = H; p.G = G; p.dp = dp; p.dvp = dvp;
+  p.chunk = chunk; p.sink = sink; p.n_splits = n_splits; p.scale_log2 = scale * 1.4426950408889634f;
+  const int items = G * ((H / G + 3) / 4) * (dvp / 4);
+  const int ni = (items + kThreads - 1) / kThreads;
+  if (ni > 4) return -1;
+  if (dt == 0) {
+    if (ni == 1) return launch_rows<__nv_bfloat16, 1>(p, R, stream);
+    if (ni == 2) return launch_rows<__nv_bfloat16, 2>(p, R, stream);
+    return launch_rows<__nv_bfloat16, 4>(p, R, stream);
+  }
+  if (ni == 1) return launch_rows<float, 1>(p, R, stream);
+  if (ni == 2) return launch_rows<float, 2>(p, R, stream);
+  return launch_rows<float, 4>(p, R, stream);
+}
+
+int bg_talk_kv_write(int dt, const float* kv, int ld, const long long* slots, void* cache, long long page_stride, int page,
+                     int row, int T, cudaStream_t stream) {
+  using namespace bg::talk;
+  if (T <= 0) return 0;
+  if (row % 8 || ld % 4 || ld < row || page <= 0 || page_stride % 8) return -1;
+  if (dt == 0)
+    bg::launch_pdl(kv_write_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, stream, kv, ld, slots,
+                   reinterpret_cast<__nv_bfloat16*>(cache), page_stride, page, row);
+  else
+    bg::launch_pdl(kv_write_kernel<float>, dim3(T), dim3(128), 0, stream, kv, ld, slots, reinterpret_cast<float*>(cache),
+                   page_stride, page, row);
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
+}  // extern "C"
+
+BG_TRACE_SETTER(talking_attn)

@@ -215,3 +215,47 @@ def bf16_gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = No
         return out
     _launch(KIND_BF16, EPI_STORE_F32 if fp32_out else EPI_STORE, x, None, 0, w, None, out, None, 1, T, N, K)
     return out
+
+
+def f32_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: Optional[torch.Tensor] = None,
+             counts: Optional[torch.Tensor] = None, max_rows: int = 0) -> torch.Tensor:
+    """out = x @ w^T in true fp32 on the CUDA cores (``csrc/gemm_f32.cu``); grouped when ``offsets`` is given (w [E, N, K],
+    at most ``max_rows`` rows in a group)."""
+    N, K = w.shape[-2], w.shape[-1]
+    assert x.dtype == w.dtype == out.dtype == torch.float32 and x.stride(1) == 1 and w.is_contiguous() and out.stride(1) == 1
+    groups = w.shape[0] if offsets is not None else 1
+    rc = _ext.lib().bg_gemm_f32(_ext.ptr(x), ctypes.c_int(x.stride(0)), _ext.ptr(w), ctypes.c_int(K), _ext.ptr(out),
+                                ctypes.c_int(out.stride(0)), _ext.ptr(offsets), _ext.ptr(counts), ctypes.c_int(groups),
+                                ctypes.c_int(x.shape[0]), ctypes.c_int(max_rows), ctypes.c_int(N), ctypes.c_int(K),
+                                _ext.stream())
+    _ext.check(rc, "bg_gemm_f32")
+    return out
+
+
+def rows_gemm(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x [T, K] @ w [N, K]^T -> fp32 [T, N] (row stride a multiple of 4): the bf16 tcgen05 GEMM with its fp32 epilogue, or
+    the CUDA-core GEMM for fp32 operands.  K is a multiple of 64 for bf16 (the caller pads weights and activations)."""
+    T, N = x.shape[0], w.shape[0]
+    if not x.is_cuda:
+        return x.float() @ w.float().t()
+    out = torch.empty(T, -(-N // 4) * 4, dtype=torch.float32, device=x.device)[:, :N]
+    if T == 0:
+        return out
+    if x.dtype == torch.float32:
+        return f32_gemm(x, w, out)
+    assert x.is_contiguous() and w.is_contiguous() and x.shape[1] == w.shape[1] and w.shape[1] % 64 == 0
+    return bf16_gemm(x, w, out=out, fp32_out=True)
+
+
+def grouped_rows_gemm(x: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, counts: torch.Tensor,
+                      max_rows: int) -> torch.Tensor:
+    """Grouped ``rows_gemm`` (w [E, N, K]; CUDA): rows past a segment's count stay undefined."""
+    E, N, K = w.shape
+    out = torch.empty(x.shape[0], -(-N // 4) * 4, dtype=torch.float32, device=x.device)
+    if x.shape[0] == 0:
+        return out
+    if x.dtype == torch.float32:
+        return f32_gemm(x, w, out[:, :N], offsets, counts, max_rows)
+    assert x.is_contiguous() and w.is_contiguous() and K % 64 == 0 and x.shape[1] == K
+    _launch(KIND_BF16, EPI_STORE_F32, x, None, 0, w.view(E * N, K), None, out, offsets, E, x.shape[0], N, K, counts=counts)
+    return out[:, :N]

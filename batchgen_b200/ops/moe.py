@@ -15,7 +15,7 @@ from typing import Optional, Tuple
 
 import torch
 
-from . import _ext, fused, gemm, ref
+from . import _ext, fused, gemm, ref, residual
 
 FP8 = torch.float8_e4m3fn
 ROW_ALIGN = 128  # grouped segments start on tile boundaries of the tcgen05 GEMM
@@ -39,6 +39,7 @@ class ExpertWeights:
     quant: str = "none"
     interleaved: bool = False
     activation: str = "silu"             # silu | swiglu_clamped (GPT-OSS) | silu_limit (DeepSeek-V4: clamp, then SiLU(gate) * up)
+                                         # | swiglu_oai | gelu_tanh (``routed_rows``: fp32 activations of layer-listed models)
     act_limit: float = 0.0               # clamp of silu_limit (0 = none)
 
     @property
@@ -99,10 +100,11 @@ def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, 
             w[nv:] = 0
         return idx, w
     T, E = logits.shape
-    logits = logits.contiguous()
+    if logits.stride(1) != 1:
+        logits = logits.contiguous()
     idx = torch.empty(T, top_k, dtype=torch.int32, device=logits.device)
     w = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
-    rc = _ext.lib().bg_router_topk(_ext.ptr(logits), _ext.ptr(bias), _ext.ptr(idx), _ext.ptr(w), ctypes.c_int(T),
+    rc = _ext.lib().bg_router_topk(_ext.ptr(logits), ctypes.c_int(logits.stride(0)), _ext.ptr(bias), _ext.ptr(idx), _ext.ptr(w), ctypes.c_int(T),
                                    ctypes.c_int(E), ctypes.c_int(top_k), ctypes.c_int(n_group),
                                    ctypes.c_int(topk_group), ctypes.c_int(int(norm_topk_prob)), ctypes.c_float(scale),
                                    ctypes.c_int(_SCORING_MODES[scoring]), _ext.ptr(num_valid), _ext.stream())
@@ -275,3 +277,39 @@ def experts_forward(hidden: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.
         if before_combine is not None:
             before_combine()
         return combine(y, pos, topk_w, extra, out_dtype or hidden.dtype)
+
+
+def routed_rows(x: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.Tensor, ew: ExpertWeights, weight_on_input: bool,
+                num_valid: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Unquantised routed experts with fp32 pre-activations and outputs.  x [T, Kp] (the experts' input, zero columns past
+    the model width) -> (y [rows, N] fp32 grouped by expert, pos [T, k] row of every (token, k) pair, -1 = none).
+    ``weight_on_input``: the routing weight scales the expert's input (it is applied to the fp32 gate and up
+    pre-activations, the same thing without rounding the product); the caller's sum over k then adds the rows as they are.
+
+    All shapes and row counts stay on the device: the call is graph capturable."""
+    E, F2, _ = ew.w13.shape
+    F = F2 // 2
+    T, K = topk_idx.shape
+    if not weight_on_input:
+        raise NotImplementedError("routed_rows covers experts whose routing weight multiplies the input")
+    kind = residual.GLU_KINDS[ew.activation]
+    if not x.is_cuda:
+        src, pos, off = permute(topk_idx, 0, E, num_valid)
+        y = torch.zeros(max(int(off[-1]), 1), ew.w2.shape[1], dtype=torch.float32)
+        wrow = torch.zeros(y.shape[0])
+        live = pos >= 0
+        wrow[pos[live].long()] = topk_w[live].float()
+        for e in range(E):
+            a, b = int(off[e]), int(off[e + 1])
+            if b > a:
+                z = x[src[a:b].long()].float() @ ew.w13[e].float().t()
+                y[a:b] = residual.glu(z, F, ew.activation, ew.act_limit, row_scale=wrow[a:b]) @ ew.w2[e].float().t()
+        return y, pos
+    assert kind is not None
+    src, pos, offsets = permute(topk_idx, 0, E, num_valid, align=8)
+    counts = offsets.real_counts
+    cap = src.shape[0]
+    xs, ws = residual.moe_gather(x, pos, topk_w, cap)
+    z = gemm.grouped_rows_gemm(xs, ew.w13, offsets, counts, max_rows=T)
+    act = residual.glu(z, F, ew.activation, ew.act_limit, row_scale=ws, total_rows=offsets[-1:], dtype=x.dtype)
+    return gemm.grouped_rows_gemm(act, ew.w2, offsets, counts, max_rows=T), pos

@@ -1,0 +1,130 @@
+"""Row operators of models with an fp32 residual stream: residual sum + RMS norm (with the embedding or the sublayers'
+outputs folded in), gated activations, operand casts, expert-row gather.
+
+CUDA tensors go to ``csrc/residual.cu``; CPU tensors to plain fp32 torch.  Operand dtype (norm output, activations) is
+bf16, or fp32 for the 32-bit form of a model.
+"""
+from __future__ import annotations
+
+import ctypes
+import math
+from typing import Optional, Tuple
+
+import torch
+
+from . import _ext
+
+_DT = {torch.bfloat16: 0, torch.float32: 1}
+GLU_KINDS = {"gelu_tanh": 0, "swiglu_oai": 1}
+
+
+def _i(v) -> ctypes.c_int:
+    return ctypes.c_int(int(v))
+
+
+def pad_to(n: int, m: int) -> int:
+    return -(-n // m) * m
+
+
+def residual_norm(x: torch.Tensor, w: torch.Tensor, eps: float, width: int, out_cols: int, dtype: torch.dtype,
+                  add: Optional[torch.Tensor] = None, routed: Optional[torch.Tensor] = None,
+                  pos: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None,
+                  embed: Optional[torch.Tensor] = None, embed_scale: float = 1.0, rows: Optional[torch.Tensor] = None,
+                  keep: bool = True) -> torch.Tensor:
+    """x [T, >= width] fp32 (+= ``add`` [T, width] fp32, += sum_k routed[pos[t, k]]; or = embed[ids] * embed_scale), then
+    y = rmsnorm(x) * w as [R, out_cols] of ``dtype`` with zero columns past ``width``.  ``rows`` (int64) picks rows of x;
+    ``keep=False`` leaves x as it was (the last norm of a step)."""
+    R = x.shape[0] if rows is None else rows.shape[0]
+    if not x.is_cuda:
+        r = rows.long() if rows is not None else torch.arange(x.shape[0])
+        cur = x[r, :width].clone()
+        if ids is not None:
+            cur = embed[ids[r].long()].float() * embed_scale
+        if add is not None:
+            cur = cur + add[r, :width]
+        if routed is not None:
+            p = pos[r].long()
+            g = routed[p.clamp_min(0), :width] * (p >= 0).unsqueeze(-1)
+            cur = cur + g.sum(1)
+        if keep:
+            x[r, :width] = cur
+        y = torch.zeros(R, out_cols, dtype=dtype)
+        y[:, :width] = (cur / torch.sqrt((cur * cur).mean(-1, keepdim=True) + eps) * w).to(dtype)
+        return y
+    y = torch.empty(R, out_cols, dtype=dtype, device=x.device)
+    for t in (add, routed):
+        assert t is None or (t.dtype == torch.float32 and t.stride(1) == 1)
+    assert x.dtype == torch.float32 and w.dtype == torch.float32 and (embed is None or embed.dtype == dtype)
+    assert (ids is None or ids.dtype == torch.int32) and (pos is None or (pos.dtype == torch.int32 and pos.is_contiguous()))
+    assert rows is None or rows.dtype == torch.int64
+    rc = _ext.lib().bg_residual_norm(
+        _i(_DT[dtype]), _ext.ptr(x), _i(x.stride(0)), _ext.ptr(rows), _ext.ptr(ids), _ext.ptr(embed),
+        _i(embed.stride(0) if embed is not None else 0), ctypes.c_float(embed_scale),
+        _i(embed.shape[0] if embed is not None else 0), _ext.ptr(add), _i(add.stride(0) if add is not None else 0),
+        _ext.ptr(routed), _i(routed.stride(0) if routed is not None else 0), _ext.ptr(pos),
+        _i(pos.shape[1] if pos is not None else 0), _ext.ptr(w), _ext.ptr(y), _i(out_cols), _i(R), _i(width),
+        ctypes.c_float(eps), _i(keep), _ext.stream())
+    _ext.check(rc, "bg_residual_norm")
+    return y
+
+
+def _glu_ref(g: torch.Tensor, u: torch.Tensor, kind: str, limit: float) -> torch.Tensor:
+    if kind == "gelu_tanh":
+        return 0.5 * g * (1 + torch.tanh(math.sqrt(2 / math.pi) * (g + 0.044715 * g ** 3))) * u
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return g * torch.sigmoid(1.702 * g) * (u + 1)
+
+
+def glu(z: torch.Tensor, F: int, kind: str, limit: float = 0.0, row_scale: Optional[torch.Tensor] = None,
+        gate: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, total_rows: Optional[torch.Tensor] = None,
+        dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """act(s * z[:, :F], s * z[:, F:2F]) * sigmoid(gate): ``kind`` gelu_tanh (tanh-GELU(g) * u) or swiglu_oai (g clamped from
+    above, u on both sides, g * sigmoid(1.702 g) * (u + 1)).  z fp32 (a column view is fine), ``row_scale`` [R] = s,
+    ``gate`` [R, 1] (a view is fine).  ``out``: [R, >= F] view, columns past F become zero."""
+    R = z.shape[0]
+    if not z.is_cuda:
+        g, u = z[:, :F].float(), z[:, F:2 * F].float()
+        if row_scale is not None:
+            g, u = g * row_scale.unsqueeze(-1), u * row_scale.unsqueeze(-1)
+        y = _glu_ref(g, u, kind, limit)
+        if gate is not None:
+            y = y * torch.sigmoid(gate.float())
+        if out is None:
+            return y.to(dtype or torch.float32)
+        out.zero_()
+        out[:, :F] = y.to(out.dtype)
+        return out
+    if out is None:
+        out = torch.empty(R, F, dtype=dtype, device=z.device)
+    assert z.dtype == torch.float32 and z.stride(1) == 1 and out.stride(1) == 1
+    rc = _ext.lib().bg_glu(_i(_DT[out.dtype]), _i(GLU_KINDS[kind]), _ext.ptr(z), _i(z.stride(0)), _i(F), _ext.ptr(out),
+                           _i(out.stride(0)), _i(R), _i(F), _i(out.shape[1]), ctypes.c_float(limit), _ext.ptr(row_scale),
+                           _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0), _ext.ptr(total_rows),
+                           _ext.stream())
+    _ext.check(rc, "bg_glu", kernels=-(-R // 65535))
+    return out
+
+
+def cast_act(x: torch.Tensor, cols: int, dtype: torch.dtype, tanh: bool = False) -> torch.Tensor:
+    """fp32 columns (a view is fine) -> [T, cols] of ``dtype``, zero past x's width; optional tanh."""
+    if not x.is_cuda:
+        y = torch.zeros(x.shape[0], cols, dtype=dtype)
+        y[:, : x.shape[1]] = (torch.tanh(x) if tanh else x).to(dtype)
+        return y
+    assert x.dtype == torch.float32 and x.stride(1) == 1
+    out = torch.empty(x.shape[0], cols, dtype=dtype, device=x.device)
+    rc = _ext.lib().bg_cast_act(_i(_DT[dtype]), _i(tanh), _ext.ptr(x), _i(x.stride(0)), _ext.ptr(out), _i(cols),
+                                _i(x.shape[0]), _i(x.shape[1]), _ext.stream())
+    _ext.check(rc, "bg_cast_act")
+    return out
+
+
+def moe_gather(x: torch.Tensor, pos: torch.Tensor, w: torch.Tensor, rows: int) -> Tuple[torch.Tensor, torch.Tensor]:
+    """CUDA: (xs [rows, cols], ws [rows]) with xs[pos[t, k]] = x[t], ws[pos[t, k]] = w[t, k]; other rows stay undefined."""
+    assert x.is_contiguous() and pos.dtype == torch.int32 and w.dtype == torch.float32
+    xs = torch.empty(rows, x.shape[1], dtype=x.dtype, device=x.device)
+    ws = torch.empty(rows, dtype=torch.float32, device=x.device)
+    rc = _ext.lib().bg_moe_gather(_i(_DT[x.dtype]), _ext.ptr(x), _i(x.shape[1]), _ext.ptr(pos), _ext.ptr(w), _ext.ptr(xs),
+                                  _ext.ptr(ws), _i(pos.shape[0]), _i(pos.shape[1]), _ext.stream())
+    _ext.check(rc, "bg_moe_gather")
+    return xs, ws

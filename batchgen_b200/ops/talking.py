@@ -1,0 +1,113 @@
+"""Paged grouped-query attention whose heads' scores are mixed before the softmax, with chunked visibility and a
+zero-score sink (``csrc/talking_attn.cu``): cache rows, and one query row per CTA for decode and short pieces.
+"""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from . import _ext
+from .residual import _DT, _i
+
+
+@dataclass
+class TalkParams:
+    """One layer's attention.  Head widths are padded to multiples of 8 with zero channels (dim_p, vdim_p)."""
+    heads: int
+    kv_heads: int
+    dim_p: int
+    vdim_p: int
+    scale: float
+    chunk: int = 0                           # 0 = every earlier key is seen
+    sink: bool = False                       # one added to the softmax denominator
+    talk: Optional[torch.Tensor] = None      # [heads, heads] fp32: score_h <- sum_g talk[h, g] score_g; None = no mixing
+
+    @property
+    def kv_row(self) -> int:
+        return self.kv_heads * (self.dim_p + self.vdim_p)
+
+
+def kv_write(kv: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor) -> None:
+    """cache[slot] = kv (fp32 columns: keys of all heads, values of all heads); cache [pages, page, row] (strided pages);
+    slots [T] int64, < 0 writes nothing."""
+    P, page, row = cache.shape
+    if not kv.is_cuda:
+        live = slots >= 0
+        s = slots[live]
+        cache[s // page, s % page] = kv[live, :row].to(cache.dtype)
+        return
+    assert kv.dtype == torch.float32 and kv.stride(1) == 1 and cache.stride(1) == row and cache.stride(2) == 1
+    assert slots.dtype == torch.int64
+    rc = _ext.lib().bg_talk_kv_write(_i(_DT[cache.dtype]), _ext.ptr(kv), _i(kv.stride(0)), _ext.ptr(slots), _ext.ptr(cache),
+                                     ctypes.c_longlong(cache.stride(0)), _i(page), _i(row), _i(kv.shape[0]), _ext.stream())
+    _ext.check(rc, "bg_talk_kv_write")
+
+
+def _rows_ref(q, p: TalkParams, cache, block_table, lens, out, row_seq):
+    H, G, d, dv = p.heads, p.kv_heads, p.dim_p, p.vdim_p
+    rep = H // G
+    page = cache.shape[1]
+    for t in range(q.shape[0]):
+        L = int(lens[t])
+        out[t, : H * dv] = 0
+        if L <= 0:
+            continue
+        first = (L - 1) // p.chunk * p.chunk if p.chunk else 0
+        pos = torch.arange(first, L)
+        bt = block_table[int(row_seq[t]) if row_seq is not None else t].long()
+        rows = cache[bt[pos // page], pos % page].float()
+        k = rows[:, : G * d].view(-1, G, d).repeat_interleave(rep, 1)
+        v = rows[:, G * d:].view(-1, G, dv).repeat_interleave(rep, 1)
+        s = torch.einsum("hd,jhd->hj", q[t, : H * d].view(H, d).float(), k) * p.scale
+        if p.talk is not None:
+            s = p.talk @ s
+        m = s.amax(-1, keepdim=True)
+        if p.sink:
+            m = m.clamp_min(0)
+        e = torch.exp(s - m)
+        den = e.sum(-1, keepdim=True) + (torch.exp(-m) if p.sink else 0)
+        out[t, : H * dv] = torch.einsum("hj,jhv->hv", e / den, v).reshape(-1).to(out.dtype)
+
+
+def _splits(rows: int, keys: int, sms: int) -> int:
+    tiles = max(1, -(-keys // 32))
+    return max(1, min(16, 3 * sms // max(rows, 1), tiles))
+
+
+def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table: torch.Tensor, lens: torch.Tensor,
+                out: torch.Tensor, row_seq: Optional[torch.Tensor] = None, row_ids: Optional[torch.Tensor] = None,
+                num_splits: int = 0) -> None:
+    """q [T, >= H * dim_p] fp32 -> out [T, >= H * vdim_p] (operand dtype, a column view is fine).  ``lens`` [T] int32 =
+    position + 1 of each row (0: no query, zero output); ``row_seq`` [R] block-table row of each query row (None: row i);
+    ``row_ids`` [R] the rows of q to compute (None: all).  The keys are in the cache already."""
+    if not q.is_cuda:
+        if row_ids is not None:
+            raise NotImplementedError("row subsets are a device path")
+        return _rows_ref(q, p, cache, block_table, lens, out, row_seq)
+    P, page, row = cache.shape
+    R = q.shape[0] if row_ids is None else row_ids.shape[0]
+    assert q.dtype == torch.float32 and q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == cache.dtype
+    assert lens.dtype == torch.int32 and block_table.dtype == torch.int32 and row == p.kv_row and cache.stride(1) == row
+    for t in (row_seq, row_ids):
+        assert t is None or t.dtype == torch.int32
+    H = p.heads
+    if num_splits <= 0:
+        keys = block_table.shape[1] * page
+        num_splits = _splits(R, min(keys, p.chunk) if p.chunk else keys, _ext.num_sms(q.device))
+    po = pml = None
+    if num_splits > 1:
+        po = torch.empty(R * num_splits * H * p.vdim_p, dtype=torch.float32, device=q.device)
+        pml = torch.empty(R * num_splits * H * 2, dtype=torch.float32, device=q.device)
+    rc = _ext.lib().bg_talk_rows(
+        _i(_DT[cache.dtype]), _ext.ptr(q), _i(q.stride(0)), _ext.ptr(p.talk), _ext.ptr(cache),
+        ctypes.c_longlong(cache.stride(0)), _i(page), _i(row), _ext.ptr(block_table), _i(block_table.stride(0)),
+        _ext.ptr(row_seq), _ext.ptr(row_ids), _ext.ptr(lens), _ext.ptr(out), _i(out.stride(0)), _ext.ptr(po),
+        _ext.ptr(pml), _i(R), _i(H), _i(p.kv_heads), _i(p.dim_p), _i(p.vdim_p), _i(p.chunk), _i(p.sink),
+        ctypes.c_float(p.scale), _i(num_splits), _ext.stream())
+    if rc in (-1, -3):
+        raise _ext.KernelError(f"attend_rows: heads {H}/{p.kv_heads}, widths {p.dim_p}/{p.vdim_p} are outside the kernel's "
+                               "contract (shared memory of one CTA, 1,024 head-column items)")
+    _ext.check(rc, "bg_talk_rows", kernels=2 if num_splits > 1 else 1)

@@ -22,6 +22,7 @@ every rank again holds every token before the next scheduling decision.
 """
 from __future__ import annotations
 
+import itertools
 import time
 from collections import OrderedDict
 from dataclasses import dataclass, field
@@ -116,13 +117,18 @@ class Engine:
             if ecfg.enable_prefix_cache:
                 raise ValueError("prefix reuse needs per-page snapshots of the window and compressor state, which "
                                  "DeepSeek-V4 layers do not keep")
+        elif self.cfg.has_state:
+            # layer-listed models: every live sequence holds one slot of recurrent state
+            state_slots = ecfg.max_state_slots or ecfg.max_decode_batch
+            if ecfg.enable_prefix_cache:
+                raise ValueError("prefix reuse needs per-page state snapshots, which recurrent layers do not keep")
         self.kv = PagedKVCache(self.cfg, n_pages, ecfg.page_size, self.device, kv_dtype, state_slots=state_slots,
                                state_heads=state_heads)
         # host tier: on a GPU the native region + asynchronous movers (a region created by the server is attached
         # through ``host_kv_fd``); the pinned torch tensor is the CPU / fallback form of the same tier
         self.host_tier = None
         if (num_host_pages or host_kv_fd is not None) and self.device.type == "cuda" \
-                and ecfg.host_kv_backend == "native" and not self.cfg.has_kda and not self.cfg.is_v4:
+                and ecfg.host_kv_backend == "native" and not self.cfg.has_state:
             from .host_tier import NativeHostTier
             self.host_tier = NativeHostTier(self.kv, num_host_pages, fd=host_kv_fd)
             self.host_kv = self.host_tier                  # same allocator face (``.alloc``)
@@ -561,6 +567,25 @@ class Engine:
 
     def _run_prefill_forward(self, rows: List[_PrefillRow]) -> None:
         """One packed prefill forward over ``rows``."""
+        group = [r.seq for r in rows if r.seq is not None]
+        ends = list(itertools.accumulate(len(r.tokens) for r in rows))
+        logit_rows = [e - 1 for e, r in zip(ends, rows) if r.seq is not None]
+        ids_t, meta, T, pad = self._rows_step(rows, logit_rows)
+        self.stats.prefill_tokens += T
+        self.step_ring.record("prefill", len(rows), T)
+        if self.sp_world > 1:
+            logits = self.model.forward_sp(ids_t, meta, self.kv)      # wanted rows that this rank owns
+            toks = self._sample_sharded(logits, group, logit_rows, T + pad) if group else []
+        else:
+            logits = self.model.forward(ids_t, meta, self.kv)
+            toks = self._sample(logits, group).tolist() if group else []
+        for s, t in zip(group, toks):
+            self.stats.prefill_cached_tokens += s.cached_prefix_tokens
+            s.num_cached_tokens = len(self._prefill_ids(s))
+            s.output_ids.append(int(t))
+
+    def _rows_step(self, rows: List[_PrefillRow], logit_rows: List[int]):
+        """(ids, metadata, tokens, padding rows) of one packed forward over ``rows``."""
         ps = self.buf.page_size
         ids: List[int] = []
         pos: List[int] = []
@@ -582,8 +607,6 @@ class Engine:
             ids += [0] * pad
             pos += [0] * pad
             slots += [-1] * pad
-        group = [r.seq for r in rows if r.seq is not None]
-        logit_rows = [cu[i + 1] - 1 for i, r in enumerate(rows) if r.seq is not None]
         has_state = self.kv.state is not None
         meta = AttnMeta(
             mode="prefill",
@@ -597,19 +620,66 @@ class Engine:
                                if has_state else None),
             logit_rows=torch.tensor(logit_rows, dtype=torch.int64, device=dev),
             num_valid=torch.tensor([T], dtype=torch.int32, device=dev) if W > 1 else None)
-        ids_t = torch.tensor(ids, dtype=torch.int32, device=dev)
-        self.stats.prefill_tokens += T
-        self.step_ring.record("prefill", len(rows), T)
-        if W > 1:
-            logits = self.model.forward_sp(ids_t, meta, self.kv)      # wanted rows that this rank owns
-            toks = self._sample_sharded(logits, group, logit_rows, T + pad) if group else []
+        return torch.tensor(ids, dtype=torch.int32, device=dev), meta, T, pad
+
+    # ------------------------------------------------------------------ caller-driven steps
+    def open_sequence(self, custom_id: str = "") -> Sequence:
+        """A sequence whose tokens the caller feeds itself (``extend``): a replayed trace, an external scheduler, a
+        scorer.  The engine's own scheduler never sees it; its pages and state slot come from the same pools."""
+        s = Sequence(global_idx=self._next_idx, prompt_ids=[], custom_id=custom_id, status=S.IN_PREFILL)
+        self._next_idx += 1
+        return s
+
+    def extend(self, pieces: Seq[tuple]) -> torch.Tensor:
+        """One step over ``pieces`` = (sequence, next tokens, wanted places among them), all in one batch: pieces of
+        prompts of any length beside single decoded tokens.  Returns fp32 logits of the wanted places, in order.
+
+        Steps in which every piece continues its sequence by one token run as decode steps; everything else runs as one
+        packed forward, in which a decoded token is a piece of length one."""
+        if self.sp_world > 1:
+            raise NotImplementedError("caller-driven steps run on one GPU per engine")
+        pieces = [(s, list(map(int, t)), list(w)) for s, t, w in pieces if len(t)]
+        ps = self.buf.page_size
+        rows: List[_PrefillRow] = []
+        want: List[int] = []
+        base = 0
+        for s, toks, w in pieces:
+            if any(not 0 <= i < len(toks) for i in w):
+                raise ValueError("a wanted place lies outside its piece")
+            need = pages_for(s.num_cached_tokens + len(toks), ps) - len(s.gpu_pages)
+            if need > 0:
+                s.gpu_pages += self._alloc_pages(need)
+            if self.kv.state is not None and s.state_slot < 0:
+                s.state_slot = self.kv.state.acquire()
+            rows.append(_PrefillRow(toks, s.num_cached_tokens, s.gpu_pages, state_slot=s.state_slot))
+            want += [base + i for i in w]
+            base += len(toks)
+        if not rows:
+            return torch.empty(0, self.cfg.vocab_size, dtype=torch.float32, device=self.device)
+        if all(len(r.tokens) == 1 and r.start > 0 for r in rows):
+            pos = [r.start for r in rows]
+            slots = [r.pages[p // ps] * ps + p % ps for r, p in zip(rows, pos)]
+            logits = self._decode_forward([s for s, _, _ in pieces], [r.tokens[0] for r in rows], pos, slots,
+                                          [p + 1 for p in pos])
+            self.stats.decode_steps += 1
+            out = logits[torch.tensor(want, dtype=torch.int64, device=logits.device)]
         else:
-            logits = self.model.forward(ids_t, meta, self.kv)
-            toks = self._sample(logits, group).tolist() if group else []
-        for s, t in zip(group, toks):
-            self.stats.prefill_cached_tokens += s.cached_prefix_tokens
-            s.num_cached_tokens = len(self._prefill_ids(s))
-            s.output_ids.append(int(t))
+            ids_t, meta, T, _ = self._rows_step(rows, want)
+            self.stats.prefill_tokens += T
+            out = self.model.forward(ids_t, meta, self.kv)
+        for s, toks, _ in pieces:
+            s.prompt_ids += toks
+            s.num_cached_tokens += len(toks)
+        self.step_ring.record("extend", len(rows), base)
+        return out
+
+    def close_sequence(self, s: Sequence) -> None:
+        """Give back what a caller-driven sequence holds."""
+        self._release_state(s)
+        if s.gpu_pages:
+            self.kv.alloc.free(s.gpu_pages)
+            s.gpu_pages = []
+        s.transition(S.COMPLETED)
 
     # ------------------------------------------------------------------ sampling
     @staticmethod
@@ -832,9 +902,29 @@ class Engine:
         lens = [p + 1 if s is not None else 0 for s, p in zip(layout, pos)]
         return layout, pos, slots, lens
 
+    def _decode_forward(self, layout: List[Optional[Sequence]], ids, pos, slots, lens, split: bool = False) -> torch.Tensor:
+        """Logits of one eager decode step over ``layout`` (``None`` entries are padding rows)."""
+        dev = self.device
+        n_real = sum(1 for s in layout if s is not None)
+        meta = AttnMeta(
+            mode="decode",
+            positions=torch.tensor(pos, dtype=torch.int32, device=dev),
+            slot_mapping=torch.tensor(slots, dtype=torch.int64, device=dev),
+            block_table=build_block_table([s.gpu_pages if s is not None else [] for s in layout], dev),
+            seqlens=torch.tensor(lens, dtype=torch.int32, device=dev),
+            state_slots=(torch.tensor([s.state_slot if s is not None else -1 for s in layout], dtype=torch.int32,
+                                      device=dev) if self.kv.state is not None else None))
+        ids_t = torch.tensor(ids, dtype=torch.int32, device=dev)
+        if self.sp_world > 1:
+            if not split and n_real != len(layout):
+                # padding rows sit at the end: the router skips them (request-split layouts pad inside the
+                # blocks instead; there the empty rows are routed like any row and dropped afterwards)
+                meta.num_valid = torch.tensor([n_real], dtype=torch.int32, device=dev)
+            return self.model.forward_sp(ids_t, meta, self.kv)
+        return self.model.forward(ids_t, meta, self.kv)
+
     def _decode_step(self, rows: List[Sequence]) -> None:
         """One synchronous decode step (the path without captured graphs)."""
-        dev = self.device
         W = self.sp_world
         split = self.model.attn_request_parallel and self.model.layout.tp_size > 1
         layout, pos, slots, lens = self._step_layout(rows)
@@ -844,24 +934,7 @@ class Engine:
             if W > 1:
                 layout = layout + [None] * (bucket - len(layout))    # the captured step covers the whole bucket
         else:
-            n_real = sum(1 for s in layout if s is not None)
-            meta = AttnMeta(
-                mode="decode",
-                positions=torch.tensor(pos, dtype=torch.int32, device=dev),
-                slot_mapping=torch.tensor(slots, dtype=torch.int64, device=dev),
-                block_table=build_block_table([s.gpu_pages if s is not None else [] for s in layout], dev),
-                seqlens=torch.tensor(lens, dtype=torch.int32, device=dev),
-                state_slots=(torch.tensor([s.state_slot if s is not None else -1 for s in layout], dtype=torch.int32,
-                                          device=dev) if self.kv.state is not None else None))
-            ids_t = torch.tensor(ids, dtype=torch.int32, device=dev)
-            if W > 1:
-                if not split and n_real != len(layout):
-                    # padding rows sit at the end: the router skips them (request-split layouts pad inside the
-                    # blocks instead; there the empty rows are routed like any row and dropped afterwards)
-                    meta.num_valid = torch.tensor([n_real], dtype=torch.int32, device=dev)
-                logits = self.model.forward_sp(ids_t, meta, self.kv)
-            else:
-                logits = self.model.forward(ids_t, meta, self.kv)
+            logits = self._decode_forward(layout, ids, pos, slots, lens, split)
         if W > 1:
             toks = self._sample_sharded(logits, layout, list(range(len(layout))), len(layout), resident=True)
         else:

@@ -90,7 +90,7 @@ class DecodeGraphRunner:
         # state slot of each row (KDA recurrent state, or DeepSeek-V4 window / compressor state); -1 = padding row: it
         # is skipped or lands in a scratch slot, so warm-up and capture touch no sequence's state
         self.state_slots = (torch.full((B,), -1, dtype=torch.int32, device=d)
-                            if (model.cfg.has_kda or model.cfg.is_v4) else None)
+                            if model.cfg.has_state else None)
         pin = torch.cuda.is_available()
         self.h_state = torch.full((B,), -1, dtype=torch.int32, pin_memory=pin)
         self.h_ids = torch.zeros(B, dtype=torch.int32, pin_memory=pin)

@@ -13,6 +13,7 @@ The native host-tier backend lives in ``core/csrc``; this module is its Python f
 """
 from __future__ import annotations
 
+import math
 from typing import Dict, List, Optional, Sequence as Seq, Tuple
 
 import torch
@@ -72,6 +73,8 @@ def host_page_bytes(cfg: ModelConfig, page_size: int, kv_elem_bytes: int = 2) ->
     if cfg.is_v4:
         return sum(v4_entries_per_page(r, page_size) * (cfg.head_dim + (cfg.index_head_dim if r == 4 else 0))
                    for r in cfg.compress_ratios if r) * kv_elem_bytes
+    if cfg.is_layered:
+        return page_size * cfg.kv_cache_dim * kv_elem_bytes
     kv_layers = sum(1 for l in range(cfg.num_layers) if not cfg.layer_is_kda(l))
     b = kv_layers * page_size * cfg.kv_cache_dim * kv_elem_bytes
     if cfg.has_dsa:
@@ -102,7 +105,15 @@ class PagedKVCache:
         self.row_dim = row_dim or cfg.kv_cache_dim
         pin = pinned and self.device.type == "cpu" and torch.cuda.is_available()
         # KDA layers keep no paged KV: layer l's rows live at index kv_index[l] of the pool
-        kv_layers = [] if cfg.is_v4 else [l for l in range(cfg.num_layers) if not cfg.layer_is_kda(l)]
+        # layer-listed models: attention layers differ in row width, so a page holds the layers' blocks [page, row_l] one
+        # after the other in one entry of the pool (``layer_rows``: layer -> (first element of a token row's share, width))
+        self.layer_rows: Dict[int, Tuple[int, int]] = {}
+        off = 0
+        for l, spec in enumerate(cfg.layer_specs):
+            if spec.mixer.kv_row:
+                self.layer_rows[l] = (off, spec.mixer.kv_row)
+                off += spec.mixer.kv_row
+        kv_layers = [] if cfg.is_v4 else [0] if cfg.is_layered else [l for l in range(cfg.num_layers) if not cfg.layer_is_kda(l)]
         self.kv_index = {l: i for i, l in enumerate(kv_layers)}
         self.kv = torch.zeros(len(kv_layers), num_pages, page_size, self.row_dim, dtype=dtype, device=self.device,
                               pin_memory=pin)
@@ -135,9 +146,17 @@ class PagedKVCache:
             self.state = StateSlotPool(cfg, state_slots, self.device, state_heads)
         elif cfg.is_v4 and state_slots:
             self.state = V4StatePool(cfg, state_slots, self.device)
+        elif cfg.recurrent_layers and state_slots:
+            self.state = FlatStatePool([((l, "S"), cfg.layer_specs[l].mixer.state_shape) for l in cfg.recurrent_layers],
+                                       state_slots, self.device)
 
     # ---- views used by the model
     def latent(self, layer: int) -> torch.Tensor:
+        if self.layer_rows:
+            off, row = self.layer_rows[layer]
+            flat = self.kv[0].view(self.num_pages, self.page_size * self.row_dim)
+            block = flat[:, off * self.page_size: (off + row) * self.page_size]
+            return block.unflatten(1, (self.page_size, row))
         return self.kv[self.kv_index[layer]]
 
     def index_keys(self, layer: int) -> Tuple[torch.Tensor, torch.Tensor]:
@@ -227,33 +246,19 @@ class StateSlotPool:
         return self.conv[i], self.rec[i]
 
 
-class V4StatePool:
-    """Per-sequence state of a DeepSeek-V4 model, one fp32 row per slot: for every layer the sliding-window ring of
-    raw KV rows ([window, D], row = position % window), and on compressed layers the compressor's pending windows
-    (projections and gate scores of the tokens not pooled yet; with overlapped windows also the previous window),
-    twice on ratio-4 layers (attention entries and index keys).  ``rec`` / ``conv`` follow ``StateSlotPool`` so the
-    host store parks a row the same way (``conv`` is an empty placeholder).
+class FlatStatePool:
+    """Per-sequence state as one fp32 row per slot, cut into named parts of any shape: ``parts`` lists ((layer, name),
+    shape).  ``rec`` / ``conv`` follow ``StateSlotPool`` so the host store parks a row the same way (``conv`` is an empty
+    placeholder).  Row ``num_slots`` is scratch for rows without a sequence."""
 
-    Reference parity: the compressed-ratio GPU KV variant and its per-sequence compressor state
-    (batchgen/kv_cache/gpu_paged_kv_manager.py, SWA / compressed-ratio variants)."""
-
-    def __init__(self, cfg: ModelConfig, num_slots: int, device):
-        self.cfg, self.num_slots = cfg, num_slots
-        D, Di, win = cfg.head_dim, cfg.index_head_dim, cfg.sliding_window
+    def __init__(self, parts, num_slots: int, device):
+        self.num_slots = num_slots
         self.offsets: Dict[Tuple[int, str], Tuple[int, Tuple[int, ...]]] = {}
         n = 0
-        for l, r in enumerate(cfg.compress_ratios):
-            parts = [("ring", (win, D))]
-            if r:
-                c = 2 if r == 4 else 1
-                parts += [("kv", (c * r, c * D)), ("score", (c * r, c * D))]
-                if r == 4:
-                    parts += [("idx_kv", (2 * r, 2 * Di)), ("idx_score", (2 * r, 2 * Di))]
-            for name, shape in parts:
-                self.offsets[(l, name)] = (n, shape)
-                n += shape[0] * shape[1]
-        assert n == cfg.v4_state_floats_per_seq()
-        # row ``num_slots`` is scratch: decode rows without a sequence park their writes there
+        for key, shape in parts:
+            self.offsets[key] = (n, tuple(shape))
+            n += (math.prod(shape) + 3) // 4 * 4                # parts start on 16-byte boundaries
+        self.row_floats = n
         self.rec = torch.zeros(1, num_slots + 1, n, dtype=torch.float32, device=device)
         self.conv = torch.zeros(1, num_slots + 1, 1, dtype=torch.float32, device=device)
         self._free = list(range(num_slots - 1, -1, -1))
@@ -274,7 +279,36 @@ class V4StatePool:
     def view(self, slot: int, layer: int, name: str) -> torch.Tensor:
         """A writable view of one part of ``slot``'s state."""
         off, shape = self.offsets[(layer, name)]
-        return self.rec[0, slot, off: off + shape[0] * shape[1]].view(shape)
+        return self.rec[0, slot, off: off + math.prod(shape)].view(shape)
+
+    def layer(self, layer: int, name: str = "S") -> torch.Tensor:
+        """One part of every slot as a strided [slots + 1, numel] view of the pool."""
+        off, shape = self.offsets[(layer, name)]
+        return self.rec[0, :, off: off + math.prod(shape)]
+
+
+class V4StatePool(FlatStatePool):
+    """Per-sequence state of a DeepSeek-V4 model: for every layer the sliding-window ring of raw KV rows ([window, D],
+    row = position % window), and on compressed layers the compressor's pending windows (projections and gate scores of
+    the tokens not pooled yet; with overlapped windows also the previous window), twice on ratio-4 layers (attention
+    entries and index keys).
+
+    Reference parity: the compressed-ratio GPU KV variant and its per-sequence compressor state
+    (batchgen/kv_cache/gpu_paged_kv_manager.py, SWA / compressed-ratio variants)."""
+
+    def __init__(self, cfg: ModelConfig, num_slots: int, device):
+        self.cfg = cfg
+        D, Di, win = cfg.head_dim, cfg.index_head_dim, cfg.sliding_window
+        parts = []
+        for l, r in enumerate(cfg.compress_ratios):
+            parts.append(((l, "ring"), (win, D)))
+            if r:
+                c = 2 if r == 4 else 1
+                parts += [((l, "kv"), (c * r, c * D)), ((l, "score"), (c * r, c * D))]
+                if r == 4:
+                    parts += [((l, "idx_kv"), (2 * r, 2 * Di)), ((l, "idx_score"), (2 * r, 2 * Di))]
+        super().__init__(parts, num_slots, device)
+        assert self.row_floats == cfg.v4_state_floats_per_seq()
 
 
 class HostStateStore:

@@ -69,6 +69,9 @@ def weight_bytes_per_rank(cfg: ModelConfig, tp: int, ep: int, sequence_parallel:
                           expert_offload_ratio: float = 0.0) -> Tuple[int, int]:
     """-> (non-expert bytes, routed-expert bytes resident on the GPU) for one rank."""
     H = cfg.hidden_size
+    if cfg.is_layered:
+        experts = sum(3 * H * s.mlp.ff * s.mlp.experts * 2 for s in cfg.layer_specs)
+        return int(cfg.param_count() * 2 - experts), int(experts)
     qb = _quant_bytes(cfg)
     lin = 1.0 + 4.0 / (128 * 128) if cfg.quant != "none" else 2.0     # attention / dense linears are FP8 or bf16
     dense = 2 * cfg.vocab_size * H * 2 / (1 if sequence_parallel else tp)
@@ -100,6 +103,8 @@ def plan_deployment(cfg: ModelConfig, ecfg: EngineConfig, machine: MachineProfil
     dense, experts = weight_bytes_per_rank(cfg, tp, ep, True, ecfg.expert_offload_ratio)
     # workspace of the largest prefill micro-batch: activations (bf16) of a few live tensors per token
     per_tok = cfg.hidden_size * 2 * 6 + cfg.num_heads // tp * (cfg.qk_head_dim + 2 * cfg.kv_cache_dim) * 2
+    if cfg.is_layered:
+        per_tok = layered_workspace_bytes(cfg)
     per_tok += cfg.num_experts_per_tok * (cfg.expert_hidden * 3 + cfg.moe_intermediate_size * 3) if cfg.n_routed_experts else 0
     workspace = int(min(ecfg.max_prefill_tokens, 32768) * per_tok * 1.25) + 2 * GiB
     graphs = int(0.5 * GiB + ecfg.cuda_graph_num_buckets * 64 * (1 << 20)) if ecfg.enable_cuda_graph else 0
@@ -121,12 +126,28 @@ def plan_deployment(cfg: ModelConfig, ecfg: EngineConfig, machine: MachineProfil
                           fits, note)
 
 
+def layered_workspace_bytes(cfg: ModelConfig) -> int:
+    """Activation bytes per prefill token of a layer-listed model: the widest layer's fp32 projections and operands, the
+    routed experts' rows, and a few rows of the model width."""
+    most = 0
+    for s in cfg.layer_specs:
+        m, f = s.mixer, s.mlp
+        n_in = 6 * m.heads * m.dim_p if m.recurrent else (m.heads + m.kv_heads) * (m.dim_p + m.vdim_p)
+        n_in += 2 * (f.shared_ff if f.kind == "moe" else f.ff) + f.experts
+        n_cat = m.heads * m.vdim_p + (f.shared_ff if f.kind == "moe" else f.ff)
+        routed = f.top * (2 * cfg.hidden_size + 8 * f.ff + 2 * f.ff + 4 * cfg.hidden_size) if f.kind == "moe" else 0
+        most = max(most, 4 * n_in + 2 * n_cat + routed)
+    return most + 16 * cfg.hidden_size
+
+
 def state_pool_bytes(cfg: ModelConfig, ecfg: EngineConfig) -> int:
     """Device bytes of the per-sequence state pool (recurrent state of KDA layers, or the window rings and compressor
     windows of DeepSeek-V4): one slot per sequence that may be live at once."""
     slots = ecfg.max_state_slots or ecfg.max_decode_batch
     if cfg.is_v4:
         return slots * 4 * cfg.v4_state_floats_per_seq()
+    if cfg.is_layered:
+        return slots * 4 * cfg.layered_state_floats_per_seq()
     return slots * cfg.kda_state_bytes_per_seq(max(ecfg.attn_tp_size, 1))
 
 
@@ -141,8 +162,10 @@ def size_kv_pool(cfg: ModelConfig, ecfg: EngineConfig, device: str, dtype) -> Tu
     if str(device).startswith("cuda"):
         free, total = torch.cuda.mem_get_info(torch.device(device))
         reserve = int(total * (1.0 - ecfg.gpu_memory_frac)) + 4 * GiB      # graphs + prefill workspace headroom
-        if cfg.has_kda or cfg.is_v4:                                       # per-sequence state slots come out of the same memory
+        if cfg.has_state:                                       # per-sequence state slots come out of the same memory
             reserve += state_pool_bytes(cfg, ecfg)
+        if cfg.is_layered:
+            reserve += int(1.25 * ecfg.max_prefill_tokens * layered_workspace_bytes(cfg))
         pages = max(16, (free - reserve) // page_bytes)
         if ecfg.max_model_len > 0:
             pages = min(pages, ecfg.max_decode_batch * (-(-ecfg.max_model_len // ecfg.page_size) + 1))
