@@ -156,6 +156,8 @@ class _Plan:
     cu_host: Optional[List[int]]
     slots: Optional[torch.Tensor]
     has_initial: Optional[torch.Tensor]
+    ctx: Optional[List[int]] = None
+    tiles: Dict[int, Tuple] = field(default_factory=dict)      # attention chunk -> (tensor-core tiles, rows of short pieces)
 
 
 class LayeredDecoder:
@@ -181,7 +183,24 @@ class LayeredDecoder:
         cu_t = torch.tensor(cu, dtype=torch.int32, device=dev)
         counts = torch.tensor([b - a for a, b in zip(cu, cu[1:])], device=dev)
         row_seq = torch.repeat_interleave(torch.arange(len(cu) - 1, dtype=torch.int32, device=dev), counts, output_size=T)
-        return _Plan((meta.positions + 1).to(torch.int32), row_seq, cu_t, list(cu), meta.state_slots, meta.state_has_initial)
+        return _Plan((meta.positions + 1).to(torch.int32), row_seq, cu_t, list(cu), meta.state_slots, meta.state_has_initial,
+                     list(meta.ctx_lens))
+
+    def _tiles(self, plan: _Plan, chunk: int, T: int):
+        """How the rows of a prompt step split over the attention kernels: pieces of a few tokens (decoded tokens among
+        them) go row by row, the rest in 128-query tiles."""
+        if chunk not in plan.tiles:
+            cu, least = plan.cu_host, talking.PREFILL_MIN_TOKENS
+            blocks = talking.work_blocks(talking.prefill_work(cu, plan.ctx, chunk, least), T, self.device)
+            short = [t for a, b in zip(cu, cu[1:]) if b - a < least for t in range(a, b)]
+            rows = seqs = None
+            if blocks and short:
+                rows = torch.tensor(short, dtype=torch.int32, device=self.device)
+                seqs = plan.row_seq[rows.long()].contiguous()
+            elif short:
+                seqs = plan.row_seq
+            plan.tiles[chunk] = (blocks, bool(short), rows, seqs)
+        return plan.tiles[chunk]
 
     # ------------------------------------------------------------------ mixers
     def _delta(self, l: int, lw: LayeredLayer, z, out, plan: _Plan, cache) -> None:
@@ -197,7 +216,14 @@ class LayeredDecoder:
         q, k = lw.seg["q"], lw.seg["k"][0]
         kv = cache.latent(l)
         talking.kv_write(z[:, k:k + lw.talk.kv_row], meta.slot_mapping, kv)
-        talking.attend_rows(z[:, q[0]:q[0] + q[1]], lw.talk, kv, meta.block_table, plan.lens, out, plan.row_seq)
+        zq = z[:, q[0]:q[0] + q[1]]
+        rows, seqs = None, plan.row_seq
+        if plan.cu is not None and z.is_cuda and talking.prefill_supported(lw.talk, kv.dtype, kv.shape[1]):
+            blocks, short, rows, seqs = self._tiles(plan, lw.talk.chunk, z.shape[0])
+            talking.attend_prefill(zq, lw.talk, kv, meta.block_table, out, blocks)
+            if not short:
+                return
+        talking.attend_rows(zq, lw.talk, kv, meta.block_table, plan.lens, out, seqs, rows)
 
     # ------------------------------------------------------------------ forward
     def forward(self, ids: torch.Tensor, meta: AttnMeta, cache) -> torch.Tensor:

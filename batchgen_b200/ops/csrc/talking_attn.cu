@@ -136,11 +136,15 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
     return (long long)bt[pos / p.page] * p.page_stride + (long long)(pos % p.page) * p.row;
   };
   auto fetch = [&](int unit, long long off) {                     // K rows of unit's key head -> this warp's buffer
-    const int c = unit / hg_n, vec = dp * (int)sizeof(KT) / 16;
-    for (int i = lane; i < NT * vec; i += 32) {                    // NT * vec is a multiple of 32: the shuffle is warp-wide
-      const int kr = i / vec, cc = i % vec;
+    const int c = unit / hg_n, vec = dp * (int)sizeof(KT) / 16;    // 16-byte pieces of a K row; NT * vec % 32 == 0
+    const int step_k = 32 / vec, step_c = 32 % vec;
+    int kr = lane / vec, cc = lane % vec;
+    for (int i = 0; i < vec; ++i) {
       const long long o = __shfl_sync(0xffffffffu, off, kr);
       if (o >= 0) cp16(kb + kr * krow + cc * 16, reinterpret_cast<const char*>(cache + o + c * dp) + cc * 16);
+      kr += step_k;
+      cc += step_c;
+      if (cc >= vec) { cc -= vec; ++kr; }
     }
     cp_commit();
   };
@@ -148,13 +152,11 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
   const int cols = dvp / 4, items = G * hg_n * cols;
   const int KG = items >= kThreads ? 1 : kThreads / items;
   const int kg = items >= kThreads ? 0 : tid / items, item0 = items >= kThreads ? tid : tid % items;
-  float acc[NI][4][4];
+  float2 acc[NI][4][2];
 #pragma unroll
   for (int n = 0; n < NI; ++n)
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) acc[n][i][j] = 0.f;
+    for (int i = 0; i < 4; ++i) acc[n][i][0] = acc[n][i][1] = make_float2(0.f, 0.f);
 
   long long off = my_lo < my_hi ? key_offset(my_lo) : -1;
   if (my_lo < my_hi && warp < units) fetch(warp, off);
@@ -167,7 +169,9 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
       cp_wait0();
       __syncwarp();
       const int c = u / hg_n, h0 = c * rep + (u % hg_n) * 4, nh = min(4, rep - (u % hg_n) * 4);
-      float s[4] = {0.f, 0.f, 0.f, 0.f};
+      float2 s[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) s[i] = make_float2(0.f, 0.f);
       const KT* kr = reinterpret_cast<const KT*>(kb + lane * krow);
       const float* qh[4];
 #pragma unroll
@@ -180,12 +184,13 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
         for (int i = 0; i < 4; ++i) {
           load8(qh[i] + e, qv);
 #pragma unroll
-          for (int j = 0; j < 8; ++j) s[i] = fmaf(qv[j], k[j], s[i]);
+          for (int j = 0; j < 8; j += 2)                           // packed FMAs (fma.rn.f32x2)
+            s[i] = __ffma2_rn(make_float2(qv[j], qv[j + 1]), make_float2(k[j], k[j + 1]), s[i]);
         }
       }
 #pragma unroll
       for (int i = 0; i < 4; ++i)
-        if (i < nh) raw[(h0 + i) * NT + lane] = s[i];
+        if (i < nh) raw[(h0 + i) * NT + lane] = s[i].x + s[i].y;
       __syncwarp();
       if (u + kWarps < units) fetch(u + kWarps, off_now);
       else if (tile + 1 < my_hi) fetch(warp, off);                 // next tile's rows fly during the rest of this tile
@@ -218,8 +223,7 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
       }
     }
     __syncthreads();
-    // O = O * alpha + P . V
-    const int j_lo = max(first - tile * NT, 0), j_hi = min(L - tile * NT, NT);
+    // O = O * alpha + P . V, four keys at a time (unseen keys have p = 0 and are not read)
     if (kg < KG) {
 #pragma unroll
       for (int n = 0; n < NI; ++n) {
@@ -234,17 +238,27 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
             const int h = h0 + min(i, nh - 1);
             ph[i] = pr + h * NT;
             const float al = a_s[h];
-#pragma unroll
-            for (int j = 0; j < 4; ++j) acc[n][i][j] *= al;
+            acc[n][i][0].x *= al; acc[n][i][0].y *= al; acc[n][i][1].x *= al; acc[n][i][1].y *= al;
           }
-#pragma unroll 8
-          for (int j = j_lo + kg; j < j_hi; j += KG) {
-            const float4 v = load4(vb + koff[j]);
+#pragma unroll 2
+          for (int j = 4 * kg; j < NT; j += 4 * KG) {
+            float4 v[4], w[4];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-              const float w = ph[i][j];
-              acc[n][i][0] = fmaf(w, v.x, acc[n][i][0]); acc[n][i][1] = fmaf(w, v.y, acc[n][i][1]);
-              acc[n][i][2] = fmaf(w, v.z, acc[n][i][2]); acc[n][i][3] = fmaf(w, v.w, acc[n][i][3]);
+            for (int x = 0; x < 4; ++x) {
+              const long long o = koff[j + x];
+              v[x] = o >= 0 ? load4(vb + o) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) w[i] = *reinterpret_cast<const float4*>(ph[i] + j);
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+              const float2 lo = make_float2(v[x].x, v[x].y), hi = make_float2(v[x].z, v[x].w);
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                const float f = x == 0 ? w[i].x : x == 1 ? w[i].y : x == 2 ? w[i].z : w[i].w;
+                acc[n][i][0] = __ffma2_rn(make_float2(f, f), lo, acc[n][i][0]);
+                acc[n][i][1] = __ffma2_rn(make_float2(f, f), hi, acc[n][i][1]);
+              }
             }
           }
         }
@@ -260,7 +274,7 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
     if (kg > 0 && kg < KG) {
 #pragma unroll
       for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(red + ((size_t)i * kThreads + tid) * 4) =
-          make_float4(acc[0][i][0], acc[0][i][1], acc[0][i][2], acc[0][i][3]);
+          make_float4(acc[0][i][0].x, acc[0][i][0].y, acc[0][i][1].x, acc[0][i][1].y);
     }
     __syncthreads();
     if (kg == 0) {
@@ -268,7 +282,7 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const float4 v = *reinterpret_cast<const float4*>(red + ((size_t)i * kThreads + k * items + tid) * 4);
-          acc[0][i][0] += v.x; acc[0][i][1] += v.y; acc[0][i][2] += v.z; acc[0][i][3] += v.w;
+          acc[0][i][0].x += v.x; acc[0][i][0].y += v.y; acc[0][i][1].x += v.z; acc[0][i][1].y += v.w;
         }
       }
     }
@@ -284,7 +298,7 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
         for (int i = 0; i < 4; ++i) {
           if (i >= nh) break;
           const int h = h0 + i, col = h * dvp + cc * 4;
-          const float4 v = make_float4(acc[n][i][0], acc[n][i][1], acc[n][i][2], acc[n][i][3]);
+          const float4 v = make_float4(acc[n][i][0].x, acc[n][i][0].y, acc[n][i][1].x, acc[n][i][1].y);
           if (p.n_splits == 1) {
             const float inv = 1.0f / (l_s[h] + (p.sink ? exp2f(-m_s[h]) : 0.f));
             put4(out + col, make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv));

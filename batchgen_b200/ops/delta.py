@@ -69,11 +69,18 @@ def delta_forward(z: torch.Tensor, offs: Tuple[int, int, int, int, int], wl: tor
     assert z.dtype == wl.dtype == state.dtype == torch.float32 and z.stride(1) == 1 and wl.stride(1) == 1
     assert out.stride(1) == 1 and state.stride(1) == 1 and slots.dtype == torch.int32
     arr = (ctypes.c_int * 5)(*offs)
-    rc = _ext.lib().bg_delta_step(
+    T = z.shape[0]
+    scratch = None
+    if cu is not None or p.dim_p > 128:
+        per = p.heads * (6 * p.dim_p + 4)                      # a token's record and its scan output
+        scratch = torch.empty(T * per, dtype=torch.float32, device=z.device)
+    rc = _ext.lib().bg_delta_forward(
         _i(_DT[out.dtype]), _ext.ptr(z), _i(z.stride(0)), arr, _ext.ptr(wl), _i(wl.stride(0)), _ext.ptr(p.w0),
         _ext.ptr(p.ab), _ext.ptr(p.norm_w), _ext.ptr(state), ctypes.c_longlong(state.stride(0)), _ext.ptr(cu),
-        _ext.ptr(slots), _ext.ptr(has_initial), _ext.ptr(out), _i(out.stride(0)), _i(slots.shape[0]), _i(p.heads),
+        _ext.ptr(slots), _ext.ptr(has_initial), _ext.ptr(out), _i(out.stride(0)), _i(T), _i(slots.shape[0]), _i(p.heads),
         _i(p.dim_p), _i(p.dim), ctypes.c_float(p.decay_scale), ctypes.c_float(p.unit_eps), ctypes.c_float(p.eps),
-        _ext.stream())
-    _ext.check(rc, "bg_delta_step")
+        _ext.ptr(scratch), _i(_ext.num_sms(z.device)), _ext.ptr(_ext.status_word(z.device)), _ext.stream())
+    if rc == -1:
+        raise _ext.KernelError(f"delta_forward: {p.heads} heads of {p.dim_p} are outside the kernels' contract (width <= 256)")
+    _ext.check(rc, "bg_delta_forward", kernels=3 if scratch is not None else 1)
     return out

@@ -1,11 +1,13 @@
 """Paged grouped-query attention whose heads' scores are mixed before the softmax, with chunked visibility and a
-zero-score sink (``csrc/talking_attn.cu``): cache rows, and one query row per CTA for decode and short pieces.
+zero-score sink: cache rows and one query row per CTA for decode and short pieces (``csrc/talking_attn.cu``), tensor-core
+flash attention over mixed queries for long pieces of prompts (``csrc/talking_prefill.cu``).
 """
 from __future__ import annotations
 
 import ctypes
+import math
 from dataclasses import dataclass
-from typing import Optional
+from typing import List, Optional, Sequence, Tuple
 
 import torch
 
@@ -73,8 +75,15 @@ def _rows_ref(q, p: TalkParams, cache, block_table, lens, out, row_seq):
 
 
 def _splits(rows: int, keys: int, sms: int) -> int:
-    tiles = max(1, -(-keys // 32))
-    return max(1, min(16, 3 * sms // max(rows, 1), tiles))
+    """Key ranges per row: whole rounds of CTAs over the SMs (two fit an SM), each range a few 32-key tiles long."""
+    slots, tiles = 2 * sms, max(1, -(-keys // 32))
+    best, score = 1, -1.0
+    for s in range(1, max(1, min(16, tiles // 4)) + 1):
+        rounds = rows * s / slots
+        v = rounds / math.ceil(rounds) - 0.004 * s             # share of the slots that work, less the merge
+        if v > score:
+            best, score = s, v
+    return best
 
 
 def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table: torch.Tensor, lens: torch.Tensor,
@@ -111,3 +120,63 @@ def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table
         raise _ext.KernelError(f"attend_rows: heads {H}/{p.kv_heads}, widths {p.dim_p}/{p.vdim_p} are outside the kernel's "
                                "contract (shared memory of one CTA, 1,024 head-column items)")
     _ext.check(rc, "bg_talk_rows", kernels=2 if num_splits > 1 else 1)
+
+
+PREFILL_MIN_TOKENS = 32      # pieces at least this long go to the tensor-core kernel
+_TILE = 128                  # queries of one CTA
+_FOLD_ROWS = 8192            # rows whose mixed queries are held at a time
+
+
+def prefill_supported(p: TalkParams, dtype: torch.dtype, page: int) -> bool:
+    """The tensor-core kernel reads bf16 pages and keeps one head's value columns in TMEM."""
+    return dtype == torch.bfloat16 and p.vdim_p <= 256 and page >= 16
+
+
+def prefill_work(cu: Sequence[int], ctx: Sequence[int], chunk: int, min_tokens: int = 1) -> List[Tuple[int, int, int, int]]:
+    """Tiles (first query row, queries, sequence, position of the first query) of every piece of at least ``min_tokens``
+    tokens, the tiles with the most visible keys first."""
+    out = []
+    for i in range(len(cu) - 1):
+        a, b = int(cu[i]), int(cu[i + 1])
+        if b - a < min_tokens:
+            continue
+        for q0 in range(a, b, _TILE):
+            out.append((q0, min(_TILE, b - q0), i, int(ctx[i]) + q0 - a))
+    out.sort(key=lambda w: -(w[3] + w[1] - (w[3] // chunk * chunk if chunk else 0)))
+    return out
+
+
+def work_blocks(work: List[Tuple[int, int, int, int]], rows: int, device) -> List[Tuple[int, int, torch.Tensor]]:
+    """Tiles grouped by ranges of query rows: (first row, rows, [n, 4] int32 tiles).  Bounds the mixed queries' memory."""
+    blocks: dict = {}
+    for w in work:
+        blocks.setdefault(w[0] // _FOLD_ROWS, []).append(w)
+    out = []
+    for b in sorted(blocks):
+        lo = b * _FOLD_ROWS
+        hi = min(rows, max(w[0] + w[1] for w in blocks[b]))
+        out.append((lo, hi - lo, torch.tensor(blocks[b], dtype=torch.int32, device=device)))
+    return out
+
+
+def attend_prefill(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table: torch.Tensor, out: torch.Tensor,
+                   blocks: List[Tuple[int, int, torch.Tensor]]) -> None:
+    """CUDA, bf16 cache: q [T, >= H * dim_p] fp32 -> out [T, >= H * vdim_p] for the rows covered by ``blocks``
+    (``work_blocks``).  The keys of every query are in the cache already."""
+    P, page, row = cache.shape
+    H, G = p.heads, p.kv_heads
+    kc = -(-G * p.dim_p // 64) * 64
+    assert q.dtype == torch.float32 and q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == cache.dtype == torch.bfloat16
+    assert row == p.kv_row and cache.stride(1) == row and block_table.dtype == torch.int32
+    L = _ext.lib()
+    for lo, n, work in blocks:
+        qf = torch.empty(n, H, kc, dtype=torch.bfloat16, device=q.device)
+        rc = L.bg_talk_fold(_ext.ptr(q[lo:]), _i(q.stride(0)), _ext.ptr(p.talk), _ext.ptr(qf), _i(n), _i(H), _i(G),
+                            _i(p.dim_p), _i(kc), ctypes.c_float(p.scale), _ext.stream())
+        _ext.check(rc, "bg_talk_fold")
+        rc = L.bg_talk_prefill(
+            _ext.ptr(qf), _ext.ptr(cache), ctypes.c_longlong(cache.stride(0)), _i(P), _i(page), _i(row),
+            _ext.ptr(block_table), _i(block_table.stride(0)), _i(block_table.shape[1]), _ext.ptr(work), _i(work.shape[0]),
+            _i(n), _i(lo), _ext.ptr(out), _i(out.stride(0)), _i(H), _i(G), _i(p.dim_p), _i(p.vdim_p), _i(kc), _i(p.chunk),
+            _i(p.sink), _ext.ptr(_ext.status_word(q.device)), _ext.stream())
+        _ext.check(rc, "bg_talk_prefill")
