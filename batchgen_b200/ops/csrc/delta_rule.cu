@@ -14,7 +14,7 @@
 // Decode (`decode_kernel`, D <= 128): a token is one read and write of the state with everything else fused around it.
 //
 // Prompts (`prep` -> `scan` -> `finish`): a value column of S evolves on its own once w, u, a * u and w * r are known, so the
-// scan splits a head's columns over CTAs of 32 columns and needs no barrier inside a token (4 lanes share a column, two
+// scan splits a head's columns over CTAs of 32 columns and needs no barrier inside a token (8 lanes share a column, three
 // shuffles sum their rows; packed fp32 FMAs).  `prep` computes the per-token vectors for all tokens in parallel and `finish`
 // applies the output norm and gate, which need whole heads.
 //
@@ -56,10 +56,12 @@ __device__ __forceinline__ float sigm(float x) { return 1.0f / (1.0f + expf(-x))
 constexpr int kMaxD = 256;
 
 // Decode, one token per sequence, persistent over (sequence, head) items.  A head's state is one contiguous block of
-// D * D * 4 bytes: bulk copies bring the next two items' blocks into a ring of three shared-memory buffers while the current
-// one is worked on in place, and a bulk copy takes it back, so the SM always has loads and stores in flight.
+// D * D * 4 bytes.  A producer thread brings blocks into a ring of three shared-memory buffers with bulk copies and takes
+// them back the same way; two groups of four warps work on alternate items in place, so one group's barriers and reductions
+// hide behind the other's arithmetic and the SM always has loads and stores in flight.
 //
-// Thread (ig, jq): value columns 4 jq .. 4 jq + 3, key rows ig, ig + RG, ... (NR of them at most).
+// A warp owns 32 value columns: lane (rg, jq) has columns 4 jq .. 4 jq + 3 of them and the key rows rg * NR .. + NR - 1
+// (two shuffles sum the four row groups), so a group needs two barriers per item: vectors ready, output norm.
 constexpr int kBufs = 3;
 
 __device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
@@ -73,155 +75,202 @@ __device__ __forceinline__ void bulk_store(void* dst, const void* src, uint32_t 
   asm volatile("cp.async.bulk.commit_group;" ::: "memory");
 }
 
-template <typename OT, int NT, int NR>
-__global__ void __launch_bounds__(NT) decode_kernel(const Params p, int items, int* status) {
+__device__ __forceinline__ void group_sync(int group) { asm volatile("bar.sync %0, 128;" ::"r"(group + 1) : "memory"); }
+__device__ __forceinline__ float4 xor_sum(float4 v, int mask) {
+  v.x += __shfl_xor_sync(0xffffffffu, v.x, mask); v.y += __shfl_xor_sync(0xffffffffu, v.y, mask);
+  v.z += __shfl_xor_sync(0xffffffffu, v.z, mask); v.w += __shfl_xor_sync(0xffffffffu, v.w, mask);
+  return v;
+}
+
+template <typename OT, int NR>
+__global__ void __launch_bounds__(288) decode_kernel(const Params p, int items, int* status) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   extern __shared__ __align__(128) float ring[];                // kBufs x D * D
-  __shared__ uint64_t full[kBufs];
+  __shared__ uint64_t full[kBufs], done[kBufs];
   __shared__ int abort_s;
-  __shared__ __align__(16) float sk[128], sw[128], sak[128], swr[128], sv[128];
-  __shared__ float red[3][4], red_o[2];
-  __shared__ __align__(16) float4 part_y[NT], part_q[NT];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int D = p.D, H = p.H, Q = D / 4, RG = NT / Q, DD = D * D;
-  const uint32_t bytes = (uint32_t)DD * 4;
-  const int jq = tid % Q, ig = tid / Q;
-  const bool active = ig < RG;
-  const int dwarps = (D + 31) / 32, owarps = (Q + 31) / 32;
+  __shared__ __align__(16) float vec[2][4][4 * NR];             // per group: k, w, a * k, w * r (zero past D)
+  __shared__ __align__(16) float sv[2][128];
+  __shared__ float red[2][3][4], red_o[2][4];
+  const int tid = threadIdx.x, lane = tid & 31;
+  const int D = p.D, H = p.H, DD = D * D, Q = D / 4;
   volatile int* abort_flag = &abort_s;
   if (tid == 0) {
-    for (int s = 0; s < kBufs; ++s) mbar_init(&full[s], 1);
+    for (int s = 0; s < kBufs; ++s) { mbar_init(&full[s], 1); mbar_init(&done[s], 1); }
     abort_s = 0;
     mbar_fence_init();
   }
+  for (int i = tid; i < 2 * 4 * 4 * NR; i += 288) (&vec[0][0][0])[i] = 0.f;
   __syncthreads();
-  auto block_of = [&](int item) { return p.state + p.slots[item / H] * p.slot_stride + (size_t)(item % H) * DD; };
-  int ahead = blockIdx.x;                                       // thread 0: next item to load (rows without a slot are skipped)
-  auto load_state = [&](int stage) {
-    while (ahead < items && p.slots[ahead / H] < 0) ahead += gridDim.x;
-    if (ahead < items) {
-      mbar_expect_tx(&full[stage], bytes);
-      bulk_load(ring + (size_t)stage * DD, block_of(ahead), bytes, &full[stage]);
-      ahead += gridDim.x;
+  if (tid >= 256) {
+    // ------------------------------------------------------------ producer (one thread): item k lives in buffer k % kBufs
+    if (tid != 256) return;
+    const uint32_t bytes = (uint32_t)DD * 4;
+    auto next_live = [&](int item) {
+      while (item < items && p.slots[item / H] < 0) item += gridDim.x;
+      return item;
+    };
+    auto block_of = [&](int item) { return p.state + p.slots[item / H] * p.slot_stride + (size_t)(item % H) * DD; };
+    int ahead = next_live(blockIdx.x);
+    auto load = [&](int k) {
+      if (ahead >= items) return;
+      mbar_expect_tx(&full[k % kBufs], bytes);
+      bulk_load(ring + (size_t)(k % kBufs) * DD, block_of(ahead), bytes, &full[k % kBufs]);
+      ahead = next_live(ahead + gridDim.x);
+    };
+    for (int k = 0; k < kBufs; ++k) load(k);
+    int k = 0;
+    for (int item = next_live(blockIdx.x); item < items; item = next_live(item + gridDim.x), ++k) {
+      if (!mbar_wait(&done[k % kBufs], (k / kBufs) & 1, abort_flag, kTimeoutProducer)) break;
+      bulk_store(block_of(item), ring + (size_t)(k % kBufs) * DD, bytes);
+      asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
+      load(k + kBufs);
     }
-  };
-  if (tid == 0) { load_state(0); load_state(1); }
-  float nr = 0.f, nk = 0.f, nv = 0.f, na = 0.f, nw = 0.f, nw0 = 0.f, nab = 0.f;
-  auto load = [&](int item) {
-    if (item < items && tid < D) {
-      const int t = item / H, hc = (item % H) * D + tid;
-      const float* zr = p.z + (size_t)t * p.ldz + hc;
-      nr = zr[p.off_r]; nk = zr[p.off_k]; nv = zr[p.off_v]; na = zr[p.off_a];
-      nw = p.wl[(size_t)t * p.ld_wl + hc];
-      nw0 = p.w0[hc];
-      nab = p.ab[hc];
-    }
-  };
-  load(blockIdx.x);
-  int n = 0;                                                    // items worked on so far
-  for (int item = blockIdx.x; item < items; item += gridDim.x) {
-    const int t = item / H, h = item % H;
-    OT* out = reinterpret_cast<OT*>(p.out) + (size_t)t * p.ldo + h * D;
-    if (p.slots[t] < 0) {
-      for (int j = tid; j < Q; j += NT) put4(out + 4 * j, make_float4(0.f, 0.f, 0.f, 0.f));
-      load(item + gridDim.x);
-      continue;
-    }
-    const int stage = n % kBufs;
-    float4 g = make_float4(0.f, 0.f, 0.f, 0.f), nw4 = g;
-    if (tid < Q) {
-      g = *reinterpret_cast<const float4*>(p.z + (size_t)t * p.ldz + p.off_g + h * D + 4 * tid);
-      nw4 = *reinterpret_cast<const float4*>(p.norm_w + h * D + 4 * tid);
-    }
-    if (warp < dwarps) {
-      const float r = nr, k = nk;
-      const float a = sigm(na + nab);
-      const float w = expf(-p.cdecay * sigm(nw + nw0));
-      if (tid < D) {
-        sk[tid] = k; sw[tid] = w; sak[tid] = a * k; swr[tid] = w * r; sv[tid] = nv;
-      }
-      const float s0 = warp_sum(tid < D ? k * k : 0.f), s1 = warp_sum(tid < D ? r * k : 0.f);
-      const float s2 = warp_sum(tid < D ? r * a * k : 0.f);
-      if (lane == 0) { red[0][warp] = s0; red[1][warp] = s1; red[2][warp] = s2; }
-    }
-    load(item + gridDim.x);
-    const bool ok = mbar_wait(&full[stage], (n / kBufs) & 1, abort_flag, kTimeoutProducer);
-    if (__syncthreads_or(!ok)) break;
-    float kk = 0.f, rk = 0.f, rak = 0.f;
-    for (int i = 0; i < dwarps; ++i) { kk += red[0][i]; rk += red[1][i]; rak += red[2][i]; }
-    const float inv2 = 1.0f / (kk + p.ueps);                    // u u^T = k k^T * inv2
-    float* Sb = ring + (size_t)stage * DD;
-    float4 S[NR], y = make_float4(0.f, 0.f, 0.f, 0.f), q = y;
-    if (active) {
-#pragma unroll
-      for (int m = 0; m < NR; ++m) {
-        const int i = ig + m * RG;
-        if (i < D) {
-          S[m] = *reinterpret_cast<const float4*>(Sb + i * D + 4 * jq);
-          const float k = sk[i], wr = swr[i];
-          y.x = fmaf(k, S[m].x, y.x); y.y = fmaf(k, S[m].y, y.y); y.z = fmaf(k, S[m].z, y.z); y.w = fmaf(k, S[m].w, y.w);
-          q.x = fmaf(wr, S[m].x, q.x); q.y = fmaf(wr, S[m].y, q.y); q.z = fmaf(wr, S[m].z, q.z); q.w = fmaf(wr, S[m].w, q.w);
-        }
-      }
-      part_y[tid] = y;
-      part_q[tid] = q;
-    }
-    __syncthreads();
-    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (active) {
-      y = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int i = 0; i < RG; ++i) {
-        const float4 v = part_y[i * Q + jq];
-        y.x += v.x; y.y += v.y; y.z += v.z; y.w += v.w;
-      }
-      y.x *= inv2; y.y *= inv2; y.z *= inv2; y.w *= inv2;
-      const float4 v = *reinterpret_cast<const float4*>(&sv[4 * jq]);
-      if (ig == 0) {
-        q = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int i = 0; i < RG; ++i) {
-          const float4 b = part_q[i * Q + jq];
-          q.x += b.x; q.y += b.y; q.z += b.z; q.w += b.w;
-        }
-        o.x = q.x - rak * y.x + rk * v.x; o.y = q.y - rak * y.y + rk * v.y;
-        o.z = q.z - rak * y.z + rk * v.z; o.w = q.w - rak * y.w + rk * v.w;
-      }
-#pragma unroll
-      for (int m = 0; m < NR; ++m) {
-        const int i = ig + m * RG;
-        if (i < D) {
-          const float k = sk[i], w = sw[i], ak = sak[i];
-          *reinterpret_cast<float4*>(Sb + i * D + 4 * jq) =
-              make_float4(fmaf(w, S[m].x, fmaf(k, v.x, -ak * y.x)), fmaf(w, S[m].y, fmaf(k, v.y, -ak * y.y)),
-                          fmaf(w, S[m].z, fmaf(k, v.z, -ak * y.z)), fmaf(w, S[m].w, fmaf(k, v.w, -ak * y.w)));
-        }
-      }
-    }
-    if (warp < owarps) {
-      const float s = warp_sum(o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w);
-      if (lane == 0) red_o[warp] = s;
-    }
-    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-    __syncthreads();
-    if (tid == 0) {
-      bulk_store(block_of(item), Sb, bytes);
-      // the block stored before this one has left its buffer: that buffer takes the item two ahead
-      asm volatile("cp.async.bulk.wait_group.read 1;" ::: "memory");
-      load_state((n + 2) % kBufs);
-    }
-    if (tid < Q) {
-      float oo = 0.f;
-      for (int i = 0; i < owarps; ++i) oo += red_o[i];
-      const float rs = 1.0f / sqrtf(oo / (float)p.Dreal + p.eps);
-      put4(out + 4 * tid, make_float4(o.x * rs * nw4.x * sigm(g.x), o.y * rs * nw4.y * sigm(g.y),
-                                      o.z * rs * nw4.z * sigm(g.z), o.w * rs * nw4.w * sigm(g.w)));
-    }
-    ++n;
-  }
-  if (tid == 0) {
     asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
     if (abort_s != 0) {
       for (uint32_t i = 0; i < (1u << 16); ++i) __nanosleep(20);     // bounded grace period for copies in flight
       if (status != nullptr) atomicMax(status, abort_s);
+    }
+    return;
+  }
+  // -------------------------------------------------------------- two groups of 128 threads
+  const int group = tid >> 7, gt = tid & 127, gw = gt >> 5, jq = lane & 7, rg = lane >> 3;
+  const int quad = gw * 8 + jq, dwarps = (D + 31) / 32;
+  const bool col_ok = quad < Q;
+  float nr = 0.f, nk = 0.f, nv = 0.f, na = 0.f, nw = 0.f, nw0 = 0.f, nab = 0.f;
+  auto fetch = [&](int item) {
+    if (item < items && gt < D) {
+      const int hc = (item % H) * D + gt;
+      const float* zr = p.z + (size_t)(item / H) * p.ldz + hc;
+      nr = zr[p.off_r]; nk = zr[p.off_k]; nv = zr[p.off_v]; na = zr[p.off_a];
+      nw = p.wl[(size_t)(item / H) * p.ld_wl + hc];
+      nw0 = p.w0[hc];
+      nab = p.ab[hc];
+    }
+  };
+  int fetched = blockIdx.x + group * gridDim.x, k = 0;          // k: live items so far; the group takes those with k % 2 == group
+  fetch(fetched);
+  int slot_next = blockIdx.x < items ? p.slots[blockIdx.x / H] : -1;
+  for (int item = blockIdx.x; item < items; item += gridDim.x) {
+    const int slot = slot_next;
+    slot_next = item + (int)gridDim.x < items ? p.slots[(item + gridDim.x) / H] : -1;
+    const int t = item / H, h = item % H;
+    OT* out = reinterpret_cast<OT*>(p.out) + (size_t)t * p.ldo + h * D;
+    if (slot < 0) {
+      if (group == 0 && gt < Q) put4(out + 4 * gt, make_float4(0.f, 0.f, 0.f, 0.f));
+      continue;
+    }
+    const int buf = k % kBufs, phase = (k / kBufs) & 1;
+    if ((k++ & 1) != group) continue;
+    if (fetched != item) fetch(item);                            // rows without a slot shifted the turns
+    float4 g = make_float4(0.f, 0.f, 0.f, 0.f), nw4 = g;
+    if (col_ok && rg == 0) {
+      g = *reinterpret_cast<const float4*>(p.z + (size_t)t * p.ldz + p.off_g + h * D + 4 * quad);
+      nw4 = *reinterpret_cast<const float4*>(p.norm_w + h * D + 4 * quad);
+    }
+    float (*v4)[4 * NR] = vec[group];
+    if (gw < dwarps) {
+      const float r = nr, kc = nk;
+      const float a = sigm(na + nab);
+      const float w = expf(-p.cdecay * sigm(nw + nw0));
+      const bool in = gt < D;
+      if (in) {
+        v4[0][gt] = kc; v4[1][gt] = w; v4[2][gt] = a * kc; v4[3][gt] = w * r;
+        sv[group][gt] = nv;
+      }
+      float s0 = in ? kc * kc : 0.f, s1 = in ? r * kc : 0.f, s2 = in ? r * a * kc : 0.f;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        s0 += __shfl_xor_sync(0xffffffffu, s0, o);
+        s1 += __shfl_xor_sync(0xffffffffu, s1, o);
+        s2 += __shfl_xor_sync(0xffffffffu, s2, o);
+      }
+      if (lane == 0) { red[group][0][gw] = s0; red[group][1][gw] = s1; red[group][2][gw] = s2; }
+    }
+    fetched = item + 2 * (int)gridDim.x;
+    fetch(fetched);
+    group_sync(group);
+    const bool ok = mbar_wait(&full[buf], phase, abort_flag, kTimeoutMma);
+    float kk = 0.f, rk = 0.f, rak = 0.f;
+    for (int i = 0; i < dwarps; ++i) { kk += red[group][0][i]; rk += red[group][1][i]; rak += red[group][2][i]; }
+    const float inv2 = 1.0f / (kk + p.ueps);                    // u u^T = k k^T * inv2
+    float* Sb = ring + (size_t)buf * DD + (size_t)rg * NR * D + 4 * quad;
+    float2 y[2], q[2];
+    y[0] = y[1] = q[0] = q[1] = make_float2(0.f, 0.f);
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    const int rows = min(NR, max(D - rg * NR, 0));
+    const bool whole = D == 4 * NR;                              // every lane has all its rows: no guards
+    auto read_row = [&](int m, float kf, float rf) {
+      const float4 s = *reinterpret_cast<const float4*>(Sb + m * D);
+      const float2 s0 = make_float2(s.x, s.y), s1 = make_float2(s.z, s.w), k2 = make_float2(kf, kf), r2 = make_float2(rf, rf);
+      y[0] = __ffma2_rn(k2, s0, y[0]); y[1] = __ffma2_rn(k2, s1, y[1]);
+      q[0] = __ffma2_rn(r2, s0, q[0]); q[1] = __ffma2_rn(r2, s1, q[1]);
+    };
+    if (ok && col_ok) {
+      const float* kv = &v4[0][rg * NR];
+      const float* rv = &v4[3][rg * NR];
+      if (whole) {
+#pragma unroll
+        for (int m = 0; m < NR; m += 4) {
+          const float4 k4 = *reinterpret_cast<const float4*>(kv + m), r4 = *reinterpret_cast<const float4*>(rv + m);
+          read_row(m, k4.x, r4.x); read_row(m + 1, k4.y, r4.y); read_row(m + 2, k4.z, r4.z); read_row(m + 3, k4.w, r4.w);
+        }
+      } else {
+        for (int m = 0; m < rows; ++m) read_row(m, kv[m], rv[m]);
+      }
+    }
+    float4 ys = make_float4(y[0].x, y[0].y, y[1].x, y[1].y), qs = make_float4(q[0].x, q[0].y, q[1].x, q[1].y);
+    ys = xor_sum(xor_sum(ys, 8), 16);
+    qs = xor_sum(xor_sum(qs, 8), 16);
+    if (ok && col_ok) {
+      ys.x *= inv2; ys.y *= inv2; ys.z *= inv2; ys.w *= inv2;
+      const float4 v = *reinterpret_cast<const float4*>(&sv[group][4 * quad]);
+      o.x = qs.x - rak * ys.x + rk * v.x; o.y = qs.y - rak * ys.y + rk * v.y;
+      o.z = qs.z - rak * ys.z + rk * v.z; o.w = qs.w - rak * ys.w + rk * v.w;
+      const float2 ny0 = make_float2(-ys.x, -ys.y), ny1 = make_float2(-ys.z, -ys.w);
+      const float2 v0 = make_float2(v.x, v.y), v1 = make_float2(v.z, v.w);
+      auto next_row = [&](const float4& s, float kf, float wf, float af) {
+        const float2 k2 = make_float2(kf, kf), w2 = make_float2(wf, wf), a2 = make_float2(af, af);
+        const float2 n0 = __ffma2_rn(w2, make_float2(s.x, s.y), __ffma2_rn(k2, v0, __fmul2_rn(a2, ny0)));
+        const float2 n1 = __ffma2_rn(w2, make_float2(s.z, s.w), __ffma2_rn(k2, v1, __fmul2_rn(a2, ny1)));
+        return make_float4(n0.x, n0.y, n1.x, n1.y);
+      };
+      const float* kv = &v4[0][rg * NR];
+      const float* wv = &v4[1][rg * NR];
+      const float* av = &v4[2][rg * NR];
+      if (whole) {
+#pragma unroll
+        for (int m = 0; m < NR; m += 8) {                        // eight rows in flight: loads first, then stores
+          float4 s[8];
+#pragma unroll
+          for (int j = 0; j < 8; ++j) s[j] = *reinterpret_cast<const float4*>(Sb + (m + j) * D);
+#pragma unroll
+          for (int j = 0; j < 8; j += 4) {
+            const float4 k4 = *reinterpret_cast<const float4*>(kv + m + j), w4 = *reinterpret_cast<const float4*>(wv + m + j);
+            const float4 a4 = *reinterpret_cast<const float4*>(av + m + j);
+            s[j] = next_row(s[j], k4.x, w4.x, a4.x);
+            s[j + 1] = next_row(s[j + 1], k4.y, w4.y, a4.y);
+            s[j + 2] = next_row(s[j + 2], k4.z, w4.z, a4.z);
+            s[j + 3] = next_row(s[j + 3], k4.w, w4.w, a4.w);
+          }
+#pragma unroll
+          for (int j = 0; j < 8; ++j) *reinterpret_cast<float4*>(Sb + (m + j) * D) = s[j];
+        }
+      } else {
+        for (int m = 0; m < rows; ++m)
+          *reinterpret_cast<float4*>(Sb + m * D) = next_row(*reinterpret_cast<const float4*>(Sb + m * D), kv[m], wv[m], av[m]);
+      }
+    }
+    const float so = warp_sum(rg == 0 ? o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w : 0.f);
+    if (lane == 0) red_o[group][gw] = so;
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    group_sync(group);
+    if (abort_s != 0) break;
+    if (gt == 0) mbar_arrive(&done[buf]);
+    if (col_ok && rg == 0) {
+      const float oo = red_o[group][0] + red_o[group][1] + red_o[group][2] + red_o[group][3];
+      const float rs = 1.0f / sqrtf(oo / (float)p.Dreal + p.eps);
+      put4(out + 4 * quad, make_float4(o.x * rs * nw4.x * sigm(g.x), o.y * rs * nw4.y * sigm(g.y),
+                                       o.z * rs * nw4.z * sigm(g.z), o.w * rs * nw4.w * sigm(g.w)));
     }
   }
 }
@@ -275,41 +324,44 @@ __global__ void __launch_bounds__(256) prep_kernel(const Params p, float* __rest
   if (lane == 0) *reinterpret_cast<float4*>(out + 5 * D) = make_float4(rak * inv, rk * inv, 0.f, 0.f);
 }
 
-constexpr int kScanCols = 32;      // value columns of a CTA: 4 warps x 8
-constexpr int kScanThreads = 128;
+constexpr int kScanCols = 32;      // value columns of a CTA
 constexpr int kScanGroup = 8;      // tokens per staged group
 
 __device__ __forceinline__ void cp16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-// Lane (cj, lr) of a warp: column cj of the warp's 8, rows 16 n + 4 lr .. + 3 for n < R / 4 (R rows a lane, D <= 4 R).
-// Shared memory of a token: w | u | au | wr (4 R floats each, zero past D) | c1 c2 . . | sv of the CTA's 32 columns.
-template <int R>
-__global__ void __launch_bounds__(kScanThreads) scan_kernel(const Params p, const float* __restrict__ rec, float* __restrict__ o_out) {
+// A lane holds R key rows x C value columns of the state: lane (cg, lr) of a warp has columns cg * C .. + C - 1 of the
+// warp's 4 C columns and rows 32 n + 4 lr .. + 3 (n < R / 4, lr < 8; D <= 8 R).  Every column's row sums meet in three
+// shuffles.  C = 4 reads the vectors once per 16 columns (many sequences); C = 2 spreads a head over twice the warps (few).
+// Shared memory of a token: w | u | au | wr (8 R floats each, zero past D) | c1 c2 . . | sv of the CTA's 32 columns.
+template <int R, int C>
+__global__ void __launch_bounds__(32 * kScanCols / (4 * C))
+scan_kernel(const Params p, const float* __restrict__ rec, float* __restrict__ o_out) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
-  constexpr int V = 4 * R, TOK = 4 * V + 4 + kScanCols;
+  constexpr int kWarps = kScanCols / (4 * C), NT = 32 * kWarps;
+  constexpr int V = 8 * R, TOK = 4 * V + 4 + kScanCols;
   extern __shared__ __align__(16) float sm[];
   const int split = blockIdx.x, h = blockIdx.y, seq = blockIdx.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane & 3, cj = lane >> 2;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane & 7, cg = lane >> 3;
   const int D = p.D, H = p.H;
   const int slot = p.slots[seq];
   const int t0 = p.cu != nullptr ? p.cu[seq] : seq;
   const int t1 = p.cu != nullptr ? p.cu[seq + 1] : seq + 1;
   if (t1 <= t0) return;
-  const int c0 = split * kScanCols, lc = warp * 8 + cj, col = c0 + lc;
+  const int c0 = split * kScanCols, lc = (warp * 4 + cg) * C, col = c0 + lc;      // D % 8 == 0: all C columns in or out
   const bool col_ok = col < D;
   if (slot < 0) {
-    if (lr == 0 && col_ok)
-      for (int t = t0; t < t1; ++t) o_out[((size_t)t * H + h) * D + col] = 0.f;
+    for (int i = tid; i < (t1 - t0) * kScanCols; i += NT)
+      if (c0 + i % kScanCols < D) o_out[((size_t)(t0 + i / kScanCols) * H + h) * D + c0 + i % kScanCols] = 0.f;
     return;
   }
-  for (int i = tid; i < 2 * kScanGroup * TOK; i += kScanThreads) sm[i] = 0.f;     // zero padding of the vectors, once
+  for (int i = tid; i < 2 * kScanGroup * TOK; i += NT) sm[i] = 0.f;               // zero padding of the vectors, once
   __syncthreads();
   const int q16 = D / 4, cols16 = min(kScanCols, D - c0) / 4;                     // 16-byte pieces of a vector / of sv
   auto fetch = [&](int g0, int buf) {                                             // tokens g0 .. of the group -> buffer
     const int n = min(kScanGroup, t1 - g0);
-    for (int tt = warp; tt < n; tt += kScanThreads / 32) {
+    for (int tt = warp; tt < n; tt += kWarps) {
       const float* src = rec + ((size_t)(g0 + tt) * H + h) * rec_floats(D);
       float* dst = sm + (buf * kScanGroup + tt) * TOK;
 #pragma unroll
@@ -318,20 +370,29 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const Params p, cons
       if (lane < cols16) cp16(dst + 4 * V + 4 + lane * 4, src + 4 * D + c0 + lane * 4);
       else if (lane == 31) cp16(dst + 4 * V, src + 5 * D);
     }
+    // a short last group is filled up with tokens that leave the state alone: w = 1, everything else 0
+    for (int tt = n + warp; tt < kScanGroup; tt += kWarps) {
+      float* dst = sm + (buf * kScanGroup + tt) * TOK;
+      for (int j = lane; j < TOK; j += 32) dst[j] = j < V ? 1.f : 0.f;
+    }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   fetch(t0, 0);
   float* Sg = p.state + slot * p.slot_stride + (size_t)h * D * D + col;
   const bool init = p.has_initial == nullptr || p.has_initial[seq] != 0;
-  float2 S[R / 2];                                                                // rows in pairs
+  float2 S[C][R / 2];                                                             // rows in pairs
 #pragma unroll
   for (int n = 0; n < R / 4; ++n)
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      const int i = 16 * n + 4 * lr + j;
-      const float v = (init && col_ok && i < D) ? Sg[(size_t)i * D] : 0.f;
-      if (j & 1) S[2 * n + j / 2].y = v;
-      else S[2 * n + j / 2].x = v;
+      const int i = 32 * n + 4 * lr + j;
+      const bool in = init && col_ok && i < D;
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        const float v = in ? Sg[(size_t)i * D + c] : 0.f;
+        if (j & 1) S[c][2 * n + j / 2].y = v;
+        else S[c][2 * n + j / 2].x = v;
+      }
     }
   int buf = 0;
   for (int g0 = t0; g0 < t1; g0 += kScanGroup, buf ^= 1) {
@@ -342,39 +403,78 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const Params p, cons
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
-    const int n_tok = min(kScanGroup, t1 - g0);
-    for (int tt = 0; tt < n_tok; ++tt) {
-      const float* tok = sm + (buf * kScanGroup + tt) * TOK;
+    // this lane's share of the group's outputs: its rows' part of q, lane 0 of a column adds -c1 y + c2 sv
+    float part[kScanGroup][C];
+    const float* base = sm + buf * kScanGroup * TOK;
+#pragma unroll
+    for (int tt = 0; tt < kScanGroup; ++tt) {
+      const float* tok = base + tt * TOK;
       const float4* w4 = reinterpret_cast<const float4*>(tok) + lr;
       const float4* u4 = w4 + V / 4;
       const float4* a4 = u4 + V / 4;
       const float4* r4 = a4 + V / 4;
-      float2 y0 = make_float2(0.f, 0.f), y1 = y0, q0 = y0, q1 = y0;
+      float2 y0[C], y1[C], q[C];
+      float4 u[R / 4];
+#pragma unroll
+      for (int c = 0; c < C; ++c) y0[c] = y1[c] = q[c] = make_float2(0.f, 0.f);
 #pragma unroll
       for (int n = 0; n < R / 4; ++n) {
-        const float4 u = u4[4 * n], r = r4[4 * n];
-        y0 = __ffma2_rn(make_float2(u.x, u.y), S[2 * n], y0);
-        y1 = __ffma2_rn(make_float2(u.z, u.w), S[2 * n + 1], y1);
-        q0 = __ffma2_rn(make_float2(r.x, r.y), S[2 * n], q0);
-        q1 = __ffma2_rn(make_float2(r.z, r.w), S[2 * n + 1], q1);
+        u[n] = u4[8 * n];
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          y0[c] = __ffma2_rn(make_float2(u[n].x, u[n].y), S[c][2 * n], y0[c]);
+          y1[c] = __ffma2_rn(make_float2(u[n].z, u[n].w), S[c][2 * n + 1], y1[c]);
+        }
       }
-      float y = (y0.x + y0.y) + (y1.x + y1.y), q = (q0.x + q0.y) + (q1.x + q1.y);
-      y += __shfl_xor_sync(0xffffffffu, y, 1);
-      q += __shfl_xor_sync(0xffffffffu, q, 1);
-      y += __shfl_xor_sync(0xffffffffu, y, 2);
-      q += __shfl_xor_sync(0xffffffffu, q, 2);
-      const float sv = tok[4 * V + 4 + lc];
-      const float2 c = *reinterpret_cast<const float2*>(tok + 4 * V);
-      const float2 ny = make_float2(-y, -y), sv2 = make_float2(sv, sv);
+      float ys[C];
+#pragma unroll
+      for (int c = 0; c < C; ++c) ys[c] = (y0[c].x + y0[c].y) + (y1[c].x + y1[c].y);
+#pragma unroll
+      for (int o = 1; o < 8; o <<= 1)
+#pragma unroll
+        for (int c = 0; c < C; ++c) ys[c] += __shfl_xor_sync(0xffffffffu, ys[c], o);
+      const float2 cc = *reinterpret_cast<const float2*>(tok + 4 * V);
+      float2 sv[C], ny[C];
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        const float s = tok[4 * V + 4 + lc + c];
+        sv[c] = make_float2(s, s);
+        ny[c] = make_float2(-ys[c], -ys[c]);
+      }
 #pragma unroll
       for (int n = 0; n < R / 4; ++n) {
-        const float4 w = w4[4 * n], u = u4[4 * n], a = a4[4 * n];
-        S[2 * n] = __ffma2_rn(make_float2(a.x, a.y), ny,
-                              __ffma2_rn(make_float2(u.x, u.y), sv2, __fmul2_rn(make_float2(w.x, w.y), S[2 * n])));
-        S[2 * n + 1] = __ffma2_rn(make_float2(a.z, a.w), ny,
-                                  __ffma2_rn(make_float2(u.z, u.w), sv2, __fmul2_rn(make_float2(w.z, w.w), S[2 * n + 1])));
+        const float4 w = w4[8 * n], a = a4[8 * n], r = r4[8 * n];
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          q[c] = __ffma2_rn(make_float2(r.x, r.y), S[c][2 * n], q[c]);
+          q[c] = __ffma2_rn(make_float2(r.z, r.w), S[c][2 * n + 1], q[c]);
+          S[c][2 * n] = __ffma2_rn(make_float2(a.x, a.y), ny[c],
+                                   __ffma2_rn(make_float2(u[n].x, u[n].y), sv[c], __fmul2_rn(make_float2(w.x, w.y), S[c][2 * n])));
+          S[c][2 * n + 1] = __ffma2_rn(make_float2(a.z, a.w), ny[c],
+                                       __ffma2_rn(make_float2(u[n].z, u[n].w), sv[c], __fmul2_rn(make_float2(w.z, w.w), S[c][2 * n + 1])));
+        }
       }
-      if (lr == 0 && col_ok) o_out[((size_t)(g0 + tt) * H + h) * D + col] = fmaf(c.y, sv, fmaf(-c.x, y, q));
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        part[tt][c] = q[c].x + q[c].y;
+        if (lr == 0) part[tt][c] += fmaf(cc.y, sv[c].x, -cc.x * ys[c]);
+      }
+    }
+    // sum over the 8 lanes of a column, handing half of the tokens to the partner at every step: lane lr keeps token lr
+#pragma unroll
+    for (int half = 4, bit = 4; half >= 1; half >>= 1, bit >>= 1)
+#pragma unroll
+      for (int tt = 0; tt < half; ++tt)
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          const bool up = lr & bit;
+          const float mine = up ? part[tt + half][c] : part[tt][c], give = up ? part[tt][c] : part[tt + half][c];
+          part[tt][c] = mine + __shfl_xor_sync(0xffffffffu, give, bit);
+        }
+    if (g0 + lr < t1 && col_ok) {
+      float* dst = o_out + ((size_t)(g0 + lr) * H + h) * D + col;
+#pragma unroll
+      for (int c = 0; c < C; ++c) dst[c] = part[0][c];
     }
     __syncthreads();
   }
@@ -383,8 +483,11 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const Params p, cons
     for (int n = 0; n < R / 4; ++n)
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const int i = 16 * n + 4 * lr + j;
-        if (i < D) Sg[(size_t)i * D] = (j & 1) ? S[2 * n + j / 2].y : S[2 * n + j / 2].x;
+        const int i = 32 * n + 4 * lr + j;
+        if (i < D) {
+#pragma unroll
+          for (int c = 0; c < C; ++c) Sg[(size_t)i * D + c] = (j & 1) ? S[c][2 * n + j / 2].y : S[c][2 * n + j / 2].x;
+        }
       }
   }
 }
@@ -418,15 +521,20 @@ __global__ void __launch_bounds__(256) finish_kernel(const Params p, const float
   }
 }
 
-template <int R>
-static int launch_scan(const Params& p, const float* rec, float* o, int nseq, cudaStream_t stream) {
-  const size_t smem = (size_t)2 * kScanGroup * (16 * R + 4 + kScanCols) * sizeof(float);
+template <int R, int C>
+static int launch_scan_as(const Params& p, const float* rec, float* o, int nseq, cudaStream_t stream) {
+  const size_t smem = (size_t)2 * kScanGroup * (32 * R + 4 + kScanCols) * sizeof(float);
   static DeviceOnce once;
-  auto kern = scan_kernel<R>;
+  auto kern = scan_kernel<R, C>;
   if (!ensure_dynamic_smem(kern, smem, once)) return -4;
   dim3 grid((p.D + kScanCols - 1) / kScanCols, p.H, nseq);
-  bg::launch_pdl(kern, grid, dim3(kScanThreads), smem, stream, p, rec, o);
+  bg::launch_pdl(kern, grid, dim3(32 * kScanCols / (4 * C)), smem, stream, p, rec, o);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+template <int R>
+static int launch_scan(const Params& p, const float* rec, float* o, int nseq, cudaStream_t stream) {
+  const long long ctas = (long long)((p.D + kScanCols - 1) / kScanCols) * p.H * nseq;
+  return ctas <= 296 ? launch_scan_as<R, 2>(p, rec, o, nseq, stream) : launch_scan_as<R, 4>(p, rec, o, nseq, stream);
 }
 
 template <typename OT>
@@ -434,35 +542,34 @@ static int launch_prompt(const Params& p, float* rec, float* o, int T, int nseq,
   const dim3 grid(T, (p.H + 7) / 8);
   bg::launch_pdl(prep_kernel, grid, dim3(256), 0, stream, p, rec);
   int rc;
-  if (p.D <= 32) rc = launch_scan<8>(p, rec, o, nseq, stream);
-  else if (p.D <= 48) rc = launch_scan<12>(p, rec, o, nseq, stream);
-  else if (p.D <= 64) rc = launch_scan<16>(p, rec, o, nseq, stream);
-  else if (p.D <= 96) rc = launch_scan<24>(p, rec, o, nseq, stream);
-  else if (p.D <= 128) rc = launch_scan<32>(p, rec, o, nseq, stream);
-  else if (p.D <= 192) rc = launch_scan<48>(p, rec, o, nseq, stream);
-  else rc = launch_scan<64>(p, rec, o, nseq, stream);
+  if (p.D <= 32) rc = launch_scan<4>(p, rec, o, nseq, stream);
+  else if (p.D <= 64) rc = launch_scan<8>(p, rec, o, nseq, stream);
+  else if (p.D <= 96) rc = launch_scan<12>(p, rec, o, nseq, stream);
+  else if (p.D <= 128) rc = launch_scan<16>(p, rec, o, nseq, stream);
+  else if (p.D <= 192) rc = launch_scan<24>(p, rec, o, nseq, stream);
+  else rc = launch_scan<32>(p, rec, o, nseq, stream);
   if (rc != 0) return rc;
   bg::launch_pdl(finish_kernel<OT>, grid, dim3(256), 0, stream, p, (const float*)o);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
-template <typename OT, int NT, int NR>
+template <typename OT, int NR>
 static int launch_decode_as(const Params& p, int nseq, int num_sms, int* status, cudaStream_t stream) {
   const size_t smem = (size_t)kBufs * p.D * p.D * sizeof(float);
   static DeviceOnce once;
-  auto kern = decode_kernel<OT, NT, NR>;
+  auto kern = decode_kernel<OT, NR>;
   if (!ensure_dynamic_smem(kern, 3 * 128 * 128 * sizeof(float), once)) return -4;
-  const int per_sm = smem > 100 * 1024 ? 1 : smem > 48 * 1024 ? 2 : 4;
+  const int per_sm = smem > 100 * 1024 || NR > 16 ? 1 : smem > 48 * 1024 ? 2 : 3;
   const int items = nseq * p.H, most = num_sms * per_sm;
-  bg::launch_pdl(kern, dim3(items < most ? items : most), dim3(NT), smem, stream, p, items, status);
+  bg::launch_pdl(kern, dim3(items < most ? items : most), dim3(288), smem, stream, p, items, status);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
 template <typename OT>
 static int launch_decode(const Params& p, int nseq, int num_sms, int* status, cudaStream_t stream) {
-  if (p.D <= 32) return launch_decode_as<OT, 128, 2>(p, nseq, num_sms, status, stream);
-  if (p.D <= 64) return launch_decode_as<OT, 256, 4>(p, nseq, num_sms, status, stream);
-  return launch_decode_as<OT, 256, 16>(p, nseq, num_sms, status, stream);
+  if (p.D <= 32) return launch_decode_as<OT, 8>(p, nseq, num_sms, status, stream);
+  if (p.D <= 64) return launch_decode_as<OT, 16>(p, nseq, num_sms, status, stream);
+  return launch_decode_as<OT, 32>(p, nseq, num_sms, status, stream);
 }
 
 }  // namespace delta
