@@ -217,6 +217,17 @@ def bf16_gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = No
     return out
 
 
+def grouped_bf16_gemm(x: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, counts: torch.Tensor) -> torch.Tensor:
+    """Ragged grouped bf16 GEMM on the GPU: x [R, K] rows grouped by expert, w [E, N, K] -> [R, N] bf16; ``counts`` rows of
+    each segment are present, the others stay undefined."""
+    E, N, K = w.shape
+    out = torch.empty(x.shape[0], N, dtype=torch.bfloat16, device=x.device)
+    if x.shape[0]:
+        _launch(KIND_BF16, EPI_STORE, x.contiguous(), None, 0, w.view(E * N, K), None, out, offsets, E, x.shape[0], N, K,
+                counts=counts)
+    return out
+
+
 def f32_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: Optional[torch.Tensor] = None,
              counts: Optional[torch.Tensor] = None, max_rows: int = 0) -> torch.Tensor:
     """out = x @ w^T in true fp32 on the CUDA cores (``csrc/gemm_f32.cu``); grouped when ``offsets`` is given (w [E, N, K],

@@ -232,8 +232,15 @@ def grouped_experts(xq, xs, offsets: torch.Tensor, ew: ExpertWeights, x_dense: O
             act = _activation(gu, ew.activation, ew.act_limit).to(x.dtype)
         with timer.timed("moe.s3_gemm"):
             return grouped_w4(act, ew.w2, ew.w2_s, offsets)
-    # unquantised experts (CPU fp32 oracle path and bf16 debugging)
+    # unquantised experts
     x = x_dense
+    if (x.is_cuda and x.dtype == torch.bfloat16 and counts is not None and ew.w13.shape[2] % 64 == 0
+            and ew.w2.shape[2] % 64 == 0):
+        with timer.timed("moe.s1_gemm"):
+            gu = gemm.grouped_bf16_gemm(x, ew.w13, offsets, counts)
+        act = _activation(gu, ew.activation, ew.act_limit).contiguous()
+        with timer.timed("moe.s3_gemm"):
+            return gemm.grouped_bf16_gemm(act, ew.w2, offsets, counts)
     out = torch.zeros(x.shape[0], ew.w2.shape[1], dtype=x.dtype, device=x.device)
     off = offsets.tolist()
     for e in range(ew.num_experts):
@@ -272,7 +279,7 @@ def experts_forward(hidden: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.
     else:
         rows = hidden[src.clamp_min(0).long()]
         rows = torch.where((src >= 0).unsqueeze(-1), rows, torch.zeros_like(rows))
-        y = grouped_experts(None, None, offsets, ew, x_dense=rows)
+        y = grouped_experts(None, None, offsets, ew, x_dense=rows, counts=getattr(offsets, "real_counts", None))
     with timer.timed("moe.combine"):
         if before_combine is not None:
             before_combine()
