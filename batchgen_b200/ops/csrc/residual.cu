@@ -145,9 +145,9 @@ glu_kernel(const float* __restrict__ z, int ldz, int u_off, OT* __restrict__ out
            const float* __restrict__ row_scale, const float* __restrict__ gate, int ld_gate,
            const int* __restrict__ total_rows) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
-  const int r = blockIdx.y;
+  const int r = blockIdx.x;
   if (total_rows != nullptr && r >= *total_rows) return;
-  const int c = (blockIdx.x * kThreads + threadIdx.x) * 4;
+  const int c = (blockIdx.y * kThreads + threadIdx.x) * 4;
   if (c >= Fo) return;
   float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
   if (c < F) {                                          // F % 4 == 0
@@ -227,24 +227,16 @@ int bg_glu(int dt, int kind, const float* z, int ldz, int u_off, void* out, int 
            const float* row_scale, const float* gate, int ld_gate, const int* total_rows, cudaStream_t stream) {
   using namespace bg::resid;
   if (R <= 0 || Fo <= 0) return 0;
-  if (F % 4 || Fo % 4 || F > Fo || ldz % 4 || u_off % 4 || ldo % 4 || ldo < Fo || R > 65535 * 32) return -1;
-  // grid.y is limited to 65535 rows: longer inputs go in pieces
-  for (int r0 = 0; r0 < R; r0 += 65535) {
-    if (r0 > 0 && total_rows != nullptr) return -1;
-    const int n = R - r0 < 65535 ? R - r0 : 65535;
-    dim3 grid((Fo / 4 + kThreads - 1) / kThreads, n);
-    const float* zr = z + (size_t)r0 * ldz;
-    const float* rs = row_scale != nullptr ? row_scale + r0 : nullptr;
-    const float* gt = gate != nullptr ? gate + (size_t)r0 * ld_gate : nullptr;
-#define BG_GLU(OT, KIND)                                                                                              \
-  bg::launch_pdl(glu_kernel<OT, KIND>, grid, dim3(kThreads), 0, stream, zr, ldz, u_off,                               \
-                 reinterpret_cast<OT*>(out) + (size_t)r0 * ldo, ldo, F, Fo, limit, rs, gt, ld_gate, total_rows)
-    if (dt == 0 && kind == 0) BG_GLU(__nv_bfloat16, 0);
-    else if (dt == 0) BG_GLU(__nv_bfloat16, 1);
-    else if (kind == 0) BG_GLU(float, 0);
-    else BG_GLU(float, 1);
+  if (F % 4 || Fo % 4 || F > Fo || ldz % 4 || u_off % 4 || ldo % 4 || ldo < Fo) return -1;
+  const dim3 grid(R, (Fo / 4 + kThreads - 1) / kThreads);
+#define BG_GLU(OT, KIND)                                                                                      \
+  bg::launch_pdl(glu_kernel<OT, KIND>, grid, dim3(kThreads), 0, stream, z, ldz, u_off, reinterpret_cast<OT*>(out), ldo, F, \
+                 Fo, limit, row_scale, gate, ld_gate, total_rows)
+  if (dt == 0 && kind == 0) BG_GLU(__nv_bfloat16, 0);
+  else if (dt == 0) BG_GLU(__nv_bfloat16, 1);
+  else if (kind == 0) BG_GLU(float, 0);
+  else BG_GLU(float, 1);
 #undef BG_GLU
-  }
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 

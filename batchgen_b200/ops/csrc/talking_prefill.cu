@@ -10,7 +10,7 @@
 // kv(h)'s.  The mixed scores leave the tensor core in fp32.
 //
 // One CTA = (tile of 128 queries of one sequence, head h).  M = 128 queries on the TMEM lanes, key tiles of 128:
-//   S (2 x 128 columns, double buffered) = Q' . K^T, both operands streamed in 64-wide K blocks through a 4-stage TMA ring
+//   S (2 x 128 columns, double buffered) = Q' . K^T, both operands streamed in 64-wide K blocks through a TMA ring
 //   O (dv columns) += P . V,  P written by the softmax threads as a swizzled K-major tile, V read N-major
 // K and V come straight from the paged cache by TMA (3-D map: column, token of the page, page).  A thread owns a query row:
 // no cross-thread reduction; O is rescaled only when the running maximum grew by more than 2^8.
@@ -24,11 +24,11 @@ namespace bg {
 namespace talkpre {
 
 constexpr int BM = 128, BN = 128;
-constexpr int kStages = 4;
+constexpr int kMaxStages = 5;                              // K-block stages: five with up to 128 value columns, else four
 constexpr int kThreads = 192;
+constexpr int kMaxBoxes = BN / 16;                         // pages of 16 tokens and more
 constexpr int kABytes = BM * 128, kBBytes = BN * 128;      // one 64-wide bf16 K block of each operand
 constexpr int kPBytes = 2 * BM * 128;
-constexpr int kVBytes = 4 * BN * 128;                      // room for 256 value columns, or two tiles of up to 128
 constexpr int kTmemCols = 512;                             // S: 2 x 128, O: up to 256
 
 struct Work {
@@ -53,8 +53,8 @@ struct Params {
 };
 
 struct Shared {
-  uint64_t full[kStages], empty[kStages];
-  uint64_t v_full[2], v_empty[2];
+  uint64_t full[kMaxStages], empty[kMaxStages];
+  uint64_t v_full, v_empty;
   uint64_t s_full[2];
   uint64_t p_full, o_done;
   uint32_t tmem_base;
@@ -105,6 +105,7 @@ __device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&v)[32
       : "memory");
 }
 
+template <int kStages>
 __global__ void __launch_bounds__(kThreads, 1)
 attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv, const Params p) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
@@ -112,7 +113,7 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
   uint8_t* a_buf = smem;
   uint8_t* b_buf = a_buf + kStages * kABytes;
   uint8_t* v_buf = b_buf + kStages * kBBytes;
-  uint8_t* p_buf = v_buf + kVBytes;
+  uint8_t* p_buf = v_buf + (p.dv64 / 64) * BN * 128;
   Shared& ss = *reinterpret_cast<Shared*>(p_buf + kPBytes);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   volatile int* abort_flag = &ss.abort_flag;
@@ -122,12 +123,13 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
   const int first = p.chunk > 0 ? w.pos0 - w.pos0 % p.chunk : 0;
   const int k0 = first - first % p.box_rows;                     // first key of tile 0: starts on a box of a page
   const int n_tiles = (last + 1 - k0 + BN - 1) / BN;
-  const int n_vbuf = p.dv64 <= 128 ? 2 : 1;
   const int v_tile_bytes = (p.dv64 / 64) * BN * 128;
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) { mbar_init(&ss.full[s], 1); mbar_init(&ss.empty[s], 1); }
-    for (int s = 0; s < 2; ++s) { mbar_init(&ss.v_full[s], 1); mbar_init(&ss.v_empty[s], 1); mbar_init(&ss.s_full[s], 1); }
+    for (int s = 0; s < 2; ++s) mbar_init(&ss.s_full[s], 1);
+    mbar_init(&ss.v_full, 1);
+    mbar_init(&ss.v_empty, 1);
     mbar_init(&ss.p_full, 128);
     mbar_init(&ss.o_done, 1);
     ss.abort_flag = 0;
@@ -151,43 +153,58 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
       const int boxes = BN / p.box_rows;
       uint32_t it = 0;
       bool ok = true;
-      // box b of tile t: tokens k0 + t * BN + b * box_rows ..; past the table's end the last page is read (masked keys)
-      auto page_of = [&](int t, int b, int& row) -> int {
-        const int pos = k0 + t * BN + b * p.box_rows;
-        row = pos % p.page;
-        return bt[min(pos / p.page, p.bt_cols - 1)];
+      // box b of tile t: tokens k0 + t * BN + b * box_rows ..; past the table's end the last page is read (masked keys).
+      // Page numbers of a tile are looked up once, one tile ahead of their use.
+      const int shift = 31 - __clz(p.page);
+      int old[kMaxBoxes], pg[kMaxBoxes] = {}, nxt[kMaxBoxes] = {};
+      auto look_up = [&](int t) {
+#pragma unroll
+        for (int b = 0; b < kMaxBoxes; ++b)
+          if (b < boxes) nxt[b] = bt[min((k0 + t * BN + b * p.box_rows) >> shift, p.bt_cols - 1)];
       };
+      const int vcol = p.v_col0 + (h / p.rep) * p.dvp;
+      auto load_v = [&](int t) -> bool {                           // values of tile t, whose pages are in `old`
+        if (!mbar_wait(&ss.v_empty, (t & 1) ^ 1, abort_flag, kTimeoutProducer)) return false;
+        mbar_expect_tx(&ss.v_full, v_tile_bytes);
+        for (int c = 0; c < p.dv64 / 64; ++c)
+#pragma unroll
+          for (int b = 0; b < kMaxBoxes; ++b)
+            if (b < boxes)
+              tma_load_3d(v_buf + (c * BN + b * p.box_rows) * 128, &tm_kv, &ss.v_full, vcol + c * 64,
+                          (k0 + t * BN + b * p.box_rows) & (p.page - 1), old[b]);
+        return true;
+      };
+      look_up(0);
+      // the MMA warp takes S(0), S(1), PV(0), S(2), PV(1), ..: values follow the next tile's keys
       for (int t = 0; ok && t < n_tiles; ++t) {
+#pragma unroll
+        for (int b = 0; b < kMaxBoxes; ++b) { old[b] = pg[b]; pg[b] = nxt[b]; }
+        if (t + 1 < n_tiles) look_up(t + 1);
+        const int pos = k0 + t * BN;
         for (int kb = 0; kb < p.KB; ++kb, ++it) {
           const int s = it % kStages;
           if (!mbar_wait(&ss.empty[s], ((it / kStages) & 1) ^ 1, abort_flag, kTimeoutProducer)) { ok = false; break; }
           mbar_expect_tx(&ss.full[s], kABytes + kBBytes);
           tma_load_2d(a_buf + s * kABytes, &tm_q, &ss.full[s], (h * p.KB + kb) * 64, w.q_row0 - p.row_shift);
-          for (int b = 0; b < boxes; ++b) {
-            int row;
-            const int pg = page_of(t, b, row);
-            tma_load_3d(b_buf + s * kBBytes + b * p.box_rows * 128, &tm_kv, &ss.full[s], kb * 64, row, pg);
-          }
+#pragma unroll
+          for (int b = 0; b < kMaxBoxes; ++b)
+            if (b < boxes)
+              tma_load_3d(b_buf + s * kBBytes + b * p.box_rows * 128, &tm_kv, &ss.full[s], kb * 64,
+                          (pos + b * p.box_rows) & (p.page - 1), pg[b]);
         }
-        if (!ok) break;
-        const int vb = t % n_vbuf;
-        if (!mbar_wait(&ss.v_empty[vb], ((t / n_vbuf) & 1) ^ 1, abort_flag, kTimeoutProducer)) { ok = false; break; }
-        mbar_expect_tx(&ss.v_full[vb], v_tile_bytes);
-        for (int c = 0; c < p.dv64 / 64; ++c)
-          for (int b = 0; b < boxes; ++b) {
-            int row;
-            const int pg = page_of(t, b, row);
-            tma_load_3d(v_buf + vb * v_tile_bytes + (c * BN + b * p.box_rows) * 128, &tm_kv, &ss.v_full[vb],
-                        p.v_col0 + (h / p.rep) * p.dvp + c * 64, row, pg);
-          }
+        if (ok && t > 0) ok = load_v(t - 1);
+      }
+      if (ok && n_tiles > 0) {
+#pragma unroll
+        for (int b = 0; b < kMaxBoxes; ++b) old[b] = pg[b];
+        ok = load_v(n_tiles - 1);
       }
       if (ok) {
         // leave only when every copy has landed and been consumed
         const uint32_t n = it < (uint32_t)kStages ? it : (uint32_t)kStages;
         for (uint32_t j = it - n; j < it; ++j)
           if (!mbar_wait(&ss.empty[j % kStages], (j / kStages) & 1, abort_flag, kTimeoutProducer)) break;
-        for (int t = max(0, n_tiles - n_vbuf); t < n_tiles; ++t)
-          if (!mbar_wait(&ss.v_empty[t % n_vbuf], (t / n_vbuf) & 1, abort_flag, kTimeoutProducer)) break;
+        if (n_tiles > 0) mbar_wait(&ss.v_empty, (n_tiles - 1) & 1, abort_flag, kTimeoutProducer);
       } else {
         for (uint32_t i = 0; i < (1u << 16); ++i) __nanosleep(20);   // bounded grace period for copies in flight
       }
@@ -219,17 +236,16 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
       for (int t = 0; ok && t < n_tiles; ++t) {
         // S of tile t + 1 goes into the buffer that the softmax of tile t - 1 has left (its P was handed over before PV(t-1))
         if (t + 1 < n_tiles && !issue_s(t + 1)) { ok = false; break; }
-        const int vb = t % n_vbuf;
-        if (!mbar_wait(&ss.v_full[vb], (t / n_vbuf) & 1, abort_flag, kTimeoutMma)) { ok = false; break; }
+        if (!mbar_wait(&ss.v_full, t & 1, abort_flag, kTimeoutMma)) { ok = false; break; }
         if (!mbar_wait(&ss.p_full, t & 1, abort_flag, kTimeoutMma)) { ok = false; break; }
         tc_fence_after();
-        const uint32_t v_base = smem_u32(v_buf + vb * v_tile_bytes);
+        const uint32_t v_base = smem_u32(v_buf);
 #pragma unroll
         for (int j = 0; j < BN / 16; ++j) {
           const uint64_t pdesc = make_smem_desc_sw128(smem_u32(p_buf + (j / 4) * BM * 128)) + 2 * (j % 4);
           mma_f16(tm_o, pdesc, desc_mn_sw128(v_base + j * 2048, BN * 128, 1024), idesc_pv, (t > 0 || j > 0) ? 1u : 0u);
         }
-        tc_commit(&ss.v_empty[vb]);
+        tc_commit(&ss.v_empty);
         tc_commit(&ss.o_done);
       }
     }
@@ -475,10 +491,14 @@ int bg_talk_prefill(const void* qf, const void* cache, long long page_stride, in
   p.block_table = block_table; p.bt_stride = bt_stride; p.bt_cols = bt_cols; p.page = page; p.box_rows = box_rows;
   p.KB = kc / 64; p.v_col0 = G * dp; p.dvp = dvp; p.dv64 = (dvp + 63) / 64 * 64; p.rep = H / G; p.chunk = chunk;
   p.sink = sink; p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo; p.row_shift = row_shift; p.status = status;
-  static bg::DeviceOnce once;
-  const size_t smem = kStages * (kABytes + kBBytes) + kVBytes + kPBytes + sizeof(Shared) + 1024;
-  if (!bg::ensure_dynamic_smem(attn_kernel, smem, once)) return -13;
-  attn_kernel<<<dim3(n_work, H), kThreads, smem, stream>>>(tq, tk, p);
+  const int stages = p.dv64 <= 128 ? 5 : 4;
+  const size_t smem = stages * (kABytes + kBBytes) + (p.dv64 / 64) * BN * 128 + kPBytes + sizeof(Shared) + 1024;
+  static bg::DeviceOnce once4, once5;
+  constexpr size_t kSmemMax = 227 * 1024;
+  if (!bg::ensure_dynamic_smem(attn_kernel<4>, kSmemMax, once4) || !bg::ensure_dynamic_smem(attn_kernel<5>, kSmemMax, once5))
+    return -13;
+  if (stages == 5) attn_kernel<5><<<dim3(n_work, H), kThreads, smem, stream>>>(tq, tk, p);
+  else attn_kernel<4><<<dim3(n_work, H), kThreads, smem, stream>>>(tq, tk, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -14;
 }
 

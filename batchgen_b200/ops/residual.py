@@ -101,7 +101,7 @@ def glu(z: torch.Tensor, F: int, kind: str, limit: float = 0.0, row_scale: Optio
                            _i(out.stride(0)), _i(R), _i(F), _i(out.shape[1]), ctypes.c_float(limit), _ext.ptr(row_scale),
                            _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0), _ext.ptr(total_rows),
                            _ext.stream())
-    _ext.check(rc, "bg_glu", kernels=-(-R // 65535))
+    _ext.check(rc, "bg_glu")
     return out
 
 
