@@ -14,7 +14,7 @@
 // Decode (`decode_kernel`, D <= 128): a token is one read and write of the state with everything else fused around it.
 //
 // Prompts (`prep` -> `scan` -> `finish`): a value column of S evolves on its own once w, u, a * u and w * r are known, so the
-// scan splits a head's columns over CTAs of 32 columns and needs no barrier inside a token (8 lanes share a column, three
+// scan splits a head's columns over CTAs of 32 columns and needs no barrier inside a token (16 lanes share a column, four
 // shuffles sum their rows; packed fp32 FMAs).  `prep` computes the per-token vectors for all tokens in parallel and `finish`
 // applies the output norm and gate, which need whole heads.
 //
@@ -331,25 +331,26 @@ __device__ __forceinline__ void cp16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-// A lane holds R key rows x C value columns of the state: lane (cg, lr) of a warp has columns cg * C .. + C - 1 of the
-// warp's 4 C columns and rows 32 n + 4 lr .. + 3 (n < R / 4, lr < 8; D <= 8 R).  Every column's row sums meet in three
-// shuffles.  C = 4 reads the vectors once per 16 columns (many sequences); C = 2 spreads a head over twice the warps (few).
-// Shared memory of a token: w | u | au | wr (8 R floats each, zero past D) | c1 c2 . . | sv of the CTA's 32 columns.
+// A lane holds R key rows x C value columns of the state; 16 lanes share a column: lane (cg, lr) of a warp has columns
+// cg * C .. + C - 1 of the warp's 2 C columns and rows 64 n + 4 lr .. + 3 (n < R / 4, lr < 16; D <= 16 R).  Few rows and many
+// columns a lane keep the shared-memory reads of the vectors, the scan's limit, small; the row sums of a column meet in four
+// shuffles.  C = 4 reads the vectors once per 8 columns (many sequences); C = 2 spreads a head over twice the warps (few).
+// Shared memory of a token: w | u | au | wr (16 R floats each, zero past D) | c1 c2 . . | sv of the CTA's 32 columns.
 template <int R, int C>
-__global__ void __launch_bounds__(32 * kScanCols / (4 * C))
+__global__ void __launch_bounds__(32 * kScanCols / (2 * C))
 scan_kernel(const Params p, const float* __restrict__ rec, float* __restrict__ o_out) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
-  constexpr int kWarps = kScanCols / (4 * C), NT = 32 * kWarps;
-  constexpr int V = 8 * R, TOK = 4 * V + 4 + kScanCols;
+  constexpr int kWarps = kScanCols / (2 * C), NT = 32 * kWarps;
+  constexpr int V = 16 * R, TOK = 4 * V + 4 + kScanCols;
   extern __shared__ __align__(16) float sm[];
   const int split = blockIdx.x, h = blockIdx.y, seq = blockIdx.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane & 7, cg = lane >> 3;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane & 15, cg = lane >> 4;
   const int D = p.D, H = p.H;
   const int slot = p.slots[seq];
   const int t0 = p.cu != nullptr ? p.cu[seq] : seq;
   const int t1 = p.cu != nullptr ? p.cu[seq + 1] : seq + 1;
   if (t1 <= t0) return;
-  const int c0 = split * kScanCols, lc = (warp * 4 + cg) * C, col = c0 + lc;      // D % 8 == 0: all C columns in or out
+  const int c0 = split * kScanCols, lc = (warp * 2 + cg) * C, col = c0 + lc;      // D % 8 == 0: all C columns in or out
   const bool col_ok = col < D;
   if (slot < 0) {
     for (int i = tid; i < (t1 - t0) * kScanCols; i += NT)
@@ -385,7 +386,7 @@ scan_kernel(const Params p, const float* __restrict__ rec, float* __restrict__ o
   for (int n = 0; n < R / 4; ++n)
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      const int i = 32 * n + 4 * lr + j;
+      const int i = 64 * n + 4 * lr + j;
       const bool in = init && col_ok && i < D;
 #pragma unroll
       for (int c = 0; c < C; ++c) {
@@ -419,7 +420,7 @@ scan_kernel(const Params p, const float* __restrict__ rec, float* __restrict__ o
       for (int c = 0; c < C; ++c) y0[c] = y1[c] = q[c] = make_float2(0.f, 0.f);
 #pragma unroll
       for (int n = 0; n < R / 4; ++n) {
-        u[n] = u4[8 * n];
+        u[n] = u4[16 * n];
 #pragma unroll
         for (int c = 0; c < C; ++c) {
           y0[c] = __ffma2_rn(make_float2(u[n].x, u[n].y), S[c][2 * n], y0[c]);
@@ -430,20 +431,22 @@ scan_kernel(const Params p, const float* __restrict__ rec, float* __restrict__ o
 #pragma unroll
       for (int c = 0; c < C; ++c) ys[c] = (y0[c].x + y0[c].y) + (y1[c].x + y1[c].y);
 #pragma unroll
-      for (int o = 1; o < 8; o <<= 1)
+      for (int o = 1; o < 16; o <<= 1)
 #pragma unroll
         for (int c = 0; c < C; ++c) ys[c] += __shfl_xor_sync(0xffffffffu, ys[c], o);
       const float2 cc = *reinterpret_cast<const float2*>(tok + 4 * V);
       float2 sv[C], ny[C];
 #pragma unroll
-      for (int c = 0; c < C; ++c) {
-        const float s = tok[4 * V + 4 + lc + c];
-        sv[c] = make_float2(s, s);
-        ny[c] = make_float2(-ys[c], -ys[c]);
+      for (int c = 0; c < C; c += 2) {
+        const float2 s = *reinterpret_cast<const float2*>(tok + 4 * V + 4 + lc + c);
+        sv[c] = make_float2(s.x, s.x);
+        sv[c + 1] = make_float2(s.y, s.y);
       }
 #pragma unroll
+      for (int c = 0; c < C; ++c) ny[c] = make_float2(-ys[c], -ys[c]);
+#pragma unroll
       for (int n = 0; n < R / 4; ++n) {
-        const float4 w = w4[8 * n], a = a4[8 * n], r = r4[8 * n];
+        const float4 w = w4[16 * n], a = a4[16 * n], r = r4[16 * n];
 #pragma unroll
         for (int c = 0; c < C; ++c) {
           q[c] = __ffma2_rn(make_float2(r.x, r.y), S[c][2 * n], q[c]);
@@ -460,7 +463,8 @@ scan_kernel(const Params p, const float* __restrict__ rec, float* __restrict__ o
         if (lr == 0) part[tt][c] += fmaf(cc.y, sv[c].x, -cc.x * ys[c]);
       }
     }
-    // sum over the 8 lanes of a column, handing half of the tokens to the partner at every step: lane lr keeps token lr
+    // sum over the 16 lanes of a column, handing half of the tokens to the partner at every step: lanes lr and lr + 8 end
+    // with token lr
 #pragma unroll
     for (int half = 4, bit = 4; half >= 1; half >>= 1, bit >>= 1)
 #pragma unroll
@@ -471,10 +475,12 @@ scan_kernel(const Params p, const float* __restrict__ rec, float* __restrict__ o
           const float mine = up ? part[tt + half][c] : part[tt][c], give = up ? part[tt][c] : part[tt + half][c];
           part[tt][c] = mine + __shfl_xor_sync(0xffffffffu, give, bit);
         }
-    if (g0 + lr < t1 && col_ok) {
+#pragma unroll
+    for (int c = 0; c < C; ++c) part[0][c] += __shfl_xor_sync(0xffffffffu, part[0][c], 8);
+    if (lr < 8 && g0 + lr < t1 && col_ok) {
       float* dst = o_out + ((size_t)(g0 + lr) * H + h) * D + col;
 #pragma unroll
-      for (int c = 0; c < C; ++c) dst[c] = part[0][c];
+      for (int c = 0; c < C; c += 2) *reinterpret_cast<float2*>(dst + c) = make_float2(part[0][c], part[0][c + 1]);
     }
     __syncthreads();
   }
@@ -483,7 +489,7 @@ scan_kernel(const Params p, const float* __restrict__ rec, float* __restrict__ o
     for (int n = 0; n < R / 4; ++n)
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const int i = 32 * n + 4 * lr + j;
+        const int i = 64 * n + 4 * lr + j;
         if (i < D) {
 #pragma unroll
           for (int c = 0; c < C; ++c) Sg[(size_t)i * D + c] = (j & 1) ? S[c][2 * n + j / 2].y : S[c][2 * n + j / 2].x;
@@ -523,12 +529,12 @@ __global__ void __launch_bounds__(256) finish_kernel(const Params p, const float
 
 template <int R, int C>
 static int launch_scan_as(const Params& p, const float* rec, float* o, int nseq, cudaStream_t stream) {
-  const size_t smem = (size_t)2 * kScanGroup * (32 * R + 4 + kScanCols) * sizeof(float);
+  const size_t smem = (size_t)2 * kScanGroup * (64 * R + 4 + kScanCols) * sizeof(float);
   static DeviceOnce once;
   auto kern = scan_kernel<R, C>;
   if (!ensure_dynamic_smem(kern, smem, once)) return -4;
   dim3 grid((p.D + kScanCols - 1) / kScanCols, p.H, nseq);
-  bg::launch_pdl(kern, grid, dim3(32 * kScanCols / (4 * C)), smem, stream, p, rec, o);
+  bg::launch_pdl(kern, grid, dim3(32 * kScanCols / (2 * C)), smem, stream, p, rec, o);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 template <int R>
@@ -542,12 +548,10 @@ static int launch_prompt(const Params& p, float* rec, float* o, int T, int nseq,
   const dim3 grid(T, (p.H + 7) / 8);
   bg::launch_pdl(prep_kernel, grid, dim3(256), 0, stream, p, rec);
   int rc;
-  if (p.D <= 32) rc = launch_scan<4>(p, rec, o, nseq, stream);
-  else if (p.D <= 64) rc = launch_scan<8>(p, rec, o, nseq, stream);
-  else if (p.D <= 96) rc = launch_scan<12>(p, rec, o, nseq, stream);
-  else if (p.D <= 128) rc = launch_scan<16>(p, rec, o, nseq, stream);
-  else if (p.D <= 192) rc = launch_scan<24>(p, rec, o, nseq, stream);
-  else rc = launch_scan<32>(p, rec, o, nseq, stream);
+  if (p.D <= 64) rc = launch_scan<4>(p, rec, o, nseq, stream);
+  else if (p.D <= 128) rc = launch_scan<8>(p, rec, o, nseq, stream);
+  else if (p.D <= 192) rc = launch_scan<12>(p, rec, o, nseq, stream);
+  else rc = launch_scan<16>(p, rec, o, nseq, stream);
   if (rc != 0) return rc;
   bg::launch_pdl(finish_kernel<OT>, grid, dim3(256), 0, stream, p, (const float*)o);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
