@@ -89,6 +89,8 @@ def model_contract(cfg, world: int, on_gpu: bool, moe_comm: str = "nccl") -> Lis
     a model outside the contract would raise ``KernelError`` at its first step (no silent library fallback); here it
     is refused before the workers start, with every violated rule in the message.  Returns notes for the log."""
     notes, bad = [], []
+    if cfg.is_layered:
+        return _layered_contract(cfg, world, on_gpu)
     if world > 1:
         if cfg.num_heads % world:
             bad.append(f"{cfg.num_heads} attention heads do not divide over {world} ranks")
@@ -142,6 +144,27 @@ def model_contract(cfg, world: int, on_gpu: bool, moe_comm: str = "nccl") -> Lis
     if bad:
         raise PreflightError("model contract: " + "; ".join(bad))
     return notes or ["model geometry within the kernels' contract"]
+
+
+def _layered_contract(cfg, world: int, on_gpu: bool) -> List[str]:
+    """Layer-listed models pad every width to what the kernels tile; what is left are the kernels' upper bounds."""
+    bad = []
+    if world > 1:
+        bad.append("layer-listed models run on one GPU per engine: raise --dp-size to the world size")
+    for i, s in enumerate(cfg.layer_specs):
+        m, f = s.mixer, s.mlp
+        if m.recurrent and m.dim > 256:
+            bad.append(f"layer {i}: delta-rule head width {m.dim} exceeds 256")
+        if not m.recurrent and m.kv_heads * -(-(m.heads // m.kv_heads) // 4) * (m.vdim_p // 4) > 1024:
+            bad.append(f"layer {i}: {m.heads} heads x {m.vdim} value channels exceed the decode attention kernel")
+        if f.kind == "moe" and (f.top > 16 or f.experts > 1024 or f.top > f.experts):
+            bad.append(f"layer {i}: top {f.top} of {f.experts} experts (the router takes up to 16 of 1,024)")
+    if bad:
+        raise PreflightError("model contract: " + "; ".join(bad))
+    if not on_gpu:
+        return ["fp32 reference path: no kernel geometry rules apply"]
+    return ["layer-listed model: tcgen05 projections, experts and prompt attention; delta-rule, decode attention and row "
+            "operators as CUDA kernels of their own"]
 
 
 def host_memory(args) -> List[str]:

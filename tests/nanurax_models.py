@@ -43,7 +43,7 @@ CONFIGS = {
     # recurrent layers only: no paged rows at all
     "recurrent": config(120, 72, [delta(2, 24, dense(72)), delta(4, 8, None)]),
     # attention only: no state slots
-    "attention": config(120, 96, [attention(6, 3, 16, 16, 50, dense(64)), attention(2, 1, 48, 48, 130, None)]),
+    "attention": config(120, 96, [attention(9, 3, 16, 16, 50, dense(64)), attention(2, 1, 48, 48, 130, None)]),
 }
 
 

@@ -239,7 +239,7 @@ def _attention_case(lens, H, G, d, dv, page, chunk, dtype, seed=0, talk=True, ed
     return q.to(DEV), p, pool["pool"].to(DEV), bt.to(DEV), want, dp, dvp
 
 
-SHAPES = [(6, 3, 48, 48, 64, 100), (4, 4, 20, 36, 16, 37), (8, 1, 64, 128, 64, 0), (32, 8, 128, 128, 64, 160),
+SHAPES = [(9, 3, 56, 48, 64, 100), (4, 4, 20, 36, 16, 37), (8, 1, 64, 128, 64, 0), (32, 8, 128, 128, 64, 160),
           (1, 1, 8, 8, 32, 16), (16, 2, 40, 200, 128, 64), (10, 2, 96, 24, 64, 1)]
 
 

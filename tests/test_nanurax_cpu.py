@@ -126,19 +126,22 @@ def test_greedy_generation_through_the_scheduler_with_chunks_holds_and_evictions
     w = nm.weights_of(d, seed=3)
     model = nm.build(d, w)
     prompts = [nm.prompt(d, n, i) for i, n in enumerate((50, 9, 33, 21))]
-    want = [_greedy(d, w, p, 12) for p in prompts]
-    params = SamplingParams(max_new_tokens=12, ignore_eos=True)
+    want = [_greedy(d, w, p, 30) for p in prompts]
+    params = SamplingParams(max_new_tokens=30, ignore_eos=True)
     assert nm.engine(model).generate(prompts, params) == want
-    # pieces of at most 16 prompt tokens, two state slots, few pages of 8 tokens: rows wait, are evicted and recomputed
-    tight = nm.engine(model, tokens=8 * 17, slots=2, page=8, max_prefill_tokens=16, initial_gpu_page_buffer=1,
+    # pieces of at most 16 prompt tokens, few state slots and pages of 8 tokens: rows wait, are evicted and recomputed
+    tight = nm.engine(model, tokens=8 * 16, slots=3, page=8, max_prefill_tokens=16, initial_gpu_page_buffer=1,
                       extension_gpu_page_buffer=1, decision_frequency_pages=1)
     assert tight.generate(prompts, params) == want
+    assert tight.stats.evictions > 0 and tight.stats.prefill_chunks > 0
     # a host tier: parked rows keep their state
     from batchgen_b200.config import EngineConfig
     from batchgen_b200.runtime.engine import Engine
-    ecfg = EngineConfig(page_size=8, max_decode_batch=2, max_state_slots=2, initial_gpu_page_buffer=1,
+    ecfg = EngineConfig(page_size=8, max_decode_batch=4, max_state_slots=3, initial_gpu_page_buffer=1,
                         extension_gpu_page_buffer=1, decision_frequency_pages=1, enable_cuda_graph=False)
-    assert Engine(model, ecfg, num_gpu_pages=14, num_host_pages=40).generate(prompts, params) == want
+    parked = Engine(model, ecfg, num_gpu_pages=16, num_host_pages=60)
+    assert parked.generate(prompts, params) == want
+    assert parked.stats.holds > 0 and parked.host_state.offloads > 0 and parked.host_state.loads > 0
 
 
 # ---------------------------------------------------------------- registry, directories, command line
@@ -215,3 +218,44 @@ def test_planner_and_preflight_know_the_design():
     plan = planner.plan_deployment(cfg, ecfg, planner.MACHINES["b200"])
     assert plan.fits and plan.expert_bytes == 3 * 64 * 3 * 2304 * 1024 * 2
     assert planner.layered_workspace_bytes(cfg) > 4 * 5 * 4096
+
+
+def test_server_serves_a_model_directory(tmp_path):
+    import time
+
+    from fastapi.testclient import TestClient
+
+    from batchgen_b200.server.http_server import create_app
+    from batchgen_b200.server.preflight import PreflightError, model_contract, run_all_preflights
+    from batchgen_b200.server.server_args import ServerArgs, ServerArgsError, validate_server_args
+    d = nm.config(300, 48, [nm.delta(2, 16, nm.dense(40)), nm.attention(4, 2, 8, 8, 24, nm.moe(24, 3, 1, 1.0, 32))])
+    w = nm.weights_of(d, seed=8)
+    _save(str(tmp_path / "m"), d, w)
+    args = validate_server_args(ServerArgs(
+        model=str(tmp_path / "m"), device="cpu", tokenizer="ids", page_size=16, num_gpu_pages=64, initial_gpu_page_buffer=2,
+        extension_gpu_page_buffer=1, decision_frequency_pages=1, storage_path=str(tmp_path / "store"), startup_timeout=120.0,
+        watchdog_timeout=0.0, max_model_len=256))
+    assert run_all_preflights(args)
+    prompts = [nm.prompt(d, n, i) for i, n in enumerate((30, 5))]
+    lines = [{"custom_id": f"r{i}", "method": "POST", "url": "/v1/completions",
+              "body": {"model": "m", "prompt": p, "max_tokens": 6, "temperature": 0, "ignore_eos": True}}
+             for i, p in enumerate(prompts)]
+    with TestClient(create_app(args)) as c:
+        data = "\n".join(map(json.dumps, lines)) + "\n"
+        f = c.post("/v1/files", files={"file": ("in.jsonl", data.encode(), "application/jsonl")}, data={"purpose": "batch"}).json()
+        b = c.post("/v1/batches", json={"input_file_id": f["id"], "endpoint": "/v1/completions"}).json()
+        for _ in range(1200):
+            b = c.get(f"/v1/batches/{b['id']}").json()
+            if b["status"] in ("completed", "failed"):
+                break
+            time.sleep(0.1)
+        assert b["status"] == "completed" and b["request_counts"]["completed"] == 2, b
+        out = {o["custom_id"]: o["response"]["body"]["choices"][0]["text"] for o in
+               map(json.loads, c.get(f"/v1/files/{b['output_file_id']}/content").text.splitlines())}
+    for i, p in enumerate(prompts):
+        assert out[f"r{i}"].split() == [str(t) for t in _greedy(d, w, p, 6)]
+    with pytest.raises(ServerArgsError):
+        validate_server_args(ServerArgs(model=str(tmp_path / "nothing")))
+    from batchgen_b200.config import get_model_config
+    with pytest.raises(PreflightError, match="one GPU"):
+        model_contract(get_model_config(str(tmp_path / "m")), 2, True)
