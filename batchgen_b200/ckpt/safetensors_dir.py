@@ -46,6 +46,32 @@ def tensor_shapes(path: str) -> Dict[str, Tuple[int, ...]]:
     return out
 
 
+def checkpoint_shapes(path: str) -> Dict[str, Tuple[int, ...]]:
+    """name -> shape of a model directory: its .safetensors files, or converted shards (``ckpt.converter``)."""
+    if _files(path):
+        return tensor_shapes(path)
+    from .converter import ConvertedCheckpoint
+    ck = ConvertedCheckpoint(path)
+    shapes = {k: tuple(e["shape"]) for k, (_, e) in ck.index.items()}
+    ck.close()
+    return shapes
+
+
+def checkpoint_loader(path: str) -> Callable[[str, Tuple[int, ...]], torch.Tensor]:
+    """Loader of a model directory in either format."""
+    if _files(path):
+        return SafetensorsDir(path).loader()
+    from .converter import ConvertedCheckpoint
+    ck = ConvertedCheckpoint(path)
+    inner = ck.loader()
+
+    def load(name, shape):
+        if name not in ck:
+            raise KeyError(f"the checkpoint has no tensor {name!r}")
+        return inner(name, shape)
+    return load
+
+
 class SafetensorsDir:
     def __init__(self, path: str):
         self.index: Dict[str, Tuple[memoryview, dict]] = {}

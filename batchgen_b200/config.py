@@ -639,8 +639,8 @@ def nanurax_config(d: Dict, name: str = "nanurax", decay_ranks: Optional[Dict[in
 
 
 def _nanurax_dir(path: str, d: Dict) -> ModelConfig:
-    from .ckpt.safetensors_dir import tensor_shapes
-    shapes = tensor_shapes(path)
+    from .ckpt.safetensors_dir import checkpoint_shapes
+    shapes = checkpoint_shapes(path)
     ranks = {i: shapes[f"l{i}.mix.w1"][0] for i in range(len(d["layers"])) if f"l{i}.mix.w1" in shapes}
     cfg = nanurax_config(d, os.path.basename(os.path.normpath(path)) or "nanurax", ranks)
     cfg.checkpoint_dir = path

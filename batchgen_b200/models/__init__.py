@@ -21,8 +21,8 @@ def build_model(cfg: ModelConfig, device="cpu", dtype="fp32", seed: int = 0, lay
     dt = _DTYPES[dtype] if isinstance(dtype, str) else dtype
     layout = layout or ParallelLayout()
     if loader is None and cfg.checkpoint_dir:
-        from ..ckpt.safetensors_dir import SafetensorsDir
-        loader = SafetensorsDir(cfg.checkpoint_dir).loader()
+        from ..ckpt.safetensors_dir import checkpoint_loader
+        loader = checkpoint_loader(cfg.checkpoint_dir)
     if loader is not None:
         from .checkpoint_names import aliased_loader
         loader = aliased_loader(cfg, loader)            # published names of the family, when they differ

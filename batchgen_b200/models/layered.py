@@ -147,6 +147,39 @@ def build_layered_weights(cfg: ModelConfig, layout: ParallelLayout, src: WeightS
     return w
 
 
+def layered_tensor_specs(cfg: ModelConfig) -> List[Tuple[str, Tuple[int, ...], str, int]]:
+    """(name, shape, init kind, layer) of every checkpoint tensor (layer -1: embedding, final norm, head)."""
+    D, V = cfg.hidden_size, cfg.vocab_size
+    out = [("embed", (V, D), "normal", -1), ("final.norm", (D,), "norm", -1), ("head", (V, D), "normal", -1)]
+    for i, s in enumerate(cfg.layer_specs):
+        m, f, p, q = s.mixer, s.mlp, f"l{i}.mix.", f"l{i}.mlp."
+        out.append((f"l{i}.norm1", (D,), "norm", i))
+        if m.recurrent:
+            n = m.heads * m.dim
+            out += [(p + x, (n, D), "normal", i) for x in ("r", "k", "v", "g", "a")]
+            out += [(p + "w1", (m.decay_rank, D), "normal", i), (p + "w2", (n, m.decay_rank), "normal", i),
+                    (p + "a.b", (n,), "bias", i), (p + "w0", (n,), "bias", i), (p + "norm", (n,), "norm", i),
+                    (p + "o", (D, n), "normal", i)]
+        else:
+            out += [(p + "q", (m.heads * m.dim, D), "normal", i), (p + "k", (m.kv_heads * m.dim, D), "normal", i),
+                    (p + "v", (m.kv_heads * m.vdim, D), "normal", i), (p + "o", (D, m.heads * m.vdim), "normal", i)]
+            if m.talking:
+                out.append((p + "talk", (m.heads, m.heads), "normal", i))
+
+        def ff(prefix, n):
+            return [(prefix + "gate", (n, D), "normal", i), (prefix + "up", (n, D), "normal", i),
+                    (prefix + "down", (D, n), "normal", i)]
+        if f.kind == "dense":
+            out += ff(q, f.ff)
+        elif f.kind == "moe":
+            out.append((q + "router", (f.experts, D), "normal", i))
+            for e in range(f.experts):
+                out += ff(f"{q}e{e}.", f.ff)
+            if f.shared_ff:
+                out += ff(q + "shared.", f.shared_ff) + [(q + "shared.sg", (1, D), "normal", i)]
+    return out
+
+
 @dataclass
 class _Plan:
     """Device tables of one step, shared by its layers."""

@@ -345,8 +345,11 @@ def build_weights(cfg: ModelConfig, layout: ParallelLayout, src: WeightSource, d
 
 
 def checkpoint_tensor_specs(cfg: ModelConfig):
-    """(name, shape, init kind, layer) of every checkpoint tensor of an MLA model, in file order
+    """(name, shape, init kind, layer) of every checkpoint tensor of an MLA, GQA or layer-listed model, in file order
     (layer -1 = embeddings / final norm / lm_head)."""
+    if cfg.is_layered:
+        from .layered import layered_tensor_specs
+        return layered_tensor_specs(cfg)
     H = cfg.hidden_size
     out = [("model.embed_tokens.weight", (cfg.vocab_size, H), "normal", -1),
            ("model.norm.weight", (H,), "norm", -1)]

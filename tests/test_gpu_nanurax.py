@@ -245,7 +245,7 @@ SHAPES = [(9, 3, 56, 48, 64, 100), (4, 4, 20, 36, 16, 37), (8, 1, 64, 128, 64, 0
 
 @pytest.mark.parametrize("H,G,d,dv,page,chunk", SHAPES)
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-def test_attention_rows_and_tiles_match_the_oracle(H, G, d, dv, page, chunk, dtype):
+def test_attention_rows_and_tiles_match_the_oracle(H, G, d, dv, page, chunk, dtype, monkeypatch):
     from batchgen_b200.ops import _ext, talking
     lens = [150, 33, 1, 300]
     q, p, pool, bt, want, dp, dvp = _attention_case(lens, H, G, d, dv, page, chunk, dtype, seed=H + d)
@@ -283,6 +283,13 @@ def test_attention_rows_and_tiles_match_the_oracle(H, G, d, dv, page, chunk, dty
     out = torch.full((T, H * dvp), 5.0, dtype=dtype, device=DEV)
     talking.attend_prefill(q, p, pool, bt, out, talking.work_blocks(talking.prefill_work(cu, [0] * 4, chunk), T, DEV))
     check(out, "tiles")
+    # mixed queries held for a few rows at a time (ranges that cut through tiles' alignment)
+    monkeypatch.setattr(talking, "_FOLD_ROWS", 100)
+    blocks = talking.work_blocks(talking.prefill_work(cu, [0] * 4, chunk), T, DEV)
+    assert len(blocks) > 2
+    out = torch.full((T, H * dvp), 5.0, dtype=dtype, device=DEV)
+    talking.attend_prefill(q, p, pool, bt, out, blocks)
+    check(out, "row ranges")
     # the last 70 queries of the long sequence as a piece of their own (cached keys before them)
     out = torch.full((T, H * dvp), 5.0, dtype=dtype, device=DEV)
     talking.attend_prefill(q, p, pool, bt[3:4].contiguous(), out,
@@ -401,6 +408,20 @@ def test_mixed_batches_equal_each_request_alone(dtype, tol):
     for g, x in zip(got, want):
         assert nm.close(torch.cat(g), x, tol, d), nm.error(torch.cat(g), x)
     assert eng.kv.alloc.num_used == 0 and eng.kv.state.num_free == 4
+
+
+@pytest.mark.parametrize("dtype,tol", [("fp32", 1e-4), ("bf16", 6e-2)])
+def test_a_long_prompt_over_many_pages_and_chunks(dtype, tol):
+    d = nm.config(150, 64, [nm.delta(2, 32, nm.dense(64)), nm.attention(4, 2, 16, 24, 700, nm.moe(40, 3, 3, 1.2, 24))])
+    w = nm.weights_of(d, seed=15)
+    toks = nm.prompt(d, 1500)
+    want = oracle.forward(d, w, toks, torch.float64)
+    eng = nm.engine(nm.build(d, w, DEV, dtype), tokens=1536 + 64)
+    for sizes in ([1500], [1390, 1], [333]):
+        s = eng.open_sequence()
+        got = nm.run_pieces(eng, s, toks, sizes)
+        eng.close_sequence(s)
+        assert nm.close(got, want, tol, d), (sizes, nm.error(got, want))
 
 
 def test_greedy_generation_in_32_bit_and_long_decoding():

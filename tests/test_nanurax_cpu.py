@@ -159,6 +159,15 @@ def test_config_directory_registry_and_validation(tmp_path):
     toks = nm.prompt(d, 40)
     eng = nm.engine(build_model(cfg))
     assert nm.error(eng.extend([(eng.open_sequence(), toks, range(40))]), oracle.forward(d, w, toks)) < 2e-5
+    # the names the framework writes are the ones it reads; a converted copy of the directory serves as well
+    from batchgen_b200.ckpt.converter import convert_dir
+    from batchgen_b200.models.weights import checkpoint_tensor_specs
+    assert {n: s for n, s, _, _ in checkpoint_tensor_specs(cfg)} == {k: tuple(t.shape) for k, t in w.items()}
+    convert_dir(str(tmp_path / "m"), str(tmp_path / "c"))
+    conv = get_model_config(str(tmp_path / "c"))
+    assert conv.layer_specs == cfg.layer_specs
+    eng = nm.engine(build_model(conv))
+    assert nm.error(eng.extend([(eng.open_sequence(), toks, range(40))]), oracle.forward(d, w, toks)) < 2e-5
     bad = json.loads(json.dumps(d))
     bad["layers"][0]["type"] = "something_else"
     with pytest.raises(ValueError, match="something_else"):
