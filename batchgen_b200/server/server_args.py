@@ -19,7 +19,7 @@ from ..config import EngineConfig, list_models
 @dataclass
 class ServerArgs:
     # model / paths
-    model: str = "tiny-deepseek-v3"         # preset name or a Hugging Face style id (config.get_model_config)
+    model: str = "tiny-deepseek-v3"         # preset name, Hugging Face style id, or model directory (config.get_model_config)
     cache_dir: str = ""                     # directory for derived files (converted shards, staged stores)
     converted_ckpt_dir: str = ""            # checkpoint in the converted format (ckpt.converter); empty = random weights
     tokenizer: str = "ids"                  # ids | bytes | a local tokenizer directory
