@@ -581,11 +581,8 @@ static int launch_decode(const Params& p, int nseq, int num_sms, int* status, cu
 
 extern "C" {
 
-// Floats of scratch per token: prompt records and the scan's outputs.
-long long bg_delta_scratch_floats(int H, int D) { return (long long)H * (bg::delta::rec_floats(D) + D); }
-
 // offs: host array of five column offsets (r, k, v, g, a).  dt: 0 = bf16 output, 1 = fp32.  D a multiple of 8, <= 256.
-// T: rows of z.  `scratch` (T * bg_delta_scratch_floats floats) selects the prompt path; null the decode kernel (D <= 128, one
+// T: rows of z.  `scratch` (T * H * (6 D + 4) floats: records, then the scan's outputs) selects the prompt path; null the decode kernel (D <= 128, one
 // token per sequence).
 int bg_delta_forward(int dt, const float* z, int ldz, const int* offs, const float* wl, int ld_wl, const float* w0,
                      const float* ab, const float* norm_w, float* state, long long slot_stride, const int* cu,
