@@ -22,21 +22,33 @@ from typing import Dict, List, Optional, Tuple
 
 @dataclass(frozen=True)
 class MixerSpec:
-    """The token mixer of one layer of a layer-listed model."""
-    kind: str                              # "attention" | "general_delta"
+    """A token mixer of a layer-listed model."""
+    kind: str                              # "attention" | "general_delta" | "channel_delta" | "mlstm" | "retention"
     heads: int
     dim: int                               # query / key width of a head
-    kv_heads: int = 0                      # attention: key / value heads (query head h reads h // (heads / kv_heads))
+    kv_heads: int = 0                      # key / value heads of attention, query / key heads of channel_delta (0 = heads)
     vdim: int = 0                          # value width of a head
     scale: float = 1.0                     # attention: factor of the scores
     chunk: int = 0                         # attention: keys are seen inside the query's own chunk of this many positions (0 = all)
     talking: bool = False                  # attention: a [heads, heads] matrix mixes the heads' scores before the softmax
     sink: bool = False                     # attention: one is added to the softmax denominator
-    decay_rank: int = 0                    # general_delta: width of the low-rank decay projection
+    out_gate: bool = False                 # attention: a sigmoid gate per head scales its output
+    rot_dims: int = 0                      # attention, retention: leading head dimensions with rotary positions (rotate half)
+    rot_base: float = 10000.0
+    decay_rank: int = 0                    # general_delta, channel_delta: width of the low-rank decay projection
+    gate_rank: int = 0                     # channel_delta: width of the low-rank output-gate projection
+    conv: int = 0                          # channel_delta: taps of the short convolutions of q, k and v
+    gate_cap: float = 0.0                  # mlstm: soft cap of the gates' pre-activations
+    decay: Tuple[float, ...] = ()          # retention: decay per head
 
     @property
     def recurrent(self) -> bool:
-        return self.kind == "general_delta"
+        return self.kind != "attention"
+
+    @property
+    def qk_heads(self) -> int:
+        """Heads of the keys (and, for recurrent mixers, of the queries)."""
+        return self.kv_heads or self.heads
 
     @property
     def dim_p(self) -> int:
@@ -57,13 +69,50 @@ class MixerSpec:
         """fp32 state [head, key channel, value channel]; empty for attention."""
         return (self.heads, self.dim_p, self.vdim_p) if self.recurrent else (0, 0, 0)
 
+    @property
+    def state_parts(self) -> Dict[str, Tuple[int, ...]]:
+        """Everything a sequence carries from token to token, by name (fp32)."""
+        if not self.recurrent:
+            return {}
+        parts: Dict[str, Tuple[int, ...]] = {"S": self.state_shape}
+        if self.kind == "mlstm":
+            parts["n"] = (self.heads, self.dim_p)                  # normaliser, decayed and written like a column of S
+            parts["m"] = (self.heads,)                             # running maximum of the log gates
+        if self.kind == "channel_delta":
+            parts["conv"] = (self.conv - 1, self.conv_channels)    # last inputs of the short convolutions, oldest first
+        return parts
+
+    @property
+    def conv_channels(self) -> int:
+        return 2 * self.qk_heads * self.dim_p + self.heads * self.vdim_p
+
+    @property
+    def in_columns(self) -> int:
+        """fp32 columns a token's projections take (a workspace estimate, padding aside)."""
+        qk, v = self.heads * self.dim_p, self.heads * self.vdim_p
+        return {"attention": qk + self.kv_heads * (self.dim_p + self.vdim_p) + self.heads,
+                "general_delta": 6 * qk,
+                "channel_delta": 2 * self.conv_channels + 2 * v + qk + self.decay_rank + self.gate_rank + self.heads,
+                "mlstm": 2 * qk + 2 * v + 2 * self.heads, "retention": 2 * qk + 2 * v}[self.kind]
+
+    def param_count(self, width: int) -> int:
+        qk, v, H = self.heads * self.dim, self.heads * self.vdim, self.heads
+        if self.kind == "attention":
+            return width * (H + self.kv_heads) * (self.dim + self.vdim) + (H * H if self.talking else 0)
+        if self.kind == "general_delta":
+            return width * (6 * qk + self.decay_rank) + self.decay_rank * qk
+        if self.kind == "channel_delta":
+            return (width * (2 * self.qk_heads * self.dim + 2 * v + H + self.decay_rank + self.gate_rank)
+                    + self.decay_rank * qk + self.gate_rank * v)
+        return width * (2 * qk + 3 * v + (2 * H if self.kind == "mlstm" else 0))
+
 
 @dataclass(frozen=True)
 class MlpSpec:
     """The feed-forward of one layer of a layer-listed model."""
     kind: str = "none"                     # none | dense | moe
     ff: int = 0                            # dense width, or width of one routed expert
-    activation: str = "gelu_tanh"          # gelu_tanh | swiglu_oai (clamped gate and up, sigmoid slope 1.702, up + 1)
+    activation: str = "gelu_tanh"          # gelu_tanh | swiglu_oai (clamped gate and up, sigmoid slope 1.702, up + 1) | relu2 (no gate)
     limit: float = 0.0                     # clamp of swiglu_oai
     experts: int = 0
     top: int = 0
@@ -76,12 +125,32 @@ class MlpSpec:
 class LayerSpec:
     mixer: MixerSpec
     mlp: MlpSpec = MlpSpec()
+    second: Optional[MixerSpec] = None     # a mixer beside the first: both outputs are RMS-normed over the width and averaged
+
+    @property
+    def mixers(self) -> Tuple[MixerSpec, ...]:
+        return (self.mixer,) if self.second is None else (self.mixer, self.second)
+
+    @property
+    def kv_row(self) -> int:
+        return sum(m.kv_row for m in self.mixers)
+
+    def state_parts(self, width: int, canon_taps: int) -> Dict[str, Tuple[int, ...]]:
+        """fp32 state of a sequence in this layer: the mixers' parts (the second mixer's names end in ".1") and, with input
+        convolutions, the last inputs of each sublayer."""
+        parts = {name + (f".{i}" if i else ""): shape for i, m in enumerate(self.mixers) for name, shape in m.state_parts.items()}
+        if canon_taps:
+            rows = (canon_taps - 1, -(-width // 4) * 4)
+            parts["canon1"] = rows
+            if self.mlp.kind != "none":
+                parts["canon2"] = rows
+        return parts
 
 
 @dataclass
 class ModelConfig:
     name: str = "tiny-deepseek-v3"
-    family: str = "deepseek_v3"  # deepseek_v3 | deepseek_v2 | deepseek_v4 | glm5 | kimi_k3 | kimi_k25 | gpt_oss | minimax | mixtral | qwen2_moe | nanurax
+    family: str = "deepseek_v3"  # deepseek_v3 | deepseek_v2 | deepseek_v4 | glm5 | kimi_k3 | kimi_k25 | gpt_oss | minimax | mixtral | qwen2_moe | nanurax | pamevik
     vocab_size: int = 1024
     hidden_size: int = 256
     num_layers: int = 2
@@ -149,10 +218,13 @@ class ModelConfig:
     # ---- quantisation of linear / expert weights
     quant: str = "none"                    # none | fp8_block | mxfp4 | int4
     quant_block: int = 128
-    # ---- layer-listed models: every layer has its own mixer and feed-forward, both reading one norm of the residual
-    # stream (parallel block), with an fp32 residual and scaled embeddings
+    # ---- layer-listed models: every layer has its own mixer and feed-forward, with an fp32 residual and scaled embeddings
     layer_specs: Tuple[LayerSpec, ...] = ()
     embed_scale: float = 1.0
+    sandwich: bool = False                 # False: mixer and feed-forward read one RMS norm and are added together (parallel
+                                           # block); True: one after the other, a norm before and after each
+    layer_norm: bool = False               # sandwich: norms subtract the mean and have biases (else RMS norms)
+    canon_taps: int = 0                    # sandwich: every sublayer reads h + conv(h), a causal convolution of this many taps
     checkpoint_dir: str = ""               # directory the config was read from (its .safetensors files are the weights)
     # ---- misc
     eos_token_id: int = 1
@@ -174,15 +246,20 @@ class ModelConfig:
 
     @property
     def recurrent_layers(self) -> Tuple[int, ...]:
-        return tuple(l for l, s in enumerate(self.layer_specs) if s.mixer.recurrent)
+        return tuple(l for l, s in enumerate(self.layer_specs) if any(m.recurrent for m in s.mixers))
 
     @property
     def has_state(self) -> bool:
         """A live sequence holds a state slot besides (or instead of) paged KV."""
-        return self.has_kda or self.is_v4 or len(self.recurrent_layers) > 0
+        return self.has_kda or self.is_v4 or len(self.layered_state_parts()) > 0
+
+    def layered_state_parts(self) -> List[Tuple[Tuple[int, str], Tuple[int, ...]]]:
+        """((layer, name), shape) of everything a sequence of a layer-listed model carries outside the paged rows."""
+        return [((l, name), shape) for l, s in enumerate(self.layer_specs)
+                for name, shape in s.state_parts(self.hidden_size, self.canon_taps).items()]
 
     def layered_state_floats_per_seq(self) -> int:
-        return sum(math.prod(self.layer_specs[l].mixer.state_shape) for l in self.recurrent_layers)
+        return sum(math.prod(shape) for _, shape in self.layered_state_parts())
 
     def v4_state_floats_per_seq(self) -> int:
         """fp32 words of per-sequence state of a DeepSeek-V4 model: per layer the window ring, the compressor's
@@ -203,7 +280,7 @@ class ModelConfig:
         if self.is_v4:
             return self.head_dim
         if self.is_layered:
-            return sum(s.mixer.kv_row for s in self.layer_specs)
+            return sum(s.kv_row for s in self.layer_specs)
         if self.num_kv_heads > 0:
             return 2 * self.num_kv_heads * self.head_dim
         return self.kv_lora_rank + self.qk_rope_head_dim
@@ -289,12 +366,9 @@ class ModelConfig:
             return n
         if self.is_layered:
             for spec in self.layer_specs:
-                m, f = spec.mixer, spec.mlp
-                if m.recurrent:
-                    n += h * (6 * m.heads * m.dim + m.decay_rank) + m.decay_rank * m.heads * m.dim
-                else:
-                    n += h * (m.heads + m.kv_heads) * (m.dim + m.vdim) + m.heads * m.heads
-                n += 3 * h * f.ff * (f.experts if f.kind == "moe" else 1) + h * f.experts + 3 * h * f.shared_ff
+                f = spec.mlp
+                n += sum(m.param_count(h) for m in spec.mixers)
+                n += (2 if f.activation == "relu2" else 3) * h * f.ff * (f.experts if f.kind == "moe" else 1) + h * f.experts + 3 * h * f.shared_ff
             return n
         for l in range(self.num_layers):
             if self.layer_is_kda(l):
@@ -330,8 +404,10 @@ class ModelConfig:
         if "compress_ratios" in kw:
             kw["compress_ratios"] = tuple(kw["compress_ratios"])
         if "layer_specs" in kw:
+            def mixer(m):
+                return None if m is None else MixerSpec(**{**m, "decay": tuple(m.get("decay", ()))})
             kw["layer_specs"] = tuple(
-                x if isinstance(x, LayerSpec) else LayerSpec(MixerSpec(**x["mixer"]), MlpSpec(**x["mlp"]))
+                x if isinstance(x, LayerSpec) else LayerSpec(mixer(x["mixer"]), MlpSpec(**x["mlp"]), mixer(x.get("second")))
                 for x in kw["layer_specs"])
         return cls(**kw)
 
@@ -647,7 +723,68 @@ def _nanurax_dir(path: str, d: Dict) -> ModelConfig:
     return cfg
 
 
-_ARCHITECTURES = {"Nanurax": _nanurax_dir}        # config.json "architecture" -> reader of the model directory
+# ------------------------------------------------------------------ Pamevik: layer-listed config.json
+def _pamevik_layer(d: Dict, index: int, ranks: Tuple[int, int]) -> LayerSpec:
+    m, kind = d["mixer"], d["type"]
+
+    def divides(x: MixerSpec) -> MixerSpec:
+        if x.heads % x.qk_heads:
+            raise ValueError(f"layer {index}: {x.heads} heads do not divide over {x.qk_heads} key heads")
+        if x.rot_dims % 2 or x.rot_dims > x.dim:
+            raise ValueError(f"layer {index}: {x.rot_dims} rotary dimensions in heads of {x.dim}")
+        return x
+
+    def rotary(x: Dict) -> Dict:
+        r = x.get("rot")
+        return {"rot_dims": int(r["dims"]), "rot_base": float(r["base"])} if r else {}
+    second = None
+    if kind == "mlstm":
+        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], vdim=m["vdim"], gate_cap=float(m["gate_cap"]))
+    elif kind == "channel_delta":
+        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], kv_heads=m.get("kv_heads", m["heads"]), vdim=m["vdim"],
+                          conv=int(m["conv"]), decay_rank=ranks[0], gate_rank=ranks[1])
+    elif kind == "parallel":
+        a, r = m["left"], m["right"]
+        mixer = MixerSpec("attention", heads=a["heads"], dim=a["dim"], kv_heads=a.get("kv_heads", a["heads"]), vdim=a["vdim"],
+                          scale=float(a["scale"]), out_gate=True, **rotary(a))
+        second = divides(MixerSpec("retention", heads=r["heads"], dim=r["dim"], vdim=r["vdim"],
+                                   decay=tuple(float(x) for x in r["decay"]), **rotary(r)))
+        if len(second.decay) != second.heads:
+            raise ValueError(f"layer {index}: {len(second.decay)} decays for {second.heads} heads")
+    else:
+        raise ValueError(f"layer {index}: unknown mixer type {kind!r}")
+    f = d.get("mlp")
+    if f and f["kind"] != "dense":
+        raise ValueError(f"layer {index}: unknown feed-forward kind {f['kind']!r}")
+    return LayerSpec(divides(mixer), MlpSpec("dense", ff=f["ff"], activation="relu2") if f else MlpSpec(), second)
+
+
+def pamevik_config(d: Dict, name: str = "pamevik", ranks: Optional[Dict[int, Tuple[int, int]]] = None) -> ModelConfig:
+    """A Pamevik config.json (parsed) as a ``ModelConfig``.  ``ranks``: per channel_delta layer the widths of its low-rank
+    decay and output-gate projections, which only the checkpoint's tensor shapes tell (default 64)."""
+    layers = tuple(_pamevik_layer(x, i, (ranks or {}).get(i, (64, 64))) for i, x in enumerate(d["layers"]))
+    att = [m for s in layers for m in s.mixers if not m.recurrent]
+    return ModelConfig(
+        name=name, family="pamevik", vocab_size=d["vocab"], hidden_size=d["width"], num_layers=len(layers), layer_specs=layers,
+        rms_eps=float(d["norm"]["eps"]), sandwich=True, layer_norm=True, canon_taps=int(d["canon"]["taps"]),
+        # summaries that planners read; the layers themselves are described by ``layer_specs``
+        num_heads=max(m.heads for s in layers for m in s.mixers), num_kv_heads=max((m.kv_heads for m in att), default=1),
+        head_dim=max(m.dim for s in layers for m in s.mixers), first_k_dense=0,
+        intermediate_size=max(s.mlp.ff for s in layers), moe_intermediate_size=0, n_routed_experts=0, n_shared_experts=0,
+        num_experts_per_tok=0, max_position_embeddings=1 << 30, eos_token_id=-1, bos_token_id=-1)
+
+
+def _pamevik_dir(path: str, d: Dict) -> ModelConfig:
+    from .ckpt.safetensors_dir import checkpoint_shapes
+    shapes = checkpoint_shapes(path)
+    ranks = {i: (shapes[f"l{i}.mix.a1"][0], shapes[f"l{i}.mix.g1"][0]) for i in range(len(d["layers"]))
+             if f"l{i}.mix.a1" in shapes and f"l{i}.mix.g1" in shapes}
+    cfg = pamevik_config(d, os.path.basename(os.path.normpath(path)) or "pamevik", ranks)
+    cfg.checkpoint_dir = path
+    return cfg
+
+
+_ARCHITECTURES = {"Nanurax": _nanurax_dir, "Pamevik": _pamevik_dir}        # config.json "architecture" -> reader of the model directory
 
 
 def load_model_dir(path: str) -> ModelConfig:
@@ -687,7 +824,35 @@ def nanurax_bench() -> ModelConfig:
         "nanurax-bench")
 
 
+def tiny_pamevik() -> ModelConfig:
+    """One layer of every mixer, with and without a feed-forward."""
+    cd = {"type": "channel_delta", "mixer": {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 40, "conv": 3}}
+    ml = {"type": "mlstm", "mixer": {"heads": 3, "dim": 20, "vdim": 32, "gate_cap": 9.0}}
+    par = {"type": "parallel", "mixer": {
+        "left": {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 24, "scale": 0.2, "rot": {"base": 5000.0, "dims": 16}},
+        "right": {"heads": 2, "dim": 16, "vdim": 40, "decay": [0.9, 0.99], "rot": {"base": 800.0, "dims": 16}}}}
+    return pamevik_config({
+        "vocab": 320, "width": 120, "norm": {"eps": 1e-5}, "canon": {"taps": 3},
+        "layers": [dict(cd, mlp={"kind": "dense", "ff": 200}), dict(par, mlp=None), dict(ml, mlp={"kind": "dense", "ff": 88})]},
+        "tiny-pamevik", {0: (12, 20)})
+
+
+def pamevik_bench() -> ModelConfig:
+    """Layers of a real model's size: channel-delta, mLSTM, channel-delta and one attention-beside-retention layer."""
+    dense = {"kind": "dense", "ff": 9216}
+    cd = {"type": "channel_delta", "mlp": dense, "mixer": {"heads": 32, "kv_heads": 32, "dim": 128, "vdim": 128, "conv": 4}}
+    ml = {"type": "mlstm", "mlp": dense, "mixer": {"heads": 32, "dim": 128, "vdim": 128, "gate_cap": 15.0}}
+    rot = {"base": 1e6, "dims": 128}
+    par = {"type": "parallel", "mlp": dense, "mixer": {
+        "left": {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": rot},
+        "right": {"heads": 32, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 7 * i / 31) for i in range(32)], "rot": rot}}}
+    return pamevik_config({"vocab": 163840, "width": 2304, "norm": {"eps": 1e-6}, "canon": {"taps": 4},
+                           "layers": [cd, ml, dict(cd), par]}, "pamevik-bench", {0: (128, 128), 2: (128, 128)})
+
+
 _PRESETS = {
+    "tiny-pamevik": tiny_pamevik,
+    "pamevik-bench": pamevik_bench,
     "tiny-nanurax": tiny_nanurax,
     "nanurax-bench": nanurax_bench,
     "tiny-deepseek-v3": tiny_deepseek_v3,
@@ -741,6 +906,7 @@ _PATTERNS = [
     (r"gpt[-_]?oss", "gpt-oss-120b"),
     (r"minimax", "minimax-m2.5"),
     (r"nanurax", "nanurax-bench"),
+    (r"pamevik", "pamevik-bench"),
 ]
 
 

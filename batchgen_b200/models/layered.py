@@ -1,82 +1,81 @@
-"""Layer-listed decoders (``ModelConfig.layer_specs``): every layer names its own token mixer and feed-forward, both read
-one norm of an fp32 residual stream, and their outputs are added together (parallel block).  Nanurax is the family built
-this way: generalised delta-rule layers (recurrent state per sequence) and chunked talking-heads attention layers (paged
-KV), dense tanh-GELU or input-weighted clamped-SwiGLU mixture feed-forwards.
+"""Layer-listed decoders (``ModelConfig.layer_specs``): every layer names its own token mixer(s) and feed-forward around an
+fp32 residual stream.  Two block forms:
+
+* parallel (Nanurax): mixer and feed-forward read one RMS norm and their outputs are added together.  Generalised delta-rule
+  layers and chunked talking-heads attention layers, dense tanh-GELU or input-weighted clamped-SwiGLU mixture feed-forwards.
+* sandwich (Pamevik, ``ModelConfig.sandwich``): mixer, then feed-forward, each between two norms (``layer_norm``: with mean and
+  bias) and behind an input convolution (``canon_taps``).  mLSTM, gated delta-rule with a decay per channel, and softmax
+  attention beside retention; squared-ReLU feed-forwards.
 
 Same calling contract as ``Transformer``: ``forward(ids [T], meta, cache) -> fp32 logits``; all state lives in the caller's
-``PagedKVCache`` (paged rows per attention layer, ``FlatStatePool`` slots for the recurrent layers), and a step may mix
-pieces of prompts with single decoded tokens (``AttnMeta`` mode "prefill") or decode one token per sequence (mode "decode",
-graph capturable).
+``PagedKVCache`` (paged rows per attention layer, ``FlatStatePool`` slots for everything else a sequence carries), and a step
+may mix pieces of prompts with single decoded tokens (``AttnMeta`` mode "prefill") or decode one token per sequence (mode
+"decode", graph capturable).
 
-A layer runs as: residual sum + norm (one kernel, which also adds the previous layer's outputs) -> one GEMM for everything
-that reads the norm (mixer projections, router, shared-expert gate, dense or shared gate / up) -> the mixer's core and the
-gated activation, written side by side -> one GEMM against [W_o | W_down], whose fp32 output is the layer's addend.  Routed
-experts add their rows in the next residual kernel.  GEMM outputs stay fp32: what enters the recurrence, the scores, the
-router and the residual sum is never rounded to 16 bits; GEMM operands are bf16, or fp32 in the 32-bit form of the model.
+A parallel block runs as: residual sum + norm (one kernel, which also adds the previous layer's outputs) -> one GEMM for
+everything that reads the norm (mixer projections, router, shared-expert gate, dense or shared gate / up) -> the mixer's core
+and the gated activation, written side by side -> one GEMM against [W_o | W_down], whose fp32 output is the layer's addend.
+Routed experts add their rows in the next residual kernel.  A sandwich block runs every sublayer as: norm of the previous
+sublayer's output + residual sum + norm + input convolution (one kernel in decode, two in prompts) -> one GEMM for everything
+that reads it -> core or activation -> one GEMM per output projection, whose fp32 output goes to the next norm kernel.  GEMM
+outputs stay fp32: what enters the recurrence, the scores, the router and the residual sum is never rounded to 16 bits; GEMM
+operands are bf16, or fp32 in the 32-bit form of the model.
 
 Widths: the contraction side of every operand is padded with zeros to a multiple of 64 (one TMA / MMA block), head widths
 to multiples of 8, so any model size runs on the same kernels.
 """
 from __future__ import annotations
 
-import math
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Tuple
 
 import torch
 
 from ..config import LayerSpec, ModelConfig
-from ..ops import delta, gemm, residual, talking
+from ..ops import conv, gemm, residual
 from ..ops import moe as moe_ops
 from ..ops.moe import ExpertWeights
 from ..ops.residual import pad_to
 from ..utils.timing import null_timer
+from .mixers import K_ALIGN, Mixer, StepPlan, build_mixer, mixer_tensor_specs, pad_cols, pad_rows, stack_parts
 from .transformer import AttnMeta
 from .weights import ParallelLayout, WeightSource
-
-DECAY_SCALE = math.exp(-0.5)       # decay = exp(-DECAY_SCALE * sigmoid(.)), so a channel keeps at least exp(-exp(-1/2)) a step
-K_ALIGN = 64
 
 
 @dataclass
 class LayeredLayer:
+    """A parallel block."""
     spec: LayerSpec = None
     norm: torch.Tensor = None                     # [width] fp32
     w_in: torch.Tensor = None                     # [sum of segments, width_p]
-    seg: Dict[str, Tuple[int, int]] = field(default_factory=dict)     # name -> (first column of the GEMM output, width)
+    seg: Dict[str, Tuple[int, int]] = field(default_factory=dict)     # feed-forward part -> (first column of the GEMM output, width)
     w_out: torch.Tensor = None                    # [width, mix_p + ff_p]: [W_o | W_down]
-    mix_cols: int = 0                             # columns the mixer writes
-    mix_p: int = 0                                # the same, padded to K_ALIGN
+    mix_p: int = 0                                # columns the mixer writes, padded to K_ALIGN
     ff_p: int = 0
-    w_decay: torch.Tensor = None                  # delta: [heads * dim_p, rank_p], second factor of the decay projection
-    delta: Optional[delta.DeltaParams] = None
-    talk: Optional[talking.TalkParams] = None
+    mixer: Mixer = None
     experts: Optional[ExpertWeights] = None
+
+
+@dataclass
+class Sublayer:
+    """One half of a sandwich block: mixer(s) side by side, or a feed-forward."""
+    norm: residual.Norm
+    post: residual.Norm
+    w_in: torch.Tensor                            # [columns, width_p]
+    w_out: List[torch.Tensor]                     # per mixer W_o, or [W_down]: [width, operand width padded to K_ALIGN]
+    mixers: List[Mixer] = field(default_factory=list)       # empty: feed-forward
+    branch_w: Optional[Tuple[torch.Tensor, torch.Tensor]] = None      # weights of two mixers' output norms
+    canon_w: Optional[torch.Tensor] = None        # [taps, width4] fp32 input convolution
+    canon_part: str = ""                          # its state part
+    ff: int = 0
 
 
 @dataclass
 class LayeredWeights:
     embed: torch.Tensor = None                    # [vocab, width]
-    final_norm: torch.Tensor = None
+    final_norm: torch.Tensor = None               # fp32 gain, or a ``residual.Norm`` (sandwich)
     lm_head: torch.Tensor = None                  # [vocab, width_p]
-    layers: List[LayeredLayer] = field(default_factory=list)
-
-
-def _pad_cols(w: torch.Tensor, cols: int) -> torch.Tensor:
-    return w if w.shape[1] == cols else torch.nn.functional.pad(w, (0, cols - w.shape[1]))
-
-
-def _pad_rows(w: torch.Tensor, rows: int) -> torch.Tensor:
-    return w if w.shape[0] == rows else torch.nn.functional.pad(w, (0, 0, 0, rows - w.shape[0]))
-
-
-def _head_rows(w: torch.Tensor, heads: int, d: int, dp: int) -> torch.Tensor:
-    """[heads * d, ...] -> [heads * dp, ...]: zero rows behind every head."""
-    if d == dp:
-        return w
-    out = w.new_zeros(heads, dp, *w.shape[1:])
-    out[:, :d] = w.view(heads, d, *w.shape[1:])
-    return out.view(heads * dp, *w.shape[1:])
+    layers: List = field(default_factory=list)    # LayeredLayer, or lists of Sublayers
 
 
 def build_layered_weights(cfg: ModelConfig, layout: ParallelLayout, src: WeightSource, dtype: torch.dtype) -> LayeredWeights:
@@ -87,90 +86,112 @@ def build_layered_weights(cfg: ModelConfig, layout: ParallelLayout, src: WeightS
     Kp = pad_to(D, K_ALIGN)
     w = LayeredWeights()
     w.embed = src.get("embed", (V, D)).to(dtype).contiguous()
-    w.final_norm = src.get("final.norm", (D,), "norm").float().contiguous()
-    w.lm_head = _pad_cols(src.get("head", (V, D)).to(dtype), Kp).contiguous()
-    for i, spec in enumerate(cfg.layer_specs):
-        m, f, p = spec.mixer, spec.mlp, f"l{i}.mix."
-        lw = LayeredLayer(spec=spec, norm=src.get(f"l{i}.norm1", (D,), "norm").float().contiguous())
-        parts: List[Tuple[str, torch.Tensor]] = []
-        if m.recurrent:
-            n, H, d, dp = m.heads * m.dim, m.heads, m.dim, m.dim_p
-            parts += [(x, _head_rows(src.get(p + x, (n, D)), H, d, dp)) for x in ("r", "k", "v", "g", "a")]
-            parts.append(("low", src.get(p + "w1", (m.decay_rank, D))))
-            vec = lambda name, kind: _head_rows(src.get(p + name, (n,), kind).float(), H, d, dp).contiguous()   # noqa: E731
-            lw.delta = delta.DeltaParams(w0=vec("w0", "bias"), ab=vec("a.b", "bias"), norm_w=vec("norm", "norm"), heads=H,
-                                         dim=d, dim_p=dp, decay_scale=DECAY_SCALE, eps=cfg.rms_eps)
-            w2 = _head_rows(src.get(p + "w2", (n, m.decay_rank)), H, d, dp)
-            lw.w_decay = _pad_cols(w2.to(dtype), pad_to(m.decay_rank, K_ALIGN)).contiguous()
-            o = src.get(p + "o", (D, n))
-            heads_o, d_o, dp_o = H, d, dp
-        else:
-            H, G = m.heads, m.kv_heads
-            parts += [("q", _head_rows(src.get(p + "q", (H * m.dim, D)), H, m.dim, m.dim_p)),
-                      ("k", _head_rows(src.get(p + "k", (G * m.dim, D)), G, m.dim, m.dim_p)),
-                      ("v", _head_rows(src.get(p + "v", (G * m.vdim, D)), G, m.vdim, m.vdim_p))]
-            talk = src.get(p + "talk", (H, H)).float().contiguous() if m.talking else None
-            lw.talk = talking.TalkParams(heads=H, kv_heads=G, dim_p=m.dim_p, vdim_p=m.vdim_p, scale=m.scale, chunk=m.chunk,
-                                         sink=m.sink, talk=talk)
-            o = src.get(p + "o", (D, H * m.vdim))
-            heads_o, d_o, dp_o = H, m.vdim, m.vdim_p
-        o = _head_rows(o.t().contiguous(), heads_o, d_o, dp_o).t()                  # [D, heads * dp]: zero columns
-        lw.mix_cols = heads_o * dp_o
-        lw.mix_p = pad_to(lw.mix_cols, K_ALIGN)
-        outs = [_pad_cols(o, lw.mix_p)]
-        q = f"l{i}.mlp."
-        ff, prefix = (f.ff, q) if f.kind == "dense" else (f.shared_ff, q + "shared.") if f.kind == "moe" else (0, "")
-        if f.kind == "moe":
-            parts.append(("router", src.get(q + "router", (f.experts, D))))
-            if ff:
-                parts.append(("gate1", src.get(prefix + "sg", (1, D))))
-            Fp = pad_to(f.ff, K_ALIGN)
-            w13, wd = [], []
-            for e in range(f.experts):
-                ep = f"{q}e{e}."
-                gu = [_pad_rows(src.get(ep + x, (f.ff, D)).to(dtype), Fp) for x in ("gate", "up")]
-                w13.append(_pad_cols(torch.cat(gu, 0), Kp))
-                wd.append(_pad_cols(src.get(ep + "down", (D, f.ff)).to(dtype), Fp))
-            lw.experts = ExpertWeights(w13=torch.stack(w13), w2=torch.stack(wd), activation=f.activation, act_limit=f.limit)
-        if ff:
-            lw.ff_p = pad_to(ff, K_ALIGN)
-            parts += [(x, _pad_rows(src.get(prefix + x, (ff, D)), lw.ff_p)) for x in ("gate", "up")]
-            outs.append(_pad_cols(src.get(prefix + "down", (D, ff)), lw.ff_p))
-        row, stack = 0, []
-        for name, t in parts:
-            lw.seg[name] = (row, t.shape[0])
-            stack.append(_pad_rows(t.to(dtype), pad_to(t.shape[0], 8)))
-            row += stack[-1].shape[0]
-        lw.w_in = _pad_cols(torch.cat(stack, 0), Kp).contiguous()
-        lw.w_out = torch.cat([t.to(dtype) for t in outs], 1).contiguous()
-        w.layers.append(lw)
+    w.final_norm = (_norm(src, "final.norm", cfg) if cfg.sandwich
+                    else src.get("final.norm", (D,), "norm").float().contiguous())
+    w.lm_head = pad_cols(src.get("head", (V, D)).to(dtype), Kp).contiguous()
+    block = _build_sandwich if cfg.sandwich else _build_parallel
+    w.layers = [block(cfg, spec, f"l{i}.", src, dtype) for i, spec in enumerate(cfg.layer_specs)]
     return w
+
+
+def _norm(src: WeightSource, name: str, cfg: ModelConfig) -> residual.Norm:
+    D = cfg.hidden_size
+
+    def vec(n, kind):
+        return torch.nn.functional.pad(src.get(n, (D,), kind).float(), (0, pad_to(D, 4) - D)).contiguous()
+    return residual.Norm(vec(name, "norm"), vec(name + ".b", "bias") if cfg.layer_norm else None, cfg.layer_norm)
+
+
+def _build_sandwich(cfg: ModelConfig, spec: LayerSpec, p: str, src: WeightSource, dtype: torch.dtype) -> List[Sublayer]:
+    D, f = cfg.hidden_size, spec.mlp
+    Kp, W4 = pad_to(D, K_ALIGN), pad_to(D, 4)
+    if f.kind not in ("none", "dense") or (f.kind == "dense" and f.activation != "relu2"):
+        raise NotImplementedError("sandwich blocks carry squared-ReLU feed-forwards")
+    prefixes = [p + "mix."] if spec.second is None else [p + "mix.left.", p + "mix.right."]
+    mixers = [build_mixer(m, q, src, cfg, dtype, i) for i, (m, q) in enumerate(zip(spec.mixers, prefixes))]
+    out = []
+    for n in (1, 2) if f.kind == "dense" else (1,):
+        s = Sublayer(_norm(src, f"{p}norm{n}", cfg), _norm(src, f"{p}norm{n}b", cfg), None, [])
+        if cfg.canon_taps:
+            s.canon_part = f"canon{n}"
+            taps = src.get(f"{p}canon{n}", (D, cfg.canon_taps)).float()
+            s.canon_w = pad_rows(taps, W4).t().contiguous()
+        if n == 1:
+            s.mixers = mixers
+            s.w_in = stack_parts([(m.seg, name, t) for m in mixers for name, t in m.parts], Kp, dtype)
+            s.w_out = [pad_cols(m.o.to(dtype), pad_to(m.cols, K_ALIGN)).contiguous() for m in mixers]
+            for m in mixers:
+                m.parts, m.o = [], None
+            if spec.second is not None:
+                s.branch_w = tuple(torch.nn.functional.pad(src.get(q + "out", (D,), "norm").float(), (0, W4 - D)).contiguous()
+                                   for q in prefixes)
+        else:
+            s.ff = f.ff
+            s.w_in = pad_cols(pad_rows(src.get(p + "mlp.up", (f.ff, D)).to(dtype), pad_to(f.ff, 8)), Kp).contiguous()
+            s.w_out = [pad_cols(src.get(p + "mlp.down", (D, f.ff)).to(dtype), pad_to(f.ff, K_ALIGN)).contiguous()]
+        out.append(s)
+    return out
+
+
+def _build_parallel(cfg: ModelConfig, spec: LayerSpec, p: str, src: WeightSource, dtype: torch.dtype) -> LayeredLayer:
+    D, f = cfg.hidden_size, spec.mlp
+    Kp = pad_to(D, K_ALIGN)
+    lw = LayeredLayer(spec=spec, norm=src.get(p + "norm1", (D,), "norm").float().contiguous())
+    mx = lw.mixer = build_mixer(spec.mixer, p + "mix.", src, cfg, dtype)
+    parts = [(mx.seg, name, t) for name, t in mx.parts]
+    lw.mix_p = pad_to(mx.cols, K_ALIGN)
+    outs = [pad_cols(mx.o, lw.mix_p)]
+    mx.parts, mx.o = [], None
+    q = p + "mlp."
+    ff, prefix = (f.ff, q) if f.kind == "dense" else (f.shared_ff, q + "shared.") if f.kind == "moe" else (0, "")
+    if f.kind == "moe":
+        parts.append((lw.seg, "router", src.get(q + "router", (f.experts, D))))
+        if ff:
+            parts.append((lw.seg, "gate1", src.get(prefix + "sg", (1, D))))
+        Fp = pad_to(f.ff, K_ALIGN)
+        w13, wd = [], []
+        for e in range(f.experts):
+            ep = f"{q}e{e}."
+            gu = [pad_rows(src.get(ep + x, (f.ff, D)).to(dtype), Fp) for x in ("gate", "up")]
+            w13.append(pad_cols(torch.cat(gu, 0), Kp))
+            wd.append(pad_cols(src.get(ep + "down", (D, f.ff)).to(dtype), Fp))
+        lw.experts = ExpertWeights(w13=torch.stack(w13), w2=torch.stack(wd), activation=f.activation, act_limit=f.limit)
+    if ff:
+        lw.ff_p = pad_to(ff, K_ALIGN)
+        parts += [(lw.seg, x, pad_rows(src.get(prefix + x, (ff, D)), lw.ff_p)) for x in ("gate", "up")]
+        outs.append(pad_cols(src.get(prefix + "down", (D, ff)), lw.ff_p))
+    lw.w_in = stack_parts(parts, Kp, dtype)
+    lw.w_out = torch.cat([t.to(dtype) for t in outs], 1).contiguous()
+    return lw
 
 
 def layered_tensor_specs(cfg: ModelConfig) -> List[Tuple[str, Tuple[int, ...], str, int]]:
     """(name, shape, init kind, layer) of every checkpoint tensor (layer -1: embedding, final norm, head)."""
     D, V = cfg.hidden_size, cfg.vocab_size
-    out = [("embed", (V, D), "normal", -1), ("final.norm", (D,), "norm", -1), ("head", (V, D), "normal", -1)]
+
+    def norm(name, l):
+        return [(name, (D,), "norm", l)] + ([(name + ".b", (D,), "bias", l)] if cfg.layer_norm else [])
+    out = [("embed", (V, D), "normal", -1), *norm("final.norm", -1), ("head", (V, D), "normal", -1)]
     for i, s in enumerate(cfg.layer_specs):
-        m, f, p, q = s.mixer, s.mlp, f"l{i}.mix.", f"l{i}.mlp."
-        out.append((f"l{i}.norm1", (D,), "norm", i))
-        if m.recurrent:
-            n = m.heads * m.dim
-            out += [(p + x, (n, D), "normal", i) for x in ("r", "k", "v", "g", "a")]
-            out += [(p + "w1", (m.decay_rank, D), "normal", i), (p + "w2", (n, m.decay_rank), "normal", i),
-                    (p + "a.b", (n,), "bias", i), (p + "w0", (n,), "bias", i), (p + "norm", (n,), "norm", i),
-                    (p + "o", (D, n), "normal", i)]
+        f, q = s.mlp, f"l{i}.mlp."
+        prefixes = [f"l{i}.mix."] if s.second is None else [f"l{i}.mix.left.", f"l{i}.mix.right."]
+        if cfg.sandwich:
+            for n in ("1", "2") if f.kind != "none" else ("1",):
+                out += norm(f"l{i}.norm{n}", i) + norm(f"l{i}.norm{n}b", i)
+                if cfg.canon_taps:
+                    out.append((f"l{i}.canon{n}", (D, cfg.canon_taps), "normal", i))
+            if s.second is not None:
+                out += [(q_ + "out", (D,), "norm", i) for q_ in prefixes]
         else:
-            out += [(p + "q", (m.heads * m.dim, D), "normal", i), (p + "k", (m.kv_heads * m.dim, D), "normal", i),
-                    (p + "v", (m.kv_heads * m.vdim, D), "normal", i), (p + "o", (D, m.heads * m.vdim), "normal", i)]
-            if m.talking:
-                out.append((p + "talk", (m.heads, m.heads), "normal", i))
+            out += norm(f"l{i}.norm1", i)
+        for m, p in zip(s.mixers, prefixes):
+            out += mixer_tensor_specs(m, p, D, i)
 
         def ff(prefix, n):
             return [(prefix + "gate", (n, D), "normal", i), (prefix + "up", (n, D), "normal", i),
                     (prefix + "down", (D, n), "normal", i)]
         if f.kind == "dense":
-            out += ff(q, f.ff)
+            out += ff(q, f.ff)[1 if f.activation == "relu2" else 0:]
         elif f.kind == "moe":
             out.append((q + "router", (f.experts, D), "normal", i))
             for e in range(f.experts):
@@ -178,19 +199,6 @@ def layered_tensor_specs(cfg: ModelConfig) -> List[Tuple[str, Tuple[int, ...], s
             if f.shared_ff:
                 out += ff(q + "shared.", f.shared_ff) + [(q + "shared.sg", (1, D), "normal", i)]
     return out
-
-
-@dataclass
-class _Plan:
-    """Device tables of one step, shared by its layers."""
-    lens: torch.Tensor                            # [T] int32: position + 1 (0 = padding row)
-    row_seq: Optional[torch.Tensor]               # [T] int32 block-table row of each token, None = identity
-    cu: Optional[torch.Tensor]                    # [nseq + 1] int32, None = one token per sequence
-    cu_host: Optional[List[int]]
-    slots: Optional[torch.Tensor]
-    has_initial: Optional[torch.Tensor]
-    ctx: Optional[List[int]] = None
-    tiles: Dict[int, Tuple] = field(default_factory=dict)      # attention chunk -> (tensor-core tiles, rows of short pieces)
 
 
 class LayeredDecoder:
@@ -207,69 +215,88 @@ class LayeredDecoder:
         self.streamer = None
         self.layer_hook = None                    # called with (layer, residual stream [T, width]) after every layer
 
-    # ------------------------------------------------------------------ step tables
-    def _plan(self, meta: AttnMeta, T: int) -> _Plan:
+    def _plan(self, meta: AttnMeta, T: int) -> StepPlan:
         if meta.mode == "decode":
-            return _Plan(meta.seqlens, None, None, None, meta.state_slots, None)
+            return StepPlan(meta.seqlens, None, None, None, meta.state_slots, None)
         dev = self.device
         cu = meta.cu_seqlens
         cu_t = torch.tensor(cu, dtype=torch.int32, device=dev)
         counts = torch.tensor([b - a for a, b in zip(cu, cu[1:])], device=dev)
         row_seq = torch.repeat_interleave(torch.arange(len(cu) - 1, dtype=torch.int32, device=dev), counts, output_size=T)
-        return _Plan((meta.positions + 1).to(torch.int32), row_seq, cu_t, list(cu), meta.state_slots, meta.state_has_initial,
-                     list(meta.ctx_lens))
+        return StepPlan((meta.positions + 1).to(torch.int32), row_seq, cu_t, list(cu), meta.state_slots, meta.state_has_initial,
+                        list(meta.ctx_lens))
 
-    def _tiles(self, plan: _Plan, chunk: int, T: int):
-        """How the rows of a prompt step split over the attention kernels: pieces of a few tokens (decoded tokens among
-        them) go row by row, the rest in 128-query tiles."""
-        if chunk not in plan.tiles:
-            cu, least = plan.cu_host, talking.PREFILL_MIN_TOKENS
-            blocks = talking.work_blocks(talking.prefill_work(cu, plan.ctx, chunk, least), T, self.device)
-            short = [t for a, b in zip(cu, cu[1:]) if b - a < least for t in range(a, b)]
-            rows = seqs = None
-            if blocks and short:
-                rows = torch.tensor(short, dtype=torch.int32, device=self.device)
-                seqs = plan.row_seq[rows.long()].contiguous()
-            elif short:
-                seqs = plan.row_seq
-            plan.tiles[chunk] = (blocks, bool(short), rows, seqs)
-        return plan.tiles[chunk]
+    def _operand(self, T: int, cols: int, cols_p: int) -> torch.Tensor:
+        """[T, cols_p] operand of an output projection whose writer fills the first ``cols`` columns."""
+        return (torch.zeros if cols != cols_p else torch.empty)(T, cols_p, dtype=self.dtype, device=self.device)
 
-    # ------------------------------------------------------------------ mixers
-    def _delta(self, l: int, lw: LayeredLayer, z, out, plan: _Plan, cache) -> None:
-        o, n = lw.seg["low"]
-        low = residual.cast_act(z[:, o:o + n], lw.w_decay.shape[1], self.dtype, tanh=True)
-        wl = gemm.rows_gemm(low, lw.w_decay)
-        if plan.slots is None:
-            raise RuntimeError("a model with recurrent layers needs AttnMeta.state_slots")
-        delta.delta_forward(z, tuple(lw.seg[x][0] for x in ("r", "k", "v", "g", "a")), wl, lw.delta, cache.state.layer(l),
-                            plan.slots, out, plan.cu, plan.cu_host, plan.has_initial)
-
-    def _attention(self, l: int, lw: LayeredLayer, z, out, plan: _Plan, meta: AttnMeta, cache) -> None:
-        q, k = lw.seg["q"], lw.seg["k"][0]
-        kv = cache.latent(l)
-        talking.kv_write(z[:, k:k + lw.talk.kv_row], meta.slot_mapping, kv)
-        zq = z[:, q[0]:q[0] + q[1]]
-        rows, seqs = None, plan.row_seq
-        if plan.cu is not None and z.is_cuda and talking.prefill_supported(lw.talk, kv.dtype, kv.shape[1]):
-            blocks, short, rows, seqs = self._tiles(plan, lw.talk.chunk, z.shape[0])
-            talking.attend_prefill(zq, lw.talk, kv, meta.block_table, out, blocks)
-            if not short:
-                return
-        talking.attend_rows(zq, lw.talk, kv, meta.block_table, plan.lens, out, seqs, rows)
-
-    # ------------------------------------------------------------------ forward
     def forward(self, ids: torch.Tensor, meta: AttnMeta, cache) -> torch.Tensor:
         """ids [T] -> fp32 logits [len(logit_rows) or T, vocab]."""
+        plan = self._plan(meta, ids.shape[0])
+        x = torch.empty(ids.shape[0], pad_to(self.cfg.hidden_size, 4), dtype=torch.float32, device=self.device)
+        y = (self._sandwich if self.cfg.sandwich else self._parallel)(x, ids.to(torch.int32), plan, meta, cache)
+        with self.timer.timed("lm_head"):
+            return gemm.rows_gemm(y, self.w.lm_head)
+
+    # ------------------------------------------------------------------ sandwich blocks
+    def _enter(self, x, s: Sublayer, l: int, plan: StepPlan, cache, pending) -> torch.Tensor:
+        """What a sublayer reads: the previous sublayer's output joins the residual stream, norm, input convolution."""
+        D, eps = self.cfg.hidden_size, self.cfg.rms_eps
+        args = (x, s.norm, eps, D, self.width_p, self.dtype)
+        if s.canon_w is None:
+            return residual.sandwich_norm(*args, **pending)
+        hist = cache.state.layer(l, s.canon_part)
+        if plan.cu is None:
+            return residual.sandwich_norm(*args, **pending, canon=residual.Canon(s.canon_w, hist, plan.slots))
+        h = residual.sandwich_norm(*args, **pending, raw=True)
+        y = torch.empty(x.shape[0], self.width_p, dtype=self.dtype, device=x.device)
+        return conv.causal_conv(h, s.canon_w, hist, plan.slots, y, "residual", plan.cu, plan.cu_host, plan.row_seq, plan.has_initial)
+
+    def _sandwich(self, x, ids, plan: StepPlan, meta: AttnMeta, cache) -> torch.Tensor:
         cfg, tm, w = self.cfg, self.timer, self.w
-        T, D = ids.shape[0], cfg.hidden_size
-        dev, dt = self.device, self.dtype
-        plan = self._plan(meta, T)
-        x = torch.empty(T, pad_to(D, 4), dtype=torch.float32, device=dev)
-        first = dict(ids=ids.to(torch.int32), embed=w.embed, embed_scale=cfg.embed_scale)
+        T, D = x.shape[0], cfg.hidden_size
+        if plan.slots is None and cfg.has_state:
+            raise RuntimeError("a model with per-sequence state needs AttnMeta.state_slots")
+        pending = dict(ids=ids, embed=w.embed, embed_scale=cfg.embed_scale)
+        for l, layer in enumerate(w.layers):
+            for i, s in enumerate(layer):
+                with tm.timed("norm", l):
+                    y = self._enter(x, s, l, plan, cache, pending)
+                if self.layer_hook is not None and l and not i:
+                    self.layer_hook(l - 1, x[:, :D])
+                with tm.timed("proj_in", l):
+                    z = gemm.rows_gemm(y, s.w_in)
+                if s.mixers:
+                    operands = []
+                    with tm.timed("mixer_" + meta.mode, l):
+                        for m, wo in zip(s.mixers, s.w_out):
+                            operands.append(self._operand(T, m.cols, wo.shape[1]))
+                            m.run(l, z, operands[-1][:, :m.cols], plan, meta, cache)
+                else:
+                    with tm.timed("act", l):
+                        operands = [residual.cast_act(z[:, :s.ff], s.w_out[0].shape[1], self.dtype, "relu2")]
+                with tm.timed("proj_out", l):
+                    outs = [gemm.rows_gemm(o, wo) for o, wo in zip(operands, s.w_out)]
+                pending = dict(add=outs[0], post=s.post)
+                if len(outs) > 1:
+                    pending.update(add2=outs[1], branch_w=s.branch_w)
+        args = (x, w.final_norm, cfg.rms_eps, D, self.width_p, self.dtype)
+        if self.layer_hook is not None:           # the last sublayer's output is only summed inside the final norm
+            residual.sandwich_norm(*args, **pending)
+            pending = {}
+            self.layer_hook(len(w.layers) - 1, x[:, :D])
+        return residual.sandwich_norm(*args, **pending, keep=False,
+                                      rows=meta.logit_rows.long() if meta.logit_rows is not None else None)
+
+    # ------------------------------------------------------------------ parallel blocks
+    def _parallel(self, x, ids, plan: StepPlan, meta: AttnMeta, cache) -> torch.Tensor:
+        cfg, tm, w = self.cfg, self.timer, self.w
+        T, D = x.shape[0], cfg.hidden_size
+        dt = self.dtype
+        first = dict(ids=ids, embed=w.embed, embed_scale=cfg.embed_scale)
         add = routed = pos = None
         for l, lw in enumerate(w.layers):
-            f = lw.spec.mlp
+            f, mx = lw.spec.mlp, lw.mixer
             with tm.timed("norm", l):
                 h = residual.residual_norm(x, lw.norm, cfg.rms_eps, D, self.width_p, dt, add=add, routed=routed, pos=pos,
                                            **first)
@@ -278,13 +305,9 @@ class LayeredDecoder:
             first = {}
             with tm.timed("proj_in", l):
                 z = gemm.rows_gemm(h, lw.w_in)
-            padded = lw.mix_cols != lw.mix_p
-            cat = (torch.zeros if padded else torch.empty)(T, lw.mix_p + lw.ff_p, dtype=dt, device=dev)
+            cat = self._operand(T, mx.cols if mx.cols != lw.mix_p else lw.mix_p + lw.ff_p, lw.mix_p + lw.ff_p)
             with tm.timed("mixer_" + meta.mode, l):
-                if lw.delta is not None:
-                    self._delta(l, lw, z, cat[:, :lw.mix_cols], plan, cache)
-                else:
-                    self._attention(l, lw, z, cat[:, :lw.mix_cols], plan, meta, cache)
+                mx.run(l, z, cat[:, :mx.cols], plan, meta, cache)
             if lw.ff_p:
                 g0, s = lw.seg["gate"][0], lw.seg.get("gate1")
                 with tm.timed("glu", l):
@@ -303,7 +326,5 @@ class LayeredDecoder:
             residual.residual_norm(x, w.final_norm, cfg.rms_eps, D, self.width_p, dt, add=add, routed=routed, pos=pos)
             add = routed = pos = None
             self.layer_hook(len(w.layers) - 1, x[:, :D])
-        y = residual.residual_norm(x, w.final_norm, cfg.rms_eps, D, self.width_p, dt, add=add, routed=routed, pos=pos,
-                                   rows=meta.logit_rows.long() if meta.logit_rows is not None else None, keep=False)
-        with tm.timed("lm_head"):
-            return gemm.rows_gemm(y, w.lm_head)
+        return residual.residual_norm(x, w.final_norm, cfg.rms_eps, D, self.width_p, dt, add=add, routed=routed, pos=pos,
+                                      rows=meta.logit_rows.long() if meta.logit_rows is not None else None, keep=False)

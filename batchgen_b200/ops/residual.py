@@ -1,5 +1,6 @@
 """Row operators of models with an fp32 residual stream: residual sum + RMS norm (with the embedding or the sublayers'
-outputs folded in), gated activations, operand casts, expert-row gather.
+outputs folded in), the same step of blocks with a norm before and after each sublayer, gated activations, operand casts,
+expert-row gather.
 
 CUDA tensors go to ``csrc/residual.cu``; CPU tensors to plain fp32 torch.  Operand dtype (norm output, activations) is
 bf16, or fp32 for the 32-bit form of a model.
@@ -8,6 +9,7 @@ from __future__ import annotations
 
 import ctypes
 import math
+from dataclasses import dataclass
 from typing import Optional, Tuple
 
 import torch
@@ -16,6 +18,7 @@ from . import _ext
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 GLU_KINDS = {"gelu_tanh": 0, "swiglu_oai": 1}
+CAST_KINDS = {"none": 0, "tanh": 1, "relu2": 2}
 
 
 def _i(v) -> ctypes.c_int:
@@ -105,18 +108,98 @@ def glu(z: torch.Tensor, F: int, kind: str, limit: float = 0.0, row_scale: Optio
     return out
 
 
-def cast_act(x: torch.Tensor, cols: int, dtype: torch.dtype, tanh: bool = False) -> torch.Tensor:
-    """fp32 columns (a view is fine) -> [T, cols] of ``dtype``, zero past x's width; optional tanh."""
+def cast_act(x: torch.Tensor, cols: int, dtype: torch.dtype, act: str = "none") -> torch.Tensor:
+    """fp32 columns (a view is fine) -> [T, cols] of ``dtype``, zero past x's width; ``act`` none, tanh or relu2 (the square
+    of the positive part)."""
     if not x.is_cuda:
         y = torch.zeros(x.shape[0], cols, dtype=dtype)
-        y[:, : x.shape[1]] = (torch.tanh(x) if tanh else x).to(dtype)
+        y[:, : x.shape[1]] = (torch.tanh(x) if act == "tanh" else x.clamp_min(0) ** 2 if act == "relu2" else x).to(dtype)
         return y
     assert x.dtype == torch.float32 and x.stride(1) == 1
     out = torch.empty(x.shape[0], cols, dtype=dtype, device=x.device)
-    rc = _ext.lib().bg_cast_act(_i(_DT[dtype]), _i(tanh), _ext.ptr(x), _i(x.stride(0)), _ext.ptr(out), _i(cols),
+    rc = _ext.lib().bg_cast_act(_i(_DT[dtype]), _i(CAST_KINDS[act]), _ext.ptr(x), _i(x.stride(0)), _ext.ptr(out), _i(cols),
                                 _i(x.shape[0]), _i(x.shape[1]), _ext.stream())
     _ext.check(rc, "bg_cast_act")
     return out
+
+
+@dataclass
+class Norm:
+    """A norm over the model width: (x - mean) / sqrt(variance + eps) * w + b when ``center``, else x / sqrt(mean square +
+    eps) * w (+ b).  Vectors are fp32, padded with zeros to a multiple of 4."""
+    w: torch.Tensor
+    b: Optional[torch.Tensor] = None
+    center: bool = False
+
+    def ref(self, x: torch.Tensor, eps: float, width: int) -> torch.Tensor:
+        if self.center:
+            x = x - x.mean(-1, keepdim=True)
+        y = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * self.w[:width]
+        return y if self.b is None else y + self.b[:width]
+
+
+@dataclass
+class Canon:
+    """Input convolution of a decode step, folded into the norm: y = h + conv(h) over this token and the stored inputs."""
+    w: torch.Tensor                 # [taps, width rounded up to 4] fp32
+    hist: torch.Tensor              # [slots, (taps - 1) * same] fp32 (strided view of the state pool), updated
+    slots: torch.Tensor             # [T] int32, < 0: no history, none kept
+
+
+def sandwich_norm(x: torch.Tensor, norm: Norm, eps: float, width: int, out_cols: int, dtype: torch.dtype,
+                  add: Optional[torch.Tensor] = None, add2: Optional[torch.Tensor] = None,
+                  branch_w: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, post: Optional[Norm] = None,
+                  ids: Optional[torch.Tensor] = None, embed: Optional[torch.Tensor] = None, embed_scale: float = 1.0,
+                  rows: Optional[torch.Tensor] = None, keep: bool = True, raw: bool = False,
+                  canon: Optional[Canon] = None) -> torch.Tensor:
+    """x [T, >= width] fp32 += post(sublayer output), then norm(x) as [R, out_cols] of ``dtype`` with zero columns past
+    ``width``, or with ``raw`` as fp32 [R, width rounded up to 4].  The sublayer's output is ``add`` [T, width] fp32, or with
+    ``add2`` half the sum of both, each RMS-normed with its weight of ``branch_w``; ``ids``: x = embed[ids] * embed_scale
+    instead.  ``canon`` (one token per sequence) applies the input convolution to the result.  ``rows`` (int64) picks rows of
+    x; ``keep=False`` leaves x as it was."""
+    R = x.shape[0] if rows is None else rows.shape[0]
+    W4 = pad_to(width, 4)
+    if not x.is_cuda:
+        r = rows.long() if rows is not None else torch.arange(x.shape[0])
+        cur = x[r, :width].clone()
+        if ids is not None:
+            cur = embed[ids[r].long()].float() * embed_scale
+        if add is not None:
+            s = add[r, :width]
+            if add2 is not None:
+                s = 0.5 * sum(t / torch.sqrt((t * t).mean(-1, keepdim=True) + eps) * g[:width]
+                              for t, g in zip((s, add2[r, :width]), branch_w))
+            cur = cur + post.ref(s, eps, width)
+        if keep:
+            x[r, :width] = cur
+        h = torch.nn.functional.pad(norm.ref(cur, eps, width), (0, W4 - width))
+        if raw:
+            return h
+        if canon is not None:
+            from .conv import causal_conv
+            return causal_conv(h, canon.w, canon.hist, canon.slots, torch.zeros(R, out_cols, dtype=dtype), "residual")
+        y = torch.zeros(R, out_cols, dtype=dtype)
+        y[:, :width] = h[:, :width].to(dtype)
+        return y
+    y = torch.empty(R, W4 if raw else out_cols, dtype=torch.float32 if raw else dtype, device=x.device)
+    for t in (add, add2):
+        assert t is None or (t.dtype == torch.float32 and t.stride(1) == 1)
+    assert x.dtype == torch.float32 and (embed is None or embed.dtype == dtype) and (add is None) == (post is None)
+    assert (ids is None or ids.dtype == torch.int32) and (rows is None or rows.dtype == torch.int64)
+    assert canon is None or (rows is None and not raw and canon.slots.dtype == torch.int32 and canon.hist.stride(1) == 1)
+    P = lambda n: (_ext.ptr(n.w if n is not None else None), _ext.ptr(n.b if n is not None else None))   # noqa: E731
+    rc = _ext.lib().bg_sandwich_norm(
+        _i(_DT[dtype]), _ext.ptr(x), _i(x.stride(0)), _ext.ptr(rows), _ext.ptr(ids), _ext.ptr(embed),
+        _i(embed.stride(0) if embed is not None else 0), ctypes.c_float(embed_scale),
+        _i(embed.shape[0] if embed is not None else 0), _ext.ptr(add), _i(add.stride(0) if add is not None else 0),
+        _ext.ptr(add2), _i(add2.stride(0) if add2 is not None else 0), _ext.ptr(branch_w[0] if add2 is not None else None),
+        _ext.ptr(branch_w[1] if add2 is not None else None), *P(post), _i(post is not None and post.center), *P(norm),
+        _i(norm.center), _ext.ptr(y), _i(y.shape[1]), _i(raw), _ext.ptr(canon.w if canon else None),
+        _ext.ptr(canon.hist if canon else None), ctypes.c_longlong(canon.hist.stride(0) if canon else 0),
+        _ext.ptr(canon.slots if canon else None), _i(canon.w.shape[0] if canon else 0), _i(R), _i(width), ctypes.c_float(eps),
+        _i(keep), _ext.stream())
+    _ext.check(rc, "bg_sandwich_norm")
+    return y
 
 
 def moe_gather(x: torch.Tensor, pos: torch.Tensor, w: torch.Tensor, rows: int) -> Tuple[torch.Tensor, torch.Tensor]:

@@ -1,5 +1,5 @@
-"""Paged grouped-query attention whose heads' scores are mixed before the softmax, with chunked visibility and a
-zero-score sink: cache rows and one query row per CTA for decode and short pieces (``csrc/talking_attn.cu``), tensor-core
+"""Paged grouped-query attention for layer-listed models.  Optional parts: heads' scores mixed before the softmax, chunked
+visibility, a zero-score sink, rotary positions on queries and keys, a sigmoid gate per head on the output.  Cache rows and one query row per CTA for decode and short pieces (``csrc/talking_attn.cu``), tensor-core
 flash attention over mixed queries for long pieces of prompts (``csrc/talking_prefill.cu``).
 """
 from __future__ import annotations
@@ -12,6 +12,7 @@ from typing import List, Optional, Sequence, Tuple
 import torch
 
 from . import _ext
+from .conv import rotate_ref
 from .residual import _DT, _i
 
 
@@ -32,11 +33,16 @@ class TalkParams:
         return self.kv_heads * (self.dim_p + self.vdim_p)
 
 
-def kv_write(kv: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor) -> None:
+def kv_write(kv: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, p: Optional[TalkParams] = None,
+             rope: Optional[torch.Tensor] = None) -> None:
     """cache[slot] = kv (fp32 columns: keys of all heads, values of all heads); cache [pages, page, row] (strided pages);
-    slots [T] int64, < 0 writes nothing."""
+    slots [T] int64, < 0 writes nothing.  ``rope`` [T, dims] (``conv.Rotary.table``) turns the keys of ``p``'s heads."""
     P, page, row = cache.shape
     if not kv.is_cuda:
+        if rope is not None:
+            n = p.kv_heads * p.dim_p
+            k = rotate_ref(kv[:, :n].view(-1, p.kv_heads, p.dim_p), rope).reshape(-1, n)
+            kv = torch.cat([k, kv[:, n:row]], 1)
         live = slots >= 0
         s = slots[live]
         cache[s // page, s % page] = kv[live, :row].to(cache.dtype)
@@ -44,12 +50,15 @@ def kv_write(kv: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor) -> None
     assert kv.dtype == torch.float32 and kv.stride(1) == 1 and cache.stride(1) == row and cache.stride(2) == 1
     assert slots.dtype == torch.int64
     rc = _ext.lib().bg_talk_kv_write(_i(_DT[cache.dtype]), _ext.ptr(kv), _i(kv.stride(0)), _ext.ptr(slots), _ext.ptr(cache),
-                                     ctypes.c_longlong(cache.stride(0)), _i(page), _i(row), _i(kv.shape[0]), _ext.stream())
+                                     ctypes.c_longlong(cache.stride(0)), _i(page), _i(row), _i(kv.shape[0]), _ext.ptr(rope),
+                                     _i(rope.shape[1] // 2 if rope is not None else 0), _i(p.kv_heads if p else 1),
+                                     _i(p.dim_p if p else 0), _ext.stream())
     _ext.check(rc, "bg_talk_kv_write")
 
 
-def _rows_ref(q, p: TalkParams, cache, block_table, lens, out, row_seq):
+def _rows_ref(q, p: TalkParams, cache, block_table, lens, out, row_seq, rope, gate):
     H, G, d, dv = p.heads, p.kv_heads, p.dim_p, p.vdim_p
+    q = rotate_ref(q[:, : H * d].float().view(-1, H, d), rope).reshape(-1, H * d)
     rep = H // G
     page = cache.shape[1]
     for t in range(q.shape[0]):
@@ -71,7 +80,10 @@ def _rows_ref(q, p: TalkParams, cache, block_table, lens, out, row_seq):
             m = m.clamp_min(0)
         e = torch.exp(s - m)
         den = e.sum(-1, keepdim=True) + (torch.exp(-m) if p.sink else 0)
-        out[t, : H * dv] = torch.einsum("hj,jhv->hv", e / den, v).reshape(-1).to(out.dtype)
+        o = torch.einsum("hj,jhv->hv", e / den, v)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[t, :H].float()).unsqueeze(-1)
+        out[t, : H * dv] = o.reshape(-1).to(out.dtype)
 
 
 def _splits(rows: int, keys: int, sms: int) -> int:
@@ -88,14 +100,15 @@ def _splits(rows: int, keys: int, sms: int) -> int:
 
 def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table: torch.Tensor, lens: torch.Tensor,
                 out: torch.Tensor, row_seq: Optional[torch.Tensor] = None, row_ids: Optional[torch.Tensor] = None,
-                num_splits: int = 0) -> None:
+                num_splits: int = 0, rope: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """q [T, >= H * dim_p] fp32 -> out [T, >= H * vdim_p] (operand dtype, a column view is fine).  ``lens`` [T] int32 =
     position + 1 of each row (0: no query, zero output); ``row_seq`` [R] block-table row of each query row (None: row i);
-    ``row_ids`` [R] the rows of q to compute (None: all).  The keys are in the cache already."""
+    ``row_ids`` [R] the rows of q to compute (None: all).  ``rope`` [T, dims] turns the queries, ``gate`` [T, >= H] fp32 scales
+    each head's output by its sigmoid.  The keys are in the cache already."""
     if not q.is_cuda:
         if row_ids is not None:
             raise NotImplementedError("row subsets are a device path")
-        return _rows_ref(q, p, cache, block_table, lens, out, row_seq)
+        return _rows_ref(q, p, cache, block_table, lens, out, row_seq, rope, gate)
     P, page, row = cache.shape
     R = q.shape[0] if row_ids is None else row_ids.shape[0]
     assert q.dtype == torch.float32 and q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == cache.dtype
@@ -115,7 +128,8 @@ def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table
         ctypes.c_longlong(cache.stride(0)), _i(page), _i(row), _ext.ptr(block_table), _i(block_table.stride(0)),
         _ext.ptr(row_seq), _ext.ptr(row_ids), _ext.ptr(lens), _ext.ptr(out), _i(out.stride(0)), _ext.ptr(po),
         _ext.ptr(pml), _i(R), _i(H), _i(p.kv_heads), _i(p.dim_p), _i(p.vdim_p), _i(p.chunk), _i(p.sink),
-        ctypes.c_float(p.scale), _i(num_splits), _ext.stream())
+        ctypes.c_float(p.scale), _i(num_splits), _ext.ptr(rope), _i(rope.shape[1] // 2 if rope is not None else 0),
+        _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0), _ext.stream())
     if rc in (-1, -3):
         raise _ext.KernelError(f"attend_rows: heads {H}/{p.kv_heads}, widths {p.dim_p}/{p.vdim_p} are outside the kernel's "
                                "contract (shared memory of one CTA, 1,024 head-column items)")
@@ -160,23 +174,34 @@ def work_blocks(work: List[Tuple[int, int, int, int]], rows: int, device) -> Lis
 
 
 def attend_prefill(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table: torch.Tensor, out: torch.Tensor,
-                   blocks: List[Tuple[int, int, torch.Tensor]]) -> None:
+                   blocks: List[Tuple[int, int, torch.Tensor]], rope: Optional[torch.Tensor] = None,
+                   gate: Optional[torch.Tensor] = None) -> None:
     """CUDA, bf16 cache: q [T, >= H * dim_p] fp32 -> out [T, >= H * vdim_p] for the rows covered by ``blocks``
-    (``work_blocks``).  The keys of every query are in the cache already."""
+    (``work_blocks``); ``rope`` and ``gate`` as for ``attend_rows``.  The keys of every query are in the cache already.
+
+    Mixed heads contract over a token's whole key block, plain heads over their own key head's columns."""
     P, page, row = cache.shape
     H, G = p.heads, p.kv_heads
-    kc = -(-G * p.dim_p // 64) * 64
+    plain = p.talk is None
+    assert plain or rope is None, "mixed heads with rotary queries are not covered"
+    kc = -(-(p.dim_p if plain else G * p.dim_p) // 64) * 64
     assert q.dtype == torch.float32 and q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == cache.dtype == torch.bfloat16
     assert row == p.kv_row and cache.stride(1) == row and block_table.dtype == torch.int32
     L = _ext.lib()
     for lo, n, work in blocks:
         qf = torch.empty(n, H, kc, dtype=torch.bfloat16, device=q.device)
-        rc = L.bg_talk_fold(_ext.ptr(q[lo:]), _i(q.stride(0)), _ext.ptr(p.talk), _ext.ptr(qf), _i(n), _i(H), _i(G),
-                            _i(p.dim_p), _i(kc), ctypes.c_float(p.scale), _ext.stream())
+        if plain:
+            rc = L.bg_talk_turn(_ext.ptr(q[lo:]), _i(q.stride(0)), _ext.ptr(rope[lo:] if rope is not None else None),
+                                _i(rope.shape[1] // 2 if rope is not None else 0), _ext.ptr(qf), _i(n), _i(H), _i(p.dim_p),
+                                _i(kc), ctypes.c_float(p.scale), _ext.stream())
+        else:
+            rc = L.bg_talk_fold(_ext.ptr(q[lo:]), _i(q.stride(0)), _ext.ptr(p.talk), _ext.ptr(qf), _i(n), _i(H), _i(G),
+                                _i(p.dim_p), _i(kc), ctypes.c_float(p.scale), _ext.stream())
         _ext.check(rc, "bg_talk_fold")
         rc = L.bg_talk_prefill(
             _ext.ptr(qf), _ext.ptr(cache), ctypes.c_longlong(cache.stride(0)), _i(P), _i(page), _i(row),
             _ext.ptr(block_table), _i(block_table.stride(0)), _i(block_table.shape[1]), _ext.ptr(work), _i(work.shape[0]),
             _i(n), _i(lo), _ext.ptr(out), _i(out.stride(0)), _i(H), _i(G), _i(p.dim_p), _i(p.vdim_p), _i(kc), _i(p.chunk),
-            _i(p.sink), _ext.ptr(_ext.status_word(q.device)), _ext.stream())
+            _i(p.sink), _i(p.dim_p if plain else 0), _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0),
+            _ext.ptr(_ext.status_word(q.device)), _ext.stream())
         _ext.check(rc, "bg_talk_prefill")

@@ -110,9 +110,9 @@ class PagedKVCache:
         self.layer_rows: Dict[int, Tuple[int, int]] = {}
         off = 0
         for l, spec in enumerate(cfg.layer_specs):
-            if spec.mixer.kv_row:
-                self.layer_rows[l] = (off, spec.mixer.kv_row)
-                off += spec.mixer.kv_row
+            if spec.kv_row:
+                self.layer_rows[l] = (off, spec.kv_row)
+                off += spec.kv_row
         kv_layers = [] if cfg.is_v4 else [0] if cfg.is_layered else [l for l in range(cfg.num_layers) if not cfg.layer_is_kda(l)]
         self.kv_index = {l: i for i, l in enumerate(kv_layers)}
         self.kv = torch.zeros(len(kv_layers), num_pages, page_size, self.row_dim, dtype=dtype, device=self.device,
@@ -146,9 +146,8 @@ class PagedKVCache:
             self.state = StateSlotPool(cfg, state_slots, self.device, state_heads)
         elif cfg.is_v4 and state_slots:
             self.state = V4StatePool(cfg, state_slots, self.device)
-        elif cfg.recurrent_layers and state_slots:
-            self.state = FlatStatePool([((l, "S"), cfg.layer_specs[l].mixer.state_shape) for l in cfg.recurrent_layers],
-                                       state_slots, self.device)
+        elif cfg.is_layered and cfg.has_state and state_slots:
+            self.state = FlatStatePool(cfg.layered_state_parts(), state_slots, self.device)
 
     # ---- views used by the model
     def latent(self, layer: int) -> torch.Tensor:

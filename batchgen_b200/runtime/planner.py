@@ -131,10 +131,12 @@ def layered_workspace_bytes(cfg: ModelConfig) -> int:
     routed experts' rows, and a few rows of the model width."""
     most = 0
     for s in cfg.layer_specs:
-        m, f = s.mixer, s.mlp
-        n_in = 6 * m.heads * m.dim_p if m.recurrent else (m.heads + m.kv_heads) * (m.dim_p + m.vdim_p)
+        f = s.mlp
+        n_in = sum(m.in_columns for m in s.mixers)
+        if any(m.recurrent and m.kind != "general_delta" for m in s.mixers):
+            n_in += max(4 * m.heads * (m.dim_p + m.vdim_p) for m in s.mixers if m.recurrent)    # records of the prompt scan
         n_in += 2 * (f.shared_ff if f.kind == "moe" else f.ff) + f.experts
-        n_cat = m.heads * m.vdim_p + (f.shared_ff if f.kind == "moe" else f.ff)
+        n_cat = sum(m.heads * m.vdim_p for m in s.mixers) + (f.shared_ff if f.kind == "moe" else f.ff)
         routed = f.top * (2 * cfg.hidden_size + 8 * f.ff + 2 * f.ff + 4 * cfg.hidden_size) if f.kind == "moe" else 0
         most = max(most, 4 * n_in + 2 * n_cat + routed)
     return most + 16 * cfg.hidden_size

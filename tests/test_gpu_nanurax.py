@@ -67,7 +67,7 @@ def test_glu_cast_and_gather(dtype):
     s = scale.unsqueeze(-1)
     a, u = (s * z[:, F:2 * F]).clamp(max=0.9), (s * z[:, 2 * F:]).clamp(-0.9, 0.9)
     assert _rel(out[:, :F], a * torch.sigmoid(1.702 * a) * (u + 1) * torch.sigmoid(gate)) < tol
-    c = residual.cast_act(zd[:, 3:20], 64, dtype, tanh=True)
+    c = residual.cast_act(zd[:, 3:20], 64, dtype, act="tanh")
     assert _rel(c[:, :17], torch.tanh(z[:, 3:20])) < tol and float(c[:, 17:].abs().sum()) == 0
     x = torch.randn(6, 64, generator=g).to(dtype)
     pos = torch.tensor([[4, 0], [1, -1], [2, 3], [5, 6], [-1, -1], [8, 7]], dtype=torch.int32)
