@@ -1,10 +1,13 @@
-// Row kernels of models with an fp32 residual stream and parallel blocks (mixer and feed-forward read one norm):
+// Row kernels of models with an fp32 residual stream:
 //
 //   residual_norm   x[t] += sum of the sublayers' fp32 outputs (dense rows and / or routed rows gathered by position),
 //                   or x[t] = embed[id] * scale for the first layer; y[t] = x[t] / sqrt(mean(x^2) + eps) * w
+//   sandwich_norm   the same for blocks with a norm before and after each sublayer: the sublayer's output (or half the sum of
+//                   two, each RMS-normed) passes its own norm before it joins x; optional mean subtraction and biases; in
+//                   decode the input convolution y = h + conv(h) of the next sublayer is folded in
 //   glu             gated activations (tanh-GELU, clamped SwiGLU with slope 1.702 and u + 1), with an optional factor on
 //                   the pre-activations (routing weight applied to the expert's input) and an optional sigmoid gate
-//   cast_act        out = f(x), f = tanh or identity: fp32 columns of a projection to the operand type of the next one
+//   cast_act        out = f(x), f = tanh, squared ReLU or identity: fp32 columns of a projection to the operand type of the next one
 //   moe_gather      token rows -> expert-grouped rows, one block per (token, k) pair, plus the pair's routing weight
 //
 // Activations are fp32 in, bf16 or fp32 out (`OT`); sums, norms and gates are fp32.
@@ -124,6 +127,175 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(const NormParam
   }
 }
 
+struct SandwichParams {
+  float* x;               // [T, ldx] residual stream
+  int ldx;
+  const long long* rows;  // [R] rows of x, or null
+  const int* ids;         // first layer: token ids (x is written, not read)
+  const void* embed;      // [V, lde]
+  int lde;
+  float escale;
+  int vocab;
+  const float *a, *b;     // the sublayer's output(s) [T, ld], or null
+  int lda, ldb;
+  const float *wa, *wb;   // with b: weights of the outputs' RMS norms
+  const float *w1, *b1;   // norm of the output; b1 may be null
+  int center1;
+  const float *w2, *b2;   // norm of x
+  int center2;
+  void* y;                // [R, ldy]
+  int ldy, raw;           // raw: y is fp32 and ends at D rounded up to 4
+  const float* cw;        // [taps, D4] input convolution, or null
+  float* hist;            // [slots, (taps - 1) * D4] rows of `hist_stride`
+  long long hist_stride;
+  const int* slots;
+  int taps;
+  int D;
+  float eps;
+  int keep;
+};
+
+constexpr int kWarps = kThreads / 32;
+// sum over the block; `red` holds kWarps floats and is not reused before the next barrier of the caller
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < kWarps; ++i) s += red[i];
+  return s;
+}
+
+// One block per row; thread i owns the 4-wide vectors i, i + 256, ... and keeps the first NV of them in registers: D <= 1024 NV.
+// Columns D .. D4 hold zeros (weights and biases are zero there).
+template <typename OT, int NV>
+__global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichParams p) {
+  bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
+  __shared__ float red[6][kWarps];
+  const int tid = threadIdx.x;
+  const long long t = p.rows != nullptr ? p.rows[blockIdx.x] : (long long)blockIdx.x;
+  float* xr = p.x + t * p.ldx;
+  const int D = p.D, nv = (D + 3) / 4;
+  const float inv_d = 1.0f / (float)D;
+  float4 f[NV], s[NV];
+  auto each = [&](auto fn) {
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int v = tid + n * kThreads;
+      if (v < nv) fn(n, v * 4);
+    }
+  };
+  auto ld4 = [](const float* q, int c) { return *reinterpret_cast<const float4*>(q + c); };
+  auto dot = [](const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
+  auto mask = [&](float4 v, int c) {                               // zero past D
+    if (c + 1 >= D) v.y = 0.f;
+    if (c + 2 >= D) v.z = 0.f;
+    if (c + 3 >= D) v.w = 0.f;
+    return v;
+  };
+  // mean and 1 / sqrt(variance + eps) of the vectors in v (mean 0 without centring)
+  auto moments = [&](float4 (&v)[NV], int center, float* r0, float* r1, float& mean, float& rstd) {
+    mean = 0.f;
+    if (center) {
+      float sum = 0.f;
+      each([&](int n, int) { sum += (v[n].x + v[n].y) + (v[n].z + v[n].w); });
+      mean = block_sum(sum, r0) * inv_d;
+    }
+    float sq = 0.f;
+    each([&](int n, int c) {
+      const float4 d = mask(make_float4(v[n].x - mean, v[n].y - mean, v[n].z - mean, v[n].w - mean), c);
+      sq += dot(d);
+    });
+    rstd = 1.0f / sqrtf(block_sum(sq, r1) * inv_d + p.eps);
+  };
+  auto norm4 = [&](const float4& v, float mean, float rstd, const float* w, const float* b, int c) {
+    const float4 g = ld4(w, c);
+    float4 o = make_float4((v.x - mean) * rstd * g.x, (v.y - mean) * rstd * g.y, (v.z - mean) * rstd * g.z, (v.w - mean) * rstd * g.w);
+    if (b != nullptr) {
+      const float4 a = ld4(b, c);
+      o.x += a.x; o.y += a.y; o.z += a.z; o.w += a.w;
+    }
+    return o;
+  };
+  if (p.ids != nullptr) {
+    const int id = min(max(p.ids[t], 0), p.vocab - 1);
+    const OT* er = reinterpret_cast<const OT*>(p.embed) + (size_t)id * p.lde;
+    each([&](int n, int c) {
+      f[n].x = to_f(er[c]) * p.escale;
+      f[n].y = c + 1 < D ? to_f(er[c + 1]) * p.escale : 0.f;
+      f[n].z = c + 2 < D ? to_f(er[c + 2]) * p.escale : 0.f;
+      f[n].w = c + 3 < D ? to_f(er[c + 3]) * p.escale : 0.f;
+    });
+  } else {
+    each([&](int n, int c) { f[n] = mask(ld4(xr, c), c); });
+  }
+  if (p.a != nullptr) {
+    const float* ar = p.a + t * p.lda;
+    each([&](int n, int c) { s[n] = mask(ld4(ar, c), c); });
+    if (p.b != nullptr) {
+      const float* br = p.b + t * p.ldb;
+      float4 u[NV];
+      float sa = 0.f, sb = 0.f;
+      each([&](int n, int c) {
+        u[n] = mask(ld4(br, c), c);
+        sa += dot(s[n]);
+        sb += dot(u[n]);
+      });
+      sa = warp_sum(sa);
+      sb = warp_sum(sb);
+      if ((tid & 31) == 0) { red[0][tid >> 5] = sa; red[1][tid >> 5] = sb; }
+      __syncthreads();
+      float ta = 0.f, tb = 0.f;
+#pragma unroll
+      for (int i = 0; i < kWarps; ++i) { ta += red[0][i]; tb += red[1][i]; }
+      const float ra = 0.5f / sqrtf(ta * inv_d + p.eps), rb = 0.5f / sqrtf(tb * inv_d + p.eps);
+      each([&](int n, int c) {
+        const float4 ga = ld4(p.wa, c), gb = ld4(p.wb, c);
+        s[n] = make_float4(s[n].x * ra * ga.x + u[n].x * rb * gb.x, s[n].y * ra * ga.y + u[n].y * rb * gb.y,
+                           s[n].z * ra * ga.z + u[n].z * rb * gb.z, s[n].w * ra * ga.w + u[n].w * rb * gb.w);
+      });
+    }
+    float mean, rstd;
+    moments(s, p.center1, red[2], red[3], mean, rstd);
+    each([&](int n, int c) {
+      const float4 o = norm4(s[n], mean, rstd, p.w1, p.b1, c);
+      f[n].x += o.x; f[n].y += o.y; f[n].z += o.z; f[n].w += o.w;
+    });
+  }
+  if (p.keep) each([&](int n, int c) { *reinterpret_cast<float4*>(xr + c) = f[n]; });
+  float mean, rstd;
+  moments(f, p.center2, red[4], red[5], mean, rstd);
+  OT* yr = reinterpret_cast<OT*>(p.y) + (size_t)blockIdx.x * p.ldy;
+  float* hr = reinterpret_cast<float*>(p.y) + (size_t)blockIdx.x * p.ldy;
+  const int slot = p.cw != nullptr ? p.slots[blockIdx.x] : -1;
+  const int D4 = nv * 4;
+  each([&](int n, int c) {
+    float4 h = norm4(f[n], mean, rstd, p.w2, p.b2, c);
+    if (p.cw != nullptr) {                                         // y = h + conv(h); the stored inputs move up by one
+      const float4 in = h;
+      auto tap = [&](int j, const float4& v) {
+        const float4 w = ld4(p.cw + (size_t)j * D4, c);
+        h.x = fmaf(w.x, v.x, h.x); h.y = fmaf(w.y, v.y, h.y); h.z = fmaf(w.z, v.z, h.z); h.w = fmaf(w.w, v.w, h.w);
+      };
+      if (slot >= 0) {
+        float* hs = p.hist + slot * p.hist_stride + c;
+        for (int j = 0; j + 1 < p.taps; ++j) {
+          const float4 old = *reinterpret_cast<const float4*>(hs + (size_t)j * D4);
+          tap(j, old);
+          if (j > 0) *reinterpret_cast<float4*>(hs + (size_t)(j - 1) * D4) = old;
+        }
+        if (p.taps > 1) *reinterpret_cast<float4*>(hs + (size_t)(p.taps - 2) * D4) = in;
+      }
+      tap(p.taps - 1, in);
+    }
+    if (p.raw) store4(hr + c, h);
+    else store4(yr + c, h);
+  });
+  if (!p.raw)
+    for (int c = D4 + tid * 4; c < p.ldy; c += kThreads * 4) store4(yr + c, make_float4(0.f, 0.f, 0.f, 0.f));
+}
+
 __device__ __forceinline__ float sigmoid_acc(float x) { return 1.0f / (1.0f + expf(-x)); }
 
 template <int KIND>
@@ -175,6 +347,7 @@ cast_act_kernel(const float* __restrict__ x, int ldx, OT* __restrict__ out, int 
   if (c < N) {
     v = x[(size_t)t * ldx + c];
     if (KIND == 1) v = tanhf(v);
+    if (KIND == 2) { v = fmaxf(v, 0.f); v *= v; }
   }
   out[(size_t)t * ldo + c] = from_f<OT>(v);
 }
@@ -222,6 +395,37 @@ int bg_residual_norm(int dt, float* x, int ldx, const long long* rows, const int
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
+// dt: 0 = bf16, 1 = fp32 (embedding table and output).  Leading dimensions: multiples of 4, at least D rounded up to 4; vectors
+// of the norms hold that many floats.  D <= 16384.  a null: nothing joins x; ids: x = embed[ids] * escale.
+int bg_sandwich_norm(int dt, float* x, int ldx, const long long* rows, const int* ids, const void* embed, int lde, float escale,
+                     int vocab, const float* a, int lda, const float* b, int ldb, const float* wa, const float* wb, const float* w1,
+                     const float* b1, int center1, const float* w2, const float* b2, int center2, void* y, int ldy, int raw,
+                     const float* cw, float* hist, long long hist_stride, const int* slots, int taps, int R, int D, float eps,
+                     int keep, cudaStream_t stream) {
+  using namespace bg::resid;
+  if (R <= 0) return 0;
+  const int D4 = (D + 3) / 4 * 4;
+  if (D <= 0 || D > 16384 || ldx % 4 || ldx < D4 || ldy % 4 || ldy < D4 || (raw && ldy != D4) || w2 == nullptr ||
+      (a != nullptr && (lda % 4 || lda < D4 || w1 == nullptr)) ||
+      (b != nullptr && (a == nullptr || ldb % 4 || ldb < D4 || wa == nullptr || wb == nullptr)) ||
+      (ids != nullptr && (embed == nullptr || vocab <= 0)) ||
+      (cw != nullptr && (slots == nullptr || taps < 1 || (taps > 1 && hist == nullptr) || hist_stride % 4 || rows != nullptr)))
+    return -1;
+  SandwichParams p;
+  p.x = x; p.ldx = ldx; p.rows = rows; p.ids = ids; p.embed = embed; p.lde = lde; p.escale = escale; p.vocab = vocab;
+  p.a = a; p.b = b; p.lda = lda; p.ldb = ldb; p.wa = wa; p.wb = wb; p.w1 = w1; p.b1 = b1; p.center1 = center1;
+  p.w2 = w2; p.b2 = b2; p.center2 = center2; p.y = y; p.ldy = ldy; p.raw = raw; p.cw = cw; p.hist = hist;
+  p.hist_stride = hist_stride; p.slots = slots; p.taps = taps; p.D = D; p.eps = eps; p.keep = keep;
+#define BG_SANDWICH(NV)                                                                                                  do {                                                                                                                     if (dt == 0) bg::launch_pdl(sandwich_norm_kernel<__nv_bfloat16, NV>, dim3(R), dim3(kThreads), 0, stream, p);           else bg::launch_pdl(sandwich_norm_kernel<float, NV>, dim3(R), dim3(kThreads), 0, stream, p);                         } while (0)
+  if (D <= 1024) BG_SANDWICH(1);
+  else if (D <= 2048) BG_SANDWICH(2);
+  else if (D <= 4096) BG_SANDWICH(4);
+  else if (D <= 8192) BG_SANDWICH(8);
+  else BG_SANDWICH(16);
+#undef BG_SANDWICH
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
 // kind 0 tanh-GELU, 1 clamped SwiGLU.  z points at the first gate column, the up column of a gate column is u_off further.
 int bg_glu(int dt, int kind, const float* z, int ldz, int u_off, void* out, int ldo, int R, int F, int Fo, float limit,
            const float* row_scale, const float* gate, int ld_gate, const int* total_rows, cudaStream_t stream) {
@@ -240,7 +444,7 @@ int bg_glu(int dt, int kind, const float* z, int ldz, int u_off, void* out, int 
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
-// out [T, ldo] = f(x[:, :N]) with zero columns N .. ldo; kind 0 identity, 1 tanh
+// out [T, ldo] = f(x[:, :N]) with zero columns N .. ldo; kind 0 identity, 1 tanh, 2 squared ReLU
 int bg_cast_act(int dt, int kind, const float* x, int ldx, void* out, int ldo, int T, int N, cudaStream_t stream) {
   using namespace bg::resid;
   if (T <= 0 || ldo <= 0) return 0;
@@ -249,9 +453,11 @@ int bg_cast_act(int dt, int kind, const float* x, int ldx, void* out, int ldo, i
 #define BG_CAST(OT, KIND) \
   bg::launch_pdl(cast_act_kernel<OT, KIND>, grid, dim3(kThreads), 0, stream, x, ldx, reinterpret_cast<OT*>(out), ldo, T, N)
   if (dt == 0 && kind == 0) BG_CAST(__nv_bfloat16, 0);
-  else if (dt == 0) BG_CAST(__nv_bfloat16, 1);
+  else if (dt == 0 && kind == 1) BG_CAST(__nv_bfloat16, 1);
+  else if (dt == 0) BG_CAST(__nv_bfloat16, 2);
   else if (kind == 0) BG_CAST(float, 0);
-  else BG_CAST(float, 1);
+  else if (kind == 1) BG_CAST(float, 1);
+  else BG_CAST(float, 2);
 #undef BG_CAST
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }

@@ -4,9 +4,11 @@
 //   s[h, j]  = scale * sum_g talk[h, g] (q[g] . k[kv(g), j])        g over all query heads, kv(g) = g / (H / G)
 //   seen     = first <= j <= position, first = position - position % chunk (chunk 0: first = 0)
 //   p[h, j]  = exp(s[h, j]) / (1 + sum exp(s[h, :]))                 (the 1 only with a sink)
-//   o[h]     = sum_j p[h, j] v[kv(h), j]
+//   o[h]     = sum_j p[h, j] v[kv(h), j], times sigmoid(gate[h]) when there is a gate
 //
-// Mixing couples all heads at a key, so a CTA takes all heads of its row.  Keys go in tiles of 32 (a lane per key); a
+// Without a mixing matrix a head keeps its own score.  Queries (on load) and keys (on the way to the cache) may carry rotary
+// positions: channel i turns with channel i + half.  Mixing couples all heads at a key, so a CTA takes all heads of its row.
+// Keys go in tiles of 32 (a lane per key); a
 // tile's steps are: raw scores (each warp takes key heads, whose K rows it stages through its own shared-memory buffer;
 // the next tile's rows are fetched while the rest of this tile runs), mixing and online softmax (a warp owns blocks of 4
 // heads, all 32 keys in its lanes), P.V (a thread owns 4 value columns of up to 4 heads that share a value head, so V is
@@ -42,6 +44,10 @@ struct Params {
   float* part_ml;               // [R, n_splits, H, 2]
   int H, G, dp, dvp, chunk, sink, n_splits;
   float scale_log2;
+  const float* rope;            // [T, 2 * half] cosines, then sines, or null
+  int half;
+  const float* gate;            // [T, ld_gate] or null
+  int ld_gate;
 };
 
 template <typename T> __device__ __forceinline__ float to_f(T v);
@@ -57,6 +63,16 @@ __device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) {
   const __nv_bfloat162* v = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
   for (int i = 0; i < 4; ++i) { const float2 a = __bfloat1622float2(v[i]); f[2 * i] = a.x; f[2 * i + 1] = a.y; }
+}
+__device__ __forceinline__ float sigm(float x) { return 1.0f / (1.0f + expf(-x)); }
+// channel e of a head whose first 2 * half channels turn
+__device__ __forceinline__ float turned(const float* x, int e, const float* rope, int half) {
+  const float a = x[e];
+  if (e >= 2 * half) return a;
+  const bool low = e < half;
+  const int i = low ? e : e - half;
+  const float b = x[low ? e + half : i], c = rope[i], s = rope[half + i];
+  return low ? a * c - b * s : a * c + b * s;
 }
 __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
 __device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
@@ -76,17 +92,18 @@ __device__ __forceinline__ void cp16(void* dst, const void* src) {
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void cp_wait0() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 
-// shared memory, in floats: q [H dp] | talk^T [H][Hp] | raw scores [H][NT] | probabilities [Hp][NT] | m, l, a [Hp] each |
+// shared memory, in floats: q [H dp] | talk^T [H][Hp] (mixed heads only) | raw scores [H][NT] | probabilities [Hp][NT] |
+// m, l, a [Hp] each |
 // key offsets [NT] (long long), then the K buffers (one per warp), reused for the last reduction
 __host__ __device__ inline int pad4(int x) { return (x + 3) / 4 * 4; }
-__host__ __device__ inline size_t smem_floats(int H, int dp) {
+__host__ __device__ inline size_t smem_floats(int H, int dp, bool mixed) {
   const int Hp = pad4(H);
-  return (size_t)pad4(H * dp) + (size_t)H * Hp + (size_t)H * NT + (size_t)Hp * NT + 3 * (size_t)Hp + 2 * NT;
+  return (size_t)pad4(H * dp) + (mixed ? (size_t)H * Hp : 0) + (size_t)H * NT + (size_t)Hp * NT + 3 * (size_t)Hp + 2 * NT;
 }
 template <typename KT>
 __host__ __device__ inline size_t kbuf_bytes(int dp) { return (size_t)NT * (dp * sizeof(KT) + 16); }
 
-template <typename KT, int NI>
+template <typename KT, int NI, bool MIX>
 __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   extern __shared__ __align__(16) float sm[];
@@ -94,7 +111,7 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
   const int H = p.H, G = p.G, dp = p.dp, dvp = p.dvp, rep = H / G, Hp = pad4(H);
   float* q_s = sm;
   float* tt = q_s + pad4(H * dp);
-  float* raw = tt + H * Hp;
+  float* raw = tt + (MIX ? H * Hp : 0);
   float* pr = raw + H * NT;
   float* m_s = pr + Hp * NT;
   float* l_s = m_s + Hp;
@@ -111,12 +128,17 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
     return;                                                       // (a split row without a query is zeroed by the merge)
   }
   const float* qr = p.q + (size_t)t * p.ldq;
-  for (int i = tid; i < H * dp / 4; i += kThreads) reinterpret_cast<float4*>(q_s)[i] = reinterpret_cast<const float4*>(qr)[i];
-  for (int i = tid; i < H * Hp; i += kThreads) {
-    const int g = i / Hp, h = i % Hp;
-    float v = 0.f;
-    if (h < H) v = p.talk != nullptr ? p.talk[h * H + g] : (h == g ? 1.f : 0.f);
-    tt[i] = v * p.scale_log2;
+  if (p.rope == nullptr) {
+    for (int i = tid; i < H * dp / 4; i += kThreads) reinterpret_cast<float4*>(q_s)[i] = reinterpret_cast<const float4*>(qr)[i];
+  } else {
+    const float* rope = p.rope + (size_t)t * 2 * p.half;
+    for (int i = tid; i < H * dp; i += kThreads) q_s[i] = turned(qr + i / dp * dp, i % dp, rope, p.half);
+  }
+  if (MIX) {
+    for (int i = tid; i < H * Hp; i += kThreads) {
+      const int g = i / Hp, h = i % Hp;
+      tt[i] = h < H ? p.talk[h * H + g] * p.scale_log2 : 0.f;
+    }
   }
   for (int i = tid; i < Hp; i += kThreads) { m_s[i] = -INFINITY; l_s[i] = 0.f; }
   const int first = p.chunk > 0 ? (L - 1) - (L - 1) % p.chunk : 0;
@@ -199,11 +221,17 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
     // mixing + online softmax
     for (int hb = warp; hb < Hp / 4; hb += kWarps) {
       float v[4] = {0.f, 0.f, 0.f, 0.f};
+      if (MIX) {
 #pragma unroll 4
-      for (int g = 0; g < H; ++g) {
-        const float sg = raw[g * NT + lane];
-        const float4 w = *reinterpret_cast<const float4*>(tt + g * Hp + hb * 4);
-        v[0] = fmaf(w.x, sg, v[0]); v[1] = fmaf(w.y, sg, v[1]); v[2] = fmaf(w.z, sg, v[2]); v[3] = fmaf(w.w, sg, v[3]);
+        for (int g = 0; g < H; ++g) {
+          const float sg = raw[g * NT + lane];
+          const float4 w = *reinterpret_cast<const float4*>(tt + g * Hp + hb * 4);
+          v[0] = fmaf(w.x, sg, v[0]); v[1] = fmaf(w.y, sg, v[1]); v[2] = fmaf(w.z, sg, v[2]); v[3] = fmaf(w.w, sg, v[3]);
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (hb * 4 + i < H) v[i] = raw[(hb * 4 + i) * NT + lane] * p.scale_log2;
       }
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
@@ -300,7 +328,8 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
           const int h = h0 + i, col = h * dvp + cc * 4;
           const float4 v = make_float4(acc[n][i][0].x, acc[n][i][0].y, acc[n][i][1].x, acc[n][i][1].y);
           if (p.n_splits == 1) {
-            const float inv = 1.0f / (l_s[h] + (p.sink ? exp2f(-m_s[h]) : 0.f));
+            float inv = 1.0f / (l_s[h] + (p.sink ? exp2f(-m_s[h]) : 0.f));
+            if (p.gate != nullptr) inv *= sigm(p.gate[(size_t)t * p.ld_gate + h]);
             put4(out + col, make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv));
           } else {
             *reinterpret_cast<float4*>(p.part_o + ((size_t)r * p.n_splits + split) * H * dvp + col) = v;
@@ -336,7 +365,8 @@ __global__ void merge_kernel(const Params p) {
     const float ms = ml[(size_t)s * p.H * 2];
     if (ms != -INFINITY) l += ml[(size_t)s * p.H * 2 + 1] * exp2f(ms - m);
   }
-  const float inv = 1.0f / l;
+  float inv = 1.0f / l;
+  if (p.gate != nullptr) inv *= sigm(p.gate[(size_t)t * p.ld_gate + h]);
   for (int i = threadIdx.x; i < p.dvp / 4; i += blockDim.x) {
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int s = 0; s < S; ++s) {
@@ -350,32 +380,48 @@ __global__ void merge_kernel(const Params p) {
   }
 }
 
-// cache[slot[t]] = kv[t] (fp32 projection columns: keys of all heads, then values); slot < 0 writes nothing
+// cache[slot[t]] = kv[t] (fp32 projection columns: keys of all G heads of dp channels, then values), the keys turned by the
+// token's row of `rope` when there is one; slot < 0 writes nothing
 template <typename KT>
 __global__ void __launch_bounds__(128)
 kv_write_kernel(const float* __restrict__ kv, int ld, const long long* __restrict__ slots, KT* __restrict__ cache,
-                long long page_stride, int page, int row) {
+                long long page_stride, int page, int row, const float* __restrict__ rope, int half, int G, int dp) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   const long long slot = slots[blockIdx.x];
   if (slot < 0) return;
   KT* dst = cache + (slot / page) * page_stride + (slot % page) * row;
-  const float4* src = reinterpret_cast<const float4*>(kv + (size_t)blockIdx.x * ld);
-  for (int i = threadIdx.x; i < row / 4; i += blockDim.x) put4(dst + 4 * i, src[i]);
+  const float* src = kv + (size_t)blockIdx.x * ld;
+  const float* rr = rope + (size_t)blockIdx.x * 2 * half;
+  for (int i = threadIdx.x; i < row / 4; i += blockDim.x) {
+    const int c = 4 * i;
+    float4 v = *reinterpret_cast<const float4*>(src + c);
+    if (rope != nullptr && c < G * dp && c % dp < 2 * half) {       // dp % 8 == 0: the four channels share a head
+      const float* head = src + c / dp * dp;
+      const int e = c % dp;
+      v = make_float4(turned(head, e, rr, half), turned(head, e + 1, rr, half), turned(head, e + 2, rr, half),
+                      turned(head, e + 3, rr, half));
+    }
+    put4(dst + c, v);
+  }
 }
 
-template <typename KT, int NI>
-static int launch_rows(const Params& p, int R, cudaStream_t stream) {
+template <typename KT, int NI, bool MIX>
+static int launch_rows_as(const Params& p, int R, cudaStream_t stream) {
   size_t kb = kWarps * kbuf_bytes<KT>(p.dp);
   const size_t red = (size_t)kThreads * 16 * sizeof(float);
   if (kb < red) kb = red;
-  const size_t smem = smem_floats(p.H, p.dp) * sizeof(float) + kb;
+  const size_t smem = smem_floats(p.H, p.dp, MIX) * sizeof(float) + kb;
   if (smem > 227 * 1024) return -3;
   static DeviceOnce once;
-  auto kern = rows_kernel<KT, NI>;
+  auto kern = rows_kernel<KT, NI, MIX>;
   if (!ensure_dynamic_smem(kern, 227 * 1024, once)) return -4;
   bg::launch_pdl(kern, dim3(R, p.n_splits), dim3(kThreads), smem, stream, p);
   if (p.n_splits > 1) bg::launch_pdl(merge_kernel<KT>, dim3(R, p.H), dim3(64), 0, stream, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+template <typename KT, int NI>
+static int launch_rows(const Params& p, int R, cudaStream_t stream) {
+  return p.talk != nullptr ? launch_rows_as<KT, NI, true>(p, R, stream) : launch_rows_as<KT, NI, false>(p, R, stream);
 }
 
 }  // namespace talk
@@ -387,11 +433,12 @@ extern "C" {
 int bg_talk_rows(int dt, const float* q, int ldq, const float* talk, const void* cache, long long page_stride, int page,
                  int row, const int* block_table, int bt_stride, const int* row_seq, const int* row_ids, const int* lens,
                  void* out, int ldo, float* part_o, float* part_ml, int R, int H, int G, int dp, int dvp, int chunk,
-                 int sink, float scale, int n_splits, cudaStream_t stream) {
+                 int sink, float scale, int n_splits, const float* rope, int half, const float* gate, int ld_gate,
+                 cudaStream_t stream) {
   using namespace bg::talk;
   if (R <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || dp <= 0 || dp % 8 || dvp <= 0 || dvp % 8 || row != G * (dp + dvp) || page <= 0 ||
-      page_stride % 8 || ldq % 4 || ldo % 4 || n_splits < 1 || n_splits > 65535 || H > 65535 ||
+      page_stride % 8 || ldq % 4 || ldo % 4 || (rope != nullptr && (half <= 0 || 2 * half > dp)) || n_splits < 1 || n_splits > 65535 || H > 65535 ||
       (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return -1;
   Params p;
@@ -399,6 +446,7 @@ int bg_talk_rows(int dt, const float* q, int ldq, const float* talk, const void*
   p.block_table = block_table; p.bt_stride = bt_stride; p.row_seq = row_seq; p.row_ids = row_ids; p.lens = lens;
   p.out = out; p.ldo = ldo; p.part_o = part_o; p.part_ml = part_ml; p.H = H; p.G = G; p.dp = dp; p.dvp = dvp;
   p.chunk = chunk; p.sink = sink; p.n_splits = n_splits; p.scale_log2 = scale * 1.4426950408889634f;
+  p.rope = rope; p.half = half; p.gate = gate; p.ld_gate = ld_gate;
   const int items = G * ((H / G + 3) / 4) * (dvp / 4);
   const int ni = (items + kThreads - 1) / kThreads;
   if (ni > 4) return -1;
@@ -413,16 +461,18 @@ int bg_talk_rows(int dt, const float* q, int ldq, const float* talk, const void*
 }
 
 int bg_talk_kv_write(int dt, const float* kv, int ld, const long long* slots, void* cache, long long page_stride, int page,
-                     int row, int T, cudaStream_t stream) {
+                     int row, int T, const float* rope, int half, int G, int dp, cudaStream_t stream) {
   using namespace bg::talk;
   if (T <= 0) return 0;
   if (row % 8 || ld % 4 || ld < row || page <= 0 || page_stride % 8) return -1;
+  if (rope != nullptr && (half <= 0 || dp % 8 || 2 * half > dp || G * dp > row)) return -1;
+  if (dp <= 0) dp = row;
   if (dt == 0)
     bg::launch_pdl(kv_write_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, stream, kv, ld, slots,
-                   reinterpret_cast<__nv_bfloat16*>(cache), page_stride, page, row);
+                   reinterpret_cast<__nv_bfloat16*>(cache), page_stride, page, row, rope, half, G, dp);
   else
     bg::launch_pdl(kv_write_kernel<float>, dim3(T), dim3(128), 0, stream, kv, ld, slots, reinterpret_cast<float*>(cache),
-                   page_stride, page, row);
+                   page_stride, page, row, rope, half, G, dp);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
