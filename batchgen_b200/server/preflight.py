@@ -152,18 +152,21 @@ def _layered_contract(cfg, world: int, on_gpu: bool) -> List[str]:
     if world > 1:
         bad.append("layer-listed models run on one GPU per engine: raise --dp-size to the world size")
     for i, s in enumerate(cfg.layer_specs):
-        m, f = s.mixer, s.mlp
-        if m.recurrent and m.dim > 256:
-            bad.append(f"layer {i}: delta-rule head width {m.dim} exceeds 256")
-        if not m.recurrent and m.kv_heads * -(-(m.heads // m.kv_heads) // 4) * (m.vdim_p // 4) > 1024:
-            bad.append(f"layer {i}: {m.heads} heads x {m.vdim} value channels exceed the decode attention kernel")
+        f = s.mlp
+        for m in s.mixers:
+            if m.recurrent and m.dim > 256:
+                bad.append(f"layer {i}: {m.kind} head width {m.dim} exceeds 256")
+            if not m.recurrent and m.kv_heads * -(-(m.heads // m.kv_heads) // 4) * (m.vdim_p // 4) > 1024:
+                bad.append(f"layer {i}: {m.heads} heads x {m.vdim} value channels exceed the decode attention kernel")
         if f.kind == "moe" and (f.top > 16 or f.experts > 1024 or f.top > f.experts):
             bad.append(f"layer {i}: top {f.top} of {f.experts} experts (the router takes up to 16 of 1,024)")
     if bad:
         raise PreflightError("model contract: " + "; ".join(bad))
     if not on_gpu:
         return ["fp32 reference path: no kernel geometry rules apply"]
-    return ["layer-listed model: tcgen05 projections, experts and prompt attention; delta-rule, decode attention and row "
+    if cfg.sandwich and cfg.hidden_size > 16384:
+        raise PreflightError(f"model contract: width {cfg.hidden_size} exceeds the norm kernel's 16384")
+    return ["layer-listed model: tcgen05 projections, experts and prompt attention; recurrences, decode attention and row "
             "operators as CUDA kernels of their own"]
 
 
