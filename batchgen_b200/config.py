@@ -838,8 +838,9 @@ def tiny_pamevik() -> ModelConfig:
 
 
 def pamevik_bench() -> ModelConfig:
-    """Layers of a real model's size: channel-delta, mLSTM, channel-delta and one attention-beside-retention layer."""
-    dense = {"kind": "dense", "ff": 9216}
+    """Layers of a real model's size: channel-delta, mLSTM, channel-delta and one attention-beside-retention layer.  The
+    feed-forward's two matrices hold as many weights as the three of a gated one of width 9216."""
+    dense = {"kind": "dense", "ff": 13824}
     cd = {"type": "channel_delta", "mlp": dense, "mixer": {"heads": 32, "kv_heads": 32, "dim": 128, "vdim": 128, "conv": 4}}
     ml = {"type": "mlstm", "mlp": dense, "mixer": {"heads": 32, "dim": 128, "vdim": 128, "gate_cap": 15.0}}
     rot = {"base": 1e6, "dims": 128}

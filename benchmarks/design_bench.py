@@ -1,13 +1,15 @@
-"""Layer-listed model (Nanurax) beside the framework's closest existing model at equal size.
+"""Layer-listed models (Nanurax, Pamevik) beside the framework's closest existing model at equal size.
 
-``bench.py --workload nanurax``: both models have four layers of a real model's size (width 2304, 32 heads of 128, 64
-experts of which 8 run, one dense and three mixture feed-forwards, bf16): three recurrent layers to one attention layer.
-Nanurax runs the generalised delta rule and chunked talking-heads attention, the other one is a Kimi-Linear cut with KDA and
-MLA layers.  Prefill is one packed forward over fresh prompts, decode is a captured step over sequences with cached context;
-random weights, CUDA events, medians, the L2 flushed before every timed call.
+``bench.py --workload nanurax | pamevik``: both models have four layers of a real model's size (width 2304, 32 heads of 128,
+bf16), three recurrent layers to one attention layer.  Nanurax runs the generalised delta rule and chunked talking-heads
+attention with one dense and three mixture feed-forwards (64 experts of which 8 run); Pamevik runs two channel-delta layers, an
+mLSTM layer and attention beside retention, with dense feed-forwards.  The other one is a Kimi-Linear cut with KDA and MLA
+layers and the same kinds of feed-forwards.  Prefill is one packed forward over fresh prompts, decode is a captured step over
+sequences with cached context; random weights, CUDA events, medians, the L2 flushed before every timed call.
 
-``kernels`` of the result times the new kernels beside their likes (recurrence against KDA, decode attention against the
-paged GQA kernel, prompt attention against the expanded MLA kernel) with the share of the measured roofline each reaches.
+``kernels`` of the result times the new kernels beside their likes (recurrences against KDA, decode attention against the
+paged GQA kernel, prompt attention against the expanded MLA kernel, norms against the fused residual norm) with the share of
+the measured roofline each reaches.
 """
 from __future__ import annotations
 
@@ -52,9 +54,10 @@ class _Timer:
         return sorted(times)[len(times) // 2]
 
 
-def _closest():
+def _closest(design: str):
     from batchgen_b200.config import get_model_config
-    return get_model_config("kimi-linear-48b", num_layers=4, kda_layers=(0, 1, 2), n_routed_experts=64, num_experts_per_tok=8)
+    mlp = dict(n_routed_experts=64, num_experts_per_tok=8) if design == "nanurax" else dict(first_k_dense=4)
+    return get_model_config("kimi-linear-48b", num_layers=4, kda_layers=(0, 1, 2), **mlp)
 
 
 def _model_rates(cfg, dev, timer: _Timer) -> Dict[str, object]:
@@ -97,78 +100,172 @@ def _model_rates(cfg, dev, timer: _Timer) -> Dict[str, object]:
     return out
 
 
-def _kernels(dev, timer: _Timer, peaks) -> List[Dict[str, object]]:
-    import torch
-    from batchgen_b200.ops import attention, delta, kda, talking
-    H, G, D, page = 32, 8, 128, 64
-    HD, bf = H * D, torch.bfloat16
-    rows: List[Dict[str, object]] = []
+class _Rows:
+    """Timed kernels with the share of the roofline each reaches."""
 
-    def add(name, size, ms, gbytes=0.0, tflop=0.0):
+    def __init__(self, peaks):
+        self.peaks, self.rows = peaks, []
+
+    def __call__(self, name, size, ms, gbytes=0.0, tflop=0.0):
         r = {"kernel": name, "size": size, "us": round(ms * 1e3, 1)}
         share = []
         if gbytes:
             r["gb_per_s"] = round(gbytes / ms * 1e3)
-            share.append(gbytes / ms * 1e3 / peaks["hbm_gbs"])
+            share.append(gbytes / ms * 1e3 / self.peaks["hbm_gbs"])
         if tflop:
             r["tflops"] = round(tflop / ms * 1e3, 1)
-            share.append(tflop / ms * 1e3 / peaks["bf16_tflops"])
-        r["of_" + peaks["source"]] = round(max(share), 3)
-        rows.append(r)
-    for B, T in ((64, 1), (256, 1), (1, 4096), (8, 1024)):
-        R, size = B * T, f"{B} x {T} tokens"
-        slots = torch.arange(B, dtype=torch.int32, device=dev)
-        cu = None if T == 1 else torch.arange(0, R + 1, T, dtype=torch.int32, device=dev)
-        init = None if T == 1 else torch.ones(B, dtype=torch.int32, device=dev)
-        z, wl = torch.randn(R, 5 * HD, device=dev), torch.randn(R, HD, device=dev)
-        p = delta.DeltaParams(torch.randn(HD, device=dev), torch.randn(HD, device=dev), torch.ones(HD, device=dev), H, D, D,
-                              math.exp(-0.5))
-        st, out = torch.zeros(B + 1, HD * D, device=dev), torch.empty(R, HD, dtype=bf, device=dev)
-        ms = timer(lambda: delta.delta_forward(z, tuple(i * HD for i in range(5)), wl, p, st, slots, out, cu, None, init))
-        add("delta rule", size, ms, (R * HD * (6 * 4 + 2) + B * HD * D * 8) / 1e9)
-        del z, wl
-        qkv, f = torch.randn(R, 4 * HD + 64, device=dev).to(bf), torch.randn(R, HD, device=dev).to(bf)
-        kp = kda.KDAParams(torch.randn(3 * HD, 4, device=dev), None, torch.randn(H, device=dev), torch.randn(HD, device=dev),
-                           torch.ones(D, device=dev))
-        cs, rs = torch.zeros(B, 3 * HD, 3, device=dev), torch.zeros(B, H, D, D, device=dev)
-        ms = timer(lambda: kda.kda_forward(qkv[:, :3 * HD], f, qkv[:, 4 * HD:4 * HD + H], qkv[:, 3 * HD:4 * HD], kp, cs, rs,
-                                           slots, cu, init, H, D, D ** -0.5, 1e-6))
-        add("  KDA", size, ms, (R * HD * 12 + B * HD * (D * 8 + 3 * 3 * 8)) / 1e9)
-    talk = torch.randn(H, H, device=dev) / 6
-    for B, ctx in ((16, 4096), (64, 4096)):
-        n = B * ctx // page
-        cache = torch.randn(n, page, 2 * G * D, device=dev).to(bf)
+            share.append(tflop / ms * 1e3 / self.peaks["bf16_tflops"])
+        r["of_" + self.peaks["source"]] = round(max(share), 3)
+        self.rows.append(r)
+
+
+H, G, D, PAGE = 32, 8, 128, 64
+HD = H * D
+STATE_CASES = [(64, 1), (256, 1), (1, 4096), (8, 1024)]        # sequences, tokens of each
+
+
+def _state_case(dev, B: int, T: int):
+    import torch
+    R = B * T
+    slots = torch.arange(B, dtype=torch.int32, device=dev)
+    cu = None if T == 1 else torch.arange(0, R + 1, T, dtype=torch.int32, device=dev)
+    init = None if T == 1 else torch.ones(B, dtype=torch.int32, device=dev)
+    return R, f"{B} x {T} tokens", slots, cu, init
+
+
+def _kda_row(dev, timer, add, B, T):
+    import torch
+    from batchgen_b200.ops import kda
+    R, size, slots, cu, init = _state_case(dev, B, T)
+    qkv, f = torch.randn(R, 4 * HD + 64, device=dev).bfloat16(), torch.randn(R, HD, device=dev).bfloat16()
+    kp = kda.KDAParams(torch.randn(3 * HD, 4, device=dev), None, torch.randn(H, device=dev), torch.randn(HD, device=dev),
+                       torch.ones(D, device=dev))
+    cs, rs = torch.zeros(B, 3 * HD, 3, device=dev), torch.zeros(B, H, D, D, device=dev)
+    ms = timer(lambda: kda.kda_forward(qkv[:, :3 * HD], f, qkv[:, 4 * HD:4 * HD + H], qkv[:, 3 * HD:4 * HD], kp, cs, rs,
+                                       slots, cu, init, H, D, D ** -0.5, 1e-6))
+    add("  KDA", size, ms, (R * HD * 12 + B * HD * (D * 8 + 3 * 3 * 8)) / 1e9)
+
+
+def _decode_attention_rows(dev, timer, add, cases, talk, **more):
+    import torch
+    from batchgen_b200.ops import attention, talking
+    for B, ctx in cases:
+        n = B * ctx // PAGE
+        cache = torch.randn(n, PAGE, 2 * G * D, device=dev).bfloat16()
         bt = torch.randperm(n, device=dev).to(torch.int32).view(B, -1).contiguous()
         lens = torch.full((B,), ctx, dtype=torch.int32, device=dev)
-        q, out = torch.randn(B, HD, device=dev), torch.empty(B, HD, dtype=bf, device=dev)
-        p = talking.TalkParams(H, G, D, D, D ** -0.5, ctx, True, talk)
+        q, out = torch.randn(B, HD, device=dev), torch.empty(B, HD, dtype=torch.bfloat16, device=dev)
+        p = talking.TalkParams(H, G, D, D, D ** -0.5, ctx if talk is not None else 0, talk is not None, talk)
+        extra = {k: f(lens) for k, f in more.items()}
         gb = B * ctx * 2 * G * D * 2 / 1e9
-        add("attention, decode", f"{B} x {ctx} keys", timer(lambda: talking.attend_rows(q, p, cache, bt, lens, out)), gb)
-        qb = q.to(bf).view(B, H, D)
+        add("attention, decode", f"{B} x {ctx} keys", timer(lambda: talking.attend_rows(q, p, cache, bt, lens, out, **extra)), gb)
+        qb = q.bfloat16().view(B, H, D)
         sinks = torch.zeros(H, device=dev)
         add("  GQA decode", f"{B} x {ctx} keys",
             timer(lambda: attention.gqa_decode(qb, cache, bt, lens, G, D ** -0.5, sinks=sinks)), gb)
-    for T, chunk in ((4096, 4096), (8192, 2048)):
-        n = T // page
-        cache = torch.randn(n, page, 2 * G * D, device=dev).to(bf)
+
+
+def _prompt_attention_rows(dev, timer, add, cases, talk, **more):
+    import torch
+    from batchgen_b200.ops import attention, talking
+    for T, chunk in cases:
+        n = T // PAGE
+        cache = torch.randn(n, PAGE, 2 * G * D, device=dev).bfloat16()
         bt = torch.arange(n, device=dev, dtype=torch.int32).view(1, -1).contiguous()
-        q, out = torch.randn(T, HD, device=dev), torch.empty(T, HD, dtype=bf, device=dev)
-        p = talking.TalkParams(H, G, D, D, D ** -0.5, chunk, True, talk)
+        q, out = torch.randn(T, HD, device=dev), torch.empty(T, HD, dtype=torch.bfloat16, device=dev)
+        mixed = talk is not None
+        p = talking.TalkParams(H, G, D, D, D ** -0.5, chunk if mixed else 0, mixed, talk)
+        extra = {k: f(torch.arange(1, T + 1, dtype=torch.int32, device=dev)) for k, f in more.items()}
         pairs = T * (chunk + 1) / 2
-        blocks = talking.work_blocks(talking.prefill_work([0, T], [0], chunk), T, dev)
-        size = f"{T} tokens, chunks of {chunk}"
-        add("attention, prompt", size, timer(lambda: talking.attend_prefill(q, p, cache, bt, out, blocks)), 0,
-            pairs * 2 * H * (2 * D + H) / 1e12)
-        q3, kv = torch.randn(T, H, 192, device=dev).to(bf), torch.randn(T, H, 256, device=dev).to(bf)
-        kpe = torch.randn(T, 64, device=dev).to(bf)
+        blocks = talking.work_blocks(talking.prefill_work([0, T], [0], p.chunk), T, dev)
+        size = f"{T} tokens" + (f", chunks of {chunk}" if mixed else "")
+        add("attention, prompt", size, timer(lambda: talking.attend_prefill(q, p, cache, bt, out, blocks, **extra)), 0,
+            pairs * 2 * H * (2 * D + (H if mixed else 0)) / 1e12)
+        q3, kv = torch.randn(T, H, 192, device=dev).bfloat16(), torch.randn(T, H, 256, device=dev).bfloat16()
+        kpe = torch.randn(T, 64, device=dev).bfloat16()
         cu = list(range(0, T + 1, chunk))
         work = attention.mha_prefill_work(cu, [0] * (len(cu) - 1), cu[:-1]).to(dev)
         add("  expanded MLA prompt", size, timer(lambda: attention.mha_prefill(q3, kv, kpe, work, 0.07)), 0,
             pairs * 2 * H * 320 / 1e12)
-    return rows
 
 
-def run(args, root: str) -> int:
+def _nanurax_kernels(dev, timer: _Timer, peaks) -> List[Dict[str, object]]:
+    import torch
+    from batchgen_b200.ops import delta
+    add = _Rows(peaks)
+    for B, T in STATE_CASES:
+        R, size, slots, cu, init = _state_case(dev, B, T)
+        z, wl = torch.randn(R, 5 * HD, device=dev), torch.randn(R, HD, device=dev)
+        p = delta.DeltaParams(torch.randn(HD, device=dev), torch.randn(HD, device=dev), torch.ones(HD, device=dev), H, D, D,
+                              math.exp(-0.5))
+        st, out = torch.zeros(B + 1, HD * D, device=dev), torch.empty(R, HD, dtype=torch.bfloat16, device=dev)
+        ms = timer(lambda: delta.delta_forward(z, tuple(i * HD for i in range(5)), wl, p, st, slots, out, cu, None, init))
+        add("delta rule", size, ms, (R * HD * (6 * 4 + 2) + B * HD * D * 8) / 1e9)
+        del z, wl
+        _kda_row(dev, timer, add, B, T)
+    talk = torch.randn(H, H, device=dev) / 6
+    _decode_attention_rows(dev, timer, add, ((16, 4096), (64, 4096)), talk)
+    _prompt_attention_rows(dev, timer, add, ((4096, 4096), (8192, 2048)), talk)
+    return add.rows
+
+
+def _pamevik_kernels(dev, timer: _Timer, peaks) -> List[Dict[str, object]]:
+    import torch
+    from batchgen_b200.ops import conv, fused, recurrent, residual
+    bf, add = torch.bfloat16, _Rows(peaks)
+    rot = conv.Rotary.make(D, 1e6, dev)
+    for B, T in STATE_CASES:
+        R, size, slots, cu, init = _state_case(dev, B, T)
+        row_seq = None if T == 1 else torch.arange(B, dtype=torch.int32, device=dev).repeat_interleave(T)
+        z, out = torch.randn(R, 5 * HD + 64, device=dev), torch.empty(R, HD, dtype=bf, device=dev)
+        S = {"S": torch.zeros(B + 1, HD * D, device=dev), "n": torch.zeros(B + 1, HD, device=dev),
+             "m": torch.zeros(B + 1, H, device=dev)}
+        q, k, v, g, low = (z[:, i * HD:(i + 1) * HD] for i in range(5))
+        gates = z[:, 5 * HD:5 * HD + H]
+        base = dict(heads=H, dim_p=D, vdim=D, vdim_p=D, norm_w=torch.ones(HD, device=dev), eps=1e-6)
+        rules = {
+            "channel_delta": (dict(rate=torch.ones(H, device=dev), dt_bias=torch.zeros(HD, device=dev)), dict(low=low, beta=gates), 5),
+            "mlstm": (dict(i_bias=torch.zeros(H, device=dev), f_bias=torch.zeros(H, device=dev), gate_cap=15.0),
+                      dict(gate_i=gates, gate_f=gates), 4),
+            "retention": (dict(decay=torch.full((H,), 0.99, device=dev), gate="silu"),
+                          dict(rope=rot.table(torch.arange(1, R + 1, dtype=torch.int32, device=dev))), 4)}
+        for rule, (kw, more, columns) in rules.items():
+            p = recurrent.RecurrentParams(rule, **base, **kw)
+            st = {n: t for n, t in S.items() if n == "S" or rule == "mlstm"}
+            ms = timer(lambda: recurrent.recurrent_forward(p, q, k, v, g, st, slots, out, cu, None, init, **more))
+            add(rule, size, ms, (R * HD * (columns * 4 + 2) + B * HD * D * 8) / 1e9)
+        _kda_row(dev, timer, add, B, T)
+        w, hist = torch.randn(4, 3 * HD, device=dev), torch.zeros(B + 1, 9 * HD, device=dev)
+        x = torch.empty(R, 3 * HD, device=dev)
+        ms = timer(lambda: conv.causal_conv(z[:, :3 * HD], w, hist, slots, x, "silu", cu, None, row_seq, init))
+        add("short convolutions", size, ms, (R * 3 * HD * 8 + B * 9 * HD * 8) / 1e9)
+        del z, x
+        Wd = 2304
+        n1 = residual.Norm(torch.ones(Wd, device=dev), torch.zeros(Wd, device=dev), True)
+        xs, a, b = (torch.randn(R, Wd, device=dev) for _ in range(3))
+        cw, ch = torch.randn(4, Wd, device=dev), torch.zeros(B + 1, 3 * Wd, device=dev)
+        pair = dict(add=a, add2=b, branch_w=(n1.w, n1.w), post=n1)
+        if T == 1:
+            canon = residual.Canon(cw, ch, slots)
+            ms = timer(lambda: residual.sandwich_norm(xs, n1, 1e-6, Wd, Wd, bf, add=a, post=n1, canon=canon))
+            add("norms + input convolution", size, ms, (R * Wd * (4 * 3 + 2) + B * Wd * 24) / 1e9)
+        else:
+            y = torch.empty(R, Wd, dtype=bf, device=dev)
+            ms = timer(lambda: conv.causal_conv(residual.sandwich_norm(xs, n1, 1e-6, Wd, Wd, bf, add=a, post=n1, raw=True), cw, ch,
+                                                slots, y, "residual", cu, None, row_seq, init))
+            add("norms + input convolution", size, ms, R * Wd * (4 * 3 + 2) / 1e9)
+        add("norms of two branches", size, timer(lambda: residual.sandwich_norm(xs, n1, 1e-6, Wd, Wd, bf, **pair)),
+            R * Wd * (4 * 4 + 2) / 1e9)
+        xb, rb = xs.to(bf), a.to(bf)
+        ms = timer(lambda: fused.rmsnorm(xb, n1.w, 1e-6, residual=rb))
+        add("  residual + RMS norm", size, ms, R * Wd * 8 / 1e9)
+    rope, gate = rot.table, lambda lens: torch.randn(lens.shape[0], H, device=dev)
+    _decode_attention_rows(dev, timer, add, ((16, 4096), (64, 4096)), None, rope=rope, gate=gate)
+    _prompt_attention_rows(dev, timer, add, ((4096, 4096), (8192, 8192)), None, rope=rope, gate=gate)
+    return add.rows
+
+
+def run(args, root: str, design: str) -> int:
     import torch
     from batchgen_b200.config import get_model_config
     from batchgen_b200.ops import _ext
@@ -182,16 +279,16 @@ def run(args, root: str) -> int:
     sampler = ClockSampler(0).start()
     l0 = _ext.LAUNCHES["count"]
     models = {}
-    for cfg in (get_model_config("nanurax-bench"), _closest()):
+    for cfg in (get_model_config(f"{design}-bench"), _closest(design)):
         models[cfg.name] = _model_rates(cfg, dev, timer)
-    kernels = _kernels(dev, timer, peaks)
+    kernels = {"nanurax": _nanurax_kernels, "pamevik": _pamevik_kernels}[design](dev, timer, peaks)
     _ext.check_status()
-    value = models["nanurax-bench"]["decode"][1]["tok_per_s"]
+    step = models[f"{design}-bench"]["decode"][1]
     print(json.dumps({
-        "metric": "decode tokens/s, 64 rows at 2,048 context, four layers (Nanurax)", "value": value, "unit": "tokens/s",
-        "n_gpus": 1, "steps": args.steps, "warmup": timer.warmup, "ms_per_step": models["nanurax-bench"]["decode"][1]["ms"],
+        "metric": f"decode tokens/s, 64 rows at 2,048 context, four layers ({design.capitalize()})", "value": step["tok_per_s"],
+        "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": timer.warmup, "ms_per_step": step["ms"],
         "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-        "config": {"model": "nanurax-bench", "closest": "kimi-linear cut to four layers", "l2": "flushed before every call",
+        "config": {"model": f"{design}-bench", "closest": "kimi-linear cut to four layers", "l2": "flushed before every call",
                    "parallelism": "1 GPU"},
         "models": models, "kernels": kernels, "peaks": peaks, "clocks": sampler.stop(),
         "gpu_launches": _ext.LAUNCHES["count"] - l0}))
