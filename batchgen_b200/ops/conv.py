@@ -28,6 +28,8 @@ def causal_conv(x: torch.Tensor, w: torch.Tensor, hist: torch.Tensor, slots: tor
     if not x.is_cuda:
         return _conv_ref(x, w, hist, slots, out, kind, cu_host, has_initial)
     assert x.dtype == w.dtype == hist.dtype == torch.float32 and x.stride(1) == out.stride(1) == hist.stride(1) == 1
+    assert x.shape[1] >= C and out.shape[0] == x.shape[0] and out.shape[1] >= C and hist.shape[1] == (taps - 1) * C
+    assert (row_seq is None or row_seq.shape[0] == x.shape[0]) and (cu is None or cu.shape[0] == slots.shape[0] + 1)
     assert w.is_contiguous() and slots.dtype == torch.int32 and (row_seq is None or row_seq.dtype == torch.int32)
     rc = _ext.lib().bg_causal_conv(
         _i(_DT[out.dtype]), _i(CONV_KINDS[kind]), _ext.ptr(x), _i(x.stride(0)), _ext.ptr(w), _ext.ptr(hist),

@@ -9,9 +9,6 @@
 // is ordinary flash attention whose keys are a cached token's whole key block (width G * dp) and whose values are head
 // kv(h)'s.  The mixed scores leave the tensor core in fp32.
 //
-// Without mixing the contraction is a head's own: queries (turned by rotary positions where there are any) against the columns
-// of key head kv(h), dp wide and rounded up to 64 (the columns past the head meet zeros of the query).
-//
 // One CTA = (tile of 128 queries of one sequence, head h).  M = 128 queries on the TMEM lanes, key tiles of 128:
 //   S (2 x 128 columns, double buffered) = Q' . K^T, both operands streamed in 64-wide K blocks through a TMA ring
 //   O (dv columns) += P . V,  P written by the softmax threads as a swizzled K-major tile, V read N-major
@@ -47,13 +44,10 @@ struct Params {
   int bt_stride, bt_cols;
   int page, box_rows;            // tokens per page, rows of one TMA box (min(page, 64))
   int KB;                        // 64-wide blocks of the contraction
-  int k_step;                    // columns between key heads (plain heads); 0: every head reads the whole key block
   int v_col0, dvp, dv64, rep;    // first value column of a cache row, head widths, heads per key head
   int chunk, sink;
   __nv_bfloat16* out;
   int ldo;
-  const float* gate;             // [T, ld_gate] or null: out[h] *= sigmoid(gate[h])
-  int ld_gate;
   int row_shift;                 // rows of Q' = rows of out - row_shift
   int* status;
 };
@@ -168,7 +162,7 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
         for (int b = 0; b < kMaxBoxes; ++b)
           if (b < boxes) nxt[b] = bt[min((k0 + t * BN + b * p.box_rows) >> shift, p.bt_cols - 1)];
       };
-      const int vcol = p.v_col0 + (h / p.rep) * p.dvp, kcol = (h / p.rep) * p.k_step;
+      const int vcol = p.v_col0 + (h / p.rep) * p.dvp;
       auto load_v = [&](int t) -> bool {                           // values of tile t, whose pages are in `old`
         if (!mbar_wait(&ss.v_empty, (t & 1) ^ 1, abort_flag, kTimeoutProducer)) return false;
         mbar_expect_tx(&ss.v_full, v_tile_bytes);
@@ -195,7 +189,7 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
 #pragma unroll
           for (int b = 0; b < kMaxBoxes; ++b)
             if (b < boxes)
-              tma_load_3d(b_buf + s * kBBytes + b * p.box_rows * 128, &tm_kv, &ss.full[s], kcol + kb * 64,
+              tma_load_3d(b_buf + s * kBBytes + b * p.box_rows * 128, &tm_kv, &ss.full[s], kb * 64,
                           (pos + b * p.box_rows) & (p.page - 1), pg[b]);
         }
         if (ok && t > 0) ok = load_v(t - 1);
@@ -335,8 +329,7 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
     if (ok) {
       tc_fence_after();
       if (p.sink && live) l_run += exp2f(-m_run);
-      float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
-      if (p.gate != nullptr && live) inv *= 1.0f / (1.0f + expf(-p.gate[(size_t)(w.q_row0 + r) * p.ld_gate + h]));
+      const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
       __nv_bfloat16* orow = p.out + (size_t)(w.q_row0 + r) * p.ldo + h * p.dvp;
 #pragma unroll 1
       for (int c = 0; c < p.dv64 / 32; ++c) {
@@ -412,37 +405,6 @@ fold_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ talk
   }
 }
 
-// q'[h] of plain heads: f * q[h], turned by the token's row of `rope` ([T, 2 * half], or null); columns dp .. kc are zero
-__global__ void __launch_bounds__(kFoldThreads)
-turn_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ rope, int half, __nv_bfloat16* __restrict__ out, int H,
-            int dp, int kc, float f) {
-  bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
-  const float* qr = q + (size_t)blockIdx.x * ldq;
-  const float* rr = rope + (size_t)blockIdx.x * 2 * half;
-  __nv_bfloat16* orow = out + (size_t)blockIdx.x * H * kc;
-  for (int i = threadIdx.x * 4; i < H * kc; i += kFoldThreads * 4) {
-    const int h = i / kc, e = i % kc;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (e < dp) {                                              // dp % 8 == 0
-      const float* head = qr + h * dp;
-      v = *reinterpret_cast<const float4*>(head + e);
-      float* x = &v.x;
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int c = e + j;
-        if (rope != nullptr && c < 2 * half) {
-          const bool low = c < half;
-          const int k = low ? c : c - half;
-          const float b = head[low ? c + half : k], co = rr[k], si = rr[half + k];
-          x[j] = low ? x[j] * co - b * si : x[j] * co + b * si;
-        }
-      }
-    }
-    __align__(8) __nv_bfloat162 o[2] = {__floats2bfloat162_rn(v.x * f, v.y * f), __floats2bfloat162_rn(v.z * f, v.w * f)};
-    *reinterpret_cast<uint2*>(orow + i) = *reinterpret_cast<const uint2*>(o);
-  }
-}
-
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
                                   const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
                                   CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
@@ -498,30 +460,16 @@ int bg_talk_fold(const float* q, int ldq, const float* talk, void* out, int R, i
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
-// Queries of R rows of plain heads: q fp32 [R, ldq], rope [R, 2 * half] or null -> out bf16 [R, H, kc] (kc = dp rounded up to
-// 64), times scale * log2(e).
-int bg_talk_turn(const float* q, int ldq, const float* rope, int half, void* out, int R, int H, int dp, int kc, float scale,
-                 cudaStream_t stream) {
-  using namespace bg::talkpre;
-  if (R <= 0) return 0;
-  if (H <= 0 || dp <= 0 || dp % 8 || kc % 64 || kc < dp || ldq % 4 || (rope != nullptr && (half <= 0 || 2 * half > dp))) return -1;
-  bg::launch_pdl(turn_kernel, dim3(R), dim3(kFoldThreads), 0, stream, q, ldq, rope, half, reinterpret_cast<__nv_bfloat16*>(out), H,
-                 dp, kc, scale * 1.4426950408889634f);
-  return cudaGetLastError() == cudaSuccess ? 0 : -2;
-}
-
 // qf [R, H, kc] bf16 mixed queries of rows row_shift .. row_shift + R of the step; cache [pages, page, row] bf16 with
 // `page_stride` elements between pages; work: n_work x 4 ints (q_row0, n_q, block-table row, position of the first query),
-// q_row0 counted in rows of the step; out [T, ldo] bf16.  k_step 0: mixed queries, kc = G * dp rounded up to 64; dp: plain heads,
-// kc = dp rounded up to 64.  gate [T, ld_gate] fp32 or null.  page: a power of two >= 16; dvp <= 256.
+// q_row0 counted in rows of the step; out [T, ldo] bf16.  page: a power of two >= 16; dvp <= 256.
 int bg_talk_prefill(const void* qf, const void* cache, long long page_stride, int n_pages, int page, int row,
                     const int* block_table, int bt_stride, int bt_cols, const int* work, int n_work, int R, int row_shift,
-                    void* out, int ldo, int H, int G, int dp, int dvp, int kc, int chunk, int sink, int k_step,
-                    const float* gate, int ld_gate, int* status, cudaStream_t stream) {
+                    void* out, int ldo, int H, int G, int dp, int dvp, int kc, int chunk, int sink, int* status,
+                    cudaStream_t stream) {
   using namespace bg::talkpre;
   if (n_work <= 0) return 0;
-  if (H <= 0 || H > 65535 || G <= 0 || H % G || dp % 8 || dvp % 8 || dvp > 256 || kc % 64 ||
-      kc < (k_step > 0 ? dp : G * dp) || (k_step != 0 && k_step != dp) || page < 16 ||
+  if (H <= 0 || H > 65535 || G <= 0 || H % G || dp % 8 || dvp % 8 || dvp > 256 || kc % 64 || kc < G * dp || page < 16 ||
       (page & (page - 1)) || row != G * (dp + dvp) || page_stride % 8 || ldo % 8 || bt_cols <= 0)
     return -1;
   const int box_rows = page < 64 ? page : 64;
@@ -541,7 +489,6 @@ int bg_talk_prefill(const void* qf, const void* cache, long long page_stride, in
   Params p;
   p.work = reinterpret_cast<const Work*>(work);
   p.block_table = block_table; p.bt_stride = bt_stride; p.bt_cols = bt_cols; p.page = page; p.box_rows = box_rows;
-  p.k_step = k_step; p.gate = gate; p.ld_gate = ld_gate;
   p.KB = kc / 64; p.v_col0 = G * dp; p.dvp = dvp; p.dv64 = (dvp + 63) / 64 * 64; p.rep = H / G; p.chunk = chunk;
   p.sink = sink; p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo; p.row_shift = row_shift; p.status = status;
   const int stages = p.dv64 <= 128 ? 5 : 4;

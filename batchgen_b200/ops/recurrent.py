@@ -91,6 +91,14 @@ def recurrent_forward(p: RecurrentParams, q: torch.Tensor, k: torch.Tensor, v: t
         assert t is None or (t.dtype == torch.float32 and t.stride(1) == 1)
     assert out.stride(1) == 1 and slots.dtype == torch.int32
     T, a = q.shape[0], _Args()
+    qk, n = p.n_qk * p.dim_p, p.heads * p.vdim_p
+    for t, cols in ((q, qk), (k, qk), (v, n), (gate, n), (out, n), (low, p.heads * p.dim_p), (beta, p.heads), (gate_i, p.heads),
+                    (gate_f, p.heads), (rope, 0)):
+        assert t is None or (t.shape[0] == T and t.shape[1] >= cols), "rows or columns of an input do not match"
+    assert S.shape[1] == p.heads * p.dim_p * p.vdim_p and (cu is None or cu.shape[0] == slots.shape[0] + 1)
+    for name, cols in (("n", p.heads * p.dim_p), ("m", p.heads)) if p.rule == "mlstm" else ():
+        t = state[name]                                       # parts of one pool: the kernels step all of them by S's slot stride
+        assert t.dtype == torch.float32 and t.stride() == S.stride() and t.shape == (S.shape[0], cols)
     scratch = None
     if cu is not None or p.dim_p > 128 or p.vdim_p > 128:
         scratch = torch.empty(scratch_floats(p, T), dtype=torch.float32, device=q.device)

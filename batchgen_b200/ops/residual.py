@@ -186,6 +186,12 @@ def sandwich_norm(x: torch.Tensor, norm: Norm, eps: float, width: int, out_cols:
         assert t is None or (t.dtype == torch.float32 and t.stride(1) == 1)
     assert x.dtype == torch.float32 and (embed is None or embed.dtype == dtype) and (add is None) == (post is None)
     assert (ids is None or ids.dtype == torch.int32) and (rows is None or rows.dtype == torch.int64)
+    assert x.shape[1] >= W4 and norm.w.shape[0] == W4 and (post is None or post.w.shape[0] == W4)
+    for t in (add, add2):
+        assert t is None or (t.shape[0] == x.shape[0] and t.stride(0) >= W4)
+    if canon is not None:
+        taps = canon.w.shape[0]
+        assert canon.w.shape[1] == W4 and canon.hist.shape[1] == (taps - 1) * W4 and canon.slots.shape[0] == R
     assert canon is None or (rows is None and not raw and canon.slots.dtype == torch.int32 and canon.hist.stride(1) == 1)
     P = lambda n: (_ext.ptr(n.w if n is not None else None), _ext.ptr(n.b if n is not None else None))   # noqa: E731
     rc = _ext.lib().bg_sandwich_norm(

@@ -1,6 +1,8 @@
 """Paged grouped-query attention for layer-listed models.  Optional parts: heads' scores mixed before the softmax, chunked
-visibility, a zero-score sink, rotary positions on queries and keys, a sigmoid gate per head on the output.  Cache rows and one query row per CTA for decode and short pieces (``csrc/talking_attn.cu``), tensor-core
-flash attention over mixed queries for long pieces of prompts (``csrc/talking_prefill.cu``).
+visibility, a zero-score sink, rotary positions on queries and keys, a sigmoid gate per head on the output.
+
+Cache rows, and one query row per CTA for decode and short pieces: ``csrc/talking_attn.cu``; tensor-core flash attention for
+long pieces of prompts, over mixed queries (``csrc/talking_prefill.cu``) or plain heads (``csrc/gqa_prefill.cu``).
 """
 from __future__ import annotations
 
@@ -142,8 +144,9 @@ _FOLD_ROWS = 8192            # rows whose mixed queries are held at a time
 
 
 def prefill_supported(p: TalkParams, dtype: torch.dtype, page: int) -> bool:
-    """The tensor-core kernel reads bf16 pages and keeps one head's value columns in TMEM."""
-    return dtype == torch.bfloat16 and p.vdim_p <= 256 and page >= 16
+    """The tensor-core kernels read bf16 pages and keep one head's value columns in TMEM (plain heads: its queries in shared
+    memory)."""
+    return dtype == torch.bfloat16 and p.vdim_p <= 256 and page >= 16 and (p.talk is not None or p.dim_p <= 256)
 
 
 def prefill_work(cu: Sequence[int], ctx: Sequence[int], chunk: int, min_tokens: int = 1) -> List[Tuple[int, int, int, int]]:
@@ -183,7 +186,7 @@ def attend_prefill(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_ta
     P, page, row = cache.shape
     H, G = p.heads, p.kv_heads
     plain = p.talk is None
-    assert plain or rope is None, "mixed heads with rotary queries are not covered"
+    assert plain or (rope is None and gate is None), "mixed heads with rotary queries or output gates are not covered"
     kc = -(-(p.dim_p if plain else G * p.dim_p) // 64) * 64
     assert q.dtype == torch.float32 and q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == cache.dtype == torch.bfloat16
     assert row == p.kv_row and cache.stride(1) == row and block_table.dtype == torch.int32
@@ -191,17 +194,20 @@ def attend_prefill(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_ta
     for lo, n, work in blocks:
         qf = torch.empty(n, H, kc, dtype=torch.bfloat16, device=q.device)
         if plain:
-            rc = L.bg_talk_turn(_ext.ptr(q[lo:]), _i(q.stride(0)), _ext.ptr(rope[lo:] if rope is not None else None),
+            rc = L.bg_gqa_prompt_queries(_ext.ptr(q[lo:]), _i(q.stride(0)), _ext.ptr(rope[lo:] if rope is not None else None),
                                 _i(rope.shape[1] // 2 if rope is not None else 0), _ext.ptr(qf), _i(n), _i(H), _i(p.dim_p),
                                 _i(kc), ctypes.c_float(p.scale), _ext.stream())
         else:
             rc = L.bg_talk_fold(_ext.ptr(q[lo:]), _i(q.stride(0)), _ext.ptr(p.talk), _ext.ptr(qf), _i(n), _i(H), _i(G),
                                 _i(p.dim_p), _i(kc), ctypes.c_float(p.scale), _ext.stream())
-        _ext.check(rc, "bg_talk_fold")
-        rc = L.bg_talk_prefill(
-            _ext.ptr(qf), _ext.ptr(cache), ctypes.c_longlong(cache.stride(0)), _i(P), _i(page), _i(row),
-            _ext.ptr(block_table), _i(block_table.stride(0)), _i(block_table.shape[1]), _ext.ptr(work), _i(work.shape[0]),
-            _i(n), _i(lo), _ext.ptr(out), _i(out.stride(0)), _i(H), _i(G), _i(p.dim_p), _i(p.vdim_p), _i(kc), _i(p.chunk),
-            _i(p.sink), _i(p.dim_p if plain else 0), _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0),
-            _ext.ptr(_ext.status_word(q.device)), _ext.stream())
-        _ext.check(rc, "bg_talk_prefill")
+        _ext.check(rc, "bg_gqa_prompt_queries" if plain else "bg_talk_fold")
+        where = (_ext.ptr(qf), _ext.ptr(cache), ctypes.c_longlong(cache.stride(0)), _i(P), _i(page), _i(row),
+                 _ext.ptr(block_table), _i(block_table.stride(0)), _i(block_table.shape[1]), _ext.ptr(work), _i(work.shape[0]),
+                 _i(n), _i(lo), _ext.ptr(out), _i(out.stride(0)), _i(H), _i(G), _i(p.dim_p), _i(p.vdim_p), _i(kc), _i(p.chunk),
+                 _i(p.sink))
+        status = _ext.ptr(_ext.status_word(q.device))
+        if plain:
+            rc = L.bg_gqa_prompt(*where, _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0), status, _ext.stream())
+        else:
+            rc = L.bg_talk_prefill(*where, status, _ext.stream())
+        _ext.check(rc, "bg_gqa_prompt" if plain else "bg_talk_prefill")

@@ -218,8 +218,8 @@ def _pamevik_kernels(dev, timer: _Timer, peaks) -> List[Dict[str, object]]:
         R, size, slots, cu, init = _state_case(dev, B, T)
         row_seq = None if T == 1 else torch.arange(B, dtype=torch.int32, device=dev).repeat_interleave(T)
         z, out = torch.randn(R, 5 * HD + 64, device=dev), torch.empty(R, HD, dtype=bf, device=dev)
-        S = {"S": torch.zeros(B + 1, HD * D, device=dev), "n": torch.zeros(B + 1, HD, device=dev),
-             "m": torch.zeros(B + 1, H, device=dev)}
+        pool = torch.zeros(B + 1, HD * D + HD + H, device=dev)
+        S = {"S": pool[:, :HD * D], "n": pool[:, HD * D:HD * (D + 1)], "m": pool[:, HD * (D + 1):]}
         q, k, v, g, low = (z[:, i * HD:(i + 1) * HD] for i in range(5))
         gates = z[:, 5 * HD:5 * HD + H]
         base = dict(heads=H, dim_p=D, vdim=D, vdim_p=D, norm_w=torch.ones(HD, device=dev), eps=1e-6)
