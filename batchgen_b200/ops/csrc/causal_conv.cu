@@ -13,6 +13,7 @@ namespace cconv {
 
 constexpr int kThreads = 128;
 constexpr int kRun = 16;        // tokens a thread walks
+constexpr int kAhead = 8;       // of them loaded ahead
 
 struct Params {
   const float* x;          // [T, ldx]
@@ -68,30 +69,41 @@ __global__ void __launch_bounds__(kThreads) piece_kernel(const Params p) {
     const int j = t - first + taps - 1;                           // row of the history
     return init && j >= 0 ? ld4(p.hist + slot * p.hist_stride + (size_t)j * p.C + c) : zero;
   };
-  for (int t = lo; t < hi; ++t) {
-    const int s = p.row_seq[t];
-    if (s != seq) {
-      seq = s;
-      first = p.cu[s];
-      slot = p.slots[s];
-      init = slot >= 0 && (p.has_initial == nullptr || p.has_initial[s] != 0);
+  for (int g = lo; g < hi; g += kAhead) {
+    float4 xs[kAhead];                                            // in flight together
+    int seqs[kAhead];
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+      const int t = min(g + i, hi - 1);
+      xs[i] = ld4(p.x + (size_t)t * p.ldx + c);
+      seqs[i] = p.row_seq[t];
+    }
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+      const int t = g + i;
+      if (t >= hi) break;
+      if (seqs[i] != seq) {
+        seq = seqs[i];
+        first = p.cu[seq];
+        slot = p.slots[seq];
+        init = slot >= 0 && (p.has_initial == nullptr || p.has_initial[seq] != 0);
+        if (TAPS > 0) {
+#pragma unroll
+          for (int j = 0; j < NW - 1; ++j) win[j + 1] = input(t - TAPS + 1 + j);
+        }
+      }
+      float4 y = zero;
       if (TAPS > 0) {
 #pragma unroll
-        for (int j = 0; j < NW - 1; ++j) win[j + 1] = input(t - TAPS + 1 + j);
+        for (int j = 0; j < NW - 1; ++j) win[j] = win[j + 1];
+        win[NW - 1] = xs[i];
+#pragma unroll
+        for (int j = 0; j < NW; ++j) fma4(y, w[j], win[j]);
+      } else {
+        for (int j = 0; j < taps; ++j) fma4(y, ld4(p.w + (size_t)j * p.C + c), input(t - taps + 1 + j));
       }
+      store4(out + (size_t)t * p.ldo, finish<KIND>(y, xs[i]));
     }
-    const float4 x = ld4(p.x + (size_t)t * p.ldx + c);
-    float4 y = zero;
-    if (TAPS > 0) {
-#pragma unroll
-      for (int j = 0; j < NW - 1; ++j) win[j] = win[j + 1];
-      win[NW - 1] = x;
-#pragma unroll
-      for (int j = 0; j < NW; ++j) fma4(y, w[j], win[j]);
-    } else {
-      for (int j = 0; j < taps; ++j) fma4(y, ld4(p.w + (size_t)j * p.C + c), input(t - taps + 1 + j));
-    }
-    store4(out + (size_t)t * p.ldo, finish<KIND>(y, x));
   }
 }
 

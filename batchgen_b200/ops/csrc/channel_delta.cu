@@ -54,10 +54,10 @@ __global__ void __launch_bounds__(256) channel_records(const Args p, float* __re
   const float* kr = p.k + (size_t)t * p.ld_k + h / p.rep * K;
   const float* lr = p.low + (size_t)t * p.ld_low + h * K;
   const float b = sigm(p.beta[(size_t)t * p.ld_beta + h]), rate = p.rate[h];
-  float4 q[2], k[2];
+  float4 q[kMaxK / 128], k[kMaxK / 128];
   float kk = 0.f, qq = 0.f, qk = 0.f;
 #pragma unroll
-  for (int n = 0; n < 2; ++n) {
+  for (int n = 0; n < kMaxK / 128; ++n) {
     const int e = n * 128 + lane * 4;
     q[n] = k[n] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (e >= K) continue;
@@ -70,7 +70,7 @@ __global__ void __launch_bounds__(256) channel_records(const Args p, float* __re
   kk = warp_sum(kk); qq = warp_sum(qq); qk = warp_sum(qk);
   const float rk = 1.0f / sqrtf(kk + p.ueps), rq = p.q_scale / sqrtf(qq + p.ueps), bk = b * rk;
 #pragma unroll
-  for (int n = 0; n < 2; ++n) {
+  for (int n = 0; n < kMaxK / 128; ++n) {
     const int e = n * 128 + lane * 4;
     if (e >= K) continue;
     const float4 l = *reinterpret_cast<const float4*>(lr + e), d = *reinterpret_cast<const float4*>(p.bias0 + h * K + e);

@@ -53,11 +53,11 @@ __global__ void __launch_bounds__(256) general_records(const Args p, float* __re
   if (h >= p.H) return;
   const int D = p.K;
   float* out = rec + ((size_t)t * p.H + h) * rec_floats<GeneralDelta>(D, D);
-  float4 k[2], au[2], v[2];
+  float4 k[kMaxK / 128], au[kMaxK / 128], v[kMaxK / 128];
   float kk = 0.f, rk = 0.f, rak = 0.f;
   auto at = [&](const float* x, int ld, int e) { return *reinterpret_cast<const float4*>(x + (size_t)t * ld + h * D + e); };
 #pragma unroll
-  for (int n = 0; n < 2; ++n) {
+  for (int n = 0; n < kMaxK / 128; ++n) {
     const int e = n * 128 + lane * 4;
     k[n] = au[n] = v[n] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (e >= D) continue;
@@ -80,7 +80,7 @@ __global__ void __launch_bounds__(256) general_records(const Args p, float* __re
   kk = warp_sum(kk); rk = warp_sum(rk); rak = warp_sum(rak);
   const float s = sqrtf(kk + p.ueps), inv = 1.0f / s;
 #pragma unroll
-  for (int n = 0; n < 2; ++n) {
+  for (int n = 0; n < kMaxK / 128; ++n) {
     const int e = n * 128 + lane * 4;
     if (e >= D) continue;
     *reinterpret_cast<float4*>(out + D + e) = make_float4(k[n].x * inv, k[n].y * inv, k[n].z * inv, k[n].w * inv);
@@ -95,7 +95,7 @@ __global__ void __launch_bounds__(256) general_records(const Args p, float* __re
 
 extern "C" {
 
-// offs: host array of five column offsets (r, k, v, g, a).  dt: 0 = bf16 output, 1 = fp32.  D a multiple of 8, <= 256.
+// offs: host array of five column offsets (r, k, v, g, a).  dt: 0 = bf16 output, 1 = fp32.  D a multiple of 8, <= 512.
 // T: rows of z.  `scratch` (T * H * (6 D + 4) floats: records, then the scan's outputs) selects the prompt path; null the
 // decode kernel (D <= 128, one token per sequence).
 int bg_delta_forward(int dt, const float* z, int ldz, const int* offs, const float* wl, int ld_wl, const float* w0,

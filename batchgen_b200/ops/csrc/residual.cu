@@ -155,59 +155,74 @@ struct SandwichParams {
   int keep;
 };
 
-constexpr int kWarps = kThreads / 32;
-// sum over the block; `red` holds kWarps floats and is not reused before the next barrier of the caller
-__device__ __forceinline__ float block_sum(float v, float* red) {
-  v = warp_sum(v);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  float s = 0.f;
-#pragma unroll
-  for (int i = 0; i < kWarps; ++i) s += red[i];
-  return s;
+constexpr int kMaxWarps = kThreads / 32;
+
+// (count, mean, sum of squared deviations) of two parts together
+struct Moments { float n, mean, m2; };
+__device__ __forceinline__ void merge(Moments& a, const Moments& b) {
+  const float n = a.n + b.n;
+  if (n == 0.f) return;
+  const float d = b.mean - a.mean, r = b.n / n;
+  a.m2 += b.m2 + d * d * a.n * r;
+  a.mean += d * r;
+  a.n = n;
 }
 
-// One block per row; thread i owns the 4-wide vectors i, i + 256, ... and keeps the first NV of them in registers: D <= 1024 NV.
-// Columns D .. D4 hold zeros (weights and biases are zero there).
+// One block of up to 256 threads per row; thread i owns the 4-wide vectors i, i + blockDim, ... (NV of them) in registers.  All
+// loads of the row are issued before any is used.  A norm's mean and variance meet in one barrier: every thread takes both of
+// its own values first, then partial moments are merged.  Columns D .. D4 hold zeros (weights and biases are zero there).
 template <typename OT, int NV>
 __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichParams p) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
-  __shared__ float red[6][kWarps];
-  const int tid = threadIdx.x;
+  __shared__ float red[2][kMaxWarps];
+  __shared__ Moments part[2][kMaxWarps];
+  const int tid = threadIdx.x, NT = blockDim.x, warps = NT >> 5;
   const long long t = p.rows != nullptr ? p.rows[blockIdx.x] : (long long)blockIdx.x;
   float* xr = p.x + t * p.ldx;
   const int D = p.D, nv = (D + 3) / 4;
   const float inv_d = 1.0f / (float)D;
-  float4 f[NV], s[NV];
+  float4 f[NV], s[NV], u[NV];
   auto each = [&](auto fn) {
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
-      const int v = tid + n * kThreads;
+      const int v = tid + n * NT;
       if (v < nv) fn(n, v * 4);
     }
   };
   auto ld4 = [](const float* q, int c) { return *reinterpret_cast<const float4*>(q + c); };
   auto dot = [](const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
-  auto mask = [&](float4 v, int c) {                               // zero past D
-    if (c + 1 >= D) v.y = 0.f;
-    if (c + 2 >= D) v.z = 0.f;
-    if (c + 3 >= D) v.w = 0.f;
-    return v;
+  auto mask = [&](float4& v, int c) {                              // zero past D
+    if (c + 4 > D) {
+      if (c + 1 >= D) v.y = 0.f;
+      if (c + 2 >= D) v.z = 0.f;
+      v.w = 0.f;
+    }
   };
   // mean and 1 / sqrt(variance + eps) of the vectors in v (mean 0 without centring)
-  auto moments = [&](float4 (&v)[NV], int center, float* r0, float* r1, float& mean, float& rstd) {
-    mean = 0.f;
-    if (center) {
-      float sum = 0.f;
-      each([&](int n, int) { sum += (v[n].x + v[n].y) + (v[n].z + v[n].w); });
-      mean = block_sum(sum, r0) * inv_d;
-    }
-    float sq = 0.f;
+  auto moments = [&](float4 (&v)[NV], int center, Moments* out, float& mean, float& rstd) {
+    Moments m = {0.f, 0.f, 0.f};
     each([&](int n, int c) {
-      const float4 d = mask(make_float4(v[n].x - mean, v[n].y - mean, v[n].z - mean, v[n].w - mean), c);
-      sq += dot(d);
+      m.mean += (v[n].x + v[n].y) + (v[n].z + v[n].w);
+      m.n += (float)min(4, D - c);
     });
-    rstd = 1.0f / sqrtf(block_sum(sq, r1) * inv_d + p.eps);
+    m.mean = center && m.n > 0.f ? m.mean / m.n : 0.f;
+    each([&](int n, int c) {
+      float4 d = make_float4(v[n].x - m.mean, v[n].y - m.mean, v[n].z - m.mean, v[n].w - m.mean);
+      mask(d, c);
+      m.m2 += dot(d);
+    });
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const Moments b = {__shfl_xor_sync(0xffffffffu, m.n, o), __shfl_xor_sync(0xffffffffu, m.mean, o),
+                         __shfl_xor_sync(0xffffffffu, m.m2, o)};
+      merge(m, b);
+    }
+    if ((tid & 31) == 0) out[tid >> 5] = m;
+    __syncthreads();
+    Moments all = out[0];
+    for (int i = 1; i < warps; ++i) merge(all, out[i]);
+    mean = all.mean;
+    rstd = 1.0f / sqrtf(all.m2 * inv_d + p.eps);
   };
   auto norm4 = [&](const float4& v, float mean, float rstd, const float* w, const float* b, int c) {
     const float4 g = ld4(w, c);
@@ -228,17 +243,18 @@ __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichP
       f[n].w = c + 3 < D ? to_f(er[c + 3]) * p.escale : 0.f;
     });
   } else {
-    each([&](int n, int c) { f[n] = mask(ld4(xr, c), c); });
+    each([&](int n, int c) { f[n] = ld4(xr, c); });
   }
   if (p.a != nullptr) {
     const float* ar = p.a + t * p.lda;
-    each([&](int n, int c) { s[n] = mask(ld4(ar, c), c); });
+    each([&](int n, int c) { s[n] = ld4(ar, c); });
     if (p.b != nullptr) {
       const float* br = p.b + t * p.ldb;
-      float4 u[NV];
+      each([&](int n, int c) { u[n] = ld4(br, c); });
       float sa = 0.f, sb = 0.f;
       each([&](int n, int c) {
-        u[n] = mask(ld4(br, c), c);
+        mask(s[n], c);
+        mask(u[n], c);
         sa += dot(s[n]);
         sb += dot(u[n]);
       });
@@ -247,25 +263,29 @@ __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichP
       if ((tid & 31) == 0) { red[0][tid >> 5] = sa; red[1][tid >> 5] = sb; }
       __syncthreads();
       float ta = 0.f, tb = 0.f;
-#pragma unroll
-      for (int i = 0; i < kWarps; ++i) { ta += red[0][i]; tb += red[1][i]; }
+      for (int i = 0; i < warps; ++i) { ta += red[0][i]; tb += red[1][i]; }
       const float ra = 0.5f / sqrtf(ta * inv_d + p.eps), rb = 0.5f / sqrtf(tb * inv_d + p.eps);
       each([&](int n, int c) {
         const float4 ga = ld4(p.wa, c), gb = ld4(p.wb, c);
         s[n] = make_float4(s[n].x * ra * ga.x + u[n].x * rb * gb.x, s[n].y * ra * ga.y + u[n].y * rb * gb.y,
                            s[n].z * ra * ga.z + u[n].z * rb * gb.z, s[n].w * ra * ga.w + u[n].w * rb * gb.w);
       });
+    } else {
+      each([&](int n, int c) { mask(s[n], c); });
     }
     float mean, rstd;
-    moments(s, p.center1, red[2], red[3], mean, rstd);
+    moments(s, p.center1, part[0], mean, rstd);
     each([&](int n, int c) {
       const float4 o = norm4(s[n], mean, rstd, p.w1, p.b1, c);
+      mask(f[n], c);
       f[n].x += o.x; f[n].y += o.y; f[n].z += o.z; f[n].w += o.w;
     });
+  } else {
+    each([&](int n, int c) { mask(f[n], c); });
   }
   if (p.keep) each([&](int n, int c) { *reinterpret_cast<float4*>(xr + c) = f[n]; });
   float mean, rstd;
-  moments(f, p.center2, red[4], red[5], mean, rstd);
+  moments(f, p.center2, part[1], mean, rstd);
   OT* yr = reinterpret_cast<OT*>(p.y) + (size_t)blockIdx.x * p.ldy;
   float* hr = reinterpret_cast<float*>(p.y) + (size_t)blockIdx.x * p.ldy;
   const int slot = p.cw != nullptr ? p.slots[blockIdx.x] : -1;
@@ -293,7 +313,7 @@ __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichP
     else store4(yr + c, h);
   });
   if (!p.raw)
-    for (int c = D4 + tid * 4; c < p.ldy; c += kThreads * 4) store4(yr + c, make_float4(0.f, 0.f, 0.f, 0.f));
+    for (int c = D4 + tid * 4; c < p.ldy; c += NT * 4) store4(yr + c, make_float4(0.f, 0.f, 0.f, 0.f));
 }
 
 __device__ __forceinline__ float sigmoid_acc(float x) { return 1.0f / (1.0f + expf(-x)); }
@@ -416,12 +436,24 @@ int bg_sandwich_norm(int dt, float* x, int ldx, const long long* rows, const int
   p.a = a; p.b = b; p.lda = lda; p.ldb = ldb; p.wa = wa; p.wb = wb; p.w1 = w1; p.b1 = b1; p.center1 = center1;
   p.w2 = w2; p.b2 = b2; p.center2 = center2; p.y = y; p.ldy = ldy; p.raw = raw; p.cw = cw; p.hist = hist;
   p.hist_stride = hist_stride; p.slots = slots; p.taps = taps; p.D = D; p.eps = eps; p.keep = keep;
-#define BG_SANDWICH(NV)                                                                                                  do {                                                                                                                     if (dt == 0) bg::launch_pdl(sandwich_norm_kernel<__nv_bfloat16, NV>, dim3(R), dim3(kThreads), 0, stream, p);           else bg::launch_pdl(sandwich_norm_kernel<float, NV>, dim3(R), dim3(kThreads), 0, stream, p);                         } while (0)
-  if (D <= 1024) BG_SANDWICH(1);
-  else if (D <= 2048) BG_SANDWICH(2);
-  else if (D <= 4096) BG_SANDWICH(4);
-  else if (D <= 8192) BG_SANDWICH(8);
-  else BG_SANDWICH(16);
+  const int nv = D4 / 4;
+#define BG_SANDWICH(NV)                                                                                             \
+  do {                                                                                                              \
+    const dim3 block(((nv + NV - 1) / NV + 31) / 32 * 32);                                                          \
+    if (dt == 0) bg::launch_pdl(sandwich_norm_kernel<__nv_bfloat16, NV>, dim3(R), block, 0, stream, p);             \
+    else bg::launch_pdl(sandwich_norm_kernel<float, NV>, dim3(R), block, 0, stream, p);                             \
+  } while (0)
+  switch ((nv + kThreads - 1) / kThreads) {
+    case 1: BG_SANDWICH(1); break;
+    case 2: BG_SANDWICH(2); break;
+    case 3: BG_SANDWICH(3); break;
+    case 4: BG_SANDWICH(4); break;
+    case 5:
+    case 6: BG_SANDWICH(6); break;
+    case 7:
+    case 8: BG_SANDWICH(8); break;
+    default: BG_SANDWICH(16); break;
+  }
 #undef BG_SANDWICH
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }

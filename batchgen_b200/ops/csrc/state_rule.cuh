@@ -44,7 +44,7 @@ struct Args {
   float q_scale, k_scale, cap, ueps, eps, den_eps;       // cap: mlstm's soft cap, general_delta's decay scale
 };
 
-constexpr int kMaxK = 256;
+constexpr int kMaxK = 512;
 
 template <typename OT> __device__ __forceinline__ void put4(OT* p, float4 v);
 template <> __device__ __forceinline__ void put4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
@@ -90,7 +90,8 @@ struct Coefs {
   float ys, os, ov, oy, us, w;
 };
 
-template <typename Rule, typename OT, int NR>
+// SQ: K = V = 4 NR, known when the kernel is compiled.
+template <typename Rule, typename OT, int NR, bool SQ>
 __global__ void __launch_bounds__(288) decode_kernel(const Args p, int items) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   extern __shared__ __align__(128) float ring[];                // kBufs x K * V
@@ -100,7 +101,7 @@ __global__ void __launch_bounds__(288) decode_kernel(const Args p, int items) {
   __shared__ __align__(16) float sv[2][128];
   __shared__ float red[2][3][4], red_o[2][4];
   const int tid = threadIdx.x, lane = tid & 31;
-  const int K = p.K, V = p.V, H = p.H, KV = K * V, Q = V / 4;
+  const int K = SQ ? 4 * NR : p.K, V = SQ ? 4 * NR : p.V, H = p.H, KV = K * V, Q = V / 4;
   volatile int* abort_flag = &abort_s;
   if (tid == 0) {
     for (int s = 0; s < kBufs; ++s) { mbar_init(&full[s], 1); mbar_init(&done[s], 1); }
@@ -203,7 +204,7 @@ __global__ void __launch_bounds__(288) decode_kernel(const Args p, int items) {
     float* Sb = ring + (size_t)buf * KV + (size_t)rg * NR * V + 4 * quad;
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
     const int rows = min(NR, max(K - rg * NR, 0));
-    const bool whole = K == 4 * NR;                              // every lane has all its rows: no guards
+    const bool whole = SQ || K == 4 * NR;                              // every lane has all its rows: no guards
     float2 y[2], q[2];
     y[0] = y[1] = q[0] = q[1] = make_float2(0.f, 0.f);
     if constexpr (Rule::kRead) {
@@ -426,7 +427,7 @@ scan_kernel(const Args p, const float* __restrict__ rec, float* __restrict__ o_o
       const bool in = init && col_ok && i < K;
 #pragma unroll
       for (int c = 0; c < C; ++c) {
-        const float v = in && col + c < width ? Sg[(size_t)i * row + c] : 0.f;
+        const float v = in && (!Rule::kDen || col + c < width) ? Sg[(size_t)i * row + c] : 0.f;
         if (j & 1) S[c][2 * n + j / 2].y = v;
         else S[c][2 * n + j / 2].x = v;
       }
@@ -446,14 +447,16 @@ scan_kernel(const Args p, const float* __restrict__ rec, float* __restrict__ o_o
 #pragma unroll
     for (int tt = 0; tt < kScanGroup; ++tt) {
       const float* tok = base + tt * TOK;
-      const float2 cc = *reinterpret_cast<const float2*>(tok + NUM);
-      float2 sv[C], q[C];
+      float2 sv[C], q[C], cc;
+      auto load_values = [&]() {
+        cc = *reinterpret_cast<const float2*>(tok + NUM);
 #pragma unroll
-      for (int c = 0; c < C; c += 2) {
-        const float2 s = *reinterpret_cast<const float2*>(tok + NUM + 4 + lc + c);
-        sv[c] = twice(s.x);
-        sv[c + 1] = twice(s.y);
-      }
+        for (int c = 0; c < C; c += 2) {
+          const float2 s = *reinterpret_cast<const float2*>(tok + NUM + 4 + lc + c);
+          sv[c] = twice(s.x);
+          sv[c + 1] = twice(s.y);
+        }
+      };
 #pragma unroll
       for (int c = 0; c < C; ++c) q[c] = make_float2(0.f, 0.f);
       if constexpr (Rule::kRead) {
@@ -481,6 +484,7 @@ scan_kernel(const Args p, const float* __restrict__ rec, float* __restrict__ o_o
         for (int o = 1; o < 16; o <<= 1)
 #pragma unroll
           for (int c = 0; c < C; ++c) ys[c] += __shfl_xor_sync(0xffffffffu, ys[c], o);
+        load_values();
         float2 ny[C];                                            // what the write vector is multiplied by
 #pragma unroll
         for (int c = 0; c < C; ++c) ny[c] = twice(Rule::kTwoTerms ? -ys[c] : sv[c].x - ys[c]);
@@ -508,6 +512,7 @@ scan_kernel(const Args p, const float* __restrict__ rec, float* __restrict__ o_o
       } else {
         const float4* k4 = reinterpret_cast<const float4*>(tok) + lr;
         const float4* r4 = k4 + W / 4;
+        load_values();
         const float2 w2 = twice(cc.x);
 #pragma unroll
         for (int n = 0; n < R / 4; ++n) {
@@ -558,7 +563,7 @@ scan_kernel(const Args p, const float* __restrict__ rec, float* __restrict__ o_o
         if (i < K) {
 #pragma unroll
           for (int c = 0; c < C; ++c)
-            if (col + c < width) Sg[(size_t)i * row + c] = (j & 1) ? S[c][2 * n + j / 2].y : S[c][2 * n + j / 2].x;
+            if (!Rule::kDen || col + c < width) Sg[(size_t)i * row + c] = (j & 1) ? S[c][2 * n + j / 2].y : S[c][2 * n + j / 2].x;
         }
       }
   }
@@ -617,7 +622,8 @@ static int launch_scan_as(const Args& p, const float* rec, float* o, float* den,
 template <typename Rule, int R>
 static int launch_scan_rows(const Args& p, const float* rec, float* o, float* den, cudaStream_t stream) {
   const long long ctas = (long long)((p.V + kScanCols - 1) / kScanCols) * p.H * p.nseq;
-  return ctas <= 296 ? launch_scan_as<Rule, R, 2>(p, rec, o, den, stream) : launch_scan_as<Rule, R, 4>(p, rec, o, den, stream);
+  if constexpr (R > 16) return launch_scan_as<Rule, R, 2>(p, rec, o, den, stream);       // registers
+  else return ctas <= 296 ? launch_scan_as<Rule, R, 2>(p, rec, o, den, stream) : launch_scan_as<Rule, R, 4>(p, rec, o, den, stream);
 }
 // records, then scan and output; `rec`, `o`, `den`, `gates` are parts of the scratch
 template <typename Rule>
@@ -626,7 +632,8 @@ static int launch_scan(const Args& p, const float* rec, float* o, float* den, co
   if (p.K <= 64) rc = launch_scan_rows<Rule, 4>(p, rec, o, den, stream);
   else if (p.K <= 128) rc = launch_scan_rows<Rule, 8>(p, rec, o, den, stream);
   else if (p.K <= 192) rc = launch_scan_rows<Rule, 12>(p, rec, o, den, stream);
-  else rc = launch_scan_rows<Rule, 16>(p, rec, o, den, stream);
+  else if (p.K <= 256) rc = launch_scan_rows<Rule, 16>(p, rec, o, den, stream);
+  else rc = launch_scan_rows<Rule, 32>(p, rec, o, den, stream);
   if (rc != 0) return rc;
   const dim3 grid(p.T, (p.H + 7) / 8);
   const float* d = Rule::kDen ? den : nullptr;
@@ -635,16 +642,21 @@ static int launch_scan(const Args& p, const float* rec, float* o, float* den, co
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
-template <typename Rule, typename OT, int NR>
-static int launch_decode_as(const Args& p, cudaStream_t stream) {
+template <typename Rule, typename OT, int NR, bool SQ>
+static int launch_decode_sized(const Args& p, cudaStream_t stream) {
   const size_t smem = (size_t)kBufs * p.K * p.V * sizeof(float);
   static DeviceOnce once;
-  auto kern = decode_kernel<Rule, OT, NR>;
+  auto kern = decode_kernel<Rule, OT, NR, SQ>;
   if (!ensure_dynamic_smem(kern, 3 * 128 * 128 * sizeof(float), once)) return -4;
   const int per_sm = smem > 100 * 1024 || NR > 16 ? 1 : smem > 48 * 1024 ? 2 : 3;
   const int items = p.nseq * p.H, most = p.num_sms * per_sm;
   bg::launch_pdl(kern, dim3(items < most ? items : most), dim3(288), smem, stream, p, items);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+template <typename Rule, typename OT, int NR>
+static int launch_decode_as(const Args& p, cudaStream_t stream) {
+  return p.K == 4 * NR && p.V == 4 * NR ? launch_decode_sized<Rule, OT, NR, true>(p, stream)
+                                        : launch_decode_sized<Rule, OT, NR, false>(p, stream);
 }
 template <typename Rule, typename OT>
 static int launch_decode_rows(const Args& p, cudaStream_t stream) {

@@ -43,6 +43,7 @@ struct Params {
   float* part_o;                // [R, n_splits, H * dvp]
   float* part_ml;               // [R, n_splits, H, 2]
   int H, G, dp, dvp, chunk, sink, n_splits;
+  int k_warps;                  // warps with a K buffer (all of them unless heads are very wide)
   float scale_log2;
   const float* rope;            // [T, 2 * half] cosines, then sines, or null
   int half;
@@ -181,13 +182,13 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
     for (int i = 0; i < 4; ++i) acc[n][i][0] = acc[n][i][1] = make_float2(0.f, 0.f);
 
   long long off = my_lo < my_hi ? key_offset(my_lo) : -1;
-  if (my_lo < my_hi && warp < units) fetch(warp, off);
+  if (my_lo < my_hi && warp < p.k_warps && warp < units) fetch(warp, off);
   __syncthreads();                                                 // q_s, tt, m_s, l_s
   for (int tile = my_lo; tile < my_hi; ++tile) {
     const long long off_now = off;
     if (warp == 0) koff[lane] = off_now;
     off = tile + 1 < my_hi ? key_offset(tile + 1) : -1;
-    for (int u = warp; u < units; u += kWarps) {
+    for (int u = warp < p.k_warps ? warp : units; u < units; u += p.k_warps) {
       cp_wait0();
       __syncwarp();
       const int c = u / hg_n, h0 = c * rep + (u % hg_n) * 4, nh = min(4, rep - (u % hg_n) * 4);
@@ -214,7 +215,7 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
       for (int i = 0; i < 4; ++i)
         if (i < nh) raw[(h0 + i) * NT + lane] = s[i].x + s[i].y;
       __syncwarp();
-      if (u + kWarps < units) fetch(u + kWarps, off_now);
+      if (u + p.k_warps < units) fetch(u + p.k_warps, off_now);
       else if (tile + 1 < my_hi) fetch(warp, off);                 // next tile's rows fly during the rest of this tile
     }
     __syncthreads();
@@ -406,12 +407,12 @@ kv_write_kernel(const float* __restrict__ kv, int ld, const long long* __restric
 }
 
 template <typename KT, int NI, bool MIX>
-static int launch_rows_as(const Params& p, int R, cudaStream_t stream) {
-  size_t kb = kWarps * kbuf_bytes<KT>(p.dp);
+static int launch_rows_as(Params p, int R, cudaStream_t stream) {
+  const size_t fixed = smem_floats(p.H, p.dp, MIX) * sizeof(float), one = kbuf_bytes<KT>(p.dp), most = 227 * 1024;
   const size_t red = (size_t)kThreads * 16 * sizeof(float);
-  if (kb < red) kb = red;
-  const size_t smem = smem_floats(p.H, p.dp, MIX) * sizeof(float) + kb;
-  if (smem > 227 * 1024) return -3;
+  for (p.k_warps = kWarps; p.k_warps > 1 && fixed + p.k_warps * one > most; --p.k_warps) {}
+  const size_t smem = fixed + (p.k_warps * one < red ? red : p.k_warps * one);
+  if (smem > most) return -3;
   static DeviceOnce once;
   auto kern = rows_kernel<KT, NI, MIX>;
   if (!ensure_dynamic_smem(kern, 227 * 1024, once)) return -4;
@@ -449,15 +450,17 @@ int bg_talk_rows(int dt, const float* q, int ldq, const float* talk, const void*
   p.rope = rope; p.half = half; p.gate = gate; p.ld_gate = ld_gate;
   const int items = G * ((H / G + 3) / 4) * (dvp / 4);
   const int ni = (items + kThreads - 1) / kThreads;
-  if (ni > 4) return -1;
+  if (ni > 8) return -1;
   if (dt == 0) {
     if (ni == 1) return launch_rows<__nv_bfloat16, 1>(p, R, stream);
     if (ni == 2) return launch_rows<__nv_bfloat16, 2>(p, R, stream);
-    return launch_rows<__nv_bfloat16, 4>(p, R, stream);
+    if (ni <= 4) return launch_rows<__nv_bfloat16, 4>(p, R, stream);
+    return launch_rows<__nv_bfloat16, 8>(p, R, stream);
   }
   if (ni == 1) return launch_rows<float, 1>(p, R, stream);
   if (ni == 2) return launch_rows<float, 2>(p, R, stream);
-  return launch_rows<float, 4>(p, R, stream);
+  if (ni <= 4) return launch_rows<float, 4>(p, R, stream);
+  return launch_rows<float, 8>(p, R, stream);
 }
 
 int bg_talk_kv_write(int dt, const float* kv, int ld, const long long* slots, void* cache, long long page_stride, int page,

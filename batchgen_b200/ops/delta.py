@@ -81,6 +81,6 @@ def delta_forward(z: torch.Tensor, offs: Tuple[int, int, int, int, int], wl: tor
         _i(p.dim_p), _i(p.dim), ctypes.c_float(p.decay_scale), ctypes.c_float(p.unit_eps), ctypes.c_float(p.eps),
         _ext.ptr(scratch), _i(_ext.num_sms(z.device)), _ext.ptr(_ext.status_word(z.device)), _ext.stream())
     if rc == -1:
-        raise _ext.KernelError(f"delta_forward: {p.heads} heads of {p.dim_p} are outside the kernels' contract (width <= 256)")
+        raise _ext.KernelError(f"delta_forward: {p.heads} heads of {p.dim_p} are outside the kernels' contract (width <= 512)")
     _ext.check(rc, "bg_delta_forward", kernels=3 if scratch is not None else 1)
     return out

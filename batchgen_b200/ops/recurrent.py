@@ -119,7 +119,7 @@ def recurrent_forward(p: RecurrentParams, q: torch.Tensor, k: torch.Tensor, v: t
     rc = _ext.lib().bg_recurrent_forward(ctypes.byref(a), _ext.stream())
     if rc == -1:
         raise _ext.KernelError(f"recurrent_forward: {p.heads} heads of {p.dim_p} x {p.vdim_p} are outside the kernels' "
-                               "contract (key width <= 256)")
+                               "contract (key width <= 512)")
     _ext.check(rc, "bg_recurrent_forward", kernels=1 if scratch is None else 4 if p.rule == "mlstm" else 3)
     return out
 

@@ -134,7 +134,7 @@ def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table
         _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0), _ext.stream())
     if rc in (-1, -3):
         raise _ext.KernelError(f"attend_rows: heads {H}/{p.kv_heads}, widths {p.dim_p}/{p.vdim_p} are outside the kernel's "
-                               "contract (shared memory of one CTA, 1,024 head-column items)")
+                               "contract (shared memory of one CTA, 2,048 head-column items)")
     _ext.check(rc, "bg_talk_rows", kernels=2 if num_splits > 1 else 1)
 
 

@@ -154,9 +154,9 @@ def _layered_contract(cfg, world: int, on_gpu: bool) -> List[str]:
     for i, s in enumerate(cfg.layer_specs):
         f = s.mlp
         for m in s.mixers:
-            if m.recurrent and m.dim > 256:
-                bad.append(f"layer {i}: {m.kind} head width {m.dim} exceeds 256")
-            if not m.recurrent and m.kv_heads * -(-(m.heads // m.kv_heads) // 4) * (m.vdim_p // 4) > 1024:
+            if m.recurrent and m.dim > 512:
+                bad.append(f"layer {i}: {m.kind} head width {m.dim} exceeds 512")
+            if not m.recurrent and m.kv_heads * -(-(m.heads // m.kv_heads) // 4) * (m.vdim_p // 4) > 2048:
                 bad.append(f"layer {i}: {m.heads} heads x {m.vdim} value channels exceed the decode attention kernel")
         if f.kind == "moe" and (f.top > 16 or f.experts > 1024 or f.top > f.experts):
             bad.append(f"layer {i}: top {f.top} of {f.experts} experts (the router takes up to 16 of 1,024)")

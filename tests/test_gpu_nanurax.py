@@ -121,7 +121,7 @@ def _delta_case(T, H, d, seed):
     return z, offs, pad(low), p, args, gate, norm, dp
 
 
-@pytest.mark.parametrize("H,d", [(3, 8), (2, 20), (5, 48), (2, 64), (3, 90), (2, 128), (1, 160), (1, 256)])
+@pytest.mark.parametrize("H,d", [(3, 8), (2, 20), (5, 48), (2, 64), (3, 90), (2, 128), (1, 160), (1, 256), (1, 392)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_delta_rule_prompts_continuations_and_decoding(H, d, dtype):
     from batchgen_b200.ops import delta

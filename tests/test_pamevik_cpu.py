@@ -261,9 +261,9 @@ def test_planner_and_preflight_know_the_design():
     assert model_contract(tiny, 1, True)
     with pytest.raises(PreflightError, match="one GPU"):
         model_contract(tiny, 2, True)
-    wide = pm.config(64, 64, [pm.mlstm(1, 264, 8, 1.0)])
+    wide = pm.config(64, 64, [pm.mlstm(1, 520, 8, 1.0)])
     from batchgen_b200.config import pamevik_config
-    with pytest.raises(PreflightError, match="256"):
+    with pytest.raises(PreflightError, match="512"):
         model_contract(pamevik_config(wide), 1, True)
 
 
