@@ -157,20 +157,11 @@ struct SandwichParams {
 
 constexpr int kMaxWarps = kThreads / 32;
 
-// (count, mean, sum of squared deviations) of two parts together
-struct Moments { float n, mean, m2; };
-__device__ __forceinline__ void merge(Moments& a, const Moments& b) {
-  const float n = a.n + b.n;
-  if (n == 0.f) return;
-  const float d = b.mean - a.mean, r = b.n / n;
-  a.m2 += b.m2 + d * d * a.n * r;
-  a.mean += d * r;
-  a.n = n;
-}
+struct Moments { float n, mean, m2; };      // of a warp's elements: count, mean, sum of squared deviations from that mean
 
 // One block of up to 256 threads per row; thread i owns the 4-wide vectors i, i + blockDim, ... (NV of them) in registers.  All
-// loads of the row are issued before any is used.  A norm's mean and variance meet in one barrier: every thread takes both of
-// its own values first, then partial moments are merged.  Columns D .. D4 hold zeros (weights and biases are zero there).
+// loads of the row are issued before any is used.  A norm's mean and variance meet in one barrier: every warp takes both of its
+// own elements first, then the warps' moments are put together.  Columns D .. D4 hold zeros (weights and biases are zero there).
 template <typename OT, int NV>
 __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichParams p) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
@@ -198,31 +189,36 @@ __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichP
       v.w = 0.f;
     }
   };
+  float warp_n = 0.f;
+  each([&](int, int c) { warp_n += (float)min(4, D - c); });
+  warp_n = warp_sum(warp_n);
+  const float inv_n = warp_n > 0.f ? 1.0f / warp_n : 0.f;
   // mean and 1 / sqrt(variance + eps) of the vectors in v (mean 0 without centring)
   auto moments = [&](float4 (&v)[NV], int center, Moments* out, float& mean, float& rstd) {
-    Moments m = {0.f, 0.f, 0.f};
-    each([&](int n, int c) {
-      m.mean += (v[n].x + v[n].y) + (v[n].z + v[n].w);
-      m.n += (float)min(4, D - c);
-    });
-    m.mean = center && m.n > 0.f ? m.mean / m.n : 0.f;
-    each([&](int n, int c) {
-      float4 d = make_float4(v[n].x - m.mean, v[n].y - m.mean, v[n].z - m.mean, v[n].w - m.mean);
-      mask(d, c);
-      m.m2 += dot(d);
-    });
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const Moments b = {__shfl_xor_sync(0xffffffffu, m.n, o), __shfl_xor_sync(0xffffffffu, m.mean, o),
-                         __shfl_xor_sync(0xffffffffu, m.m2, o)};
-      merge(m, b);
+    float own = 0.f, m2 = 0.f;
+    if (center) {
+      each([&](int n, int) { own += (v[n].x + v[n].y) + (v[n].z + v[n].w); });
+      own = warp_sum(own) * inv_n;
     }
-    if ((tid & 31) == 0) out[tid >> 5] = m;
+    each([&](int n, int c) {
+      float4 d = make_float4(v[n].x - own, v[n].y - own, v[n].z - own, v[n].w - own);
+      mask(d, c);
+      m2 += dot(d);
+    });
+    m2 = warp_sum(m2);
+    if ((tid & 31) == 0) out[tid >> 5] = {warp_n, own, m2};
     __syncthreads();
-    Moments all = out[0];
-    for (int i = 1; i < warps; ++i) merge(all, out[i]);
-    mean = all.mean;
-    rstd = 1.0f / sqrtf(all.m2 * inv_d + p.eps);
+    mean = 0.f;
+    if (center) {
+      for (int i = 0; i < warps; ++i) mean += out[i].n * out[i].mean;
+      mean *= inv_d;
+    }
+    m2 = 0.f;
+    for (int i = 0; i < warps; ++i) {
+      const float d = out[i].mean - mean;
+      m2 += out[i].m2 + out[i].n * d * d;
+    }
+    rstd = 1.0f / sqrtf(m2 * inv_d + p.eps);
   };
   auto norm4 = [&](const float4& v, float mean, float rstd, const float* w, const float* b, int c) {
     const float4 g = ld4(w, c);
