@@ -44,6 +44,8 @@ struct ChannelDelta {
 };
 
 // records: g | g k | b k | g q | b (k . q), k and q normalised
+// N: K <= 128 N
+template <int N>
 __global__ void __launch_bounds__(256) channel_records(const Args p, float* __restrict__ rec) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   const int t = blockIdx.x, h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -54,10 +56,10 @@ __global__ void __launch_bounds__(256) channel_records(const Args p, float* __re
   const float* kr = p.k + (size_t)t * p.ld_k + h / p.rep * K;
   const float* lr = p.low + (size_t)t * p.ld_low + h * K;
   const float b = sigm(p.beta[(size_t)t * p.ld_beta + h]), rate = p.rate[h];
-  float4 q[kMaxK / 128], k[kMaxK / 128];
+  float4 q[N], k[N];
   float kk = 0.f, qq = 0.f, qk = 0.f;
 #pragma unroll
-  for (int n = 0; n < kMaxK / 128; ++n) {
+  for (int n = 0; n < N; ++n) {
     const int e = n * 128 + lane * 4;
     q[n] = k[n] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (e >= K) continue;
@@ -70,7 +72,7 @@ __global__ void __launch_bounds__(256) channel_records(const Args p, float* __re
   kk = warp_sum(kk); qq = warp_sum(qq); qk = warp_sum(qk);
   const float rk = 1.0f / sqrtf(kk + p.ueps), rq = p.q_scale / sqrtf(qq + p.ueps), bk = b * rk;
 #pragma unroll
-  for (int n = 0; n < kMaxK / 128; ++n) {
+  for (int n = 0; n < N; ++n) {
     const int e = n * 128 + lane * 4;
     if (e >= K) continue;
     const float4 l = *reinterpret_cast<const float4*>(lr + e), d = *reinterpret_cast<const float4*>(p.bias0 + h * K + e);
@@ -88,7 +90,9 @@ int channel_delta_forward(const Args& p, cudaStream_t stream) {
   if (p.low == nullptr || p.beta == nullptr || p.rate == nullptr || p.bias0 == nullptr) return -1;
   if (p.scratch == nullptr) return launch_decode<ChannelDelta>(p, stream);
   float* o = p.scratch + (size_t)p.T * p.H * rec_floats<ChannelDelta>(p.K, p.V);
-  bg::launch_pdl(channel_records, dim3(p.T, (p.H + 7) / 8), dim3(256), 0, stream, p, p.scratch);
+  if (p.K <= 128) bg::launch_pdl(channel_records<1>, dim3(p.T, (p.H + 7) / 8), dim3(256), 0, stream, p, p.scratch);
+  else if (p.K <= 256) bg::launch_pdl(channel_records<2>, dim3(p.T, (p.H + 7) / 8), dim3(256), 0, stream, p, p.scratch);
+  else bg::launch_pdl(channel_records<4>, dim3(p.T, (p.H + 7) / 8), dim3(256), 0, stream, p, p.scratch);
   return launch_scan<ChannelDelta>(p, p.scratch, o, nullptr, nullptr, stream);
 }
 

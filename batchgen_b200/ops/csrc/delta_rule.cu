@@ -47,17 +47,19 @@ struct GeneralDelta {
 };
 
 // records: w | u | a * u | w * r | c1, c2, 0, 0 | v * sqrt(kk + ueps), so that k v^T = u sv^T and o = q - c1 y + c2 sv
+// N: K <= 128 N
+template <int N>
 __global__ void __launch_bounds__(256) general_records(const Args p, float* __restrict__ rec) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   const int t = blockIdx.x, h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (h >= p.H) return;
   const int D = p.K;
   float* out = rec + ((size_t)t * p.H + h) * rec_floats<GeneralDelta>(D, D);
-  float4 k[kMaxK / 128], au[kMaxK / 128], v[kMaxK / 128];
+  float4 k[N], au[N], v[N];
   float kk = 0.f, rk = 0.f, rak = 0.f;
   auto at = [&](const float* x, int ld, int e) { return *reinterpret_cast<const float4*>(x + (size_t)t * ld + h * D + e); };
 #pragma unroll
-  for (int n = 0; n < kMaxK / 128; ++n) {
+  for (int n = 0; n < N; ++n) {
     const int e = n * 128 + lane * 4;
     k[n] = au[n] = v[n] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (e >= D) continue;
@@ -80,7 +82,7 @@ __global__ void __launch_bounds__(256) general_records(const Args p, float* __re
   kk = warp_sum(kk); rk = warp_sum(rk); rak = warp_sum(rak);
   const float s = sqrtf(kk + p.ueps), inv = 1.0f / s;
 #pragma unroll
-  for (int n = 0; n < kMaxK / 128; ++n) {
+  for (int n = 0; n < N; ++n) {
     const int e = n * 128 + lane * 4;
     if (e >= D) continue;
     *reinterpret_cast<float4*>(out + D + e) = make_float4(k[n].x * inv, k[n].y * inv, k[n].z * inv, k[n].w * inv);
@@ -114,7 +116,9 @@ int bg_delta_forward(int dt, const float* z, int ldz, const int* offs, const flo
   if (check_args(p) != 0 || offs[4] % 4) return -1;
   if (scratch == nullptr) return launch_decode<GeneralDelta>(p, stream);
   float* o = scratch + (size_t)T * H * rec_floats<GeneralDelta>(D, D);
-  bg::launch_pdl(general_records, dim3(T, (H + 7) / 8), dim3(256), 0, stream, p, scratch);
+  if (p.K <= 128) bg::launch_pdl(general_records<1>, dim3(T, (H + 7) / 8), dim3(256), 0, stream, p, scratch);
+  else if (p.K <= 256) bg::launch_pdl(general_records<2>, dim3(T, (H + 7) / 8), dim3(256), 0, stream, p, scratch);
+  else bg::launch_pdl(general_records<4>, dim3(T, (H + 7) / 8), dim3(256), 0, stream, p, scratch);
   return launch_scan<GeneralDelta>(p, scratch, o, nullptr, nullptr, stream);
 }
 

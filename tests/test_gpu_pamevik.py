@@ -150,7 +150,7 @@ def test_rotary_table_is_exact_far_away():
 
 
 # ---------------------------------------------------------------- recurrences
-RULE_SHAPES = [(3, 12, 20, 3), (6, 24, 40, 2), (2, 64, 32, 2), (2, 128, 128, 1), (3, 90, 60, 3), (4, 32, 128, 4), (2, 136, 48, 1),
+RULE_SHAPES = [(3, 12, 20, 3), (6, 24, 40, 2), (2, 64, 24, 2), (2, 128, 128, 1), (3, 90, 60, 3), (4, 32, 128, 4), (2, 136, 48, 1),
                (1, 40, 200, 1), (2, 160, 136, 2), (1, 200, 264, 1), (1, 256, 8, 1), (2, 392, 24, 1), (1, 512, 40, 1)]
 
 
@@ -404,7 +404,7 @@ def _attention_case(lens, H, G, d, dv, rd, page, dtype, seed=0, edit=None):
     return q, p, pool, bt.to(DEV), want, dict(rope=rope, gate=torch.cat(gates).to(DEV)), (pos + 1).to(torch.int32).to(DEV), seq, T
 
 
-SHAPES = [(9, 3, 56, 48, 56, 64), (4, 4, 20, 36, 6, 16), (8, 1, 64, 128, 32, 64), (32, 8, 128, 128, 128, 64), (1, 1, 8, 8, 2, 32),
+SHAPES = [(9, 3, 56, 48, 56, 64), (4, 4, 20, 36, 6, 16), (8, 1, 80, 128, 32, 64), (32, 8, 128, 128, 128, 64), (1, 1, 8, 8, 2, 32),
           (16, 2, 40, 200, 24, 128), (10, 2, 96, 24, 96, 64), (6, 2, 136, 264, 60, 64), (2, 1, 384, 40, 128, 64), (12, 12, 8, 512, 8, 32)]
 
 
