@@ -30,11 +30,18 @@ class MixerSpec:
     vdim: int = 0                          # value width of a head
     scale: float = 1.0                     # attention: factor of the scores
     chunk: int = 0                         # attention: keys are seen inside the query's own chunk of this many positions (0 = all)
+    window: int = 0                        # attention: the last so many positions are seen, the query's own among them (0 = all)
+    keep_first: int = 0                    # attention with a window: this many first positions of a sequence stay visible
+    bias: bool = False                     # attention: biases on the q, k, v and output projections
+    qk_norm: bool = False                  # attention: RMS norm of every query and key head, weights shared by the heads
     talking: bool = False                  # attention: a [heads, heads] matrix mixes the heads' scores before the softmax
     sink: bool = False                     # attention: one is added to the softmax denominator
     out_gate: bool = False                 # attention: a sigmoid gate per head scales its output
-    rot_dims: int = 0                      # attention, retention: leading head dimensions with rotary positions (rotate half)
+    rot_dims: int = 0                      # attention, retention: leading head dimensions with rotary positions
     rot_base: float = 10000.0
+    rot_interleaved: bool = False          # pairs (2 i, 2 i + 1) turn together; else (i, i + rot_dims / 2)
+    yarn: Tuple[float, ...] = ()           # YaRN frequencies: (factor, original positions, fast turns, slow turns); () = plain ones
+    out_scale: float = 1.0                 # factor of the mixer's output
     decay_rank: int = 0                    # general_delta, channel_delta: width of the low-rank decay projection
     gate_rank: int = 0                     # channel_delta: width of the low-rank output-gate projection
     conv: int = 0                          # channel_delta: taps of the short convolutions of q, k and v
@@ -98,7 +105,9 @@ class MixerSpec:
     def param_count(self, width: int) -> int:
         qk, v, H = self.heads * self.dim, self.heads * self.vdim, self.heads
         if self.kind == "attention":
-            return width * (H + self.kv_heads) * (self.dim + self.vdim) + (H * H if self.talking else 0)
+            n = width * (H + self.kv_heads) * (self.dim + self.vdim) + (H * H if self.talking else 0)
+            n += (H + self.kv_heads) * self.dim + self.kv_heads * self.vdim + width if self.bias else 0
+            return n + (2 * self.dim if self.qk_norm else 0)
         if self.kind == "general_delta":
             return width * (6 * qk + self.decay_rank) + self.decay_rank * qk
         if self.kind == "channel_delta":
@@ -112,20 +121,30 @@ class MlpSpec:
     """The feed-forward of one layer of a layer-listed model."""
     kind: str = "none"                     # none | dense | moe
     ff: int = 0                            # dense width, or width of one routed expert
-    activation: str = "gelu_tanh"          # gelu_tanh | swiglu_oai (clamped gate and up, sigmoid slope 1.702, up + 1) | relu2 (no gate)
+    activation: str = "gelu_tanh"          # gelu_tanh | silu | swiglu_oai (clamped gate and up, sigmoid slope 1.702, up + 1) | relu2 (no gate)
     limit: float = 0.0                     # clamp of swiglu_oai
     experts: int = 0
     top: int = 0
     weight_on_input: bool = False          # the routing weight scales the expert's input instead of its output
-    shared_ff: int = 0                     # shared expert (0 = none), same activation, scaled by a sigmoid gate per token
+    shared_ff: int = 0                     # shared expert (0 = none), same activation
     shared_limit: float = 0.0
+    shared_gate: bool = True               # the shared expert's output is scaled by a sigmoid gate per token
+    scoring: str = "sigmoid"               # router scores: sigmoid | softmax_all (over all experts)
+    correction: bool = False               # a bias per expert takes part in the choice, not in the weights
+    groups: int = 1                        # experts form this many groups, of which the best ``keep_groups`` take part
+    keep_groups: int = 1
+    group_score: str = "top2"              # a group counts with the sum of its two best choice scores, or its "max"
+    norm_weights: bool = False             # weights are divided by their sum
+    router_scale: float = 1.0
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: MixerSpec
     mlp: MlpSpec = MlpSpec()
-    second: Optional[MixerSpec] = None     # a mixer beside the first: both outputs are RMS-normed over the width and averaged
+    second: Optional[MixerSpec] = None     # a mixer beside the first: sandwich blocks average both RMS-normed outputs, hyper-
+                                           # connected blocks add them (``MixerSpec.out_scale``)
+    weights_of: int = -1                   # >= 0: the layer whose tensors this one uses, with a cache and state of its own
 
     @property
     def mixers(self) -> Tuple[MixerSpec, ...]:
@@ -150,7 +169,7 @@ class LayerSpec:
 @dataclass
 class ModelConfig:
     name: str = "tiny-deepseek-v3"
-    family: str = "deepseek_v3"  # deepseek_v3 | deepseek_v2 | deepseek_v4 | glm5 | kimi_k3 | kimi_k25 | gpt_oss | minimax | mixtral | qwen2_moe | nanurax | pamevik
+    family: str = "deepseek_v3"  # deepseek_v3 | deepseek_v2 | deepseek_v4 | glm5 | kimi_k3 | kimi_k25 | gpt_oss | minimax | mixtral | qwen2_moe | nanurax | pamevik | bolisun
     vocab_size: int = 1024
     hidden_size: int = 256
     num_layers: int = 2
@@ -224,6 +243,8 @@ class ModelConfig:
     sandwich: bool = False                 # False: mixer and feed-forward read one RMS norm and are added together (parallel
                                            # block); True: one after the other, a norm before and after each
     layer_norm: bool = False               # sandwich: norms subtract the mean and have biases (else RMS norms)
+    streams: int = 0                       # > 0: pre-norm blocks (mixer, then feed-forward) around this many residual streams with
+                                           # hyper-connections of fixed weights
     canon_taps: int = 0                    # sandwich: every sublayer reads h + conv(h), a causal convolution of this many taps
     checkpoint_dir: str = ""               # directory the config was read from (its .safetensors files are the weights)
     # ---- misc
@@ -350,7 +371,7 @@ class ModelConfig:
 
     def param_count(self) -> int:
         h = self.hidden_size
-        n = 2 * self.vocab_size * h
+        n = (1 if self.tie_word_embeddings and self.is_layered else 2) * self.vocab_size * h
         if self.is_v4:
             D, Di = self.head_dim, self.index_head_dim
             for l, r in enumerate(self.compress_ratios):
@@ -366,6 +387,8 @@ class ModelConfig:
             return n
         if self.is_layered:
             for spec in self.layer_specs:
+                if spec.weights_of >= 0:
+                    continue
                 f = spec.mlp
                 n += sum(m.param_count(h) for m in spec.mixers)
                 n += (2 if f.activation == "relu2" else 3) * h * f.ff * (f.experts if f.kind == "moe" else 1) + h * f.experts + 3 * h * f.shared_ff
@@ -405,9 +428,10 @@ class ModelConfig:
             kw["compress_ratios"] = tuple(kw["compress_ratios"])
         if "layer_specs" in kw:
             def mixer(m):
-                return None if m is None else MixerSpec(**{**m, "decay": tuple(m.get("decay", ()))})
+                return None if m is None else MixerSpec(**{**m, **{k: tuple(m.get(k, ())) for k in ("decay", "yarn")}})
             kw["layer_specs"] = tuple(
-                x if isinstance(x, LayerSpec) else LayerSpec(mixer(x["mixer"]), MlpSpec(**x["mlp"]), mixer(x.get("second")))
+                x if isinstance(x, LayerSpec) else LayerSpec(mixer(x["mixer"]), MlpSpec(**x["mlp"]), mixer(x.get("second")),
+                                                             x.get("weights_of", -1))
                 for x in kw["layer_specs"])
         return cls(**kw)
 
@@ -784,7 +808,80 @@ def _pamevik_dir(path: str, d: Dict) -> ModelConfig:
     return cfg
 
 
-_ARCHITECTURES = {"Nanurax": _nanurax_dir, "Pamevik": _pamevik_dir}        # config.json "architecture" -> reader of the model directory
+# ------------------------------------------------------------------ Bolisun: layer-listed config.json
+def _bolisun_layer(d: Dict, index: int) -> LayerSpec:
+    if d["type"] != "parallel":
+        raise ValueError(f"layer {index}: unknown mixer type {d['type']!r}")
+    m, f = d["mixer"], d.get("mlp")
+    a, r, rot, mask = m["left"], m["right"], m["left"].get("rot") or {}, m["left"].get("mask") or {}
+    sc = rot.get("scaling")
+    left = MixerSpec(
+        "attention", heads=a["heads"], dim=a["dim"], kv_heads=a.get("kv_heads", a["heads"]), vdim=a["vdim"], scale=float(a["scale"]),
+        window=int(mask.get("size", 0)), keep_first=int(mask.get("keep_first", 0)), bias=True, qk_norm=True,
+        rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)), rot_interleaved=True,
+        yarn=tuple(float(sc[k]) for k in ("factor", "original", "fast", "slow")) if sc else (), out_scale=float(m["left_scale"]))
+    right = MixerSpec("retention", heads=r["heads"], dim=r["dim"], vdim=r["vdim"], decay=tuple(float(x) for x in r["decay"]),
+                      out_scale=float(m["right_scale"]))
+    if left.heads % left.kv_heads:
+        raise ValueError(f"layer {index}: {left.heads} heads do not divide over {left.kv_heads} key heads")
+    if left.rot_dims % 2 or left.rot_dims > left.dim:
+        raise ValueError(f"layer {index}: {left.rot_dims} rotary dimensions in heads of {left.dim}")
+    if mask and left.window < 1:
+        raise ValueError(f"layer {index}: a window of {left.window} positions")
+    if len(right.decay) != right.heads:
+        raise ValueError(f"layer {index}: {len(right.decay)} decays for {right.heads} heads")
+    mlp = MlpSpec()
+    if f and f["kind"] == "dense":
+        mlp = MlpSpec("dense", ff=f["ff"], activation="swiglu_oai", limit=float(f["limit"]))
+    elif f and f["kind"] == "moe":
+        ro = f["router"]
+        g = ro.get("groups") or {"count": 1, "keep": 1}
+        mlp = MlpSpec("moe", ff=f["expert"]["ff"], activation="silu", experts=ro["experts"], top=ro["top"],
+                      shared_ff=(f.get("shared") or {}).get("ff", 0), shared_gate=False, scoring="softmax_all", correction=True,
+                      groups=g["count"], keep_groups=g["keep"], group_score="max", norm_weights=True, router_scale=float(ro["scale"]))
+        if mlp.experts % mlp.groups or mlp.keep_groups > mlp.groups or mlp.top > mlp.experts // mlp.groups * mlp.keep_groups:
+            raise ValueError(f"layer {index}: top {mlp.top} of {mlp.experts} experts in the best {mlp.keep_groups} of {mlp.groups} groups")
+    elif f:
+        raise ValueError(f"layer {index}: unknown feed-forward kind {f['kind']!r}")
+    return LayerSpec(left, mlp, right)
+
+
+def bolisun_config(d: Dict, name: str = "bolisun") -> ModelConfig:
+    """A Bolisun config.json (parsed) as a ``ModelConfig``."""
+    layers = []
+    for i, x in enumerate(d["layers"]):
+        j, seen = i, {i}
+        while d["layers"][j].get("weights_of") is not None:
+            j = d["layers"][j]["weights_of"]
+            if not 0 <= j < len(d["layers"]) or j in seen:
+                raise ValueError(f"layer {i}: weights of layer {j}")
+            seen.add(j)
+        spec = _bolisun_layer({**d["layers"][j], **x}, i)
+        if j != i:
+            if spec != _bolisun_layer(d["layers"][j], j):
+                raise ValueError(f"layer {i} differs from layer {j}, whose weights it uses")
+            spec = dataclasses.replace(spec, weights_of=j)
+        layers.append(spec)
+    moe = [s.mlp for s in layers if s.mlp.kind == "moe"]
+    return ModelConfig(
+        name=name, family="bolisun", vocab_size=d["vocab"], hidden_size=d["width"], num_layers=len(layers), layer_specs=tuple(layers),
+        embed_scale=float(d["embedding"]["scale"]), rms_eps=float(d["norm"]["eps"]), streams=int(d["streams"]), tie_word_embeddings=True,
+        # summaries that planners read; the layers themselves are described by ``layer_specs``
+        num_heads=max(m.heads for s in layers for m in s.mixers), num_kv_heads=max(s.mixer.kv_heads for s in layers),
+        head_dim=max(m.dim for s in layers for m in s.mixers), sliding_window=max(s.mixer.window for s in layers), first_k_dense=0,
+        intermediate_size=max((s.mlp.ff for s in layers if s.mlp.kind == "dense"), default=0),
+        moe_intermediate_size=max((f.ff for f in moe), default=0), n_routed_experts=max((f.experts for f in moe), default=0),
+        num_experts_per_tok=max((f.top for f in moe), default=0), n_shared_experts=int(any(f.shared_ff for f in moe)),
+        attention_bias=True, scoring_func="softmax_all", max_position_embeddings=1 << 30, eos_token_id=-1, bos_token_id=-1)
+
+
+def _bolisun_dir(path: str, d: Dict) -> ModelConfig:
+    cfg = bolisun_config(d, os.path.basename(os.path.normpath(path)) or "bolisun")
+    cfg.checkpoint_dir = path
+    return cfg
+
+
+_ARCHITECTURES = {"Nanurax": _nanurax_dir, "Pamevik": _pamevik_dir, "Bolisun": _bolisun_dir}        # config.json "architecture" -> reader of the model directory
 
 
 def load_model_dir(path: str) -> ModelConfig:
@@ -851,7 +948,41 @@ def pamevik_bench() -> ModelConfig:
                            "layers": [cd, ml, dict(cd), par]}, "pamevik-bench", {0: (128, 128), 2: (128, 128)})
 
 
+def tiny_bolisun() -> ModelConfig:
+    """A dense layer, a mixture layer that runs twice, a layer without a feed-forward."""
+    def layer(window, keep, mlp):
+        return {"type": "parallel", "mlp": mlp, "mixer": {
+            "left_scale": 0.7, "right_scale": 1.1,
+            "left": {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 24, "scale": 0.2, "mask": {"size": window, "keep_first": keep},
+                     "rot": {"base": 9000.0, "dims": 16, "scaling": {"factor": 4.0, "original": 64, "fast": 8.0, "slow": 1.0}}},
+            "right": {"heads": 3, "dim": 16, "vdim": 40, "decay": [0.9, 0.97, 0.995]}}}
+    moe = {"kind": "moe", "expert": {"ff": 40}, "shared": {"ff": 56},
+           "router": {"experts": 8, "top": 2, "scale": 1.5, "groups": {"count": 4, "keep": 2}}}
+    return bolisun_config({
+        "vocab": 320, "width": 120, "streams": 3, "norm": {"eps": 1e-5}, "embedding": {"scale": 2.0},
+        "layers": [layer(33, 5, {"kind": "dense", "ff": 200, "limit": 2.0}), layer(20, 0, moe), dict(layer(20, 0, moe), weights_of=1),
+                   layer(50, 2, None)]}, "tiny-bolisun")
+
+
+def bolisun_bench() -> ModelConfig:
+    """Layers of a real model's size: four layers of windowed attention beside retention, one dense and three mixture
+    feed-forwards (64 experts of which 8 run, and a shared one), the last mixture layer with the weights of the one before."""
+    dense = {"kind": "dense", "ff": 9216, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": 1024}, "shared": {"ff": 1024},
+           "router": {"experts": 64, "top": 8, "scale": 2.5, "groups": {"count": 8, "keep": 4}}}
+    par = {"type": "parallel", "mixer": {
+        "left_scale": 0.5, "right_scale": 0.5,
+        "left": {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024, "keep_first": 64},
+                 "rot": {"base": 1e6, "dims": 128, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}},
+        "right": {"heads": 32, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 7 * i / 31) for i in range(32)]}}}
+    return bolisun_config({"vocab": 163840, "width": 2304, "streams": 2, "norm": {"eps": 1e-6}, "embedding": {"scale": 48.0},
+                           "layers": [dict(par, mlp=dense), dict(par, mlp=moe), dict(par, mlp=moe), dict(par, mlp=moe, weights_of=2)]},
+                          "bolisun-bench")
+
+
 _PRESETS = {
+    "tiny-bolisun": tiny_bolisun,
+    "bolisun-bench": bolisun_bench,
     "tiny-pamevik": tiny_pamevik,
     "pamevik-bench": pamevik_bench,
     "tiny-nanurax": tiny_nanurax,
@@ -908,6 +1039,7 @@ _PATTERNS = [
     (r"minimax", "minimax-m2.5"),
     (r"nanurax", "nanurax-bench"),
     (r"pamevik", "pamevik-bench"),
+    (r"bolisun", "bolisun-bench"),
 ]
 
 

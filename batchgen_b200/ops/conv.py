@@ -4,7 +4,7 @@ from __future__ import annotations
 import ctypes
 import math
 from dataclasses import dataclass
-from typing import Optional, Sequence
+from typing import Optional, Sequence, Tuple
 
 import torch
 
@@ -62,36 +62,59 @@ def _conv_ref(x, w, hist, slots, out, kind, cu_host, has_initial):
 
 @dataclass
 class Rotary:
-    """Rotary positions of the leading ``dims`` dimensions, pairs (i, i + dims / 2), angle position * base^(-2 i / dims)."""
+    """Rotary positions of the leading ``dims`` dimensions, angle position * base^(-2 i / dims) of pair i: dimensions
+    (i, i + dims / 2), or (2 i, 2 i + 1) when ``interleaved``.  ``yarn`` (factor, original positions, fast, slow): frequencies of
+    pairs that turn fewer than ``slow`` times within the original positions are divided by ``factor``, those of pairs that turn
+    more than ``fast`` times stay, with a ramp between them, and cosines and sines grow by 0.1 ln(factor) + 1."""
     dims: int
     base: float
-    turns: torch.Tensor = None             # [dims / 2] float64: base^(-2 i / dims) / (2 pi)
+    turns: torch.Tensor = None             # [dims / 2] float64: turns per position
+    interleaved: bool = False
+    yarn: Tuple[float, ...] = ()
+    mult: float = 1.0                      # of cosines and sines
 
     @classmethod
-    def make(cls, dims: int, base: float, device) -> Optional["Rotary"]:
+    def make(cls, dims: int, base: float, device, interleaved: bool = False, yarn: Tuple[float, ...] = ()) -> Optional["Rotary"]:
         if not dims:
             return None
         i = torch.arange(dims // 2, dtype=torch.float64)
-        return cls(dims, base, (torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * i / dims) / (2 * math.pi)).to(device))
+        f, mult = torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * i / dims), 1.0
+        if yarn:
+            factor, original, fast, slow = yarn
+
+            def pair_of(turns):            # the pair that makes this many turns within the original positions
+                return dims * math.log(original / (2 * math.pi * turns)) / (2 * math.log(base))
+            lo, hi = max(math.floor(pair_of(fast)), 0), min(math.ceil(pair_of(slow)), dims - 1)
+            ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+            f, mult = f / factor * ramp + f * (1 - ramp), 0.1 * math.log(factor) + 1.0
+        return cls(dims, base, (f / (2 * math.pi)).to(device), interleaved, tuple(yarn), mult)
+
+    @property
+    def key(self) -> Tuple:
+        """Rotaries with equal keys have equal tables."""
+        return self.dims, self.base, self.yarn
 
     def table(self, lens: torch.Tensor) -> torch.Tensor:
         """[T, dims] fp32 of the positions ``lens`` - 1: cosines, then sines.  The turn is reduced before it is rounded to
         32 bits, so far positions keep exact angles."""
         if not lens.is_cuda:
             a = (lens.double() - 1).unsqueeze(1) * self.turns * (2 * math.pi)
-            return torch.cat([a.cos(), a.sin()], 1).float()
+            return (torch.cat([a.cos(), a.sin()], 1) * self.mult).float()
         out = torch.empty(lens.shape[0], self.dims, dtype=torch.float32, device=lens.device)
         rc = _ext.lib().bg_rope_table(_ext.ptr(lens), _ext.ptr(self.turns), _ext.ptr(out), _i(lens.shape[0]),
-                                      _i(self.dims // 2), _ext.stream())
+                                      _i(self.dims // 2), ctypes.c_float(self.mult), _ext.stream())
         _ext.check(rc, "bg_rope_table")
         return out
 
 
-def rotate_ref(x: torch.Tensor, rope: Optional[torch.Tensor]) -> torch.Tensor:
+def rotate_ref(x: torch.Tensor, rope: Optional[torch.Tensor], interleaved: bool = False) -> torch.Tensor:
     """x [T, heads, d] turned by ``rope`` (``Rotary.table``)."""
     if rope is None:
         return x
     half = rope.shape[1] // 2
     c, s = rope[:, None, :half], rope[:, None, half:]
+    if interleaved:
+        u, v = x[..., 0:2 * half:2], x[..., 1:2 * half:2]
+        return torch.cat([torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2), x[..., 2 * half:]], -1)
     u, v = x[..., :half], x[..., half:2 * half]
     return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1)

@@ -153,15 +153,15 @@ __global__ void __launch_bounds__(kThreads) step_kernel(const Params p) {
 }
 
 __global__ void __launch_bounds__(kThreads)
-rope_kernel(const int* __restrict__ lens, const double* __restrict__ turns, float* __restrict__ out, int T, int half) {
+rope_kernel(const int* __restrict__ lens, const double* __restrict__ turns, float* __restrict__ out, int T, int half, float mult) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   const int i = blockIdx.x * kThreads + threadIdx.x, t = i / half, j = i % half;
   if (t >= T) return;
   const double a = (double)(lens[t] - 1) * turns[j];
   float s, c;
   sincospif(2.0f * (float)(a - rint(a)), &s, &c);
-  out[(size_t)t * 2 * half + j] = c;
-  out[(size_t)t * 2 * half + half + j] = s;
+  out[(size_t)t * 2 * half + j] = c * mult;
+  out[(size_t)t * 2 * half + half + j] = s * mult;
 }
 
 template <typename OT, int KIND>
@@ -213,13 +213,13 @@ int bg_causal_conv(int dt, int kind, const float* x, int ldx, const float* w, fl
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
-// lens [T]: position + 1; turns [half] turns per position -> out [T, 2 * half]: cosines, then sines
-int bg_rope_table(const int* lens, const double* turns, float* out, int T, int half, cudaStream_t stream) {
+// lens [T]: position + 1; turns [half] turns per position -> out [T, 2 * half]: cosines, then sines, times mult
+int bg_rope_table(const int* lens, const double* turns, float* out, int T, int half, float mult, cudaStream_t stream) {
   using namespace bg::cconv;
   if (T <= 0 || half <= 0) return 0;
   if ((long long)T * half > 0x7fffffffll) return -1;
   bg::launch_pdl(rope_kernel, dim3((unsigned)(((long long)T * half + kThreads - 1) / kThreads)), dim3(kThreads), 0, stream, lens,
-                 turns, out, T, half);
+                 turns, out, T, half, mult);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
