@@ -1,11 +1,14 @@
 """Layer-listed decoders (``ModelConfig.layer_specs``): every layer names its own token mixer(s) and feed-forward around an
-fp32 residual stream.  Two block forms:
+fp32 residual stream.  Three block forms:
 
 * parallel (Nanurax): mixer and feed-forward read one RMS norm and their outputs are added together.  Generalised delta-rule
   layers and chunked talking-heads attention layers, dense tanh-GELU or input-weighted clamped-SwiGLU mixture feed-forwards.
 * sandwich (Pamevik, ``ModelConfig.sandwich``): mixer, then feed-forward, each between two norms (``layer_norm``: with mean and
   bias) and behind an input convolution (``canon_taps``).  mLSTM, gated delta-rule with a decay per channel, and softmax
   attention beside retention; squared-ReLU feed-forwards.
+* hyper-connected (Bolisun, ``ModelConfig.streams``): mixer, then feed-forward, each behind an RMS norm that reads a weighted sum of
+  several residual streams; its output joins all streams, which are mixed with one another.  Windowed attention with normed heads
+  beside retention; clamped-SwiGLU feed-forwards and mixtures of experts; layers may share their weights.
 
 Same calling contract as ``Transformer``: ``forward(ids [T], meta, cache) -> fp32 logits``; all state lives in the caller's
 ``PagedKVCache`` (paged rows per attention layer, ``FlatStatePool`` slots for everything else a sequence carries), and a step
@@ -17,8 +20,9 @@ everything that reads the norm (mixer projections, router, shared-expert gate, d
 and the gated activation, written side by side -> one GEMM against [W_o | W_down], whose fp32 output is the layer's addend.
 Routed experts add their rows in the next residual kernel.  A sandwich block runs every sublayer as: norm of the previous
 sublayer's output + residual sum + norm + input convolution (one kernel in decode, two in prompts) -> one GEMM for everything
-that reads it -> core or activation -> one GEMM per output projection, whose fp32 output goes to the next norm kernel.  GEMM
-outputs stay fp32: what enters the recurrence, the scores, the router and the residual sum is never rounded to 16 bits; GEMM
+that reads it -> core or activation -> one GEMM per output projection, whose fp32 output goes to the next norm kernel.  A hyper-
+connected block does the same with one GEMM against both mixers' output projections side by side (their scales are in the
+operands), and its norm kernel mixes the streams and gathers the routed experts' rows.  GEMM outputs stay fp32: what enters the recurrence, the scores, the router and the residual sum is never rounded to 16 bits; GEMM
 operands are bf16, or fp32 in the 32-bit form of the model.
 
 Widths: the contraction side of every operand is padded with zeros to a multiple of 64 (one TMA / MMA block), head widths
@@ -31,7 +35,7 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from ..config import LayerSpec, ModelConfig
+from ..config import LayerSpec, MlpSpec, ModelConfig
 from ..ops import conv, gemm, residual
 from ..ops import moe as moe_ops
 from ..ops.moe import ExpertWeights
@@ -58,22 +62,29 @@ class LayeredLayer:
 
 @dataclass
 class Sublayer:
-    """One half of a sandwich block: mixer(s) side by side, or a feed-forward."""
+    """One half of a sandwich or hyper-connected block: mixer(s) side by side, or a feed-forward."""
     norm: residual.Norm
-    post: residual.Norm
+    post: Optional[residual.Norm]                 # sandwich: norm of the output
     w_in: torch.Tensor                            # [columns, width_p]
-    w_out: List[torch.Tensor]                     # per mixer W_o, or [W_down]: [width, operand width padded to K_ALIGN]
+    w_out: List[torch.Tensor]                     # per mixer W_o (hyper-connected: one matrix), or [W_down]: [width, operand width
+                                                  # padded to K_ALIGN]
     mixers: List[Mixer] = field(default_factory=list)       # empty: feed-forward
     branch_w: Optional[Tuple[torch.Tensor, torch.Tensor]] = None      # weights of two mixers' output norms
     canon_w: Optional[torch.Tensor] = None        # [taps, width4] fp32 input convolution
     canon_part: str = ""                          # its state part
-    ff: int = 0
+    ff: int = 0                                   # width of the dense or shared feed-forward (hyper-connected: padded to K_ALIGN)
+    hc: Optional[residual.Hyper] = None           # hyper-connected blocks, with what follows
+    bias: Optional[torch.Tensor] = None           # [width4] fp32, added to the output
+    mlp: Optional[MlpSpec] = None
+    seg: Dict[str, Tuple[int, int]] = field(default_factory=dict)     # feed-forward part -> (first column of the GEMM output, width)
+    correction: Optional[torch.Tensor] = None     # [experts] fp32
+    experts: Optional[ExpertWeights] = None
 
 
 @dataclass
 class LayeredWeights:
     embed: torch.Tensor = None                    # [vocab, width]
-    final_norm: torch.Tensor = None               # fp32 gain, or a ``residual.Norm`` (sandwich)
+    final_norm: torch.Tensor = None               # fp32 gain, or a ``residual.Norm`` (sandwich, hyper-connected)
     lm_head: torch.Tensor = None                  # [vocab, width_p]
     layers: List = field(default_factory=list)    # LayeredLayer, or lists of Sublayers
 
@@ -86,11 +97,12 @@ def build_layered_weights(cfg: ModelConfig, layout: ParallelLayout, src: WeightS
     Kp = pad_to(D, K_ALIGN)
     w = LayeredWeights()
     w.embed = src.get("embed", (V, D)).to(dtype).contiguous()
-    w.final_norm = (_norm(src, "final.norm", cfg) if cfg.sandwich
+    w.final_norm = (_norm(src, "final.norm", cfg) if cfg.sandwich or cfg.streams
                     else src.get("final.norm", (D,), "norm").float().contiguous())
-    w.lm_head = pad_cols(src.get("head", (V, D)).to(dtype), Kp).contiguous()
-    block = _build_sandwich if cfg.sandwich else _build_parallel
-    w.layers = [block(cfg, spec, f"l{i}.", src, dtype) for i, spec in enumerate(cfg.layer_specs)]
+    w.lm_head = pad_cols(w.embed if cfg.tie_word_embeddings else src.get("head", (V, D)).to(dtype), Kp).contiguous()
+    block = _build_hyper if cfg.streams else _build_sandwich if cfg.sandwich else _build_parallel
+    own = {i: block(cfg, spec, f"l{i}.", src, dtype) for i, spec in enumerate(cfg.layer_specs) if spec.weights_of < 0}
+    w.layers = [own[i if spec.weights_of < 0 else spec.weights_of] for i, spec in enumerate(cfg.layer_specs)]
     return w
 
 
@@ -133,6 +145,56 @@ def _build_sandwich(cfg: ModelConfig, spec: LayerSpec, p: str, src: WeightSource
     return out
 
 
+def _experts(f: MlpSpec, q: str, src: WeightSource, D: int, dtype: torch.dtype) -> ExpertWeights:
+    Kp, Fp = pad_to(D, K_ALIGN), pad_to(f.ff, K_ALIGN)
+    w13, wd = [], []
+    for e in range(f.experts):
+        ep = f"{q}e{e}."
+        gu = [pad_rows(src.get(ep + x, (f.ff, D)).to(dtype), Fp) for x in ("gate", "up")]
+        w13.append(pad_cols(torch.cat(gu, 0), Kp))
+        wd.append(pad_cols(src.get(ep + "down", (D, f.ff)).to(dtype), Fp))
+    return ExpertWeights(w13=torch.stack(w13), w2=torch.stack(wd), activation=f.activation, act_limit=f.limit)
+
+
+def _build_hyper(cfg: ModelConfig, spec: LayerSpec, p: str, src: WeightSource, dtype: torch.dtype) -> List[Sublayer]:
+    D, f, S = cfg.hidden_size, spec.mlp, cfg.streams
+    Kp, W4 = pad_to(D, K_ALIGN), pad_to(D, 4)
+
+    def sublayer(n):
+        hc = [src.get(f"{p}hc{n}.{x}", shape, kind).float().contiguous()
+              for x, shape, kind in (("in", (S,), "norm"), ("mix", (S, S), "mix"), ("out", (S,), "norm"))]
+        return Sublayer(_norm(src, f"{p}norm{n}", cfg), None, None, [], hc=residual.Hyper(*hc))
+    s = sublayer(1)
+    prefixes = [p + "mix."] if spec.second is None else [p + "mix.left.", p + "mix.right."]
+    s.mixers = [build_mixer(m, q, src, cfg, dtype, i) for i, (m, q) in enumerate(zip(spec.mixers, prefixes))]
+    s.w_in = stack_parts([(m.seg, name, t) for m in s.mixers for name, t in m.parts], Kp, dtype)
+    s.w_out = [torch.cat([pad_cols(m.o.to(dtype), pad_to(m.cols, K_ALIGN)) for m in s.mixers], 1).contiguous()]
+    for m in s.mixers:
+        m.parts, m.o = [], None
+        if m.o_bias is not None:
+            b = torch.nn.functional.pad(m.o_bias, (0, W4 - D))
+            s.bias, m.o_bias = b if s.bias is None else s.bias + b, None
+    out = [s]
+    if f.kind == "none":
+        return out
+    s = sublayer(2)
+    s.mlp, q, parts = f, p + "mlp.", []
+    ff, prefix = (f.ff, q) if f.kind == "dense" else (f.shared_ff, q + "shared.")
+    if f.kind == "moe":
+        parts.append((s.seg, "router", src.get(q + "router", (f.experts, D))))
+        if f.correction:
+            s.correction = src.get(q + "correction", (f.experts,), "bias").float().contiguous()
+        s.experts = _experts(f, q, src, D, dtype)
+        if ff and f.shared_gate:
+            raise NotImplementedError("hyper-connected blocks carry shared experts without a gate")
+    if ff:
+        s.ff = pad_to(ff, K_ALIGN)
+        parts += [(s.seg, x, pad_rows(src.get(prefix + x, (ff, D)), s.ff)) for x in ("gate", "up")]
+        s.w_out = [pad_cols(src.get(prefix + "down", (D, ff)).to(dtype), s.ff).contiguous()]
+    s.w_in = stack_parts(parts, Kp, dtype)
+    return out + [s]
+
+
 def _build_parallel(cfg: ModelConfig, spec: LayerSpec, p: str, src: WeightSource, dtype: torch.dtype) -> LayeredLayer:
     D, f = cfg.hidden_size, spec.mlp
     Kp = pad_to(D, K_ALIGN)
@@ -148,14 +210,7 @@ def _build_parallel(cfg: ModelConfig, spec: LayerSpec, p: str, src: WeightSource
         parts.append((lw.seg, "router", src.get(q + "router", (f.experts, D))))
         if ff:
             parts.append((lw.seg, "gate1", src.get(prefix + "sg", (1, D))))
-        Fp = pad_to(f.ff, K_ALIGN)
-        w13, wd = [], []
-        for e in range(f.experts):
-            ep = f"{q}e{e}."
-            gu = [pad_rows(src.get(ep + x, (f.ff, D)).to(dtype), Fp) for x in ("gate", "up")]
-            w13.append(pad_cols(torch.cat(gu, 0), Kp))
-            wd.append(pad_cols(src.get(ep + "down", (D, f.ff)).to(dtype), Fp))
-        lw.experts = ExpertWeights(w13=torch.stack(w13), w2=torch.stack(wd), activation=f.activation, act_limit=f.limit)
+        lw.experts = _experts(f, q, src, D, dtype)
     if ff:
         lw.ff_p = pad_to(ff, K_ALIGN)
         parts += [(lw.seg, x, pad_rows(src.get(prefix + x, (ff, D)), lw.ff_p)) for x in ("gate", "up")]
@@ -171,8 +226,11 @@ def layered_tensor_specs(cfg: ModelConfig) -> List[Tuple[str, Tuple[int, ...], s
 
     def norm(name, l):
         return [(name, (D,), "norm", l)] + ([(name + ".b", (D,), "bias", l)] if cfg.layer_norm else [])
-    out = [("embed", (V, D), "normal", -1), *norm("final.norm", -1), ("head", (V, D), "normal", -1)]
+    out = [("embed", (V, D), "normal", -1), *norm("final.norm", -1)]
+    out += [] if cfg.tie_word_embeddings else [("head", (V, D), "normal", -1)]
     for i, s in enumerate(cfg.layer_specs):
+        if s.weights_of >= 0:
+            continue
         f, q = s.mlp, f"l{i}.mlp."
         prefixes = [f"l{i}.mix."] if s.second is None else [f"l{i}.mix.left.", f"l{i}.mix.right."]
         if cfg.sandwich:
@@ -182,6 +240,11 @@ def layered_tensor_specs(cfg: ModelConfig) -> List[Tuple[str, Tuple[int, ...], s
                     out.append((f"l{i}.canon{n}", (D, cfg.canon_taps), "normal", i))
             if s.second is not None:
                 out += [(q_ + "out", (D,), "norm", i) for q_ in prefixes]
+        elif cfg.streams:
+            S = cfg.streams
+            for n in ("1", "2") if f.kind != "none" else ("1",):
+                out += norm(f"l{i}.norm{n}", i)
+                out += [(f"l{i}.hc{n}.in", (S,), "norm", i), (f"l{i}.hc{n}.out", (S,), "norm", i), (f"l{i}.hc{n}.mix", (S, S), "mix", i)]
         else:
             out += norm(f"l{i}.norm1", i)
         for m, p in zip(s.mixers, prefixes):
@@ -194,10 +257,11 @@ def layered_tensor_specs(cfg: ModelConfig) -> List[Tuple[str, Tuple[int, ...], s
             out += ff(q, f.ff)[1 if f.activation == "relu2" else 0:]
         elif f.kind == "moe":
             out.append((q + "router", (f.experts, D), "normal", i))
+            out += [(q + "correction", (f.experts,), "bias", i)] if f.correction else []
             for e in range(f.experts):
                 out += ff(f"{q}e{e}.", f.ff)
             if f.shared_ff:
-                out += ff(q + "shared.", f.shared_ff) + [(q + "shared.sg", (1, D), "normal", i)]
+                out += ff(q + "shared.", f.shared_ff) + ([(q + "shared.sg", (1, D), "normal", i)] if f.shared_gate else [])
     return out
 
 
@@ -233,8 +297,12 @@ class LayeredDecoder:
     def forward(self, ids: torch.Tensor, meta: AttnMeta, cache) -> torch.Tensor:
         """ids [T] -> fp32 logits [len(logit_rows) or T, vocab]."""
         plan = self._plan(meta, ids.shape[0])
-        x = torch.empty(ids.shape[0], pad_to(self.cfg.hidden_size, 4), dtype=torch.float32, device=self.device)
-        y = (self._sandwich if self.cfg.sandwich else self._parallel)(x, ids.to(torch.int32), plan, meta, cache)
+        cfg = self.cfg
+        W4 = pad_to(cfg.hidden_size, 4)
+        x = torch.empty(*((ids.shape[0], cfg.streams, W4) if cfg.streams else (ids.shape[0], W4)), dtype=torch.float32,
+                        device=self.device)
+        block = self._hyper if cfg.streams else self._sandwich if cfg.sandwich else self._parallel
+        y = block(x, ids.to(torch.int32), plan, meta, cache)
         with self.timer.timed("lm_head"):
             return gemm.rows_gemm(y, self.w.lm_head)
 
@@ -287,6 +355,53 @@ class LayeredDecoder:
             self.layer_hook(len(w.layers) - 1, x[:, :D])
         return residual.sandwich_norm(*args, **pending, keep=False,
                                       rows=meta.logit_rows.long() if meta.logit_rows is not None else None)
+
+    # ------------------------------------------------------------------ hyper-connected blocks
+    def _hyper(self, x, ids, plan: StepPlan, meta: AttnMeta, cache) -> torch.Tensor:
+        cfg, tm, w, dt = self.cfg, self.timer, self.w, self.dtype
+        T, D = x.shape[0], cfg.hidden_size
+        args = (D, self.width_p, dt)
+        pending = dict(ids=ids, embed=w.embed, embed_scale=cfg.embed_scale)
+        for l, layer in enumerate(w.layers):
+            for i, s in enumerate(layer):
+                with tm.timed("norm", l):
+                    y = residual.hyper_norm(x, s.norm.w, cfg.rms_eps, *args, read=s.hc.read, **pending)
+                if self.layer_hook is not None and l and not i:
+                    self.layer_hook(l - 1, x[..., :D].sum(1))
+                with tm.timed("proj_in", l):
+                    z = gemm.rows_gemm(y, s.w_in)
+                pending = dict(hc=s.hc, bias=s.bias)
+                operand = None
+                if s.mixers:
+                    spans = [pad_to(m.cols, K_ALIGN) for m in s.mixers]
+                    operand = self._operand(T, sum(m.cols for m in s.mixers), sum(spans))
+                    with tm.timed("mixer_" + meta.mode, l):
+                        at = 0
+                        for m, n in zip(s.mixers, spans):
+                            m.run(l, z, operand[:, at:at + m.cols], plan, meta, cache)
+                            at += n
+                elif s.ff:
+                    with tm.timed("glu", l):
+                        operand = residual.glu(z[:, s.seg["gate"][0]:], s.ff, s.mlp.activation,
+                                               s.mlp.limit if s.mlp.kind == "dense" else s.mlp.shared_limit, dtype=dt)
+                if s.experts is not None:
+                    f, r0 = s.mlp, s.seg["router"][0]
+                    with tm.timed("moe", l):
+                        idx, rw = moe_ops.router_topk(z[:, r0:r0 + f.experts], s.correction, f.top, f.groups, f.keep_groups,
+                                                      "always" if f.norm_weights else False, f.router_scale, f.scoring,
+                                                      meta.num_valid, f.group_score)
+                        routed, pos = moe_ops.routed_rows(y, idx, rw, s.experts, False, meta.num_valid)
+                    pending.update(routed=routed, pos=pos, route_w=rw)
+                if operand is not None:
+                    with tm.timed("proj_out", l):
+                        pending["add"] = gemm.rows_gemm(operand, s.w_out[0])
+        final = (x, w.final_norm.w, cfg.rms_eps, *args)
+        if self.layer_hook is not None:           # the last sublayer's output only joins the streams inside the final norm
+            residual.hyper_norm(*final, **pending)
+            pending = {}
+            self.layer_hook(len(w.layers) - 1, x[..., :D].sum(1))
+        return residual.hyper_norm(*final, **pending, keep=False,
+                                   rows=meta.logit_rows.long() if meta.logit_rows is not None else None)
 
     # ------------------------------------------------------------------ parallel blocks
     def _parallel(self, x, ids, plan: StepPlan, meta: AttnMeta, cache) -> torch.Tensor:

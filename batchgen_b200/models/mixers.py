@@ -31,22 +31,22 @@ class StepPlan:
     slots: Optional[torch.Tensor]
     has_initial: Optional[torch.Tensor]
     ctx: Optional[List[int]] = None
-    tiles: Dict[int, Tuple] = field(default_factory=dict)      # attention chunk -> (tensor-core tiles, rows of short pieces)
-    ropes: Dict[Tuple[int, float], torch.Tensor] = field(default_factory=dict)
+    tiles: Dict[Tuple[int, int], Tuple] = field(default_factory=dict)      # chunk, window -> (tensor-core tiles, rows of short pieces)
+    ropes: Dict[Tuple, torch.Tensor] = field(default_factory=dict)
 
     def rope(self, r: Optional[conv.Rotary]) -> Optional[torch.Tensor]:
         if r is None:
             return None
-        if (r.dims, r.base) not in self.ropes:
-            self.ropes[(r.dims, r.base)] = r.table(self.lens)
-        return self.ropes[(r.dims, r.base)]
+        if r.key not in self.ropes:
+            self.ropes[r.key] = r.table(self.lens)
+        return self.ropes[r.key]
 
-    def attention_tiles(self, chunk: int, T: int):
+    def attention_tiles(self, chunk: int, T: int, window: int = 0):
         """How the rows of a prompt step split over the attention kernels: pieces of a few tokens (decoded tokens among
         them) go row by row, the rest in 128-query tiles."""
-        if chunk not in self.tiles:
+        if (chunk, window) not in self.tiles:
             cu, least, dev = self.cu_host, talking.PREFILL_MIN_TOKENS, self.lens.device
-            blocks = talking.work_blocks(talking.prefill_work(cu, self.ctx, chunk, least), T, dev)
+            blocks = talking.work_blocks(talking.prefill_work(cu, self.ctx, chunk, least, window), T, dev)
             short = [t for a, b in zip(cu, cu[1:]) if b - a < least for t in range(a, b)]
             rows = seqs = None
             if blocks and short:
@@ -54,8 +54,8 @@ class StepPlan:
                 seqs = self.row_seq[rows.long()].contiguous()
             elif short:
                 seqs = self.row_seq
-            self.tiles[chunk] = (blocks, bool(short), rows, seqs)
-        return self.tiles[chunk]
+            self.tiles[chunk, window] = (blocks, bool(short), rows, seqs)
+        return self.tiles[chunk, window]
 
 
 @dataclass
@@ -71,6 +71,8 @@ class Mixer:
     rot: Optional[conv.Rotary] = None
     delta: Optional[delta.DeltaParams] = None
     talk: Optional[talking.TalkParams] = None
+    prep: Optional[talking.HeadPrep] = None       # attention with biases or norms of its heads
+    o_bias: Optional[torch.Tensor] = None         # [width] fp32 bias of the output projection, times the output's scale
     rec: Optional[recurrent.RecurrentParams] = None
 
     def column(self, z: torch.Tensor, name: str) -> torch.Tensor:
@@ -111,16 +113,23 @@ class Mixer:
     def _attention(self, l: int, z, out, plan: StepPlan, meta, cache) -> None:
         k, p = self.seg["k"][0], self.talk
         kv, rope = cache.latent(l), plan.rope(self.rot)
-        talking.kv_write(z[:, k:k + p.kv_row], meta.slot_mapping, kv, p, rope)
         zq = self.column(z, "q")
-        rows, seqs = None, plan.row_seq
-        more = dict(rope=rope, gate=self.column(z, "gate") if "gate" in self.seg else None)
+        blocks, short, rows, seqs = [], True, None, plan.row_seq
         if plan.cu is not None and z.is_cuda and talking.prefill_supported(p, kv.dtype, kv.shape[1]):
-            blocks, short, rows, seqs = plan.attention_tiles(p.chunk, z.shape[0])
-            talking.attend_prefill(zq, p, kv, meta.block_table, out, blocks, **more)
-            if not short:
-                return
-        talking.attend_rows(zq, p, kv, meta.block_table, plan.lens, out, seqs, rows, **more)
+            blocks, short, rows, seqs = plan.attention_tiles(p.chunk, z.shape[0], p.window)
+        more = dict(rope=rope, gate=self.column(z, "gate") if "gate" in self.seg else None)
+        operand = None
+        if self.prep is not None:
+            q0 = self.seg["q"][0]
+            operand = talking.prepare_heads(z[:, q0:q0 + p.heads * p.dim_p + p.kv_row], meta.slot_mapping, kv, p, self.prep, rope,
+                                            short, bool(blocks))
+            more["rope"] = None                   # the queries have turned
+        else:
+            talking.kv_write(z[:, k:k + p.kv_row], meta.slot_mapping, kv, p, rope)
+        if blocks:
+            talking.attend_prefill(zq, p, kv, meta.block_table, out, blocks, operand=operand, **more)
+        if short:
+            talking.attend_rows(zq, p, kv, meta.block_table, plan.lens, out, seqs, rows, **more)
 
 
 # ---------------------------------------------------------------- weights
@@ -167,7 +176,16 @@ def build_mixer(m: MixerSpec, p: str, src: WeightSource, cfg: ModelConfig, dtype
         if m.out_gate:
             mx.parts.append(("gate", src.get(p + "g", (H, D))))
         talk = src.get(p + "talk", (H, H)).float().contiguous() if m.talking else None
-        mx.talk = talking.TalkParams(heads=H, kv_heads=G, dim_p=dp, vdim_p=dvp, scale=m.scale, chunk=m.chunk, sink=m.sink, talk=talk)
+        mx.talk = talking.TalkParams(heads=H, kv_heads=G, dim_p=dp, vdim_p=dvp, scale=m.scale, chunk=m.chunk, sink=m.sink, talk=talk,
+                                     window=m.window, keep=m.keep_first if m.window else 0, out_scale=m.out_scale)
+        if m.bias or m.qk_norm or m.rot_interleaved:
+            mx.prep = talking.HeadPrep(dim=d, eps=cfg.rms_eps, interleaved=m.rot_interleaved)
+        if m.bias:
+            mx.prep.bias = torch.cat([vector(x + ".b", n, w, wp, "bias") for x, n, w, wp in (("q", H, d, dp), ("k", G, d, dp),
+                                                                                        ("v", G, dv, dvp))])
+            mx.o_bias = src.get(p + "o.b", (D,), "bias").float() * m.out_scale
+        if m.qk_norm:
+            mx.prep.q_norm, mx.prep.k_norm = (vector(x + ".norm", 1, d, dp, "norm") for x in "qk")
     elif m.kind == "general_delta":
         mx.parts = [(x, rows(x, H, d, dp)) for x in ("r", "k", "v", "g", "a")]
         mx.parts.append(("low", src.get(p + "w1", (m.decay_rank, D))))
@@ -200,9 +218,9 @@ def build_mixer(m: MixerSpec, p: str, src: WeightSource, cfg: ModelConfig, dtype
                                                f_bias=src.get(p + "f.b", (H,), "bias").float().contiguous())
         else:
             mx.parts.append(("g", rows("g", H, dv, dvp)))
-            mx.rec = recurrent.RecurrentParams(**base, norm_w=torch.ones(H * dvp, device=dev), gate="silu", k_scale=d ** -0.5,
+            mx.rec = recurrent.RecurrentParams(**base, norm_w=torch.full((H * dvp,), m.out_scale, device=dev), gate="silu", k_scale=d ** -0.5,
                                                decay=torch.tensor(m.decay, dtype=torch.float32, device=dev))
-    mx.rot = conv.Rotary.make(m.rot_dims, m.rot_base, dev)
+    mx.rot = conv.Rotary.make(m.rot_dims, m.rot_base, dev, m.rot_interleaved, m.yarn)
     mx.o = head_rows(src.get(p + "o", (D, H * dv)).t().contiguous(), H, dv, dvp).t()       # [D, heads * dvp]: zero columns
     return mx
 
@@ -214,6 +232,8 @@ def mixer_tensor_specs(m: MixerSpec, p: str, D: int, layer: int) -> List[Tuple[s
         out = [("q", (qk, D), "normal"), ("k", (kv, D), "normal"), ("v", (m.kv_heads * m.vdim, D), "normal")]
         out += [("talk", (H, H), "normal")] if m.talking else []
         out += [("g", (H, D), "normal")] if m.out_gate else []
+        out += [("q.b", (qk,), "bias"), ("k.b", (kv,), "bias"), ("v.b", (m.kv_heads * m.vdim,), "bias"), ("o.b", (D,), "bias")] if m.bias else []
+        out += [("q.norm", (m.dim,), "norm"), ("k.norm", (m.dim,), "norm")] if m.qk_norm else []
     elif m.kind == "general_delta":
         out = [(x, (qk, D), "normal") for x in ("r", "k", "v", "g", "a")]
         out += [("w1", (m.decay_rank, D), "normal"), ("w2", (qk, m.decay_rank), "normal"), ("a.b", (qk,), "bias"),

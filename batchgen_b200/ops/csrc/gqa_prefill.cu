@@ -1,5 +1,5 @@
-// Prompt attention of grouped-query heads over a paged K/V cache, on tcgen05: causal, optionally with chunked visibility, a
-// zero-score sink, rotary queries and a sigmoid gate per head on the output.
+// Prompt attention of grouped-query heads over a paged K/V cache, on tcgen05: causal, optionally with chunked visibility or a
+// sliding window that keeps a sequence's first keys, a zero-score sink, rotary queries and a sigmoid gate per head on the output.
 //
 //   S[q, k] = Q[q, :] . K[k, kv(h)]      (M = 128 queries, N = 64 keys; Q resident, K streamed, both K-major)
 //   O[q, :] += P[q, k] . V[k, kv(h)]     (V read N-major, P written by the softmax threads as a swizzled K-major tile)
@@ -43,7 +43,8 @@ struct Params {
   int KB, VB;                    // 64-wide blocks of a key / value head
   int stages, tmem_cols;
   int dp, dvp, v_col0, rep;      // head widths, first value column of a cache row, heads per key head
-  int chunk, sink;
+  int chunk, window, keep, sink;  // keys seen: from the query's chunk, within the window, and the first `keep`
+  float out_scale;
   __nv_bfloat16* out;
   int ldo;
   const float* gate;             // [T, ld_gate] or null: out[h] *= sigmoid(gate[h])
@@ -132,9 +133,13 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
   const Work w = p.work[blockIdx.y];
   const int h = blockIdx.x;
   const int last = w.pos0 + w.n_q - 1;
-  const int first = p.chunk > 0 ? w.pos0 - w.pos0 % p.chunk : 0;
-  const int k0 = first - first % p.box_rows;                     // first key of tile 0: starts on a box of a page
-  const int n_tiles = (last + 1 - k0 + BN - 1) / BN;
+  int first = p.chunk > 0 ? w.pos0 - w.pos0 % p.chunk : 0;
+  if (p.window > 0) first = max(first, w.pos0 + 1 - p.window);
+  int k0 = first - first % p.box_rows;                           // first key of the tiles: starts on a box of a page
+  if (p.keep > k0) k0 = 0;
+  const int n_keep = k0 > 0 ? (p.keep + BN - 1) / BN : 0;        // kept keys that end before k0 have tiles of their own
+  const int n_tiles = n_keep + (last + 1 - k0 + BN - 1) / BN;
+  auto first_key = [&](int t) { return t < n_keep ? t * BN : k0 + (t - n_keep) * BN; };
   const int ST = p.stages;
 
   if (threadIdx.x == 0) {
@@ -166,13 +171,13 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
       const int* bt = p.block_table + (size_t)w.seq * p.bt_stride;
       const int boxes = BN / p.box_rows, shift = 31 - __clz(p.page);
       const int kcol = (h / p.rep) * p.dp, vcol = p.v_col0 + (h / p.rep) * p.dvp;
-      // box b of tile t: tokens k0 + t * BN + b * box_rows ..; past the table's end the last page is read (masked keys).
+      // box b of tile t: tokens first_key(t) + b * box_rows ..; past the table's end the last page is read (masked keys).
       // Page numbers of a tile are looked up once, one tile ahead of their use.
       int old[kMaxBoxes], pg[kMaxBoxes] = {}, nxt[kMaxBoxes] = {};
       auto look_up = [&](int t) {
 #pragma unroll
         for (int b = 0; b < kMaxBoxes; ++b)
-          if (b < boxes) nxt[b] = bt[min((k0 + t * BN + b * p.box_rows) >> shift, p.bt_cols - 1)];
+          if (b < boxes) nxt[b] = bt[min((first_key(t) + b * p.box_rows) >> shift, p.bt_cols - 1)];
       };
       auto load = [&](uint8_t* dst, uint64_t* full, int blocks, int col, int t, const int (&pages)[kMaxBoxes]) {
         mbar_expect_tx(full, blocks * kBlockBytes);
@@ -181,7 +186,7 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
           for (int b = 0; b < kMaxBoxes; ++b)
             if (b < boxes)
               tma_load_3d(dst + c * kBlockBytes + b * p.box_rows * 128, &tm_kv, full, col + c * 64,
-                          (k0 + t * BN + b * p.box_rows) & (p.page - 1), pages[b]);
+                          (first_key(t) + b * p.box_rows) & (p.page - 1), pages[b]);
       };
       auto load_v = [&](int t) -> bool {                           // values of tile t, whose pages are in `old`
         const int s = t % ST;
@@ -267,8 +272,8 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
     const uint32_t tm_o = tmem_base + 2 * BN + lane_addr;
     const int pos = w.pos0 + r;
     const bool live = r < w.n_q;
-    const int vis_lo = live ? (p.chunk > 0 ? pos - pos % p.chunk : 0) - k0 : 0;     // keys [vis_lo, vis_hi) from k0
-    const int vis_hi = live ? pos + 1 - k0 : 0;
+    int vis_lo = p.chunk > 0 ? pos - pos % p.chunk : 0;            // keys [vis_lo, pos] and those before `keep`
+    if (p.window > 0) vis_lo = max(vis_lo, pos + 1 - p.window);
     float m_run = -INFINITY, l_run = 0.f;
     uint8_t* prow = p_buf + (r >> 3) * 1024 + (r & 7) * 128;
     bool ok = true;
@@ -279,11 +284,14 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
       tmem_ld32(tmem_base + lane_addr + (t & 1) * BN, sv);
       tmem_ld32(tmem_base + lane_addr + (t & 1) * BN + 32, sv + 32);
       tmem_ld_wait();
-      const int lo = vis_lo - t * BN, hi = vis_hi - t * BN;
-      if (!__all_sync(0xffffffffu, lo <= 0 && hi >= BN)) {
+      const int kt = first_key(t);
+      const bool kept = t < n_keep;
+      const int lo = kept ? 0 : vis_lo - kt, hi = !live ? 0 : kept ? p.keep - kt : pos + 1 - kt;
+      const int below = n_keep > 0 ? 0 : p.keep - kt;              // kept keys among this tile's
+      if (!__all_sync(0xffffffffu, (lo <= 0 || below >= BN) && hi >= BN)) {
 #pragma unroll
         for (int j = 0; j < BN; ++j)
-          if (j < lo || j >= hi) sv[j] = 0xff800000u;              // minus infinity
+          if ((j < lo && j >= below) || j >= hi) sv[j] = 0xff800000u;              // minus infinity
       }
       float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -328,7 +336,7 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
     if (ok) {
       tc_fence_after();
       if (p.sink && live) l_run += exp2f(-m_run);
-      float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+      float inv = l_run > 0.f ? p.out_scale / l_run : 0.f;
       if (p.gate != nullptr && live) inv *= 1.0f / (1.0f + expf(-p.gate[(size_t)(w.q_row0 + r) * p.ld_gate + h]));
       __nv_bfloat16* orow = p.out + (size_t)(w.q_row0 + r) * p.ldo + h * p.dvp;
 #pragma unroll 1
@@ -438,11 +446,11 @@ int bg_gqa_prompt_queries(const float* q, int ldq, const float* rope, int half, 
 // dp, dvp <= 256, multiples of 8.
 int bg_gqa_prompt(const void* qf, const void* cache, long long page_stride, int n_pages, int page, int row, const int* block_table,
                   int bt_stride, int bt_cols, const int* work, int n_work, int R, int row_shift, void* out, int ldo, int H, int G,
-                  int dp, int dvp, int kc, int chunk, int sink, const float* gate, int ld_gate, int* status, cudaStream_t stream) {
+                  int dp, int dvp, int kc, int chunk, int sink, int window, int keep, float out_scale, const float* gate, int ld_gate, int* status, cudaStream_t stream) {
   using namespace bg::gqapre;
   if (n_work <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || dp <= 0 || dp % 8 || dp > 256 || dvp <= 0 || dvp % 8 || dvp > 256 || kc != (dp + 63) / 64 * 64 ||
-      page < 16 || (page & (page - 1)) || row != G * (dp + dvp) || page_stride % 8 || ldo % 8 || bt_cols <= 0 || n_work > 65535)
+      page < 16 || (page & (page - 1)) || row != G * (dp + dvp) || page_stride % 8 || ldo % 8 || bt_cols <= 0 || n_work > 65535 || window < 0 || keep < 0)
     return -1;
   const int box_rows = page < 64 ? page : 64;
   CUtensorMap tq, tk;
@@ -462,6 +470,7 @@ int bg_gqa_prompt(const void* qf, const void* cache, long long page_stride, int 
   p.work = reinterpret_cast<const Work*>(work);
   p.block_table = block_table; p.bt_stride = bt_stride; p.bt_cols = bt_cols; p.page = page; p.box_rows = box_rows;
   p.KB = kc / 64; p.VB = (dvp + 63) / 64; p.dp = dp; p.dvp = dvp; p.v_col0 = G * dp; p.rep = H / G; p.chunk = chunk; p.sink = sink;
+  p.window = window; p.keep = keep; p.out_scale = out_scale;
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo; p.gate = gate; p.ld_gate = ld_gate; p.row_shift = row_shift;
   p.status = status;
   // two CTAs an SM when two stages and half of TMEM are enough, otherwise one with as many stages as fit

@@ -22,7 +22,7 @@ constexpr int kMaxTopK = 16;
 __global__ void __launch_bounds__(128)
 router_topk_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ bias, int* __restrict__ idx_out,
                    float* __restrict__ w_out, int T, int E, int K, int n_group, int topk_group, int norm, float scale,
-                   int softmax_mode, const int* __restrict__ num_valid) {
+                   int softmax_mode, int group_max, const int* __restrict__ num_valid) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   __shared__ float choice_s[4][kMaxExperts];
   __shared__ float score_s[4][kMaxExperts];
@@ -75,7 +75,7 @@ router_topk_kernel(const float* __restrict__ logits, int ldl, const float* __res
         const float v = choice[lane * gs + i];
         if (v > m1) { m2 = m1; m1 = v; } else if (v > m2) { m2 = v; }
       }
-      group_s[warp][lane] = softmax_mode == 2 ? m1 : m1 + m2;   // softmax_all ranks a group by its best expert
+      group_s[warp][lane] = group_max ? m1 : m1 + m2;
     }
     __syncwarp();
     // keep the topk_group best groups (ties -> lower index); lane g decides for group g
@@ -122,7 +122,7 @@ router_topk_kernel(const float* __restrict__ logits, int ldl, const float* __res
   if (lane < K) {
     float wv = my_w;
     if (softmax_mode == 1) wv = wv / wsum;
-    else if (norm && K > 1) wv = wv / (wsum + 1e-20f);
+    else if (norm == 2 || (norm && K > 1)) wv = wv / (wsum + 1e-20f);
     idx_out[(size_t)t * K + lane] = my_i;
     w_out[(size_t)t * K + lane] = wv * scale;
   }
@@ -285,15 +285,16 @@ moe_combine_kernel(const __nv_bfloat16* __restrict__ y, int ldy, const int* __re
 
 extern "C" {
 
-// logits: rows of E values, ldl apart
+// logits: rows of E values, ldl apart; norm: weights divided by their sum, 1 unless K is 1, 2 always; group_max: a group counts with
+// its best expert instead of its best two
 int bg_router_topk(const float* logits, int ldl, const float* bias, int* idx, float* w, int T, int E, int K, int n_group,
-                   int topk_group, int norm, float scale, int softmax_mode, const int* num_valid,
+                   int topk_group, int norm, float scale, int softmax_mode, int group_max, const int* num_valid,
                    cudaStream_t stream) {
   using namespace bg;
   if (T <= 0) return 0;
   if (E > kMaxExperts || K > kMaxTopK || K > E || ldl < E || n_group > 32 || (n_group > 1 && E % n_group != 0)) return -1;
   bg::launch_pdl(router_topk_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, ldl, bias, idx, w, T, E, K, n_group, topk_group, norm, scale,
-                                                      softmax_mode, num_valid);
+                                                      softmax_mode, group_max, num_valid);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 

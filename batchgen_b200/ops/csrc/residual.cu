@@ -5,7 +5,9 @@
 //   sandwich_norm   the same for blocks with a norm before and after each sublayer: the sublayer's output (or half the sum of
 //                   two, each RMS-normed) passes its own norm before it joins x; optional mean subtraction and biases; in
 //                   decode the input convolution y = h + conv(h) of the next sublayer is folded in
-//   glu             gated activations (tanh-GELU, clamped SwiGLU with slope 1.702 and u + 1), with an optional factor on
+//   hyper_norm      the same for several residual streams: every stream becomes a weighted sum of all of them plus its share of
+//                   the sublayer's output; the norm reads another weighted sum
+//   glu             gated activations (tanh-GELU, SwiGLU, clamped SwiGLU with slope 1.702 and u + 1), with an optional factor on
 //                   the pre-activations (routing weight applied to the expert's input) and an optional sigmoid gate
 //   cast_act        out = f(x), f = tanh, squared ReLU or identity: fp32 columns of a projection to the operand type of the next one
 //   moe_gather      token rows -> expert-grouped rows, one block per (token, k) pair, plus the pair's routing weight
@@ -312,6 +314,143 @@ __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichP
     for (int c = D4 + tid * 4; c < p.ldy; c += NT * 4) store4(yr + c, make_float4(0.f, 0.f, 0.f, 0.f));
 }
 
+struct HyperParams {
+  float* x;               // [T, S, D4] residual streams
+  const long long* rows;  // [R] rows of x, or null
+  const int* ids;         // first layer: token ids (every stream is written, none read)
+  const void* embed;      // [V, lde]
+  int lde;
+  float escale;
+  int vocab;
+  const float* mix;       // [S, S] (from, to), or null: the streams stay
+  const float* share;     // [S] factors of the sublayer's output
+  const float* add;       // dense part of the output [T, ld_add], or null
+  int ld_add;
+  const float* bias;      // [D4] added to the output, or null
+  const float* routed;    // rows of the routed experts [*, ld_routed], or null
+  int ld_routed;
+  const int* pos;         // [T, K] row of every (token, k) pair, < 0 = none
+  const float* route_w;   // [T, K] factors of those rows
+  int K;
+  const float* read;      // [S] factors of the streams in what the norm reads, or null: all 1
+  const float* w;         // [D4] gain
+  void* y;                // [R, ldy]; columns D .. ldy are zero
+  int ldy;
+  int D, S;
+  float eps;
+  int keep;               // write the streams back
+};
+
+constexpr int kMaxStreams = 16;
+
+// One block per row; thread i owns the 4-wide vectors i, i + blockDim, ... of every stream.  SM: streams, or an upper bound of them
+// (above 4).  What the norm reads waits in shared memory for its root mean square.
+template <typename OT, int SM>
+__global__ void __launch_bounds__(kThreads) hyper_norm_kernel(const HyperParams p) {
+  bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
+  extern __shared__ float row[];
+  __shared__ float red[kThreads / 32];
+  __shared__ float mix[SM * SM], share[SM], read[SM], rw[kMaxK];
+  __shared__ int pos_s[kMaxK];
+  const int tid = threadIdx.x, NT = blockDim.x, S = SM <= 4 ? SM : p.S;
+  const long long t = p.rows != nullptr ? p.rows[blockIdx.x] : (long long)blockIdx.x;
+  const int D = p.D, nv = (D + 3) / 4, D4 = nv * 4;
+  float* xr = p.x + t * S * D4;
+  const bool pending = p.mix != nullptr;
+  for (int i = tid; i < SM * SM; i += NT) mix[i] = pending && i / SM < S && i % SM < S ? p.mix[i / SM * S + i % SM] : 0.f;
+  if (tid < SM) {
+    share[tid] = pending && tid < S ? p.share[tid] : 0.f;
+    read[tid] = tid >= S ? 0.f : p.read != nullptr ? p.read[tid] : 1.0f;
+  }
+  if (p.routed != nullptr && tid < p.K) {
+    pos_s[tid] = p.pos[t * p.K + tid];
+    rw[tid] = p.route_w[t * p.K + tid];
+  }
+  __syncthreads();
+  const OT* er = nullptr;
+  if (p.ids != nullptr) {
+    const int id = min(max(p.ids[t], 0), p.vocab - 1);
+    er = reinterpret_cast<const OT*>(p.embed) + (size_t)id * p.lde;
+  }
+  float ss = 0.f;
+  for (int v = tid; v < nv; v += NT) {
+    const int c = v * 4;
+    float4 f[SM];
+    if (er != nullptr) {
+      float4 e;
+      e.x = to_f(er[c]) * p.escale;
+      e.y = c + 1 < D ? to_f(er[c + 1]) * p.escale : 0.f;
+      e.z = c + 2 < D ? to_f(er[c + 2]) * p.escale : 0.f;
+      e.w = c + 3 < D ? to_f(er[c + 3]) * p.escale : 0.f;
+#pragma unroll
+      for (int s = 0; s < SM; ++s) f[s] = e;
+    } else {
+#pragma unroll
+      for (int s = 0; s < SM; ++s)
+        f[s] = s < S ? *reinterpret_cast<const float4*>(xr + (size_t)s * D4 + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (pending) {
+      float4 o = p.add != nullptr ? *reinterpret_cast<const float4*>(p.add + t * p.ld_add + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      if (p.bias != nullptr) {
+        const float4 b = *reinterpret_cast<const float4*>(p.bias + c);
+        o.x += b.x; o.y += b.y; o.z += b.z; o.w += b.w;
+      }
+      if (p.routed != nullptr) {
+#pragma unroll 4
+        for (int k = 0; k < p.K; ++k) {
+          const int r = pos_s[k];
+          if (r < 0) continue;
+          const float4 a = *reinterpret_cast<const float4*>(p.routed + (size_t)r * p.ld_routed + c);
+          const float g = rw[k];
+          o.x = fmaf(g, a.x, o.x); o.y = fmaf(g, a.y, o.y); o.z = fmaf(g, a.z, o.z); o.w = fmaf(g, a.w, o.w);
+        }
+      }
+      if (c + 1 >= D) o.y = 0.f;
+      if (c + 2 >= D) o.z = 0.f;
+      if (c + 3 >= D) o.w = 0.f;
+      float4 n[SM];
+#pragma unroll
+      for (int u = 0; u < SM; ++u) {
+        const float g = share[u];
+        n[u] = make_float4(g * o.x, g * o.y, g * o.z, g * o.w);
+#pragma unroll
+        for (int s = 0; s < SM; ++s) {
+          const float m = mix[s * SM + u];
+          n[u].x = fmaf(m, f[s].x, n[u].x); n[u].y = fmaf(m, f[s].y, n[u].y);
+          n[u].z = fmaf(m, f[s].z, n[u].z); n[u].w = fmaf(m, f[s].w, n[u].w);
+        }
+      }
+#pragma unroll
+      for (int s = 0; s < SM; ++s) f[s] = n[s];
+    }
+    float4 h = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int s = 0; s < SM; ++s) {
+      const float g = read[s];
+      h.x = fmaf(g, f[s].x, h.x); h.y = fmaf(g, f[s].y, h.y); h.z = fmaf(g, f[s].z, h.z); h.w = fmaf(g, f[s].w, h.w);
+      if (p.keep && s < S) *reinterpret_cast<float4*>(xr + (size_t)s * D4 + c) = f[s];
+    }
+    *reinterpret_cast<float4*>(row + c) = h;
+    ss += h.x * h.x + h.y * h.y + h.z * h.z + h.w * h.w;
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+  for (int i = 0; i < NT / 32; ++i) tot += red[i];
+  const float rstd = 1.0f / sqrtf(tot / (float)D + p.eps);
+  OT* yr = reinterpret_cast<OT*>(p.y) + (size_t)blockIdx.x * p.ldy;
+  for (int v = tid; v < p.ldy / 4; v += NT) {
+    const int c = v * 4;
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < D) {                                        // gains and the row are zero from D to D4
+      const float4 h = *reinterpret_cast<const float4*>(row + c), g = *reinterpret_cast<const float4*>(p.w + c);
+      o = make_float4(h.x * rstd * g.x, h.y * rstd * g.y, h.z * rstd * g.z, h.w * rstd * g.w);
+    }
+    store4(yr + c, o);
+  }
+}
+
 __device__ __forceinline__ float sigmoid_acc(float x) { return 1.0f / (1.0f + expf(-x)); }
 
 template <int KIND>
@@ -320,6 +459,7 @@ __device__ __forceinline__ float glu_one(float g, float u, float limit) {
     const float t = tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g));
     return 0.5f * g * (1.0f + t) * u;
   }
+  if (KIND == 2) return g * sigmoid_acc(g) * u;        // SiLU(g) * u
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g * sigmoid_acc(1.702f * g) * (u + 1.0f);
@@ -454,7 +594,43 @@ int bg_sandwich_norm(int dt, float* x, int ldx, const long long* rows, const int
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
-// kind 0 tanh-GELU, 1 clamped SwiGLU.  z points at the first gate column, the up column of a gate column is u_off further.
+// x [T, S, D4] (D4 = D rounded up to 4); the other leading dimensions: multiples of 4, at least D4; bias and w hold D4 floats.
+// D4 <= 8192, S <= 16.  mix null: nothing joins the streams; ids: every stream = embed[ids] * escale.
+int bg_hyper_norm(int dt, float* x, const long long* rows, const int* ids, const void* embed, int lde, float escale, int vocab,
+                  const float* mix, const float* share, const float* add, int ld_add, const float* bias, const float* routed,
+                  int ld_routed, const int* pos, const float* route_w, int K, const float* read, const float* w, void* y, int ldy,
+                  int R, int D, int S, float eps, int keep, cudaStream_t stream) {
+  using namespace bg::resid;
+  if (R <= 0) return 0;
+  const int D4 = (D + 3) / 4 * 4;
+  if (D <= 0 || D4 > 8192 || S <= 0 || S > kMaxStreams || ldy % 4 || ldy < D4 || (add != nullptr && (ld_add % 4 || ld_add < D4)) ||
+      (routed != nullptr && (ld_routed % 4 || ld_routed < D4 || K <= 0 || K > kMaxK || pos == nullptr || route_w == nullptr)) ||
+      (ids != nullptr && (embed == nullptr || vocab <= 0)) || (mix != nullptr && share == nullptr) ||
+      (mix == nullptr && (add != nullptr || routed != nullptr || bias != nullptr)))
+    return -1;
+  HyperParams p;
+  p.x = x; p.rows = rows; p.ids = ids; p.embed = embed; p.lde = lde; p.escale = escale; p.vocab = vocab; p.mix = mix;
+  p.share = share; p.add = add; p.ld_add = ld_add; p.bias = bias; p.routed = routed; p.ld_routed = ld_routed; p.pos = pos;
+  p.route_w = route_w; p.K = K; p.read = read; p.w = w; p.y = y; p.ldy = ldy; p.D = D; p.S = S; p.eps = eps; p.keep = keep;
+  const int nv = D4 / 4, per = (nv + kThreads - 1) / kThreads;
+  const dim3 block(((nv + per - 1) / per + 31) / 32 * 32);
+  const size_t smem = (size_t)D4 * sizeof(float);
+#define BG_HYPER(SM)                                                                                              \
+  do {                                                                                                            \
+    if (dt == 0) bg::launch_pdl(hyper_norm_kernel<__nv_bfloat16, SM>, dim3(R), block, smem, stream, p);            \
+    else bg::launch_pdl(hyper_norm_kernel<float, SM>, dim3(R), block, smem, stream, p);                            \
+  } while (0)
+  if (S == 1) BG_HYPER(1);
+  else if (S == 2) BG_HYPER(2);
+  else if (S == 3) BG_HYPER(3);
+  else if (S == 4) BG_HYPER(4);
+  else if (S <= 8) BG_HYPER(8);
+  else BG_HYPER(16);
+#undef BG_HYPER
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
+// kind 0 tanh-GELU, 1 clamped SwiGLU, 2 SwiGLU.  z points at the first gate column, the up column of a gate column is u_off further.
 int bg_glu(int dt, int kind, const float* z, int ldz, int u_off, void* out, int ldo, int R, int F, int Fo, float limit,
            const float* row_scale, const float* gate, int ld_gate, const int* total_rows, cudaStream_t stream) {
   using namespace bg::resid;
@@ -465,9 +641,11 @@ int bg_glu(int dt, int kind, const float* z, int ldz, int u_off, void* out, int 
   bg::launch_pdl(glu_kernel<OT, KIND>, grid, dim3(kThreads), 0, stream, z, ldz, u_off, reinterpret_cast<OT*>(out), ldo, F, \
                  Fo, limit, row_scale, gate, ld_gate, total_rows)
   if (dt == 0 && kind == 0) BG_GLU(__nv_bfloat16, 0);
-  else if (dt == 0) BG_GLU(__nv_bfloat16, 1);
+  else if (dt == 0 && kind == 1) BG_GLU(__nv_bfloat16, 1);
+  else if (dt == 0) BG_GLU(__nv_bfloat16, 2);
   else if (kind == 0) BG_GLU(float, 0);
-  else BG_GLU(float, 1);
+  else if (kind == 1) BG_GLU(float, 1);
+  else BG_GLU(float, 2);
 #undef BG_GLU
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }

@@ -2,9 +2,10 @@
 // sink, one query row per CTA (decode, short pieces of prompts, and the fp32 form).
 //
 //   s[h, j]  = scale * sum_g talk[h, g] (q[g] . k[kv(g), j])        g over all query heads, kv(g) = g / (H / G)
-//   seen     = first <= j <= position, first = position - position % chunk (chunk 0: first = 0)
+//   seen     = j <= position and (j >= first or j < keep), first = position - position % chunk (chunk 0: first = 0), with a
+//              window not before position - window + 1
 //   p[h, j]  = exp(s[h, j]) / (1 + sum exp(s[h, :]))                 (the 1 only with a sink)
-//   o[h]     = sum_j p[h, j] v[kv(h), j], times sigmoid(gate[h]) when there is a gate
+//   o[h]     = sum_j p[h, j] v[kv(h), j], times out_scale, times sigmoid(gate[h]) when there is a gate
 //
 // Without a mixing matrix a head keeps its own score.  Queries (on load) and keys (on the way to the cache) may carry rotary
 // positions: channel i turns with channel i + half.  Mixing couples all heads at a key, so a CTA takes all heads of its row.
@@ -42,9 +43,9 @@ struct Params {
   int ldo;
   float* part_o;                // [R, n_splits, H * dvp]
   float* part_ml;               // [R, n_splits, H, 2]
-  int H, G, dp, dvp, chunk, sink, n_splits;
+  int H, G, dp, dvp, chunk, window, keep, sink, n_splits;
   int k_warps;                  // warps with a K buffer (all of them unless heads are very wide)
-  float scale_log2;
+  float scale_log2, out_scale;
   const float* rope;            // [T, 2 * half] cosines, then sines, or null
   int half;
   const float* gate;            // [T, ld_gate] or null
@@ -142,10 +143,15 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
     }
   }
   for (int i = tid; i < Hp; i += kThreads) { m_s[i] = -INFINITY; l_s[i] = 0.f; }
-  const int first = p.chunk > 0 ? (L - 1) - (L - 1) % p.chunk : 0;
-  const int t_lo = first / NT, n_t = (L + NT - 1) / NT - t_lo;
-  const int my_lo = t_lo + (int)(((long long)n_t * split) / p.n_splits);
-  const int my_hi = t_lo + (int)(((long long)n_t * (split + 1)) / p.n_splits);
+  int first = p.chunk > 0 ? (L - 1) - (L - 1) % p.chunk : 0;
+  if (p.window > 0) first = max(first, L - p.window);
+  // kept first keys that end before the tile of `first` have tiles of their own, ahead of the others
+  int t_lo = first / NT, n_keep = 0;
+  if (p.keep > t_lo * NT) t_lo = 0;
+  else n_keep = (p.keep + NT - 1) / NT;
+  const int n_t = n_keep + (L + NT - 1) / NT - t_lo, past_keep = t_lo - n_keep;
+  const int my_lo = (int)(((long long)n_t * split) / p.n_splits);
+  const int my_hi = (int)(((long long)n_t * (split + 1)) / p.n_splits);
   const int* bt = p.block_table + (size_t)(p.row_seq != nullptr ? p.row_seq[r] : r) * p.bt_stride;
   const KT* cache = reinterpret_cast<const KT*>(p.cache);
 
@@ -154,8 +160,8 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
   const int krow = dp * (int)sizeof(KT) + 16;                     // bytes of a staged K row
   char* kb = kb_all + (size_t)warp * kbuf_bytes<KT>(dp);
   auto key_offset = [&](int tile) -> long long {                  // element offset of this lane's key, < 0 = not seen
-    const int pos = tile * NT + lane;
-    if (pos < first || pos >= L) return -1;
+    const int pos = (tile < n_keep ? tile : tile + past_keep) * NT + lane;
+    if (pos >= L || (pos < first && pos >= p.keep)) return -1;
     return (long long)bt[pos / p.page] * p.page_stride + (long long)(pos % p.page) * p.row;
   };
   auto fetch = [&](int unit, long long off) {                     // K rows of unit's key head -> this warp's buffer
@@ -329,7 +335,7 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
           const int h = h0 + i, col = h * dvp + cc * 4;
           const float4 v = make_float4(acc[n][i][0].x, acc[n][i][0].y, acc[n][i][1].x, acc[n][i][1].y);
           if (p.n_splits == 1) {
-            float inv = 1.0f / (l_s[h] + (p.sink ? exp2f(-m_s[h]) : 0.f));
+            float inv = p.out_scale / (l_s[h] + (p.sink ? exp2f(-m_s[h]) : 0.f));
             if (p.gate != nullptr) inv *= sigm(p.gate[(size_t)t * p.ld_gate + h]);
             put4(out + col, make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv));
           } else {
@@ -366,7 +372,7 @@ __global__ void merge_kernel(const Params p) {
     const float ms = ml[(size_t)s * p.H * 2];
     if (ms != -INFINITY) l += ml[(size_t)s * p.H * 2 + 1] * exp2f(ms - m);
   }
-  float inv = 1.0f / l;
+  float inv = p.out_scale / l;
   if (p.gate != nullptr) inv *= sigm(p.gate[(size_t)t * p.ld_gate + h]);
   for (int i = threadIdx.x; i < p.dvp / 4; i += blockDim.x) {
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -434,19 +440,20 @@ extern "C" {
 int bg_talk_rows(int dt, const float* q, int ldq, const float* talk, const void* cache, long long page_stride, int page,
                  int row, const int* block_table, int bt_stride, const int* row_seq, const int* row_ids, const int* lens,
                  void* out, int ldo, float* part_o, float* part_ml, int R, int H, int G, int dp, int dvp, int chunk,
-                 int sink, float scale, int n_splits, const float* rope, int half, const float* gate, int ld_gate,
+                 int window, int keep, int sink, float scale, float out_scale, int n_splits, const float* rope, int half, const float* gate, int ld_gate,
                  cudaStream_t stream) {
   using namespace bg::talk;
   if (R <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || dp <= 0 || dp % 8 || dvp <= 0 || dvp % 8 || row != G * (dp + dvp) || page <= 0 ||
       page_stride % 8 || ldq % 4 || ldo % 4 || (rope != nullptr && (half <= 0 || 2 * half > dp)) || n_splits < 1 || n_splits > 65535 || H > 65535 ||
+      window < 0 || keep < 0 ||
       (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return -1;
   Params p;
   p.q = q; p.ldq = ldq; p.talk = talk; p.cache = cache; p.page_stride = page_stride; p.page = page; p.row = row;
   p.block_table = block_table; p.bt_stride = bt_stride; p.row_seq = row_seq; p.row_ids = row_ids; p.lens = lens;
   p.out = out; p.ldo = ldo; p.part_o = part_o; p.part_ml = part_ml; p.H = H; p.G = G; p.dp = dp; p.dvp = dvp;
-  p.chunk = chunk; p.sink = sink; p.n_splits = n_splits; p.scale_log2 = scale * 1.4426950408889634f;
+  p.chunk = chunk; p.window = window; p.keep = keep; p.out_scale = out_scale; p.sink = sink; p.n_splits = n_splits; p.scale_log2 = scale * 1.4426950408889634f;
   p.rope = rope; p.half = half; p.gate = gate; p.ld_gate = ld_gate;
   const int items = G * ((H / G + 3) / 4) * (dvp / 4);
   const int ni = (items + kThreads - 1) / kThreads;

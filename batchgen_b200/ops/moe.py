@@ -11,7 +11,7 @@ from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
-from typing import Optional, Tuple
+from typing import Optional, Tuple, Union
 
 import torch
 
@@ -39,7 +39,7 @@ class ExpertWeights:
     quant: str = "none"
     interleaved: bool = False
     activation: str = "silu"             # silu | swiglu_clamped (GPT-OSS) | silu_limit (DeepSeek-V4: clamp, then SiLU(gate) * up)
-                                         # | swiglu_oai | gelu_tanh (``routed_rows``: fp32 activations of layer-listed models)
+                                         # | swiglu_oai | gelu_tanh | silu (``routed_rows``: fp32 activations of layer-listed models)
     act_limit: float = 0.0               # clamp of silu_limit (0 = none)
 
     @property
@@ -88,12 +88,14 @@ _SCORING_MODES = {"sigmoid": 0, "softmax": 1, "softmax_all": 2, "sqrtsoftplus": 
 
 
 def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, n_group: int = 1,
-                topk_group: int = 1, norm_topk_prob: bool = True, scale: float = 1.0, scoring: str = "sigmoid",
-                num_valid: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
-    """-> (idx [T, k] int32, w [T, k] fp32).  ``num_valid`` (device int32 scalar) marks rows >= it as
+                topk_group: int = 1, norm_topk_prob: Union[bool, str] = True, scale: float = 1.0, scoring: str = "sigmoid",
+                num_valid: Optional[torch.Tensor] = None, group_score: str = "") -> Tuple[torch.Tensor, torch.Tensor]:
+    """-> (idx [T, k] int32, w [T, k] fp32).  ``norm_topk_prob``: weights are divided by their sum (a single one only with
+    "always").  ``group_score``: how groups are ranked, "top2" (sum of the best two choice scores) or "max"; default "max" for
+    softmax_all, else "top2".  ``num_valid`` (device int32 scalar) marks rows >= it as
     padding: they get idx -1 / weight 0 and are ignored by dispatch."""
     if not logits.is_cuda:
-        idx, w = ref.router_topk(logits, bias, top_k, n_group, topk_group, norm_topk_prob, scale, scoring)
+        idx, w = ref.router_topk(logits, bias, top_k, n_group, topk_group, norm_topk_prob, scale, scoring, group_score)
         if num_valid is not None:
             nv = int(num_valid)
             idx[nv:] = -1
@@ -102,12 +104,14 @@ def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, 
     T, E = logits.shape
     if logits.stride(1) != 1:
         logits = logits.contiguous()
+    by_max = (group_score or ("max" if scoring == "softmax_all" else "top2")) == "max"
     idx = torch.empty(T, top_k, dtype=torch.int32, device=logits.device)
     w = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
     rc = _ext.lib().bg_router_topk(_ext.ptr(logits), ctypes.c_int(logits.stride(0)), _ext.ptr(bias), _ext.ptr(idx), _ext.ptr(w), ctypes.c_int(T),
                                    ctypes.c_int(E), ctypes.c_int(top_k), ctypes.c_int(n_group),
-                                   ctypes.c_int(topk_group), ctypes.c_int(int(norm_topk_prob)), ctypes.c_float(scale),
-                                   ctypes.c_int(_SCORING_MODES[scoring]), _ext.ptr(num_valid), _ext.stream())
+                                   ctypes.c_int(topk_group), ctypes.c_int(2 if norm_topk_prob == "always" else int(norm_topk_prob)),
+                                   ctypes.c_float(scale), ctypes.c_int(_SCORING_MODES[scoring]), ctypes.c_int(by_max),
+                                   _ext.ptr(num_valid), _ext.stream())
     _ext.check(rc, "bg_router_topk")
     return idx, w
 
@@ -292,13 +296,12 @@ def routed_rows(x: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.Tensor, e
     the model width) -> (y [rows, N] fp32 grouped by expert, pos [T, k] row of every (token, k) pair, -1 = none).
     ``weight_on_input``: the routing weight scales the expert's input (it is applied to the fp32 gate and up
     pre-activations, the same thing without rounding the product); the caller's sum over k then adds the rows as they are.
+    Without it the rows carry no weight and the caller's sum applies ``topk_w``.
 
     All shapes and row counts stay on the device: the call is graph capturable."""
     E, F2, _ = ew.w13.shape
     F = F2 // 2
     T, K = topk_idx.shape
-    if not weight_on_input:
-        raise NotImplementedError("routed_rows covers experts whose routing weight multiplies the input")
     kind = residual.GLU_KINDS[ew.activation]
     if not x.is_cuda:
         src, pos, off = permute(topk_idx, 0, E, num_valid)
@@ -310,7 +313,7 @@ def routed_rows(x: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.Tensor, e
             a, b = int(off[e]), int(off[e + 1])
             if b > a:
                 z = x[src[a:b].long()].float() @ ew.w13[e].float().t()
-                y[a:b] = residual.glu(z, F, ew.activation, ew.act_limit, row_scale=wrow[a:b]) @ ew.w2[e].float().t()
+                y[a:b] = residual.glu(z, F, ew.activation, ew.act_limit, row_scale=wrow[a:b] if weight_on_input else None) @ ew.w2[e].float().t()
         return y, pos
     assert kind is not None
     src, pos, offsets = permute(topk_idx, 0, E, num_valid, align=8)
@@ -318,5 +321,6 @@ def routed_rows(x: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.Tensor, e
     cap = src.shape[0]
     xs, ws = residual.moe_gather(x, pos, topk_w, cap)
     z = gemm.grouped_rows_gemm(xs, ew.w13, offsets, counts, max_rows=T)
-    act = residual.glu(z, F, ew.activation, ew.act_limit, row_scale=ws, total_rows=offsets[-1:], dtype=x.dtype)
+    act = residual.glu(z, F, ew.activation, ew.act_limit, row_scale=ws if weight_on_input else None, total_rows=offsets[-1:],
+                       dtype=x.dtype)
     return gemm.grouped_rows_gemm(act, ew.w2, offsets, counts, max_rows=T), pos

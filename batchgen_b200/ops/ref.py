@@ -193,7 +193,7 @@ def apply_rope(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, interleave
 # --------------------------------------------------------------------------- router
 def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, n_group: int = 1,
                 topk_group: int = 1, norm_topk_prob: bool = True, scale: float = 1.0,
-                scoring: str = "sigmoid") -> Tuple[torch.Tensor, torch.Tensor]:
+                scoring: str = "sigmoid", group_score: str = "") -> Tuple[torch.Tensor, torch.Tensor]:
     """logits: [T, E] fp32 -> (idx [T, k] int32 sorted by descending choice score, w [T, k] fp32).
 
     sigmoid scoring (DeepSeek-V3, GLM, Kimi): choice = sigmoid(logit) + bias; group-limited selection keeps
@@ -204,7 +204,8 @@ def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, 
     ranks groups by their best expert; the weights are the selected probabilities, renormalised only when
     ``norm_topk_prob`` is set.
     sqrtsoftplus scoring (DeepSeek-V4): score = sqrt(softplus(logit)), chosen with the bias added, weights
-    from the unbiased score."""
+    from the unbiased score.
+    ``group_score``: "top2" or "max" instead of the scoring's own; ``norm_topk_prob`` "always" covers top_k = 1 too."""
     T, E = logits.shape
     lf = logits.float()
     if scoring == "softmax":
@@ -221,14 +222,14 @@ def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: int, 
     choice = scores if bias is None else scores + bias.float().unsqueeze(0)
     if n_group > 1:
         g = choice.view(T, n_group, E // n_group)
-        gscore = g.max(-1)[0] if scoring == "softmax_all" else g.topk(2, dim=-1)[0].sum(-1)
+        gscore = g.max(-1)[0] if (group_score or ("max" if scoring == "softmax_all" else "top2")) == "max" else g.topk(2, dim=-1)[0].sum(-1)
         gidx = gscore.topk(topk_group, dim=-1)[1]
         gmask = torch.zeros_like(gscore).scatter_(1, gidx, 1.0)
         emask = gmask.unsqueeze(-1).expand(T, n_group, E // n_group).reshape(T, E)
         choice = choice.masked_fill(emask == 0, float("-inf"))
     _, idx = torch.topk(choice, top_k, dim=-1)
     w = scores.gather(1, idx)
-    if top_k > 1 and norm_topk_prob:
+    if norm_topk_prob == "always" or (top_k > 1 and norm_topk_prob):
         w = w / (w.sum(-1, keepdim=True) + 1e-20)
     return idx.to(torch.int32), w * scale
 

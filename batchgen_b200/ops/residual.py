@@ -1,6 +1,6 @@
 """Row operators of models with an fp32 residual stream: residual sum + RMS norm (with the embedding or the sublayers'
-outputs folded in), the same step of blocks with a norm before and after each sublayer, gated activations, operand casts,
-expert-row gather.
+outputs folded in), the same step of blocks with a norm before and after each sublayer and of hyper-connected residual streams,
+gated activations, operand casts, expert-row gather.
 
 CUDA tensors go to ``csrc/residual.cu``; CPU tensors to plain fp32 torch.  Operand dtype (norm output, activations) is
 bf16, or fp32 for the 32-bit form of a model.
@@ -17,7 +17,7 @@ import torch
 from . import _ext
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
-GLU_KINDS = {"gelu_tanh": 0, "swiglu_oai": 1}
+GLU_KINDS = {"gelu_tanh": 0, "swiglu_oai": 1, "silu": 2}
 CAST_KINDS = {"none": 0, "tanh": 1, "relu2": 2}
 
 
@@ -74,6 +74,8 @@ def residual_norm(x: torch.Tensor, w: torch.Tensor, eps: float, width: int, out_
 def _glu_ref(g: torch.Tensor, u: torch.Tensor, kind: str, limit: float) -> torch.Tensor:
     if kind == "gelu_tanh":
         return 0.5 * g * (1 + torch.tanh(math.sqrt(2 / math.pi) * (g + 0.044715 * g ** 3))) * u
+    if kind == "silu":
+        return g * torch.sigmoid(g) * u
     g, u = g.clamp(max=limit), u.clamp(-limit, limit)
     return g * torch.sigmoid(1.702 * g) * (u + 1)
 
@@ -81,7 +83,7 @@ def _glu_ref(g: torch.Tensor, u: torch.Tensor, kind: str, limit: float) -> torch
 def glu(z: torch.Tensor, F: int, kind: str, limit: float = 0.0, row_scale: Optional[torch.Tensor] = None,
         gate: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, total_rows: Optional[torch.Tensor] = None,
         dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """act(s * z[:, :F], s * z[:, F:2F]) * sigmoid(gate): ``kind`` gelu_tanh (tanh-GELU(g) * u) or swiglu_oai (g clamped from
+    """act(s * z[:, :F], s * z[:, F:2F]) * sigmoid(gate): ``kind`` gelu_tanh (tanh-GELU(g) * u), silu (SiLU(g) * u) or swiglu_oai (g clamped from
     above, u on both sides, g * sigmoid(1.702 g) * (u + 1)).  z fp32 (a column view is fine), ``row_scale`` [R] = s,
     ``gate`` [R, 1] (a view is fine).  ``out``: [R, >= F] view, columns past F become zero."""
     R = z.shape[0]
@@ -205,6 +207,68 @@ def sandwich_norm(x: torch.Tensor, norm: Norm, eps: float, width: int, out_cols:
         _ext.ptr(canon.slots if canon else None), _i(canon.w.shape[0] if canon else 0), _i(R), _i(width), ctypes.c_float(eps),
         _i(keep), _ext.stream())
     _ext.check(rc, "bg_sandwich_norm")
+    return y
+
+
+@dataclass
+class Hyper:
+    """Fixed hyper-connections of one sublayer over s residual streams (fp32): it reads sum_s read[s] x_s, then stream t becomes
+    sum_s mix[s, t] x_s + share[t] * output."""
+    read: torch.Tensor              # [s]
+    mix: torch.Tensor               # [s, s]
+    share: torch.Tensor             # [s]
+
+
+def hyper_norm(x: torch.Tensor, w: torch.Tensor, eps: float, width: int, out_cols: int, dtype: torch.dtype,
+               read: Optional[torch.Tensor] = None, hc: Optional[Hyper] = None, add: Optional[torch.Tensor] = None,
+               bias: Optional[torch.Tensor] = None, routed: Optional[torch.Tensor] = None, pos: Optional[torch.Tensor] = None,
+               route_w: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None, embed: Optional[torch.Tensor] = None,
+               embed_scale: float = 1.0, rows: Optional[torch.Tensor] = None, keep: bool = True) -> torch.Tensor:
+    """x [T, s, width rounded up to 4] fp32 residual streams.  With ``hc`` the previous sublayer's output joins them: ``add``
+    [T, width] fp32, plus ``bias``, plus sum_k route_w[t, k] * routed[pos[t, k]] (each optional).  ``ids``: every stream =
+    embed[ids] * embed_scale instead.  Then rmsnorm(sum_s read[s] x_s) * w as [R, out_cols] of ``dtype``, zero past ``width``
+    (``read`` None: the plain sum).  Vectors of the width are padded with zeros to a multiple of 4.  ``rows`` (int64) picks rows
+    of x; ``keep=False`` leaves x as it was."""
+    T, S, W4 = x.shape
+    R = T if rows is None else rows.shape[0]
+    if not x.is_cuda:
+        r = rows.long() if rows is not None else torch.arange(T)
+        cur = x[r, :, :width].clone()
+        if ids is not None:
+            cur = (embed[ids[r].long()].float() * embed_scale).unsqueeze(1).repeat(1, S, 1)
+        if hc is not None:
+            o = torch.zeros(R, width) if add is None else add[r, :width]
+            if bias is not None:
+                o = o + bias[:width]
+            if routed is not None:
+                at = pos[r].long()
+                o = o + (routed[at.clamp_min(0), :width] * (route_w[r] * (at >= 0)).unsqueeze(-1)).sum(1)
+            cur = torch.einsum("st,rsd->rtd", hc.mix, cur) + hc.share.view(1, S, 1) * o.unsqueeze(1)
+        if keep:
+            x[r, :, :width] = cur
+        u = cur.sum(1) if read is None else torch.einsum("s,rsd->rd", read, cur)
+        y = torch.zeros(R, out_cols, dtype=dtype)
+        y[:, :width] = (u / torch.sqrt((u * u).mean(-1, keepdim=True) + eps) * w[:width]).to(dtype)
+        return y
+    y = torch.empty(R, out_cols, dtype=dtype, device=x.device)
+    f32 = [t for t in (add, routed) if t is not None]
+    assert all(t.dtype == torch.float32 and t.stride(1) == 1 and t.stride(0) >= W4 for t in f32)
+    assert x.dtype == torch.float32 and x.is_contiguous() and W4 == pad_to(width, 4) and w.shape[0] == W4
+    assert (embed is None or embed.dtype == dtype) and (ids is None or (ids.dtype == torch.int32 and ids.shape[0] == T))
+    assert (rows is None or rows.dtype == torch.int64) and (add is None or add.shape[0] == T) and (bias is None or bias.shape[0] == W4)
+    assert hc is None or (hc.mix.shape == (S, S) and hc.share.shape[0] == S and hc.mix.is_contiguous())
+    assert read is None or read.shape[0] == S
+    if routed is not None:
+        assert pos.dtype == torch.int32 and pos.is_contiguous() and route_w.is_contiguous() and route_w.dtype == torch.float32
+        assert pos.shape == route_w.shape and pos.shape[0] == T
+    rc = _ext.lib().bg_hyper_norm(
+        _i(_DT[dtype]), _ext.ptr(x), _ext.ptr(rows), _ext.ptr(ids), _ext.ptr(embed), _i(embed.stride(0) if embed is not None else 0),
+        ctypes.c_float(embed_scale), _i(embed.shape[0] if embed is not None else 0), _ext.ptr(hc.mix if hc else None),
+        _ext.ptr(hc.share if hc else None), _ext.ptr(add), _i(add.stride(0) if add is not None else 0), _ext.ptr(bias),
+        _ext.ptr(routed), _i(routed.stride(0) if routed is not None else 0), _ext.ptr(pos), _ext.ptr(route_w),
+        _i(pos.shape[1] if pos is not None else 0), _ext.ptr(read), _ext.ptr(w), _ext.ptr(y), _i(out_cols), _i(R), _i(width), _i(S),
+        ctypes.c_float(eps), _i(keep), _ext.stream())
+    _ext.check(rc, "bg_hyper_norm")
     return y
 
 

@@ -1,5 +1,6 @@
 """Paged grouped-query attention for layer-listed models.  Optional parts: heads' scores mixed before the softmax, chunked
-visibility, a zero-score sink, rotary positions on queries and keys, a sigmoid gate per head on the output.
+visibility, a sliding window that keeps a sequence's first keys, a zero-score sink, rotary positions on queries and keys, a sigmoid
+gate per head on the output; biases and norms of query and key heads (``prepare_heads``, ``csrc/head_prep.cu``).
 
 Cache rows, and one query row per CTA for decode and short pieces: ``csrc/talking_attn.cu``; tensor-core flash attention for
 long pieces of prompts, over mixed queries (``csrc/talking_prefill.cu``) or plain heads (``csrc/gqa_prefill.cu``).
@@ -26,13 +27,27 @@ class TalkParams:
     dim_p: int
     vdim_p: int
     scale: float
-    chunk: int = 0                           # 0 = every earlier key is seen
+    chunk: int = 0                           # keys are seen from the query's own chunk on; 0 = every earlier key
+    window: int = 0                          # the last so many positions are seen, the query's own among them; 0 = all
+    keep: int = 0                            # with a window: so many first positions stay visible
+    out_scale: float = 1.0                   # factor of the output
     sink: bool = False                       # one added to the softmax denominator
     talk: Optional[torch.Tensor] = None      # [heads, heads] fp32: score_h <- sum_g talk[h, g] score_g; None = no mixing
 
     @property
     def kv_row(self) -> int:
         return self.kv_heads * (self.dim_p + self.vdim_p)
+
+    def first(self, pos: int) -> int:
+        """First position that a query at ``pos`` sees, kept first ones aside."""
+        first = pos - pos % self.chunk if self.chunk else 0
+        return max(first, pos + 1 - self.window) if self.window else first
+
+    def most_keys(self, keys: int) -> int:
+        """An upper bound of the keys a query sees out of ``keys``."""
+        for n in (self.chunk, self.window + self.keep if self.window else 0):
+            keys = min(keys, n) if n else keys
+        return keys
 
 
 def kv_write(kv: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, p: Optional[TalkParams] = None,
@@ -58,6 +73,54 @@ def kv_write(kv: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, p: Opti
     _ext.check(rc, "bg_talk_kv_write")
 
 
+@dataclass
+class HeadPrep:
+    """What happens to a layer's heads between their projections and the scores, rotary positions aside.  Vectors are fp32, padded
+    like the heads with zeros."""
+    dim: int                                 # real width of query and key heads
+    eps: float = 1e-6
+    bias: Optional[torch.Tensor] = None      # [heads * dim_p + kv_row], columns as projected: queries, keys, values
+    q_norm: Optional[torch.Tensor] = None    # [dim_p] gains of the RMS norms of query and key heads
+    k_norm: Optional[torch.Tensor] = None
+    interleaved: bool = False                # rotary pairs (2 i, 2 i + 1), else (i, i + dims / 2)
+
+
+def prepare_heads(z: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, p: TalkParams, h: HeadPrep,
+                  rope: Optional[torch.Tensor] = None, write_q: bool = True, operand: bool = False) -> Optional[torch.Tensor]:
+    """z [T, >= heads * dim_p + kv_row] fp32 columns of queries, keys and values: bias, norms and rotary positions; keys and values
+    go to cache[slot] (slots [T] int64, < 0: nowhere), queries back to z (``write_q``) and, with ``operand``, into the prompt
+    kernel's bf16 queries, which are returned."""
+    H, G, dp = p.heads, p.kv_heads, p.dim_p
+    P, page, row = cache.shape
+    if not z.is_cuda:
+        n = H * dp
+        x = z[:, :n + row] if h.bias is None else z[:, :n + row] + h.bias
+
+        def turn(t, heads, w):
+            t = t.reshape(-1, heads, dp)
+            if w is not None:
+                t = t / torch.sqrt((t * t).sum(-1, keepdim=True) / h.dim + h.eps) * w
+            return rotate_ref(t, rope, h.interleaved).reshape(-1, heads * dp)
+        kv_write(torch.cat([turn(x[:, n:n + G * dp], G, h.k_norm), x[:, n + G * dp:]], 1), slots, cache)
+        z[:, :n] = turn(x[:, :n], H, h.q_norm)
+        return None
+    T = z.shape[0]
+    assert z.dtype == torch.float32 and z.stride(1) == 1 and z.shape[1] >= H * dp + row and row == p.kv_row
+    assert cache.stride(1) == row and cache.stride(2) == 1 and slots.dtype == torch.int64 and slots.shape[0] == T
+    assert rope is None or (rope.is_contiguous() and rope.shape[0] == T)
+    assert h.bias is None or h.bias.shape[0] == H * dp + row
+    assert all(w is None or w.shape[0] == dp for w in (h.q_norm, h.k_norm))
+    kc = -(-dp // 64) * 64
+    qf = torch.empty(T, H, kc, dtype=torch.bfloat16, device=z.device) if operand else None
+    rc = _ext.lib().bg_head_prep(
+        _i(_DT[cache.dtype]), _ext.ptr(z), _i(z.stride(0)), _ext.ptr(h.bias), _ext.ptr(h.q_norm), _ext.ptr(h.k_norm),
+        ctypes.c_float(h.eps), _i(h.dim), _ext.ptr(rope), _i(rope.shape[1] // 2 if rope is not None else 0), _i(h.interleaved),
+        _ext.ptr(slots), _ext.ptr(cache), ctypes.c_longlong(cache.stride(0)), _i(page), _i(row), _i(write_q), _ext.ptr(qf), _i(kc),
+        ctypes.c_float(p.scale), _i(T), _i(H), _i(G), _i(dp), _i(p.vdim_p), _ext.stream())
+    _ext.check(rc, "bg_head_prep")
+    return qf
+
+
 def _rows_ref(q, p: TalkParams, cache, block_table, lens, out, row_seq, rope, gate):
     H, G, d, dv = p.heads, p.kv_heads, p.dim_p, p.vdim_p
     q = rotate_ref(q[:, : H * d].float().view(-1, H, d), rope).reshape(-1, H * d)
@@ -68,8 +131,8 @@ def _rows_ref(q, p: TalkParams, cache, block_table, lens, out, row_seq, rope, ga
         out[t, : H * dv] = 0
         if L <= 0:
             continue
-        first = (L - 1) // p.chunk * p.chunk if p.chunk else 0
-        pos = torch.arange(first, L)
+        pos = torch.arange(L)
+        pos = pos[(pos >= p.first(L - 1)) | (pos < p.keep)]
         bt = block_table[int(row_seq[t]) if row_seq is not None else t].long()
         rows = cache[bt[pos // page], pos % page].float()
         k = rows[:, : G * d].view(-1, G, d).repeat_interleave(rep, 1)
@@ -82,7 +145,7 @@ def _rows_ref(q, p: TalkParams, cache, block_table, lens, out, row_seq, rope, ga
             m = m.clamp_min(0)
         e = torch.exp(s - m)
         den = e.sum(-1, keepdim=True) + (torch.exp(-m) if p.sink else 0)
-        o = torch.einsum("hj,jhv->hv", e / den, v)
+        o = torch.einsum("hj,jhv->hv", e / den, v) * p.out_scale
         if gate is not None:
             o = o * torch.sigmoid(gate[t, :H].float()).unsqueeze(-1)
         out[t, : H * dv] = o.reshape(-1).to(out.dtype)
@@ -120,7 +183,7 @@ def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table
     H = p.heads
     if num_splits <= 0:
         keys = block_table.shape[1] * page
-        num_splits = _splits(R, min(keys, p.chunk) if p.chunk else keys, _ext.num_sms(q.device))
+        num_splits = _splits(R, p.most_keys(keys), _ext.num_sms(q.device))
     po = pml = None
     if num_splits > 1:
         po = torch.empty(R * num_splits * H * p.vdim_p, dtype=torch.float32, device=q.device)
@@ -129,8 +192,8 @@ def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table
         _i(_DT[cache.dtype]), _ext.ptr(q), _i(q.stride(0)), _ext.ptr(p.talk), _ext.ptr(cache),
         ctypes.c_longlong(cache.stride(0)), _i(page), _i(row), _ext.ptr(block_table), _i(block_table.stride(0)),
         _ext.ptr(row_seq), _ext.ptr(row_ids), _ext.ptr(lens), _ext.ptr(out), _i(out.stride(0)), _ext.ptr(po),
-        _ext.ptr(pml), _i(R), _i(H), _i(p.kv_heads), _i(p.dim_p), _i(p.vdim_p), _i(p.chunk), _i(p.sink),
-        ctypes.c_float(p.scale), _i(num_splits), _ext.ptr(rope), _i(rope.shape[1] // 2 if rope is not None else 0),
+        _ext.ptr(pml), _i(R), _i(H), _i(p.kv_heads), _i(p.dim_p), _i(p.vdim_p), _i(p.chunk), _i(p.window),
+        _i(p.keep), _i(p.sink), ctypes.c_float(p.scale), ctypes.c_float(p.out_scale), _i(num_splits), _ext.ptr(rope), _i(rope.shape[1] // 2 if rope is not None else 0),
         _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0), _ext.stream())
     if rc in (-1, -3):
         raise _ext.KernelError(f"attend_rows: heads {H}/{p.kv_heads}, widths {p.dim_p}/{p.vdim_p} are outside the kernel's "
@@ -149,7 +212,8 @@ def prefill_supported(p: TalkParams, dtype: torch.dtype, page: int) -> bool:
     return dtype == torch.bfloat16 and p.vdim_p <= 256 and page >= 16 and (p.talk is not None or p.dim_p <= 256)
 
 
-def prefill_work(cu: Sequence[int], ctx: Sequence[int], chunk: int, min_tokens: int = 1) -> List[Tuple[int, int, int, int]]:
+def prefill_work(cu: Sequence[int], ctx: Sequence[int], chunk: int, min_tokens: int = 1,
+                 window: int = 0) -> List[Tuple[int, int, int, int]]:
     """Tiles (first query row, queries, sequence, position of the first query) of every piece of at least ``min_tokens``
     tokens, the tiles with the most visible keys first."""
     out = []
@@ -159,7 +223,9 @@ def prefill_work(cu: Sequence[int], ctx: Sequence[int], chunk: int, min_tokens: 
             continue
         for q0 in range(a, b, _TILE):
             out.append((q0, min(_TILE, b - q0), i, int(ctx[i]) + q0 - a))
-    out.sort(key=lambda w: -(w[3] + w[1] - (w[3] // chunk * chunk if chunk else 0)))
+    def first(pos):
+        return max(pos // chunk * chunk if chunk else 0, pos + 1 - window if window else 0)
+    out.sort(key=lambda w: -(w[3] + w[1] - first(w[3])))
     return out
 
 
@@ -178,36 +244,43 @@ def work_blocks(work: List[Tuple[int, int, int, int]], rows: int, device) -> Lis
 
 def attend_prefill(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table: torch.Tensor, out: torch.Tensor,
                    blocks: List[Tuple[int, int, torch.Tensor]], rope: Optional[torch.Tensor] = None,
-                   gate: Optional[torch.Tensor] = None) -> None:
+                   gate: Optional[torch.Tensor] = None, operand: Optional[torch.Tensor] = None) -> None:
     """CUDA, bf16 cache: q [T, >= H * dim_p] fp32 -> out [T, >= H * vdim_p] for the rows covered by ``blocks``
     (``work_blocks``); ``rope`` and ``gate`` as for ``attend_rows``.  The keys of every query are in the cache already.
+    ``operand``: the queries as ``prepare_heads`` returns them, instead of q and ``rope``.
 
     Mixed heads contract over a token's whole key block, plain heads over their own key head's columns."""
     P, page, row = cache.shape
     H, G = p.heads, p.kv_heads
     plain = p.talk is None
-    assert plain or (rope is None and gate is None), "mixed heads with rotary queries or output gates are not covered"
+    assert plain or (rope is None and gate is None and not p.window and p.out_scale == 1.0), \
+        "mixed heads with rotary queries, windows, output gates or scales are not covered"
     kc = -(-(p.dim_p if plain else G * p.dim_p) // 64) * 64
     assert q.dtype == torch.float32 and q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == cache.dtype == torch.bfloat16
     assert row == p.kv_row and cache.stride(1) == row and block_table.dtype == torch.int32
+    assert operand is None or (plain and rope is None and operand.is_contiguous() and operand.shape == (q.shape[0], H, kc))
     L = _ext.lib()
     for lo, n, work in blocks:
-        qf = torch.empty(n, H, kc, dtype=torch.bfloat16, device=q.device)
-        if plain:
+        qf = torch.empty(n, H, kc, dtype=torch.bfloat16, device=q.device) if operand is None else operand[lo:lo + n]
+        if operand is not None:
+            rc = 0
+        elif plain:
             rc = L.bg_gqa_prompt_queries(_ext.ptr(q[lo:]), _i(q.stride(0)), _ext.ptr(rope[lo:] if rope is not None else None),
                                 _i(rope.shape[1] // 2 if rope is not None else 0), _ext.ptr(qf), _i(n), _i(H), _i(p.dim_p),
                                 _i(kc), ctypes.c_float(p.scale), _ext.stream())
         else:
             rc = L.bg_talk_fold(_ext.ptr(q[lo:]), _i(q.stride(0)), _ext.ptr(p.talk), _ext.ptr(qf), _i(n), _i(H), _i(G),
                                 _i(p.dim_p), _i(kc), ctypes.c_float(p.scale), _ext.stream())
-        _ext.check(rc, "bg_gqa_prompt_queries" if plain else "bg_talk_fold")
+        if operand is None:
+            _ext.check(rc, "bg_gqa_prompt_queries" if plain else "bg_talk_fold")
         where = (_ext.ptr(qf), _ext.ptr(cache), ctypes.c_longlong(cache.stride(0)), _i(P), _i(page), _i(row),
                  _ext.ptr(block_table), _i(block_table.stride(0)), _i(block_table.shape[1]), _ext.ptr(work), _i(work.shape[0]),
                  _i(n), _i(lo), _ext.ptr(out), _i(out.stride(0)), _i(H), _i(G), _i(p.dim_p), _i(p.vdim_p), _i(kc), _i(p.chunk),
                  _i(p.sink))
         status = _ext.ptr(_ext.status_word(q.device))
         if plain:
-            rc = L.bg_gqa_prompt(*where, _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0), status, _ext.stream())
+            rc = L.bg_gqa_prompt(*where, _i(p.window), _i(p.keep), ctypes.c_float(p.out_scale), _ext.ptr(gate),
+                                 _i(gate.stride(0) if gate is not None else 0), status, _ext.stream())
         else:
             rc = L.bg_talk_prefill(*where, status, _ext.stream())
         _ext.check(rc, "bg_gqa_prompt" if plain else "bg_talk_prefill")

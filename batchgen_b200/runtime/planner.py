@@ -70,7 +70,7 @@ def weight_bytes_per_rank(cfg: ModelConfig, tp: int, ep: int, sequence_parallel:
     """-> (non-expert bytes, routed-expert bytes resident on the GPU) for one rank."""
     H = cfg.hidden_size
     if cfg.is_layered:
-        experts = sum(3 * H * s.mlp.ff * s.mlp.experts * 2 for s in cfg.layer_specs)
+        experts = sum(3 * H * s.mlp.ff * s.mlp.experts * 2 for s in cfg.layer_specs if s.weights_of < 0)
         return int(cfg.param_count() * 2 - experts), int(experts)
     qb = _quant_bytes(cfg)
     lin = 1.0 + 4.0 / (128 * 128) if cfg.quant != "none" else 2.0     # attention / dense linears are FP8 or bf16
@@ -139,7 +139,7 @@ def layered_workspace_bytes(cfg: ModelConfig) -> int:
         n_cat = sum(m.heads * m.vdim_p for m in s.mixers) + (f.shared_ff if f.kind == "moe" else f.ff)
         routed = f.top * (2 * cfg.hidden_size + 8 * f.ff + 2 * f.ff + 4 * cfg.hidden_size) if f.kind == "moe" else 0
         most = max(most, 4 * n_in + 2 * n_cat + routed)
-    return most + 16 * cfg.hidden_size
+    return most + (12 + 4 * max(cfg.streams, 1)) * cfg.hidden_size
 
 
 def state_pool_bytes(cfg: ModelConfig, ecfg: EngineConfig) -> int:

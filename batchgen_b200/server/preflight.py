@@ -160,12 +160,19 @@ def _layered_contract(cfg, world: int, on_gpu: bool) -> List[str]:
                 bad.append(f"layer {i}: {m.heads} heads x {m.vdim} value channels exceed the decode attention kernel")
         if f.kind == "moe" and (f.top > 16 or f.experts > 1024 or f.top > f.experts):
             bad.append(f"layer {i}: top {f.top} of {f.experts} experts (the router takes up to 16 of 1,024)")
+        if f.kind == "moe" and f.groups > 32:
+            bad.append(f"layer {i}: {f.groups} groups of experts (the router takes up to 32)")
+        if any(not m.recurrent and (m.bias or m.qk_norm or m.rot_interleaved) and m.dim_p > 1024 for m in s.mixers):
+            bad.append(f"layer {i}: attention head width {s.mixer.dim} exceeds 1024")
     if bad:
         raise PreflightError("model contract: " + "; ".join(bad))
     if not on_gpu:
         return ["fp32 reference path: no kernel geometry rules apply"]
     if cfg.sandwich and cfg.hidden_size > 16384:
         raise PreflightError(f"model contract: width {cfg.hidden_size} exceeds the norm kernel's 16384")
+    if cfg.streams > 16 or (cfg.streams and cfg.hidden_size > 8192):
+        raise PreflightError(f"model contract: {cfg.streams} residual streams of width {cfg.hidden_size} (the norm kernel takes up to "
+                             "16 of 8192)")
     return ["layer-listed model: tcgen05 projections, experts and prompt attention; recurrences, decode attention and row "
             "operators as CUDA kernels of their own"]
 
