@@ -2,7 +2,7 @@
 // head, rotary positions; keys and values go to the paged cache, queries back to their columns (fp32, for the row kernel) and / or
 // into the bf16 operand of the prompt kernel, times scale * log2(e).
 //
-// A warp takes one head of one token.  Norms and rotations are fp32; channels past the real width stay zero (zero weights and
+// A warp takes kHeads heads of one token, whose loads are all issued before any is used.  Norms and rotations are fp32; channels past the real width stay zero (zero weights and
 // biases).  Pairs that turn together: (i, i + half), or (2 i, 2 i + 1) when interleaved.
 #define BG_FILE_TAG 30     // kernel-trace ids of this file are (tag << 16) | line
 #include "common.cuh"
@@ -11,6 +11,7 @@ namespace bg {
 namespace heads {
 
 constexpr int kWarps = 8;
+constexpr int kHeads = 2;      // of a warp: u and u + kWarps
 constexpr int kMaxWidth = 1024;
 
 struct Params {
@@ -38,94 +39,126 @@ __device__ __forceinline__ void put4(__nv_bfloat16* p, float4 v) {
   *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(o);
 }
 __device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 biased(const float* z, const float* b, int c) {
-  float4 v = ld4(z + c);
-  if (b != nullptr) {
-    const float4 a = ld4(b + c);
-    v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
-  }
-  return v;
-}
 
-template <typename KT>
+// NV: 4-wide vectors of a head in a lane's registers (widths up to 128 NV)
+template <typename KT, int NV, bool INTER>
 __global__ void __launch_bounds__(kWarps * 32) prep_kernel(const Params p) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   extern __shared__ __align__(16) float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t = blockIdx.x, u = blockIdx.y * kWarps + warp;
-  if (u >= p.H + 2 * p.G) return;
-  const bool query = u < p.H;
-  const long long slot = query ? -1 : p.slots[t];
-  if (!query && slot < 0) return;
-  KT* dst = query ? nullptr : reinterpret_cast<KT*>(p.cache) + (slot / p.page) * p.page_stride + (slot % p.page) * p.row;
-  const int qk = (p.H + p.G) * p.dp;
-  if (u >= p.H + p.G) {                                          // a value head: bias only
-    const int g = u - p.H - p.G;
-    const float* z = p.z + (size_t)t * p.ld + qk + g * p.dvp;
-    const float* b = p.bias != nullptr ? p.bias + qk + g * p.dvp : nullptr;
-    for (int c = lane * 4; c < p.dvp; c += 128) put4(dst + p.G * p.dp + g * p.dvp + c, biased(z, b, c));
-    return;
-  }
-  float* z = p.z + (size_t)t * p.ld + u * p.dp;
-  const float* b = p.bias != nullptr ? p.bias + u * p.dp : nullptr;
-  const float* w = query ? p.wq : p.wk;
-  float* head = sm + warp * p.dp;
-  float ss = 0.f;
-  for (int c = lane * 4; c < p.dp; c += 128) {
-    const float4 v = biased(z, b, c);
-    put4(head + c, v);
-    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-  }
-  if (w != nullptr) {
-    const float rstd = 1.0f / sqrtf(warp_sum(ss) * p.inv_d + p.eps);
-    for (int c = lane * 4; c < p.dp; c += 128) {
-      const float4 v = ld4(head + c), g = ld4(w + c);
-      put4(head + c, make_float4(v.x * rstd * g.x, v.y * rstd * g.y, v.z * rstd * g.z, v.w * rstd * g.w));
-    }
-  }
-  __syncwarp();
+  const int t = blockIdx.x, units = p.H + 2 * p.G, qk = (p.H + p.G) * p.dp;
+  const float* zr = p.z + (size_t)t * p.ld;
   const float* cs = p.rope != nullptr ? p.rope + (size_t)t * 2 * p.half : nullptr;
-  auto turned = [&](int c) -> float4 {                           // channels c .. c + 3
-    float4 v = ld4(head + c);
-    if (cs == nullptr || c >= 2 * p.half) return v;
-    float* x = &v.x;
-    if (p.interleaved) {
+  const long long slot = p.slots[t];
+  float4 v[kHeads][NV];
+  int off[kHeads], width[kHeads];                                 // first column, 0 = no head
 #pragma unroll
-      for (int j = 0; j < 4; j += 2) {
-        const int i = (c + j) >> 1;
-        if (i < p.half) {
-          const float a = x[j], d = x[j + 1], co = cs[i], si = cs[p.half + i];
-          x[j] = a * co - d * si;
-          x[j + 1] = d * co + a * si;
-        }
+  for (int i = 0; i < kHeads; ++i) {
+    const int u = blockIdx.y * kWarps * kHeads + i * kWarps + warp, g = u - p.H - p.G;
+    off[i] = g < 0 ? u * p.dp : qk + g * p.dvp;
+    width[i] = u >= units || (u >= p.H && slot < 0) ? 0 : g < 0 ? p.dp : p.dvp;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int c = lane * 4 + n * 128;
+      v[i][n] = c < width[i] ? ld4(zr + off[i] + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  }
+  KT* dst = reinterpret_cast<KT*>(p.cache) + (slot / p.page) * p.page_stride + (slot % p.page) * p.row;
+#pragma unroll
+  for (int i = 0; i < kHeads; ++i) {
+    if (width[i] == 0) continue;                                  // the same for all lanes of the warp
+    const int u = blockIdx.y * kWarps * kHeads + i * kWarps + warp;
+    const bool query = u < p.H, value = u >= p.H + p.G;
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int c = lane * 4 + n * 128;
+      if (c < width[i] && p.bias != nullptr) {
+        const float4 a = ld4(p.bias + off[i] + c);
+        v[i][n].x += a.x; v[i][n].y += a.y; v[i][n].z += a.z; v[i][n].w += a.w;
       }
-    } else {
+      ss += v[i][n].x * v[i][n].x + v[i][n].y * v[i][n].y + v[i][n].z * v[i][n].z + v[i][n].w * v[i][n].w;
+    }
+    if (value) {
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int e = c + j;
-        if (e < 2 * p.half) {
-          const bool low = e < p.half;
-          const int i = low ? e : e - p.half;
-          const float other = head[low ? e + p.half : i], co = cs[i], si = cs[p.half + i];
-          x[j] = low ? x[j] * co - other * si : x[j] * co + other * si;
+      for (int n = 0; n < NV; ++n)
+        if (lane * 4 + n * 128 < p.dvp) put4(dst + off[i] - p.H * p.dp + lane * 4 + n * 128, v[i][n]);
+      continue;
+    }
+    const float* w = query ? p.wq : p.wk;
+    if (w != nullptr) {
+      const float rstd = 1.0f / sqrtf(warp_sum(ss) * p.inv_d + p.eps);
+#pragma unroll
+      for (int n = 0; n < NV; ++n) {
+        const int c = lane * 4 + n * 128;
+        if (c < p.dp) {
+          const float4 g = ld4(w + c);
+          v[i][n] = make_float4(v[i][n].x * rstd * g.x, v[i][n].y * rstd * g.y, v[i][n].z * rstd * g.z, v[i][n].w * rstd * g.w);
         }
       }
     }
-    return v;
-  };
-  if (!query) {
-    KT* k = dst + (u - p.H) * p.dp;
-    for (int c = lane * 4; c < p.dp; c += 128) put4(k + c, turned(c));
-    return;
+    float* head = sm + warp * p.dp;                               // (i, i + half): the partner may sit in another lane
+    if (cs != nullptr && !INTER) {
+      __syncwarp();
+#pragma unroll
+      for (int n = 0; n < NV; ++n)
+        if (lane * 4 + n * 128 < p.dp) put4(head + lane * 4 + n * 128, v[i][n]);
+      __syncwarp();
+    }
+    __nv_bfloat16* qf = query && p.qf != nullptr ? p.qf + ((size_t)t * p.H + u) * p.kc : nullptr;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int c = lane * 4 + n * 128;
+      if (c >= p.dp) continue;
+      float* x = &v[i][n].x;
+      if (cs != nullptr) {
+        if (INTER) {
+#pragma unroll
+          for (int j = 0; j < 4; j += 2) {
+            const int k = (c + j) >> 1;
+            if (k < p.half) {
+              const float a = x[j], d = x[j + 1], co = cs[k], si = cs[p.half + k];
+              x[j] = a * co - d * si;
+              x[j + 1] = d * co + a * si;
+            }
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const int e = c + j;
+            if (e < 2 * p.half) {
+              const bool low = e < p.half;
+              const int k = low ? e : e - p.half;
+              const float other = head[low ? e + p.half : k], co = cs[k], si = cs[p.half + k];
+              x[j] = low ? x[j] * co - other * si : x[j] * co + other * si;
+            }
+          }
+        }
+      }
+      if (!query) {
+        put4(dst + off[i] - p.H * p.dp + c, v[i][n]);
+        continue;
+      }
+      if (p.write_q) put4(p.z + (size_t)t * p.ld + off[i] + c, v[i][n]);
+      if (qf != nullptr) put4(qf + c, make_float4(x[0] * p.q_scale, x[1] * p.q_scale, x[2] * p.q_scale, x[3] * p.q_scale));
+    }
+    if (qf != nullptr)
+      for (int c = p.dp + lane * 4; c < p.kc; c += 128) put4(qf + c, make_float4(0.f, 0.f, 0.f, 0.f));
   }
-  __nv_bfloat16* qf = p.qf != nullptr ? p.qf + ((size_t)t * p.H + u) * p.kc : nullptr;
-  for (int c = lane * 4; c < p.dp; c += 128) {
-    const float4 v = turned(c);
-    if (p.write_q) put4(z + c, v);
-    if (qf != nullptr) put4(qf + c, make_float4(v.x * p.q_scale, v.y * p.q_scale, v.z * p.q_scale, v.w * p.q_scale));
-  }
-  if (qf != nullptr)
-    for (int c = p.dp + lane * 4; c < p.kc; c += 128) put4(qf + c, make_float4(0.f, 0.f, 0.f, 0.f));
+}
+
+template <typename KT, int NV>
+static void launch(const Params& p, dim3 grid, size_t smem, cudaStream_t stream) {
+  if (p.interleaved) bg::launch_pdl(prep_kernel<KT, NV, true>, grid, dim3(kWarps * 32), 0, stream, p);
+  else bg::launch_pdl(prep_kernel<KT, NV, false>, grid, dim3(kWarps * 32), smem, stream, p);
+}
+template <typename KT>
+static void launch(const Params& p, dim3 grid, size_t smem, cudaStream_t stream) {
+  const int w = p.dp > p.dvp ? p.dp : p.dvp;
+  if (w <= 128) launch<KT, 1>(p, grid, smem, stream);
+  else if (w <= 256) launch<KT, 2>(p, grid, smem, stream);
+  else if (w <= 512) launch<KT, 4>(p, grid, smem, stream);
+  else launch<KT, 8>(p, grid, smem, stream);
 }
 
 }  // namespace heads
@@ -140,7 +173,7 @@ int bg_head_prep(int dt, float* z, int ld, const float* bias, const float* wq, c
                  void* qf, int kc, float scale, int T, int H, int G, int dp, int dvp, cudaStream_t stream) {
   using namespace bg::heads;
   if (T <= 0) return 0;
-  if (H <= 0 || G <= 0 || dp <= 0 || dp % 8 || dp > kMaxWidth || d <= 0 || d > dp || dvp <= 0 || dvp % 8 || row != G * (dp + dvp) ||
+  if (H <= 0 || G <= 0 || dp <= 0 || dp % 8 || dp > kMaxWidth || d <= 0 || d > dp || dvp <= 0 || dvp % 8 || dvp > kMaxWidth || row != G * (dp + dvp) ||
       ld % 4 || ld < H * dp + row || page <= 0 || page_stride % 8 || (rope != nullptr && (half <= 0 || 2 * half > dp)) ||
       (qf != nullptr && (kc < dp || kc % 8)) || (wq == nullptr) != (wk == nullptr) || reinterpret_cast<uintptr_t>(z) % 16)
     return -1;
@@ -149,11 +182,11 @@ int bg_head_prep(int dt, float* z, int ld, const float* bias, const float* wq, c
   p.interleaved = interleaved; p.slots = slots; p.cache = cache; p.page_stride = page_stride; p.page = page; p.row = row;
   p.write_q = write_q; p.qf = reinterpret_cast<__nv_bfloat16*>(qf); p.kc = kc; p.q_scale = scale * 1.4426950408889634f;
   p.H = H; p.G = G; p.dp = dp; p.dvp = dvp;
-  const dim3 grid(T, (H + 2 * G + kWarps - 1) / kWarps), block(kWarps * 32);
+  const dim3 grid(T, (H + 2 * G + kWarps * kHeads - 1) / (kWarps * kHeads));
   if (grid.y > 65535) return -1;
   const size_t smem = (size_t)kWarps * dp * sizeof(float);
-  if (dt == 0) bg::launch_pdl(prep_kernel<__nv_bfloat16>, grid, block, smem, stream, p);
-  else bg::launch_pdl(prep_kernel<float>, grid, block, smem, stream, p);
+  if (dt == 0) launch<__nv_bfloat16>(p, grid, smem, stream);
+  else launch<float>(p, grid, smem, stream);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 

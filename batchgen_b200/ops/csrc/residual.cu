@@ -342,14 +342,15 @@ struct HyperParams {
 };
 
 constexpr int kMaxStreams = 16;
+constexpr int kHyperThreads = 640;
 
 // One block per row; thread i owns the 4-wide vectors i, i + blockDim, ... of every stream.  SM: streams, or an upper bound of them
 // (above 4).  What the norm reads waits in shared memory for its root mean square.
 template <typename OT, int SM>
-__global__ void __launch_bounds__(kThreads) hyper_norm_kernel(const HyperParams p) {
+__global__ void __launch_bounds__(SM <= 4 ? kHyperThreads : kThreads) hyper_norm_kernel(const HyperParams p) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   extern __shared__ float row[];
-  __shared__ float red[kThreads / 32];
+  __shared__ float red[kHyperThreads / 32];
   __shared__ float mix[SM * SM], share[SM], read[SM], rw[kMaxK];
   __shared__ int pos_s[kMaxK];
   const int tid = threadIdx.x, NT = blockDim.x, S = SM <= 4 ? SM : p.S;
@@ -396,13 +397,18 @@ __global__ void __launch_bounds__(kThreads) hyper_norm_kernel(const HyperParams 
         o.x += b.x; o.y += b.y; o.z += b.z; o.w += b.w;
       }
       if (p.routed != nullptr) {
-#pragma unroll 4
-        for (int k = 0; k < p.K; ++k) {
-          const int r = pos_s[k];
-          if (r < 0) continue;
-          const float4 a = *reinterpret_cast<const float4*>(p.routed + (size_t)r * p.ld_routed + c);
-          const float g = rw[k];
-          o.x = fmaf(g, a.x, o.x); o.y = fmaf(g, a.y, o.y); o.z = fmaf(g, a.z, o.z); o.w = fmaf(g, a.w, o.w);
+        for (int k0 = 0; k0 < p.K; k0 += 4) {            // four rows' loads at a time
+          float4 a[4];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const int r = k0 + k < p.K ? pos_s[k0 + k] : -1;
+            a[k] = r >= 0 ? *reinterpret_cast<const float4*>(p.routed + (size_t)r * p.ld_routed + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float g = k0 + k < p.K ? rw[k0 + k] : 0.f;
+            o.x = fmaf(g, a[k].x, o.x); o.y = fmaf(g, a[k].y, o.y); o.z = fmaf(g, a[k].z, o.z); o.w = fmaf(g, a[k].w, o.w);
+          }
         }
       }
       if (c + 1 >= D) o.y = 0.f;
@@ -612,7 +618,9 @@ int bg_hyper_norm(int dt, float* x, const long long* rows, const int* ids, const
   p.x = x; p.rows = rows; p.ids = ids; p.embed = embed; p.lde = lde; p.escale = escale; p.vocab = vocab; p.mix = mix;
   p.share = share; p.add = add; p.ld_add = ld_add; p.bias = bias; p.routed = routed; p.ld_routed = ld_routed; p.pos = pos;
   p.route_w = route_w; p.K = K; p.read = read; p.w = w; p.y = y; p.ldy = ldy; p.D = D; p.S = S; p.eps = eps; p.keep = keep;
-  const int nv = D4 / 4, per = (nv + kThreads - 1) / kThreads;
+  // few rows: as many threads as vectors, so that a row's loads fly together
+  const int most = R <= 296 && S <= 4 ? kHyperThreads : kThreads;
+  const int nv = D4 / 4, per = (nv + most - 1) / most;
   const dim3 block(((nv + per - 1) / per + 31) / 32 * 32);
   const size_t smem = (size_t)D4 * sizeof(float);
 #define BG_HYPER(SM)                                                                                              \

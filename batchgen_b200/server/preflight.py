@@ -162,8 +162,8 @@ def _layered_contract(cfg, world: int, on_gpu: bool) -> List[str]:
             bad.append(f"layer {i}: top {f.top} of {f.experts} experts (the router takes up to 16 of 1,024)")
         if f.kind == "moe" and f.groups > 32:
             bad.append(f"layer {i}: {f.groups} groups of experts (the router takes up to 32)")
-        if any(not m.recurrent and (m.bias or m.qk_norm or m.rot_interleaved) and m.dim_p > 1024 for m in s.mixers):
-            bad.append(f"layer {i}: attention head width {s.mixer.dim} exceeds 1024")
+        if any(not m.recurrent and (m.bias or m.qk_norm or m.rot_interleaved) and max(m.dim_p, m.vdim_p) > 1024 for m in s.mixers):
+            bad.append(f"layer {i}: attention head widths {s.mixer.dim}, {s.mixer.vdim} exceed 1024")
     if bad:
         raise PreflightError("model contract: " + "; ".join(bad))
     if not on_gpu:

@@ -1,14 +1,17 @@
-"""Layer-listed models (Nanurax, Pamevik) beside the framework's closest existing model at equal size.
+"""Layer-listed models (Nanurax, Pamevik, Bolisun) beside the framework's closest existing model at equal size.
 
-``bench.py --workload nanurax | pamevik``: both models have four layers of a real model's size (width 2304, 32 heads of 128,
+``bench.py --workload nanurax | pamevik | bolisun``: both models have four layers of a real model's size (width 2304, 32 heads of 128,
 bf16), three recurrent layers to one attention layer.  Nanurax runs the generalised delta rule and chunked talking-heads
 attention with one dense and three mixture feed-forwards (64 experts of which 8 run); Pamevik runs two channel-delta layers, an
 mLSTM layer and attention beside retention, with dense feed-forwards.  The other one is a Kimi-Linear cut with KDA and MLA
-layers and the same kinds of feed-forwards.  Prefill is one packed forward over fresh prompts, decode is a captured step over
+layers and the same kinds of feed-forwards.  Bolisun runs four layers of windowed attention beside retention, with one dense and
+three mixture feed-forwards; next to the Kimi-Linear cut (mixtures of the same size) it has Pamevik with four layers of attention
+beside retention, whose dense feed-forwards hold as many weights as a token's experts.  Prefill is one packed forward over fresh prompts, decode is a captured step over
 sequences with cached context; random weights, CUDA events, medians, the L2 flushed before every timed call.
 
 ``kernels`` of the result times the new kernels beside their likes (recurrences against KDA, decode attention against the
-paged GQA kernel, prompt attention against the expanded MLA kernel, norms against the fused residual norm) with the share of
+paged GQA kernel, prompt attention against the expanded MLA kernel, norms against the fused residual norm; Bolisun's against
+Pamevik's and Nanurax's) with the share of
 the measured roofline each reaches.
 """
 from __future__ import annotations
@@ -55,9 +58,14 @@ class _Timer:
 
 
 def _closest(design: str):
+    import dataclasses
     from batchgen_b200.config import get_model_config
-    mlp = dict(n_routed_experts=64, num_experts_per_tok=8) if design == "nanurax" else dict(first_k_dense=4)
-    return get_model_config("kimi-linear-48b", num_layers=4, kda_layers=(0, 1, 2), **mlp)
+    mlp = dict(first_k_dense=4) if design == "pamevik" else dict(n_routed_experts=64, num_experts_per_tok=8)
+    out = [get_model_config("kimi-linear-48b", num_layers=4, kda_layers=(0, 1, 2), **mlp)]
+    if design == "bolisun":
+        cfg = get_model_config("pamevik-bench")
+        out.insert(0, dataclasses.replace(cfg, name="pamevik-beside", layer_specs=cfg.layer_specs[-1:] * 4))
+    return out
 
 
 def _model_rates(cfg, dev, timer: _Timer) -> Dict[str, object]:
@@ -265,6 +273,100 @@ def _pamevik_kernels(dev, timer: _Timer, peaks) -> List[Dict[str, object]]:
     return add.rows
 
 
+def _bolisun_kernels(dev, timer: _Timer, peaks) -> List[Dict[str, object]]:
+    import torch
+    from batchgen_b200.config import get_model_config
+    from batchgen_b200.ops import conv, moe, recurrent, residual, talking
+    bf, add = torch.bfloat16, _Rows(peaks)
+    row, W, E, K, Fe = 2 * G * D, 2304, 64, 8, 1024
+    left = get_model_config("bolisun-bench").layer_specs[0].mixer
+    win, keep = left.window, left.keep_first
+    rot = conv.Rotary.make(D, 1e6, dev, True, left.yarn)
+    half = conv.Rotary.make(D, 1e6, dev)
+    norm, bias = torch.ones(D, device=dev), torch.zeros(HD + row, device=dev)
+    prep = talking.HeadPrep(D, 1e-6, bias, norm, norm, True)
+    full = talking.TalkParams(H, G, D, D, D ** -0.5)
+    near = talking.TalkParams(H, G, D, D, D ** -0.5, window=win, keep=keep, out_scale=0.5)
+    gains = residual.Norm(torch.ones(W, device=dev), torch.zeros(W, device=dev), True)
+    for B, T in STATE_CASES:
+        R, size, slots, cu, init = _state_case(dev, B, T)
+        prompt = T > 1
+        z, out = torch.randn(R, 4 * HD, device=dev), torch.empty(R, HD, dtype=bf, device=dev)
+        S = torch.zeros(B + 1, HD * D, device=dev)
+        p = recurrent.RecurrentParams("retention", H, D, D, D, torch.full((HD,), 0.5, device=dev), 1e-6, "silu",
+                                      decay=torch.full((H,), 0.99, device=dev))
+        q, k, v, g = (z[:, i * HD:(i + 1) * HD] for i in range(4))
+        ms = timer(lambda: recurrent.recurrent_forward(p, q, k, v, g, {"S": S}, slots, out, cu, None, init))
+        add("retention", size, ms, (R * HD * 18 + B * HD * D * 8) / 1e9)
+        _kda_row(dev, timer, add, B, T)
+        # heads between projections and scores, beside the rotary cache write (and, in prompts, the query operand)
+        n = -(-R // PAGE)
+        cache, at = torch.zeros(n, PAGE, row, dtype=bf, device=dev), torch.arange(R, device=dev)
+        lens = torch.arange(1, R + 1, dtype=torch.int32, device=dev)
+        tab, tab2 = rot.table(lens), half.table(lens)
+        gb = R * (HD + row) * 4 / 1e9 + R * (row * 2 + HD * (2 if prompt else 4) + D * 4) / 1e9
+        ms = timer(lambda: talking.prepare_heads(z, at, cache, near, prep, tab, not prompt, prompt))
+        add("heads: bias, norm, rotation, cache", size, ms, gb)
+        if not prompt:
+            ms = timer(lambda: talking.kv_write(z[:, :row], at, cache, full, tab2))
+            add("  rotary cache write", size, ms, R * (row * 6 + D * 4) / 1e9)
+        x, a = torch.randn(R, 2, W, device=dev), torch.randn(R, W, device=dev)
+        ones, mix = torch.ones(2, device=dev), torch.eye(2, device=dev)
+        hc = residual.Hyper(ones, mix, ones)
+        ms = timer(lambda: residual.hyper_norm(x, gains.w, 1e-6, W, W, bf, read=ones, hc=hc, add=a, bias=gains.b))
+        add("hyper-connection + norm", size, ms, R * W * (4 * 5 + 2) / 1e9)
+        routed = torch.randn(R * K, W, device=dev)
+        pos = torch.randperm(R * K, device=dev).to(torch.int32).view(R, K).contiguous()
+        rw = torch.rand(R, K, device=dev)
+        ms = timer(lambda: residual.hyper_norm(x, gains.w, 1e-6, W, W, bf, read=ones, hc=hc, add=a, routed=routed, pos=pos, route_w=rw))
+        add("hyper-connection + norm + experts' rows", size, ms, R * W * (4 * (5 + K) + 2) / 1e9)
+        x1 = x[:, 0].contiguous()
+        ms = timer(lambda: residual.sandwich_norm(x1, gains, 1e-6, W, W, bf, add=a, post=gains))
+        add("  norms of a sandwich block", size, ms, R * W * (4 * 3 + 2) / 1e9)
+        ms = timer(lambda: residual.residual_norm(x1, gains.w, 1e-6, W, W, bf, add=a, routed=routed, pos=pos))
+        add("  residual + norm + experts' rows", size, ms, R * W * (4 * (3 + K) + 2) / 1e9)
+        logits, corr = torch.randn(R, E, device=dev), torch.zeros(E, device=dev)
+        gb = R * (E * 4 + K * 8) / 1e9
+        add("router", size, timer(lambda: moe.router_topk(logits, corr, K, 8, 4, "always", 2.5, "softmax_all", None, "max")), gb)
+        add("  router, sigmoid", size, timer(lambda: moe.router_topk(logits, None, K, norm_topk_prob=False)), gb)
+        idx, rw = moe.router_topk(logits, corr, K, 8, 4, "always", 2.5, "softmax_all", None, "max")
+        h = torch.randn(R, W, device=dev).to(bf)
+        w13, w2 = (torch.randn(E, *s, device=dev, dtype=bf) * 0.02 for s in ((2 * Fe, W), (W, Fe)))
+        gb, tf = E * 3 * W * Fe * 2 / 1e9 + R * K * W * 4 / 1e9, R * K * 6 * W * Fe / 1e12
+        for name, kind, on_input in (("experts", "silu", False), ("  experts, weighted input", "swiglu_oai", True)):
+            ew = moe.ExpertWeights(w13, w2, activation=kind, act_limit=7.0)
+            add(name, size, timer(lambda: moe.routed_rows(h, idx, rw, ew, on_input)), gb, tf)
+        del x, a, routed, z, w13, w2
+    for B, ctx in ((16, 4096), (64, 4096), (256, 4096)):
+        n = B * ctx // PAGE
+        cache = torch.randn(n, PAGE, row, device=dev).bfloat16()
+        bt = torch.randperm(n, device=dev).to(torch.int32).view(B, -1).contiguous()
+        lens = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+        q, out = torch.randn(B, HD, device=dev), torch.empty(B, HD, dtype=bf, device=dev)
+        for name, p, keys in (("attention, decode, window", near, win + keep), ("  attention, decode", full, ctx)):
+            add(name, f"{B} x {keys} of {ctx} keys", timer(lambda: talking.attend_rows(q, p, cache, bt, lens, out)),
+                B * keys * row * 2 / 1e9)
+        bts = bt[:, :(win + keep) // PAGE].contiguous()              # as many keys, one after the other
+        short = torch.full((B,), win + keep, dtype=torch.int32, device=dev)
+        add("  attention, decode", f"{B} x {win + keep} keys", timer(lambda: talking.attend_rows(q, full, cache, bts, short, out)),
+            B * (win + keep) * row * 2 / 1e9)
+        del cache
+    for B, T in ((1, 4096), (8, 1024), (1, 16384)):
+        n, R = T // PAGE, B * T
+        cache = torch.randn(B * n, PAGE, row, device=dev).bfloat16()
+        bt = torch.arange(B * n, device=dev, dtype=torch.int32).view(B, n).contiguous()
+        qf = torch.randn(R, H, D, device=dev).bfloat16()
+        q, out = torch.empty(R, HD, device=dev), torch.empty(R, HD, dtype=bf, device=dev)
+        cu = list(range(0, R + 1, T))
+        for name, p in (("attention, prompt, window", near), ("  attention, prompt", full)):
+            blocks = talking.work_blocks(talking.prefill_work(cu, [0] * B, 0, 1, p.window), R, dev)
+            seen = B * sum(p.most_keys(t) for t in range(1, T + 1))
+            add(name, f"{B} x {T} tokens", timer(lambda: talking.attend_prefill(q, p, cache, bt, out, blocks, operand=qf)), 0,
+                seen * 4 * H * D / 1e12)
+        del cache, q, qf
+    return add.rows
+
+
 def run(args, root: str, design: str) -> int:
     import torch
     from batchgen_b200.config import get_model_config
@@ -279,16 +381,16 @@ def run(args, root: str, design: str) -> int:
     sampler = ClockSampler(0).start()
     l0 = _ext.LAUNCHES["count"]
     models = {}
-    for cfg in (get_model_config(f"{design}-bench"), _closest(design)):
+    for cfg in (get_model_config(f"{design}-bench"), *_closest(design)):
         models[cfg.name] = _model_rates(cfg, dev, timer)
-    kernels = {"nanurax": _nanurax_kernels, "pamevik": _pamevik_kernels}[design](dev, timer, peaks)
+    kernels = {"nanurax": _nanurax_kernels, "pamevik": _pamevik_kernels, "bolisun": _bolisun_kernels}[design](dev, timer, peaks)
     _ext.check_status()
     step = models[f"{design}-bench"]["decode"][1]
     print(json.dumps({
         "metric": f"decode tokens/s, 64 rows at 2,048 context, four layers ({design.capitalize()})", "value": step["tok_per_s"],
         "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": timer.warmup, "ms_per_step": step["ms"],
         "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-        "config": {"model": f"{design}-bench", "closest": "kimi-linear cut to four layers", "l2": "flushed before every call",
+        "config": {"model": f"{design}-bench", "closest": list(models)[1:], "l2": "flushed before every call",
                    "parallelism": "1 GPU"},
         "models": models, "kernels": kernels, "peaks": peaks, "clocks": sampler.stop(),
         "gpu_launches": _ext.LAUNCHES["count"] - l0}))
