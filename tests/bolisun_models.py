@@ -1,4 +1,5 @@
 """Small Bolisun configurations and models for the tests."""
+import json
 import random
 
 import bolisun_oracle as oracle
@@ -70,6 +71,16 @@ CONFIGS = {
 }
 
 
+def without_choices(d):
+    """The same design with every expert chosen: rounding flips nothing."""
+    d = json.loads(json.dumps(d))
+    for x in d["layers"]:
+        if (x["mlp"] or {}).get("kind") == "moe":
+            x["mlp"]["router"].pop("groups", None)
+            x["mlp"]["router"]["top"] = x["mlp"]["router"]["experts"]
+    return d
+
+
 def random_config(seed):
     """A design of random sizes, constants and order of layers."""
     r = random.Random(seed)
@@ -97,8 +108,8 @@ def random_config(seed):
     return config(r.randint(30, 300), r.randint(9, 140), r.randint(1, 6), layers, 10 ** r.uniform(-6, -4), r.uniform(0.5, 4))
 
 
-def weights_of(d, seed=0):
-    return oracle.random_weights(d, seed)
+def weights_of(d, seed=0, settled=False):
+    return oracle.random_weights(d, seed, settled)
 
 
 def build(d, weights, device="cpu", dtype="fp32"):

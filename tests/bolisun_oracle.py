@@ -203,9 +203,10 @@ def tensor_shapes(cfg):
     return out
 
 
-def random_weights(cfg, seed=0):
-    """Weights with every mechanism in play: gains near 1, biases of visible size, streams that differ, router corrections of
-    both signs.  Values are representable in bf16."""
+def random_weights(cfg, seed=0, settled=False):
+    """Weights with every mechanism in play: gains near 1, biases of visible size, streams that differ, router corrections that
+    make choice scores of both signs.  ``settled``: corrections far apart, so that few choices are close.  Values are representable
+    in bf16."""
     g = torch.Generator().manual_seed(seed)
     w = {}
     for name, shape in sorted(tensor_shapes(cfg).items()):
@@ -222,7 +223,7 @@ def random_weights(cfg, seed=0):
         elif leaf == "mix":
             t = 0.8 * torch.eye(shape[0]) + 0.2 * t / shape[0] ** 0.5
         elif leaf == "correction":
-            t = 0.1 * t - 0.15
+            t = (1.0 if settled else 0.1) * t - 0.15
         elif leaf != "embed":
             t = t * (2.5 if leaf == "router" else 1.3) * shape[1] ** -0.5
         w[name] = t.bfloat16().float()
