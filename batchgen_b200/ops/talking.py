@@ -28,11 +28,11 @@ class TalkParams:
     vdim_p: int
     scale: float
     chunk: int = 0                           # keys are seen from the query's own chunk on; 0 = every earlier key
+    sink: bool = False                       # one added to the softmax denominator
+    talk: Optional[torch.Tensor] = None      # [heads, heads] fp32: score_h <- sum_g talk[h, g] score_g; None = no mixing
     window: int = 0                          # the last so many positions are seen, the query's own among them; 0 = all
     keep: int = 0                            # with a window: so many first positions stay visible
     out_scale: float = 1.0                   # factor of the output
-    sink: bool = False                       # one added to the softmax denominator
-    talk: Optional[torch.Tensor] = None      # [heads, heads] fp32: score_h <- sum_g talk[h, g] score_g; None = no mixing
 
     @property
     def kv_row(self) -> int:
