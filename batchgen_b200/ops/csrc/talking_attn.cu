@@ -7,7 +7,7 @@
 //   p[h, j]  = exp(s[h, j]) / (1 + sum exp(s[h, :]))                 (the 1 only with a sink)
 //   o[h]     = sum_j p[h, j] v[kv(h), j], times out_scale, times sigmoid(gate[h]) when there is a gate
 //
-// Without a mixing matrix a head keeps its own score.  Queries (on load) and keys (on the way to the cache) may carry rotary
+// Without a mixing matrix a head keeps its own score (bf16 heads up to 128 wide then run on gqa_rows.cuh instead).  Queries (on load) and keys (on the way to the cache) may carry rotary
 // positions: channel i turns with channel i + half.  Mixing couples all heads at a key, so a CTA takes all heads of its row.
 // Keys go in tiles of 32 (a lane per key); a
 // tile's steps are: raw scores (each warp takes key heads, whose K rows it stages through its own shared-memory buffer;
@@ -434,6 +434,8 @@ static int launch_rows(const Params& p, int R, cudaStream_t stream) {
 }  // namespace talk
 }  // namespace bg
 
+#include "gqa_rows.cuh"
+
 extern "C" {
 
 // dt: 0 = bf16 cache and output, 1 = fp32.  -1: sizes out of contract; -3: heads x width need more shared memory than a CTA has.
@@ -457,8 +459,9 @@ int bg_talk_rows(int dt, const float* q, int ldq, const float* talk, const void*
   p.rope = rope; p.half = half; p.gate = gate; p.ld_gate = ld_gate;
   const int items = G * ((H / G + 3) / 4) * (dvp / 4);
   const int ni = (items + kThreads - 1) / kThreads;
-  if (ni > 8) return -1;
+  if (ni > 8 && !(dt == 0 && plain::supported(p))) return -1;
   if (dt == 0) {
+    if (plain::supported(p)) return plain::launch(p, R, stream);
     if (ni == 1) return launch_rows<__nv_bfloat16, 1>(p, R, stream);
     if (ni == 2) return launch_rows<__nv_bfloat16, 2>(p, R, stream);
     if (ni <= 4) return launch_rows<__nv_bfloat16, 4>(p, R, stream);

@@ -2,7 +2,8 @@
 visibility, a sliding window that keeps a sequence's first keys, a zero-score sink, rotary positions on queries and keys, a sigmoid
 gate per head on the output; biases and norms of query and key heads (``prepare_heads``, ``csrc/head_prep.cu``).
 
-Cache rows, and one query row per CTA for decode and short pieces: ``csrc/talking_attn.cu``; tensor-core flash attention for
+Cache rows, and one query row per CTA for decode and short pieces: ``csrc/talking_attn.cu`` (plain bf16 heads on the tensor
+cores, ``csrc/gqa_rows.cuh``); tensor-core flash attention for
 long pieces of prompts, over mixed queries (``csrc/talking_prefill.cu``) or plain heads (``csrc/gqa_prefill.cu``).
 """
 from __future__ import annotations
@@ -151,6 +152,17 @@ def _rows_ref(q, p: TalkParams, cache, block_table, lens, out, row_seq, rope, ga
         out[t, : H * dv] = o.reshape(-1).to(out.dtype)
 
 
+def rows_on_tensor_cores(p: TalkParams, dtype: torch.dtype) -> bool:
+    """The row kernel of plain bf16 heads up to 128 wide (``csrc/gqa_rows.cuh``)."""
+    return dtype == torch.bfloat16 and p.talk is None and p.dim_p <= 128 and p.vdim_p <= 128
+
+
+def _ranges(ctas: int, keys: int, sms: int) -> int:
+    """Key ranges per row for ``gqa_rows.cuh``: rounds of CTAs over the SMs (two fit an SM), of which each takes as long as its
+    keys and some 256 more to start and end."""
+    return min(range(1, max(1, min(16, keys // 64)) + 1), key=lambda s: math.ceil(ctas * s / (2 * sms)) * (keys / s + 256))
+
+
 def _splits(rows: int, keys: int, sms: int) -> int:
     """Key ranges per row: whole rounds of CTAs over the SMs (two fit an SM), each range a few 32-key tiles long."""
     slots, tiles = 2 * sms, max(1, -(-keys // 32))
@@ -183,7 +195,11 @@ def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table
     H = p.heads
     if num_splits <= 0:
         keys = block_table.shape[1] * page
-        num_splits = _splits(R, p.most_keys(keys), _ext.num_sms(q.device))
+        if rows_on_tensor_cores(p, cache.dtype):
+            heads = p.kv_heads * -(-(H // p.kv_heads) // 16)              # CTAs of a row and key range
+            num_splits = _ranges(R * heads, p.most_keys(keys), _ext.num_sms(q.device))
+        else:
+            num_splits = _splits(R, p.most_keys(keys), _ext.num_sms(q.device))
     po = pml = None
     if num_splits > 1:
         po = torch.empty(R * num_splits * H * p.vdim_p, dtype=torch.float32, device=q.device)
