@@ -25,7 +25,7 @@ struct Params {
   const long long* slots; // [T] cache slots, < 0: not written
   void* cache;            // [pages, page, row]
   long long page_stride;
-  int page, row;
+  int page, shift, row;   // tokens per page = 2^shift, elements per token
   int write_q;            // queries go back to z
   __nv_bfloat16* qf;      // [T, H, kc] or null
   int kc;
@@ -63,7 +63,7 @@ __global__ void __launch_bounds__(kWarps * 32) prep_kernel(const Params p) {
       v[i][n] = c < width[i] ? ld4(zr + off[i] + c) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   }
-  KT* dst = reinterpret_cast<KT*>(p.cache) + (slot / p.page) * p.page_stride + (slot % p.page) * p.row;
+  KT* dst = reinterpret_cast<KT*>(p.cache) + (slot >> p.shift) * p.page_stride + (int)(slot & (p.page - 1)) * (long long)p.row;
 #pragma unroll
   for (int i = 0; i < kHeads; ++i) {
     if (width[i] == 0) continue;                                  // the same for all lanes of the warp
@@ -166,7 +166,7 @@ static void launch(const Params& p, dim3 grid, size_t smem, cudaStream_t stream)
 
 extern "C" {
 
-// dt: 0 = bf16 cache, 1 = fp32.  z: T rows of ld floats, the heads' columns first; row = G (dp + dvp); d: real width of query and
+// dt: 0 = bf16 cache, 1 = fp32.  page: a power of two.  z: T rows of ld floats, the heads' columns first; row = G (dp + dvp); d: real width of query and
 // key heads (for the norms).  qf [T, H, kc] bf16 or null.
 int bg_head_prep(int dt, float* z, int ld, const float* bias, const float* wq, const float* wk, float eps, int d, const float* rope,
                  int half, int interleaved, const long long* slots, void* cache, long long page_stride, int page, int row, int write_q,
@@ -174,13 +174,14 @@ int bg_head_prep(int dt, float* z, int ld, const float* bias, const float* wq, c
   using namespace bg::heads;
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || dp <= 0 || dp % 8 || dp > kMaxWidth || d <= 0 || d > dp || dvp <= 0 || dvp % 8 || dvp > kMaxWidth || row != G * (dp + dvp) ||
-      ld % 4 || ld < H * dp + row || page <= 0 || page_stride % 8 || (rope != nullptr && (half <= 0 || 2 * half > dp)) ||
+      ld % 4 || ld < H * dp + row || page <= 0 || (page & (page - 1)) || page_stride % 8 || (rope != nullptr && (half <= 0 || 2 * half > dp)) ||
       (qf != nullptr && (kc < dp || kc % 8)) || (wq == nullptr) != (wk == nullptr) || reinterpret_cast<uintptr_t>(z) % 16)
     return -1;
   Params p;
   p.z = z; p.ld = ld; p.bias = bias; p.wq = wq; p.wk = wk; p.eps = eps; p.inv_d = 1.0f / (float)d; p.rope = rope; p.half = half;
   p.interleaved = interleaved; p.slots = slots; p.cache = cache; p.page_stride = page_stride; p.page = page; p.row = row;
   p.write_q = write_q; p.qf = reinterpret_cast<__nv_bfloat16*>(qf); p.kc = kc; p.q_scale = scale * 1.4426950408889634f;
+  for (p.shift = 0; (1 << p.shift) < page; ++p.shift) {}
   p.H = H; p.G = G; p.dp = dp; p.dvp = dvp;
   const dim3 grid(T, (H + 2 * G + kWarps * kHeads - 1) / (kWarps * kHeads));
   if (grid.y > 65535) return -1;

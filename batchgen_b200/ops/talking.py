@@ -3,8 +3,8 @@ visibility, a sliding window that keeps a sequence's first keys, a zero-score si
 gate per head on the output; biases and norms of query and key heads (``prepare_heads``, ``csrc/head_prep.cu``).
 
 Cache rows, and one query row per CTA for decode and short pieces: ``csrc/talking_attn.cu`` (plain bf16 heads on the tensor
-cores, ``csrc/gqa_rows.cuh``); tensor-core flash attention for
-long pieces of prompts, over mixed queries (``csrc/talking_prefill.cu``) or plain heads (``csrc/gqa_prefill.cu``).
+cores, ``csrc/gqa_rows.cuh``); tensor-core flash attention for long pieces of prompts, over mixed queries
+(``csrc/talking_prefill.cu``) or plain heads (``csrc/gqa_prefill.cu``).
 """
 from __future__ import annotations
 

@@ -189,7 +189,8 @@ class _Attention:
 
 SHAPES = [(9, 3, 56, 48, 56, 64, 64), (4, 4, 20, 36, 6, 16, 33), (8, 1, 80, 128, 32, 64, 100), (32, 8, 128, 128, 128, 64, 128),
           (1, 1, 8, 8, 2, 32, 1), (16, 2, 40, 200, 24, 128, 17), (10, 2, 96, 24, 96, 64, 250), (6, 2, 136, 264, 60, 64, 90),
-          (2, 1, 384, 40, 128, 64, 65), (12, 12, 8, 512, 8, 32, 40), (20, 4, 128, 64, 128, 64, 700)]
+          (2, 1, 384, 40, 128, 64, 65), (12, 12, 8, 512, 8, 32, 40), (20, 4, 128, 64, 128, 64, 700),
+          (20, 1, 120, 88, 64, 16, 75), (24, 2, 64, 56, 64, 64, 130)]
 
 
 @pytest.mark.parametrize("H,G,d,dv,rd,page,window", SHAPES)
@@ -229,6 +230,32 @@ def test_windowed_attention_rows_and_tiles(H, G, d, dv, rd, page, window, dtype)
                 [(a.T - n + i, min(128, n - i), 0, 500 - n + i) for i in range(0, n, 128)], a.T, DEV), operand=qf)
             assert _rel(a.heads(out)[-n:], full[-n:]) < tol and float((out[: a.T - n] - 5).abs().sum()) == 0
     _ext.check_status()
+
+
+@pytest.mark.parametrize("H,G,d,dv", [(6, 2, 24, 40), (33, 1, 128, 128), (10, 1, 64, 8)])
+def test_row_kernel_of_plain_heads_with_chunks_a_sink_and_gates(H, G, d, dv):
+    """The parts of the row kernel that other designs use."""
+    from batchgen_b200.ops import talking
+    g, n, chunk = _gen(H), 200, 70
+    r = lambda *s: torch.randn(*s, generator=g)      # noqa: E731
+    q, k, v, gate = r(n, H, d), r(n, G, d).to(BF).float(), r(n, G, dv).to(BF).float(), r(n, H)
+    p = talking.TalkParams(H, G, d, dv, d ** -0.5, chunk, True, out_scale=1.5)
+    pool = torch.zeros(4, 64, p.kv_row, dtype=BF, device=DEV)
+    pool.view(256, -1)[:n] = torch.cat([k.reshape(n, -1), v.reshape(n, -1)], 1).to(DEV)
+    i, j = torch.arange(n).view(-1, 1), torch.arange(n).view(1, -1)
+    seen = torch.cat([(j <= i) & (j // chunk == i // chunk), torch.ones(n, 1, dtype=torch.bool)], 1)
+    more = [torch.cat([x.double(), torch.zeros(1, *x.shape[1:], dtype=F64)]) for x in (k, v)]        # the sink: a score of 0, a value of 0
+    want = oracle.attention(q.double(), *more, d ** -0.5, seen) * 1.5 * torch.sigmoid(gate.double()).unsqueeze(-1)
+    lens = torch.arange(1, n + 1, dtype=torch.int32)
+    lens[13] = 0
+    for splits in (1, 2, 5):
+        out = torch.full((n, H * dv), 5.0, dtype=BF, device=DEV)
+        talking.attend_rows(q.reshape(n, -1).to(DEV), p, pool, _i32([[0, 1, 2, 3]]), lens.to(DEV), out, torch.zeros(n, dtype=torch.int32,
+                            device=DEV), num_splits=splits, gate=gate.to(DEV))
+        got = out.view(n, H, dv)
+        assert float(got[13].abs().sum()) == 0
+        keep = [t for t in range(n) if t != 13]
+        assert _rel(got[keep], want[keep]) < 1e-2, splits
 
 
 def test_heads_without_norms_turn_halves_too():
