@@ -3,11 +3,13 @@
 //   residual_norm   x[t] += sum of the sublayers' fp32 outputs (dense rows and / or routed rows gathered by position),
 //                   or x[t] = embed[id] * scale for the first layer; y[t] = x[t] / sqrt(mean(x^2) + eps) * w
 //   sandwich_norm   the same for blocks with a norm before and after each sublayer: the sublayer's output (or half the sum of
-//                   two, each RMS-normed) passes its own norm before it joins x; optional mean subtraction and biases; in
-//                   decode the input convolution y = h + conv(h) of the next sublayer is folded in
+//                   two, each RMS-normed, or the weighted rows of routed experts) passes its own norm before it joins x; optional
+//                   mean subtraction and biases; the norm before may be absent; in decode the input convolution y = h + conv(h)
+//                   of the next sublayer (or its token shift, a convolution of two taps) is folded in
 //   hyper_norm      the same for several residual streams: every stream becomes a weighted sum of all of them plus its share of
 //                   the sublayer's output; the norm reads another weighted sum
-//   glu             gated activations (tanh-GELU, SwiGLU, clamped SwiGLU with slope 1.702 and u + 1), with an optional factor on
+//   token_side      tanh-GELU(z) * the token's row of a table
+//   glu             gated activations (tanh-GELU, SwiGLU, clamped SwiGLU with slope 1.702 and u + 1; squared ReLU without a gate), with an optional factor on
 //                   the pre-activations (routing weight applied to the expert's input) and an optional sigmoid gate
 //   cast_act        out = f(x), f = tanh, squared ReLU or identity: fp32 columns of a projection to the operand type of the next one
 //   moe_gather      token rows -> expert-grouped rows, one block per (token, k) pair, plus the pair's routing weight
@@ -141,11 +143,16 @@ struct SandwichParams {
   const float *a, *b;     // the sublayer's output(s) [T, ld], or null
   int lda, ldb;
   const float *wa, *wb;   // with b: weights of the outputs' RMS norms
+  const float* routed;    // instead of a: rows of the routed experts [*, ld_routed], or null
+  int ld_routed;
+  const int* pos;         // [T, K] row of every (token, k) pair, < 0 = none
+  const float* route_w;   // [T, K] factors of those rows
+  int K;
   const float *w1, *b1;   // norm of the output; b1 may be null
   int center1;
-  const float *w2, *b2;   // norm of x
+  const float *w2, *b2;   // norm of x; w2 null: x itself
   int center2;
-  void* y;                // [R, ldy]
+  void* y;                // [R, ldy], or null: only x
   int ldy, raw;           // raw: y is fp32 and ends at D rounded up to 4
   const float* cw;        // [taps, D4] input convolution, or null
   float* hist;            // [slots, (taps - 1) * D4] rows of `hist_stride`
@@ -169,6 +176,8 @@ __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichP
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   __shared__ float red[2][kMaxWarps];
   __shared__ Moments part[2][kMaxWarps];
+  __shared__ int pos_s[kMaxK];
+  __shared__ float rw[kMaxK];
   const int tid = threadIdx.x, NT = blockDim.x, warps = NT >> 5;
   const long long t = p.rows != nullptr ? p.rows[blockIdx.x] : (long long)blockIdx.x;
   float* xr = p.x + t * p.ldx;
@@ -243,9 +252,34 @@ __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichP
   } else {
     each([&](int n, int c) { f[n] = ld4(xr, c); });
   }
-  if (p.a != nullptr) {
-    const float* ar = p.a + t * p.lda;
-    each([&](int n, int c) { s[n] = ld4(ar, c); });
+  if (p.a != nullptr || p.routed != nullptr) {
+    if (p.routed != nullptr) {
+      if (tid < p.K) {
+        pos_s[tid] = p.pos[t * p.K + tid];
+        rw[tid] = p.route_w[t * p.K + tid];
+      }
+      __syncthreads();
+      each([&](int n, int) { s[n] = make_float4(0.f, 0.f, 0.f, 0.f); });
+      for (int k0 = 0; k0 < p.K; k0 += 4) {                          // four rows' loads at a time
+        each([&](int n, int c) {
+          float4 a[4];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const int r = k0 + k < p.K ? pos_s[k0 + k] : -1;
+            a[k] = r >= 0 ? ld4(p.routed + (size_t)r * p.ld_routed, c) : make_float4(0.f, 0.f, 0.f, 0.f);
+          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float g = k0 + k < p.K ? rw[k0 + k] : 0.f;
+            s[n].x = fmaf(g, a[k].x, s[n].x); s[n].y = fmaf(g, a[k].y, s[n].y);
+            s[n].z = fmaf(g, a[k].z, s[n].z); s[n].w = fmaf(g, a[k].w, s[n].w);
+          }
+        });
+      }
+    } else {
+      const float* ar = p.a + t * p.lda;
+      each([&](int n, int c) { s[n] = ld4(ar, c); });
+    }
     if (p.b != nullptr) {
       const float* br = p.b + t * p.ldb;
       each([&](int n, int c) { u[n] = ld4(br, c); });
@@ -282,14 +316,15 @@ __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(const SandwichP
     each([&](int n, int c) { mask(f[n], c); });
   }
   if (p.keep) each([&](int n, int c) { *reinterpret_cast<float4*>(xr + c) = f[n]; });
+  if (p.y == nullptr) return;
   float mean, rstd;
-  moments(f, p.center2, part[1], mean, rstd);
+  if (p.w2 != nullptr) moments(f, p.center2, part[1], mean, rstd);
   OT* yr = reinterpret_cast<OT*>(p.y) + (size_t)blockIdx.x * p.ldy;
   float* hr = reinterpret_cast<float*>(p.y) + (size_t)blockIdx.x * p.ldy;
   const int slot = p.cw != nullptr ? p.slots[blockIdx.x] : -1;
   const int D4 = nv * 4;
   each([&](int n, int c) {
-    float4 h = norm4(f[n], mean, rstd, p.w2, p.b2, c);
+    float4 h = p.w2 != nullptr ? norm4(f[n], mean, rstd, p.w2, p.b2, c) : f[n];
     if (p.cw != nullptr) {                                         // y = h + conv(h); the stored inputs move up by one
       const float4 in = h;
       auto tap = [&](int j, const float4& v) {
@@ -466,6 +501,10 @@ __device__ __forceinline__ float glu_one(float g, float u, float limit) {
     return 0.5f * g * (1.0f + t) * u;
   }
   if (KIND == 2) return g * sigmoid_acc(g) * u;        // SiLU(g) * u
+  if (KIND == 3) {                                     // squared ReLU, no gate
+    g = fmaxf(g, 0.f);
+    return g * g;
+  }
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g * sigmoid_acc(1.702f * g) * (u + 1.0f);
@@ -489,13 +528,27 @@ glu_kernel(const float* __restrict__ z, int ldz, int u_off, OT* __restrict__ out
     const float m = gate != nullptr ? sigmoid_acc(gate[(size_t)r * ld_gate]) : 1.0f;
     const float* zr = z + (size_t)r * ldz + c;
     const float4 g = *reinterpret_cast<const float4*>(zr);
-    const float4 u = *reinterpret_cast<const float4*>(zr + u_off);
+    const float4 u = KIND == 3 ? g : *reinterpret_cast<const float4*>(zr + u_off);
     o.x = glu_one<KIND>(g.x * s, u.x * s, limit) * m;
     o.y = glu_one<KIND>(g.y * s, u.y * s, limit) * m;
     o.z = glu_one<KIND>(g.z * s, u.z * s, limit) * m;
     o.w = glu_one<KIND>(g.w * s, u.w * s, limit) * m;
   }
   store4(out + (size_t)r * ldo + c, o);
+}
+
+// out[t, c] = tanh-GELU(z[t, c]) * table[ids[t], c], zero for c >= n
+template <typename OT>
+__global__ void __launch_bounds__(kThreads)
+token_side_kernel(const float* __restrict__ z, int ldz, const OT* __restrict__ table, long long ldt, const int* __restrict__ ids, int vocab,
+                  OT* __restrict__ out, int ldo, int T, int n) {
+  bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
+  const int i = blockIdx.x * kThreads + threadIdx.x;
+  const int t = i / ldo, c = i % ldo;
+  if (t >= T) return;
+  float v = 0.f;
+  if (c < n) v = glu_one<0>(z[(size_t)t * ldz + c], to_f(table[min(max(ids[t], 0), vocab - 1) * ldt + c]), 0.f);
+  out[(size_t)t * ldo + c] = from_f<OT>(v);
 }
 
 template <typename OT, int KIND>
@@ -558,24 +611,27 @@ int bg_residual_norm(int dt, float* x, int ldx, const long long* rows, const int
 }
 
 // dt: 0 = bf16, 1 = fp32 (embedding table and output).  Leading dimensions: multiples of 4, at least D rounded up to 4; vectors
-// of the norms hold that many floats.  D <= 16384.  a null: nothing joins x; ids: x = embed[ids] * escale.
+// of the norms hold that many floats.  D <= 16384.  a and routed null: nothing joins x; ids: x = embed[ids] * escale; w2 null: no
+// norm of x; y null: only x is written.
 int bg_sandwich_norm(int dt, float* x, int ldx, const long long* rows, const int* ids, const void* embed, int lde, float escale,
-                     int vocab, const float* a, int lda, const float* b, int ldb, const float* wa, const float* wb, const float* w1,
-                     const float* b1, int center1, const float* w2, const float* b2, int center2, void* y, int ldy, int raw,
+                     int vocab, const float* a, int lda, const float* b, int ldb, const float* wa, const float* wb, const float* routed,
+                     int ld_routed, const int* pos, const float* route_w, int K, const float* w1, const float* b1, int center1, const float* w2, const float* b2, int center2, void* y, int ldy, int raw,
                      const float* cw, float* hist, long long hist_stride, const int* slots, int taps, int R, int D, float eps,
                      int keep, cudaStream_t stream) {
   using namespace bg::resid;
   if (R <= 0) return 0;
   const int D4 = (D + 3) / 4 * 4;
-  if (D <= 0 || D > 16384 || ldx % 4 || ldx < D4 || ldy % 4 || ldy < D4 || (raw && ldy != D4) || w2 == nullptr ||
-      (a != nullptr && (lda % 4 || lda < D4 || w1 == nullptr)) ||
+  if (D <= 0 || D > 16384 || ldx % 4 || ldx < D4 || ldy % 4 || ldy < D4 || (raw && ldy != D4) || (y == nullptr && cw != nullptr) ||
+      (a != nullptr && (lda % 4 || lda < D4 || w1 == nullptr || routed != nullptr)) ||
+      (routed != nullptr && (ld_routed % 4 || ld_routed < D4 || K <= 0 || K > kMaxK || pos == nullptr || route_w == nullptr || w1 == nullptr)) ||
       (b != nullptr && (a == nullptr || ldb % 4 || ldb < D4 || wa == nullptr || wb == nullptr)) ||
       (ids != nullptr && (embed == nullptr || vocab <= 0)) ||
       (cw != nullptr && (slots == nullptr || taps < 1 || (taps > 1 && hist == nullptr) || hist_stride % 4 || rows != nullptr)))
     return -1;
   SandwichParams p;
   p.x = x; p.ldx = ldx; p.rows = rows; p.ids = ids; p.embed = embed; p.lde = lde; p.escale = escale; p.vocab = vocab;
-  p.a = a; p.b = b; p.lda = lda; p.ldb = ldb; p.wa = wa; p.wb = wb; p.w1 = w1; p.b1 = b1; p.center1 = center1;
+  p.a = a; p.b = b; p.lda = lda; p.ldb = ldb; p.wa = wa; p.wb = wb; p.routed = routed; p.ld_routed = ld_routed; p.pos = pos;
+  p.route_w = route_w; p.K = K; p.w1 = w1; p.b1 = b1; p.center1 = center1;
   p.w2 = w2; p.b2 = b2; p.center2 = center2; p.y = y; p.ldy = ldy; p.raw = raw; p.cw = cw; p.hist = hist;
   p.hist_stride = hist_stride; p.slots = slots; p.taps = taps; p.D = D; p.eps = eps; p.keep = keep;
   const int nv = D4 / 4;
@@ -638,7 +694,7 @@ int bg_hyper_norm(int dt, float* x, const long long* rows, const int* ids, const
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
-// kind 0 tanh-GELU, 1 clamped SwiGLU, 2 SwiGLU.  z points at the first gate column, the up column of a gate column is u_off further.
+// kind 0 tanh-GELU, 1 clamped SwiGLU, 2 SwiGLU, 3 squared ReLU (no up column).  z points at the first gate column, the up column of a gate column is u_off further.
 int bg_glu(int dt, int kind, const float* z, int ldz, int u_off, void* out, int ldo, int R, int F, int Fo, float limit,
            const float* row_scale, const float* gate, int ld_gate, const int* total_rows, cudaStream_t stream) {
   using namespace bg::resid;
@@ -650,11 +706,29 @@ int bg_glu(int dt, int kind, const float* z, int ldz, int u_off, void* out, int 
                  Fo, limit, row_scale, gate, ld_gate, total_rows)
   if (dt == 0 && kind == 0) BG_GLU(__nv_bfloat16, 0);
   else if (dt == 0 && kind == 1) BG_GLU(__nv_bfloat16, 1);
-  else if (dt == 0) BG_GLU(__nv_bfloat16, 2);
+  else if (dt == 0 && kind == 2) BG_GLU(__nv_bfloat16, 2);
+  else if (dt == 0) BG_GLU(__nv_bfloat16, 3);
   else if (kind == 0) BG_GLU(float, 0);
   else if (kind == 1) BG_GLU(float, 1);
-  else BG_GLU(float, 2);
+  else if (kind == 2) BG_GLU(float, 2);
+  else BG_GLU(float, 3);
 #undef BG_GLU
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
+// z [T, ldz] fp32, table rows of ldt elements (the first n count), ids [T] -> out [T, ldo]
+int bg_token_side(int dt, const float* z, int ldz, const void* table, long long ldt, const int* ids, int vocab, void* out, int ldo, int T,
+                  int n, cudaStream_t stream) {
+  using namespace bg::resid;
+  if (T <= 0 || ldo <= 0) return 0;
+  if (n < 0 || n > ldo || n > ldz || n > ldt || vocab <= 0 || (long long)T * ldo > 0x7fffffffll) return -1;
+  const dim3 grid((unsigned)(((long long)T * ldo + kThreads - 1) / kThreads));
+  if (dt == 0)
+    bg::launch_pdl(token_side_kernel<__nv_bfloat16>, grid, dim3(kThreads), 0, stream, z, ldz, reinterpret_cast<const __nv_bfloat16*>(table),
+                   ldt, ids, vocab, reinterpret_cast<__nv_bfloat16*>(out), ldo, T, n);
+  else
+    bg::launch_pdl(token_side_kernel<float>, grid, dim3(kThreads), 0, stream, z, ldz, reinterpret_cast<const float*>(table), ldt, ids, vocab,
+                   reinterpret_cast<float*>(out), ldo, T, n);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 

@@ -17,7 +17,7 @@ import torch
 from . import _ext
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
-GLU_KINDS = {"gelu_tanh": 0, "swiglu_oai": 1, "silu": 2}
+GLU_KINDS = {"gelu_tanh": 0, "swiglu_oai": 1, "silu": 2, "relu2": 3}        # relu2: no gate
 CAST_KINDS = {"none": 0, "tanh": 1, "relu2": 2}
 
 
@@ -76,6 +76,8 @@ def _glu_ref(g: torch.Tensor, u: torch.Tensor, kind: str, limit: float) -> torch
         return 0.5 * g * (1 + torch.tanh(math.sqrt(2 / math.pi) * (g + 0.044715 * g ** 3))) * u
     if kind == "silu":
         return g * torch.sigmoid(g) * u
+    if kind == "relu2":
+        return g.clamp_min(0) ** 2
     g, u = g.clamp(max=limit), u.clamp(-limit, limit)
     return g * torch.sigmoid(1.702 * g) * (u + 1)
 
@@ -83,12 +85,12 @@ def _glu_ref(g: torch.Tensor, u: torch.Tensor, kind: str, limit: float) -> torch
 def glu(z: torch.Tensor, F: int, kind: str, limit: float = 0.0, row_scale: Optional[torch.Tensor] = None,
         gate: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, total_rows: Optional[torch.Tensor] = None,
         dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """act(s * z[:, :F], s * z[:, F:2F]) * sigmoid(gate): ``kind`` gelu_tanh (tanh-GELU(g) * u), silu (SiLU(g) * u) or swiglu_oai (g clamped from
-    above, u on both sides, g * sigmoid(1.702 g) * (u + 1)).  z fp32 (a column view is fine), ``row_scale`` [R] = s,
+    """act(s * z[:, :F], s * z[:, F:2F]) * sigmoid(gate): ``kind`` gelu_tanh (tanh-GELU(g) * u), silu (SiLU(g) * u), swiglu_oai (g clamped from
+    above, u on both sides, g * sigmoid(1.702 g) * (u + 1)) or relu2 (the square of g's positive part, no u).  z fp32 (a column view is fine), ``row_scale`` [R] = s,
     ``gate`` [R, 1] (a view is fine).  ``out``: [R, >= F] view, columns past F become zero."""
     R = z.shape[0]
     if not z.is_cuda:
-        g, u = z[:, :F].float(), z[:, F:2 * F].float()
+        g, u = z[:, :F].float(), z[:, :F].float() if kind == "relu2" else z[:, F:2 * F].float()
         if row_scale is not None:
             g, u = g * row_scale.unsqueeze(-1), u * row_scale.unsqueeze(-1)
         y = _glu_ref(g, u, kind, limit)
@@ -148,16 +150,17 @@ class Canon:
     slots: torch.Tensor             # [T] int32, < 0: no history, none kept
 
 
-def sandwich_norm(x: torch.Tensor, norm: Norm, eps: float, width: int, out_cols: int, dtype: torch.dtype,
+def sandwich_norm(x: torch.Tensor, norm: Optional[Norm], eps: float, width: int, out_cols: int, dtype: torch.dtype,
                   add: Optional[torch.Tensor] = None, add2: Optional[torch.Tensor] = None,
                   branch_w: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, post: Optional[Norm] = None,
                   ids: Optional[torch.Tensor] = None, embed: Optional[torch.Tensor] = None, embed_scale: float = 1.0,
                   rows: Optional[torch.Tensor] = None, keep: bool = True, raw: bool = False,
-                  canon: Optional[Canon] = None) -> torch.Tensor:
-    """x [T, >= width] fp32 += post(sublayer output), then norm(x) as [R, out_cols] of ``dtype`` with zero columns past
-    ``width``, or with ``raw`` as fp32 [R, width rounded up to 4].  The sublayer's output is ``add`` [T, width] fp32, or with
-    ``add2`` half the sum of both, each RMS-normed with its weight of ``branch_w``; ``ids``: x = embed[ids] * embed_scale
-    instead.  ``canon`` (one token per sequence) applies the input convolution to the result.  ``rows`` (int64) picks rows of
+                  canon: Optional[Canon] = None, routed: Optional[torch.Tensor] = None, pos: Optional[torch.Tensor] = None,
+                  route_w: Optional[torch.Tensor] = None, emit: bool = True) -> Optional[torch.Tensor]:
+    """x [T, >= width] fp32 += post(sublayer output), then norm(x) (None: x itself) as [R, out_cols] of ``dtype`` with zero columns
+    past ``width``, or with ``raw`` as fp32 [R, width rounded up to 4], or with ``emit=False`` nothing.  The sublayer's output is
+    ``add`` [T, width] fp32, or with ``add2`` half the sum of both, each RMS-normed with its weight of ``branch_w``, or
+    sum_k route_w[t, k] * routed[pos[t, k]]; ``ids``: x = embed[ids] * embed_scale instead.  ``canon`` (one token per sequence) applies the input convolution to the result.  ``rows`` (int64) picks rows of
     x; ``keep=False`` leaves x as it was."""
     R = x.shape[0] if rows is None else rows.shape[0]
     W4 = pad_to(width, 4)
@@ -166,7 +169,10 @@ def sandwich_norm(x: torch.Tensor, norm: Norm, eps: float, width: int, out_cols:
         cur = x[r, :width].clone()
         if ids is not None:
             cur = embed[ids[r].long()].float() * embed_scale
-        if add is not None:
+        if routed is not None:
+            at = pos[r].long()
+            cur = cur + post.ref((routed[at.clamp_min(0), :width] * (route_w[r] * (at >= 0)).unsqueeze(-1)).sum(1), eps, width)
+        elif add is not None:
             s = add[r, :width]
             if add2 is not None:
                 s = 0.5 * sum(t / torch.sqrt((t * t).mean(-1, keepdim=True) + eps) * g[:width]
@@ -174,7 +180,9 @@ def sandwich_norm(x: torch.Tensor, norm: Norm, eps: float, width: int, out_cols:
             cur = cur + post.ref(s, eps, width)
         if keep:
             x[r, :width] = cur
-        h = torch.nn.functional.pad(norm.ref(cur, eps, width), (0, W4 - width))
+        if not emit:
+            return None
+        h = torch.nn.functional.pad(cur if norm is None else norm.ref(cur, eps, width), (0, W4 - width))
         if raw:
             return h
         if canon is not None:
@@ -183,12 +191,16 @@ def sandwich_norm(x: torch.Tensor, norm: Norm, eps: float, width: int, out_cols:
         y = torch.zeros(R, out_cols, dtype=dtype)
         y[:, :width] = h[:, :width].to(dtype)
         return y
-    y = torch.empty(R, W4 if raw else out_cols, dtype=torch.float32 if raw else dtype, device=x.device)
-    for t in (add, add2):
+    y = torch.empty(R, W4 if raw else out_cols, dtype=torch.float32 if raw else dtype, device=x.device) if emit else None
+    for t in (add, add2, routed):
         assert t is None or (t.dtype == torch.float32 and t.stride(1) == 1)
-    assert x.dtype == torch.float32 and (embed is None or embed.dtype == dtype) and (add is None) == (post is None)
+    assert x.dtype == torch.float32 and (embed is None or embed.dtype == dtype)
+    assert (add is None and routed is None) == (post is None) and (add is None or routed is None) and (emit or keep)
+    if routed is not None:
+        assert pos.dtype == torch.int32 and pos.is_contiguous() and route_w.is_contiguous() and route_w.dtype == torch.float32
+        assert pos.shape == route_w.shape and pos.shape[0] == x.shape[0] and routed.stride(0) >= W4
     assert (ids is None or ids.dtype == torch.int32) and (rows is None or rows.dtype == torch.int64)
-    assert x.shape[1] >= W4 and norm.w.shape[0] == W4 and (post is None or post.w.shape[0] == W4)
+    assert x.shape[1] >= W4 and all(n is None or n.w.shape[0] == W4 for n in (norm, post))
     for t in (add, add2):
         assert t is None or (t.shape[0] == x.shape[0] and t.stride(0) >= W4)
     if canon is not None:
@@ -201,13 +213,32 @@ def sandwich_norm(x: torch.Tensor, norm: Norm, eps: float, width: int, out_cols:
         _i(embed.stride(0) if embed is not None else 0), ctypes.c_float(embed_scale),
         _i(embed.shape[0] if embed is not None else 0), _ext.ptr(add), _i(add.stride(0) if add is not None else 0),
         _ext.ptr(add2), _i(add2.stride(0) if add2 is not None else 0), _ext.ptr(branch_w[0] if add2 is not None else None),
-        _ext.ptr(branch_w[1] if add2 is not None else None), *P(post), _i(post is not None and post.center), *P(norm),
-        _i(norm.center), _ext.ptr(y), _i(y.shape[1]), _i(raw), _ext.ptr(canon.w if canon else None),
+        _ext.ptr(branch_w[1] if add2 is not None else None), _ext.ptr(routed), _i(routed.stride(0) if routed is not None else 0),
+        _ext.ptr(pos), _ext.ptr(route_w), _i(pos.shape[1] if pos is not None else 0), *P(post), _i(post is not None and post.center),
+        *P(norm), _i(norm is not None and norm.center), _ext.ptr(y), _i(y.shape[1] if emit else W4), _i(raw), _ext.ptr(canon.w if canon else None),
         _ext.ptr(canon.hist if canon else None), ctypes.c_longlong(canon.hist.stride(0) if canon else 0),
         _ext.ptr(canon.slots if canon else None), _i(canon.w.shape[0] if canon else 0), _i(R), _i(width), ctypes.c_float(eps),
         _i(keep), _ext.stream())
     _ext.check(rc, "bg_sandwich_norm")
     return y
+
+
+def token_side(z: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, out_cols: int, dtype: torch.dtype) -> torch.Tensor:
+    """tanh-GELU(z) * table[ids] as [T, out_cols] of ``dtype``, zero past the table's width: z [T, >= n] fp32 (a column view is
+    fine), table [vocab, n] (a column view is fine), ids [T] int32 (clamped to the table)."""
+    n = table.shape[1]
+    if not z.is_cuda:
+        g = z[:, :n].float()
+        y = torch.zeros(z.shape[0], out_cols, dtype=dtype)
+        y[:, :n] = (_glu_ref(g, table[ids.long().clamp(0, table.shape[0] - 1)].float(), "gelu_tanh", 0.0)).to(dtype)
+        return y
+    assert z.dtype == torch.float32 and z.stride(1) == 1 and table.stride(1) == 1 and table.dtype == dtype
+    assert ids.dtype == torch.int32 and ids.shape[0] == z.shape[0] and z.shape[1] >= n and out_cols >= n
+    out = torch.empty(z.shape[0], out_cols, dtype=dtype, device=z.device)
+    rc = _ext.lib().bg_token_side(_i(_DT[dtype]), _ext.ptr(z), _i(z.stride(0)), _ext.ptr(table), ctypes.c_longlong(table.stride(0)),
+                                  _ext.ptr(ids), _i(table.shape[0]), _ext.ptr(out), _i(out_cols), _i(z.shape[0]), _i(n), _ext.stream())
+    _ext.check(rc, "bg_token_side")
+    return out
 
 
 @dataclass
