@@ -16,7 +16,7 @@ __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1
 
 struct ChannelDelta {
   static constexpr int kVecs = 4;
-  static constexpr bool kRead = true, kTwoTerms = false, kDen = false, kOwnV = false;
+  static constexpr bool kRead = true, kTwoTerms = false, kForget = false, kDen = false, kOwnV = false;
   struct Regs { float q, k, low, dtb, beta, rate; };
   struct Scal { float b; };
   static __device__ __forceinline__ void fetch(const Args& p, int t, int h, int c, Regs& x) {

@@ -21,7 +21,7 @@ namespace rec {
 
 struct GeneralDelta {
   static constexpr int kVecs = 4;
-  static constexpr bool kRead = true, kTwoTerms = true, kDen = false, kOwnV = true;
+  static constexpr bool kRead = true, kTwoTerms = true, kForget = false, kDen = false, kOwnV = true;
   struct Regs { float r, k, a, w, w0, ab; };
   struct Scal {};
   static __device__ __forceinline__ void fetch(const Args& p, int t, int h, int c, Regs& x) {

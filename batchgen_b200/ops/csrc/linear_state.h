@@ -7,6 +7,7 @@ namespace rec {
 
 int channel_delta_forward(const Args& p, cudaStream_t stream);      // channel_delta.cu
 int mlstm_forward(const Args& p, cudaStream_t stream);              // mlstm.cu
+int hgrn2_forward(const Args& p, cudaStream_t stream);              // hgrn2.cu
 
 }  // namespace rec
 }  // namespace bg

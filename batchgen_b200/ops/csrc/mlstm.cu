@@ -19,7 +19,7 @@ __device__ __forceinline__ float soft_cap(float x, float cap) { return cap * tan
 
 struct MLstm {
   static constexpr int kVecs = 2;
-  static constexpr bool kRead = false, kTwoTerms = false, kDen = true, kOwnV = false;
+  static constexpr bool kRead = false, kTwoTerms = false, kForget = false, kDen = true, kOwnV = false;
   struct Regs { float q, k, gi, gf, bi, bf, n, m; };
   struct Scal { float keep, put, m; };
   static __device__ __forceinline__ void fetch(const Args& p, int t, int h, int c, Regs& x) {

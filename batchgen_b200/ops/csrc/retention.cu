@@ -18,7 +18,7 @@ __device__ __forceinline__ float turned(const float* x, int c, const float* rope
 
 struct Retention {
   static constexpr int kVecs = 2;
-  static constexpr bool kRead = false, kTwoTerms = false, kDen = false, kOwnV = false;
+  static constexpr bool kRead = false, kTwoTerms = false, kForget = false, kDen = false, kOwnV = false;
   struct Regs { float q, k, w; };
   struct Scal { float w; };
   static __device__ __forceinline__ void fetch(const Args& p, int t, int h, int c, Regs& x) {
@@ -68,7 +68,7 @@ static int retention_forward(const Args& p, cudaStream_t stream) {
 }  // namespace rec
 }  // namespace bg
 
-// rule: 0 channel_delta, 1 mlstm, 2 retention.  -1: sizes or strides outside the kernels' contract
+// rule: 0 channel_delta, 1 mlstm, 2 retention, 3 hgrn2.  -1: sizes or strides outside the kernels' contract
 extern "C" int bg_recurrent_forward(const bg::rec::Args* a, cudaStream_t stream) {
   using namespace bg::rec;
   if (a->nseq <= 0 || a->T <= 0) return 0;
@@ -77,6 +77,7 @@ extern "C" int bg_recurrent_forward(const bg::rec::Args* a, cudaStream_t stream)
     case 0: return channel_delta_forward(*a, stream);
     case 1: return mlstm_forward(*a, stream);
     case 2: return retention_forward(*a, stream);
+    case 3: return hgrn2_forward(*a, stream);
     default: return -1;
   }
 }

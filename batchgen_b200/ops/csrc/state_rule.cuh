@@ -3,6 +3,7 @@
 //
 //   kVecs         vectors of K channels a token contributes
 //   kRead         the update needs y = (read vector)^T S of the old state; otherwise the decay is one number per token
+//   kForget       without kRead: the decay f is a vector over the key channels and the write vector is 1 - f (HGRN2)
 //   kTwoTerms     the correction by y and the new value are written along different vectors
 //   kDen          a normaliser vector is carried like one more value column with value 1 (mLSTM)
 //   Regs, fetch   what a thread loads of a token ahead of its turn (thread = channel)
@@ -20,12 +21,13 @@ namespace bg {
 namespace rec {
 
 struct Args {
-  const float *q, *k, *v, *gate;   // fp32 column views of the step's projections
+  const float *q, *k, *v, *gate;   // fp32 column views of the step's projections; gate null: the output has none
   const float* low;                // [T, H * K] decay pre-activation
   const float* beta;               // write strength (channel_delta, [T, H]) or removal rate (general_delta, [T, H * K])
   const float *gate_i, *gate_f;    // mlstm: [T, H]
-  const float *bias0, *bias1;      // general_delta: decay and removal offsets; channel_delta: dt_bias; mlstm: gate biases
-  const float* rate;               // channel_delta: exp(A_log) [H]; retention: decay [H]
+  const float *bias0, *bias1;      // general_delta: decay and removal offsets; channel_delta: dt_bias; mlstm: gate biases; hgrn2:
+                                   // forget bias (k: its pre-activation)
+  const float* rate;               // channel_delta: exp(A_log) [H]; retention: decay [H]; hgrn2: lower bounds [H * K]
   const float* rope;               // retention: [T, 2 * half] cosines, then sines
   const float* norm_w;             // [H * V] gain of the output norm
   float* state;                    // this layer's S [H, K, V] in slot 0; slots are `slot_stride` floats apart
@@ -54,6 +56,12 @@ template <> __device__ __forceinline__ void put4<__nv_bfloat16>(__nv_bfloat16* p
 }
 __device__ __forceinline__ float sigm(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float gate_act(float x, int silu) { return silu ? x * sigm(x) : sigm(x); }
+// factors of 4 output channels; g null: no gate
+__device__ __forceinline__ float4 gate4(const float* g, int silu) {
+  if (g == nullptr) return make_float4(1.f, 1.f, 1.f, 1.f);
+  const float4 v = *reinterpret_cast<const float4*>(g);
+  return make_float4(gate_act(v.x, silu), gate_act(v.y, silu), gate_act(v.z, silu), gate_act(v.w, silu));
+}
 __device__ __forceinline__ float2 twice(float x) { return make_float2(x, x); }
 
 // ---------------------------------------------------------------- decode
@@ -85,7 +93,7 @@ __device__ __forceinline__ float4 xor_sum(float4 v, int mask) {
 
 // What a column's outputs and its next state are made of, from the token's sums (filled by `Rule::coefs`):
 //   kRead:  y' = ys * y;  o = os * q + ov * v - oy * y'  (kTwoTerms)   or   u = us * (v - y'), o = os * q + ov * u
-//   linear: S' = w S + k v, o = os * (q^T S')
+//   linear: S' = w S + k v, o = os * (q^T S')   (kForget: w and k per key channel, f and 1 - f)
 struct Coefs {
   float ys, os, ov, oy, us, w;
 };
@@ -171,7 +179,7 @@ __global__ void __launch_bounds__(288) decode_kernel(const Args p, int items) {
     if (fetched != item) fetch(item);                            // rows without a slot shifted the turns
     float4 g = make_float4(0.f, 0.f, 0.f, 0.f), nw4 = g;
     if (col_ok && rg == 0) {
-      g = *reinterpret_cast<const float4*>(p.gate + (size_t)t * p.ld_gate + h * V + 4 * quad);
+      g = gate4(p.gate != nullptr ? p.gate + (size_t)t * p.ld_gate + h * V + 4 * quad : nullptr, p.silu);
       nw4 = *reinterpret_cast<const float4*>(p.norm_w + h * V + 4 * quad);
     }
     float (*v4)[4 * NR] = vec[group];
@@ -289,9 +297,10 @@ __global__ void __launch_bounds__(288) decode_kernel(const Args p, int items) {
       // one sweep: S' = w S + k v, o = q^T S'
       if (ok && col_ok) {
         const float4 v = *reinterpret_cast<const float4*>(&sv[group][4 * quad]);
-        const float2 va = make_float2(v.x, v.y), vb = make_float2(v.z, v.w), w2 = twice(cf.w);
+        const float2 va = make_float2(v.x, v.y), vb = make_float2(v.z, v.w);
         auto step = [&](float4& s, float kf, float rf) {
-          const float2 k2 = twice(kf), r2 = twice(rf);
+          const float2 k2 = twice(Rule::kForget ? 1.0f - kf : kf), r2 = twice(rf);
+          const float2 w2 = twice(Rule::kForget ? kf : cf.w);
           const float2 n0 = __ffma2_rn(w2, make_float2(s.x, s.y), __fmul2_rn(k2, va));
           const float2 n1 = __ffma2_rn(w2, make_float2(s.z, s.w), __fmul2_rn(k2, vb));
           q[0] = __ffma2_rn(r2, n0, q[0]); q[1] = __ffma2_rn(r2, n1, q[1]);
@@ -334,8 +343,7 @@ __global__ void __launch_bounds__(288) decode_kernel(const Args p, int items) {
     if (col_ok && rg == 0) {
       const float oo = red_o[group][0] + red_o[group][1] + red_o[group][2] + red_o[group][3];
       const float rs = 1.0f / sqrtf(oo / (float)p.v_real + p.eps);
-      put4(out + 4 * quad, make_float4(o.x * rs * nw4.x * gate_act(g.x, p.silu), o.y * rs * nw4.y * gate_act(g.y, p.silu),
-                                       o.z * rs * nw4.z * gate_act(g.z, p.silu), o.w * rs * nw4.w * gate_act(g.w, p.silu)));
+      put4(out + 4 * quad, make_float4(o.x * rs * nw4.x * g.x, o.y * rs * nw4.y * g.y, o.z * rs * nw4.z * g.z, o.w * rs * nw4.w * g.w));
     }
   }
 }
@@ -345,6 +353,7 @@ __global__ void __launch_bounds__(288) decode_kernel(const Args p, int items) {
 //   general (kTwoTerms):  w | u | a u | w r, numbers c1 c2;  S' = w S - (a u) y + u v, y = u^T S, o = (w r)^T S - c1 y + c2 v
 //   kRead:                w | read | write | w r, number c;  S' = w S + write (v - y), y = read^T S, o = (w r)^T S + c (v - y)
 //   linear:               k | r, number w;                   S' = w S + k v, o = r^T S'
+//   kForget:              f | r;                             S' = f S + (1 - f) v, o = r^T S'
 template <typename Rule>
 __host__ __device__ inline int rec_floats(int K, int V) { return Rule::kVecs * K + 4 + (Rule::kOwnV ? V : 0); }
 
@@ -409,7 +418,7 @@ scan_kernel(const Args p, const float* __restrict__ rec, float* __restrict__ o_o
     // a short last group is filled up with tokens that leave the state alone: decay 1, everything else 0
     for (int tt = n + warp; tt < kScanGroup; tt += kWarps) {
       float* dst = sm + (buf * kScanGroup + tt) * TOK;
-      for (int j = lane; j < TOK; j += 32) dst[j] = (Rule::kRead ? j < W : j == NUM) ? 1.f : 0.f;
+      for (int j = lane; j < TOK; j += 32) dst[j] = (Rule::kRead || Rule::kForget ? j < W : j == NUM) ? 1.f : 0.f;
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -519,8 +528,13 @@ scan_kernel(const Args p, const float* __restrict__ rec, float* __restrict__ o_o
           const float4 k = k4[16 * n], r = r4[16 * n];
 #pragma unroll
           for (int c = 0; c < C; ++c) {
-            S[c][2 * n] = __ffma2_rn(make_float2(k.x, k.y), sv[c], __fmul2_rn(w2, S[c][2 * n]));
-            S[c][2 * n + 1] = __ffma2_rn(make_float2(k.z, k.w), sv[c], __fmul2_rn(w2, S[c][2 * n + 1]));
+            if constexpr (Rule::kForget) {
+              S[c][2 * n] = __ffma2_rn(make_float2(k.x, k.y), S[c][2 * n], __fmul2_rn(make_float2(1.0f - k.x, 1.0f - k.y), sv[c]));
+              S[c][2 * n + 1] = __ffma2_rn(make_float2(k.z, k.w), S[c][2 * n + 1], __fmul2_rn(make_float2(1.0f - k.z, 1.0f - k.w), sv[c]));
+            } else {
+              S[c][2 * n] = __ffma2_rn(make_float2(k.x, k.y), sv[c], __fmul2_rn(w2, S[c][2 * n]));
+              S[c][2 * n + 1] = __ffma2_rn(make_float2(k.z, k.w), sv[c], __fmul2_rn(w2, S[c][2 * n + 1]));
+            }
             q[c] = __ffma2_rn(make_float2(r.x, r.y), S[c][2 * n], q[c]);
             q[c] = __ffma2_rn(make_float2(r.z, r.w), S[c][2 * n + 1], q[c]);
           }
@@ -600,11 +614,10 @@ finish_kernel(const Args p, const float* __restrict__ o_in, const float* __restr
       v = *reinterpret_cast<const float4*>(o + e);
       v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
     }
-    const float4 g = *reinterpret_cast<const float4*>(p.gate + (size_t)t * p.ld_gate + h * V + e);
+    const float4 g = gate4(p.gate != nullptr ? p.gate + (size_t)t * p.ld_gate + h * V + e : nullptr, p.silu);
     const float4 nw = *reinterpret_cast<const float4*>(p.norm_w + h * V + e);
     put4(reinterpret_cast<OT*>(p.out) + (size_t)t * p.ld_out + h * V + e,
-         make_float4(v.x * rs * nw.x * gate_act(g.x, p.silu), v.y * rs * nw.y * gate_act(g.y, p.silu),
-                     v.z * rs * nw.z * gate_act(g.z, p.silu), v.w * rs * nw.w * gate_act(g.w, p.silu)));
+         make_float4(v.x * rs * nw.x * g.x, v.y * rs * nw.y * g.y, v.z * rs * nw.z * g.z, v.w * rs * nw.w * g.w));
   }
 }
 

@@ -1,7 +1,7 @@
 """Linear-attention recurrences with a matrix state per head (``csrc/linear_state.cu``): the gated delta rule with a decay per
-key channel, the mLSTM cell with its running maximum and normaliser, and retention with a fixed decay per head.  All of them
-decay the rows of S [key channels x value channels], add a rank-one write and read S^T q; the output is divided by its root
-mean square per head, scaled by a weight and gated.
+key channel, the mLSTM cell with its running maximum and normaliser, retention with a fixed decay per head, and HGRN2, whose forget
+gate per key channel is also what is not written.  All of them decay the rows of S [key channels x value channels], add a rank-one
+write and read S^T q; the output is divided by its root mean square per head, scaled by a weight and (except HGRN2's) gated.
 
 The generalised delta rule (``ops/delta.py``) runs on the same state kernels.
 """
@@ -18,7 +18,7 @@ from . import _ext
 from .conv import rotate_ref
 from .residual import _DT
 
-RULES = {"channel_delta": 0, "mlstm": 1, "retention": 2}
+RULES = {"channel_delta": 0, "mlstm": 1, "retention": 2, "hgrn2": 3}
 _GATES = {"sigmoid": torch.sigmoid, "silu": F.silu}
 
 
@@ -42,6 +42,7 @@ class RecurrentParams:
     f_bias: Optional[torch.Tensor] = None
     gate_cap: float = 1.0
     decay: Optional[torch.Tensor] = None      # retention: [heads]
+    f_lower: Optional[torch.Tensor] = None    # hgrn2: [heads * dim_p] lower bounds of the forget gate (its bias is ``f_bias``, as wide)
     unit_eps: float = 1e-6                    # channel_delta: inside the root of the unit vectors
     den_eps: float = 1e-6                     # mlstm: added to the denominator
 
@@ -67,20 +68,21 @@ def scratch_floats(p: RecurrentParams, T: int) -> int:
     return T * p.heads * (vectors * p.dim_p + 4 + p.vdim_p + (8 if p.rule == "mlstm" else 0))
 
 
-def recurrent_forward(p: RecurrentParams, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor,
+def recurrent_forward(p: RecurrentParams, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: Optional[torch.Tensor],
                       state: Dict[str, torch.Tensor], slots: torch.Tensor, out: torch.Tensor,
                       cu: Optional[torch.Tensor] = None, cu_host: Optional[Sequence[int]] = None,
                       has_initial: Optional[torch.Tensor] = None, *, low: Optional[torch.Tensor] = None,
                       beta: Optional[torch.Tensor] = None, gate_i: Optional[torch.Tensor] = None,
                       gate_f: Optional[torch.Tensor] = None, rope: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """q, k [T, qk_heads * dim_p], v, gate [T, heads * vdim_p]: fp32 column views; ``out`` [T, >= heads * vdim_p] in the operand
+    """q, k [T, qk_heads * dim_p], v, gate [T, heads * vdim_p] (None: no gate): fp32 column views; ``out`` [T, >= heads * vdim_p] in the operand
     dtype.  ``state``: "S" [slots, heads * dim_p * vdim_p] (and mLSTM's "n", "m"), strided views of the pool; slots [nseq] int32
     (< 0: skipped, zero output); ``cu`` [nseq + 1] int32 token ranges, None = one token per sequence; ``has_initial`` [nseq]
     int32, None = continue from the slot.
 
     channel_delta: ``low`` [T, heads * dim_p] decay pre-activation, ``beta`` [T, >= heads] write strength before its sigmoid.
     mlstm: ``gate_i`` / ``gate_f`` [T, >= heads] gate pre-activations without their biases.
-    retention: ``rope`` [T, dims] (``conv.Rotary.table``) turns q and k."""
+    retention: ``rope`` [T, dims] (``conv.Rotary.table``) turns q and k.
+    hgrn2: ``k`` is the pre-activation of the forget gate without its bias, q is read through SiLU."""
     if not q.is_cuda:
         nseq = len(slots)
         bounds = list(range(nseq + 1)) if cu is None and cu_host is None else list(cu_host if cu_host is not None else cu.tolist())
@@ -99,12 +101,14 @@ def recurrent_forward(p: RecurrentParams, q: torch.Tensor, k: torch.Tensor, v: t
     for name, cols in (("n", p.heads * p.dim_p), ("m", p.heads)) if p.rule == "mlstm" else ():
         t = state[name]                                       # parts of one pool: the kernels step all of them by S's slot stride
         assert t.dtype == torch.float32 and t.stride() == S.stride() and t.shape == (S.shape[0], cols)
+    if p.rule == "hgrn2":
+        assert p.f_bias.shape[0] == p.f_lower.shape[0] == p.heads * p.dim_p and p.f_bias.dtype == p.f_lower.dtype == torch.float32
     scratch = None
     if cu is not None or p.dim_p > 128 or p.vdim_p > 128:
         scratch = torch.empty(scratch_floats(p, T), dtype=torch.float32, device=q.device)
     tensors = dict(q=q, k=k, v=v, gate=gate, low=low, beta=beta, gate_i=gate_i, gate_f=gate_f,
-                   bias0=p.dt_bias if p.rule == "channel_delta" else p.i_bias, bias1=p.f_bias,
-                   rate=p.decay if p.rule == "retention" else p.rate, rope=rope, norm_w=p.norm_w, state=S,
+                   bias0={"channel_delta": p.dt_bias, "hgrn2": p.f_bias}.get(p.rule, p.i_bias), bias1=p.f_bias,
+                   rate={"retention": p.decay, "hgrn2": p.f_lower}.get(p.rule, p.rate), rope=rope, norm_w=p.norm_w, state=S,
                    norm_state=state.get("n"), max_state=state.get("m"), cu=cu, slots=slots, has_initial=has_initial, out=out,
                    scratch=scratch, status=_ext.status_word(q.device))
     for n, t in tensors.items():
@@ -138,6 +142,9 @@ def _step_inputs(p, q, k, v, low, beta, gate_i, gate_f, rope):
         def cap(x, b):
             return p.gate_cap * torch.tanh((x[:, :H].float() + b) / p.gate_cap)
         extra = (cap(gate_i, p.i_bias), F.logsigmoid(cap(gate_f, p.f_bias)))
+    elif p.rule == "hgrn2":
+        f = p.f_lower + (1 - p.f_lower) * torch.sigmoid(k.reshape(-1, H * K) + p.f_bias)
+        q, extra = F.silu(q), (f.view(-1, H, K),)
     else:
         q, k, extra = rotate_ref(q, rope), rotate_ref(k, rope), ()
     return (q * p.q_scale).repeat_interleave(rep, 1), (k * p.k_scale).repeat_interleave(rep, 1), v, extra
@@ -175,11 +182,17 @@ def _forward_ref(p, q, k, v, gate, state, slots, out, cu, has_initial, low, beta
                 n, m = keep.view(H, 1) * n + put.view(H, 1) * ks[t], new
                 den = torch.maximum((n * qs[t]).sum(-1).abs(), torch.exp(-m)) + p.den_eps
                 o = torch.einsum("hkv,hk->hv", S, qs[t]) / den.unsqueeze(-1)
+            elif p.rule == "hgrn2":
+                f = extra[0][t].unsqueeze(-1)
+                S = f * S + (1 - f) * vs[t].unsqueeze(1)
+                o = torch.einsum("hkv,hk->hv", S, qs[t])
             else:
                 S = p.decay.view(H, 1, 1) * S + write * vs[t].unsqueeze(1)
                 o = torch.einsum("hkv,hk->hv", S, qs[t])
             o = o / torch.sqrt((o * o).sum(-1, keepdim=True) / p.vdim + p.eps)
-            o = o.reshape(-1) * p.norm_w * act(gate[t, :H * V].float())
+            o = o.reshape(-1) * p.norm_w
+            if gate is not None:
+                o = o * act(gate[t, :H * V].float())
             out[t, :H * V] = o.to(out.dtype)
         state["S"][slot] = S.reshape(-1)
         if p.rule == "mlstm":
