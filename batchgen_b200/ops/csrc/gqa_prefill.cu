@@ -1,5 +1,6 @@
 // Prompt attention of grouped-query heads over a paged K/V cache, on tcgen05: causal, optionally with chunked visibility or a
-// sliding window that keeps a sequence's first keys, a zero-score sink, rotary queries and a sigmoid gate per head on the output.
+// sliding window that keeps a sequence's first keys, a sink (score zero or one per head), rotary queries and a sigmoid gate per head
+// or per element on the output.
 //
 //   S[q, k] = Q[q, :] . K[k, kv(h)]      (M = 128 queries, N = 64 keys; Q resident, K streamed, both K-major)
 //   O[q, :] += P[q, k] . V[k, kv(h)]     (V read N-major, P written by the softmax threads as a swizzled K-major tile)
@@ -47,8 +48,9 @@ struct Params {
   float out_scale;
   __nv_bfloat16* out;
   int ldo;
-  const float* gate;             // [T, ld_gate] or null: out[h] *= sigmoid(gate[h])
-  int ld_gate;
+  const float* gate;             // [T, ld_gate] or null: out[h] *= sigmoid(gate[h]), or per element
+  int ld_gate, gate_cols;        // columns of a head: 1 or dvp
+  const float* sinks;            // [H] scores of the sink, or null: zero
   int row_shift;                 // rows of Q = rows of out - row_shift
   int smem_bytes;
   int* status;
@@ -335,9 +337,11 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
     if (ok && n_tiles > 0) ok = !vote_any_128(!mbar_wait(&ss.o_done, (n_tiles - 1) & 1, abort_flag, kTimeoutEpilogue));
     if (ok) {
       tc_fence_after();
-      if (p.sink && live) l_run += exp2f(-m_run);
+      if (p.sink && live) l_run += exp2f((p.sinks != nullptr ? p.sinks[h] * 1.4426950408889634f : 0.f) - m_run);
       float inv = l_run > 0.f ? p.out_scale / l_run : 0.f;
-      if (p.gate != nullptr && live) inv *= 1.0f / (1.0f + expf(-p.gate[(size_t)(w.q_row0 + r) * p.ld_gate + h]));
+      const float* gate = p.gate != nullptr ? p.gate + (size_t)(w.q_row0 + r) * p.ld_gate + h * p.gate_cols : nullptr;
+      const bool each = gate != nullptr && p.gate_cols > 1;
+      if (gate != nullptr && !each && live) inv *= 1.0f / (1.0f + expf(-gate[0]));
       __nv_bfloat16* orow = p.out + (size_t)(w.q_row0 + r) * p.ldo + h * p.dvp;
 #pragma unroll 1
       for (int c = 0; c < p.VB * 2; ++c) {
@@ -349,6 +353,16 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
           for (int j = 0; j < 32; j += 8) {
             if (c * 32 + j < p.dvp) {                          // dvp is a multiple of 8
               __align__(16) __nv_bfloat162 o[4];
+              if (each) {
+#pragma unroll
+                for (int q = 0; q < 8; q += 4) {
+                  const float4 g = *reinterpret_cast<const float4*>(gate + c * 32 + j + q);
+                  ov[j + q] = __float_as_uint(__uint_as_float(ov[j + q]) / (1.0f + expf(-g.x)));
+                  ov[j + q + 1] = __float_as_uint(__uint_as_float(ov[j + q + 1]) / (1.0f + expf(-g.y)));
+                  ov[j + q + 2] = __float_as_uint(__uint_as_float(ov[j + q + 2]) / (1.0f + expf(-g.z)));
+                  ov[j + q + 3] = __float_as_uint(__uint_as_float(ov[j + q + 3]) / (1.0f + expf(-g.w)));
+                }
+              }
 #pragma unroll
               for (int q = 0; q < 4; ++q)
                 o[q] = __floats2bfloat162_rn(__uint_as_float(ov[j + 2 * q]) * inv, __uint_as_float(ov[j + 2 * q + 1]) * inv);
@@ -446,11 +460,13 @@ int bg_gqa_prompt_queries(const float* q, int ldq, const float* rope, int half, 
 // dp, dvp <= 256, multiples of 8.
 int bg_gqa_prompt(const void* qf, const void* cache, long long page_stride, int n_pages, int page, int row, const int* block_table,
                   int bt_stride, int bt_cols, const int* work, int n_work, int R, int row_shift, void* out, int ldo, int H, int G,
-                  int dp, int dvp, int kc, int chunk, int sink, int window, int keep, float out_scale, const float* gate, int ld_gate, int* status, cudaStream_t stream) {
+                  int dp, int dvp, int kc, int chunk, int sink, int window, int keep, float out_scale, const float* gate, int ld_gate, int gate_cols, const float* sinks,
+                  int* status, cudaStream_t stream) {
   using namespace bg::gqapre;
   if (n_work <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || dp <= 0 || dp % 8 || dp > 256 || dvp <= 0 || dvp % 8 || dvp > 256 || kc != (dp + 63) / 64 * 64 ||
-      page < 16 || (page & (page - 1)) || row != G * (dp + dvp) || page_stride % 8 || ldo % 8 || bt_cols <= 0 || n_work > 65535 || window < 0 || keep < 0)
+      page < 16 || (page & (page - 1)) || row != G * (dp + dvp) || page_stride % 8 || ldo % 8 || bt_cols <= 0 || n_work > 65535 || window < 0 || keep < 0 ||
+      (gate != nullptr && gate_cols != 1 && (gate_cols != dvp || ld_gate % 4 || reinterpret_cast<uintptr_t>(gate) % 16)))
     return -1;
   const int box_rows = page < 64 ? page : 64;
   CUtensorMap tq, tk;
@@ -471,7 +487,7 @@ int bg_gqa_prompt(const void* qf, const void* cache, long long page_stride, int 
   p.block_table = block_table; p.bt_stride = bt_stride; p.bt_cols = bt_cols; p.page = page; p.box_rows = box_rows;
   p.KB = kc / 64; p.VB = (dvp + 63) / 64; p.dp = dp; p.dvp = dvp; p.v_col0 = G * dp; p.rep = H / G; p.chunk = chunk; p.sink = sink;
   p.window = window; p.keep = keep; p.out_scale = out_scale;
-  p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo; p.gate = gate; p.ld_gate = ld_gate; p.row_shift = row_shift;
+  p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo; p.gate = gate; p.ld_gate = ld_gate; p.gate_cols = gate_cols; p.sinks = sinks; p.row_shift = row_shift;
   p.status = status;
   // two CTAs an SM when two stages and half of TMEM are enough, otherwise one with as many stages as fit
   const bool two = p.VB <= 2 && tile_bytes(p.KB, p.VB, 2) + (int)sizeof(Shared) <= kSmemTwo;

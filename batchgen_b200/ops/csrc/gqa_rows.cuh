@@ -96,7 +96,7 @@ __global__ void __launch_bounds__(kRowWarps * 32, 2) gqa_rows_kernel(const Param
   auto fetch = [&](int tile, int slot, long long off) {
     if (tile < my_hi) {
       copy_rows(ring_u + slot * sb, kb, dp, cache + c * dp, off);
-      copy_rows(ring_u + slot * sb + kTile * kb, vb, dvp, cache + (size_t)G * dp + (size_t)c * dvp, off);
+      copy_rows(ring_u + slot * sb + kTile * kb, vb, dvp, cache + (size_t)p.v_col0 + (size_t)c * dvp, off);
     }
     cp_commit();                                                   // an empty group keeps the count of groups in step
   };
@@ -239,9 +239,8 @@ __global__ void __launch_bounds__(kRowWarps * 32, 2) gqa_rows_kernel(const Param
       a.x += f * v.x; a.y += f * v.y; a.z += f * v.z; a.w += f * v.w;
     }
     if (p.n_splits == 1) {
-      float inv = p.out_scale / (ll + (p.sink ? exp2f(-mm) : 0.f));
-      if (p.gate != nullptr) inv *= sigm(p.gate[(size_t)t * p.ld_gate + h]);
-      put4(out + 4 * i, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv));
+      const float inv = p.out_scale / (ll + (p.sink ? exp2f(sink_score(p, h) - mm) : 0.f));
+      put4(out + 4 * i, gated4(p, t, h, col, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv)));
     } else {
       *reinterpret_cast<float4*>(p.part_o + (((size_t)r * p.n_splits + split) * H + h) * dvp + col) = a;
       if (col == 0) *reinterpret_cast<float2*>(p.part_ml + (((size_t)r * p.n_splits + split) * H + h) * 2) = make_float2(mm, ll);
@@ -265,7 +264,7 @@ static int launch_heads(const Params& p, int R, int groups, cudaStream_t stream)
 }
 static bool supported(const Params& p) {
   const int groups = (p.H / p.G + 15) / 16;
-  return p.talk == nullptr && p.dp <= kMaxWidth && p.dvp <= kMaxWidth && (long long)p.G * groups <= 65535;
+  return p.talk == nullptr && p.v_col0 == p.G * p.dp && p.dp <= kMaxWidth && p.dvp <= kMaxWidth && (long long)p.G * groups <= 65535;
 }
 static int launch(const Params& p, int R, cudaStream_t stream) {
   const int groups = (p.H / p.G + 15) / 16;

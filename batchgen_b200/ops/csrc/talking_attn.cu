@@ -4,8 +4,8 @@
 //   s[h, j]  = scale * sum_g talk[h, g] (q[g] . k[kv(g), j])        g over all query heads, kv(g) = g / (H / G)
 //   seen     = j <= position and (j >= first or j < keep), first = position - position % chunk (chunk 0: first = 0), with a
 //              window not before position - window + 1
-//   p[h, j]  = exp(s[h, j]) / (1 + sum exp(s[h, :]))                 (the 1 only with a sink)
-//   o[h]     = sum_j p[h, j] v[kv(h), j], times out_scale, times sigmoid(gate[h]) when there is a gate
+//   p[h, j]  = exp(s[h, j]) / (exp(sink[h]) + sum exp(s[h, :]))      (the sink's term only with a sink; without numbers of its own it is 1)
+//   o[h]     = sum_j p[h, j] v[kv(h), j], times out_scale, times sigmoid(gate[h]) (or a gate per element) when there is a gate
 //
 // Without a mixing matrix a head keeps its own score (bf16 heads up to 128 wide then run on gqa_rows.cuh instead).  Queries (on load) and keys (on the way to the cache) may carry rotary
 // positions: channel i turns with channel i + half.  Mixing couples all heads at a key, so a CTA takes all heads of its row.
@@ -16,7 +16,7 @@
 // read once).  With `n_splits` > 1 the key range is split over CTAs and merged by a second kernel.
 //
 // The cache row of a token holds the keys of all G heads (dp each), then the values (dvp each); dp and dvp are the head
-// widths padded to multiples of 8 with zero channels.
+// widths padded to multiples of 8 with zero channels.  The values may also be the first columns of the keys (a cached latent).
 #define BG_FILE_TAG 23     // kernel-trace ids of this file are (tag << 16) | line
 #include "common.cuh"
 
@@ -49,7 +49,10 @@ struct Params {
   const float* rope;            // [T, 2 * half] cosines, then sines, or null
   int half;
   const float* gate;            // [T, ld_gate] or null
-  int ld_gate;
+  int ld_gate, gate_cols;       // columns of a head: 1 or dvp
+  const float* sinks;           // [H] or null: all zero
+  int v_col0;                   // first value column of a cache row
+  const __nv_bfloat16* qb;      // latent_rows.cuh: [R, H, row] queries
 };
 
 template <typename T> __device__ __forceinline__ float to_f(T v);
@@ -67,6 +70,20 @@ __device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) {
   for (int i = 0; i < 4; ++i) { const float2 a = __bfloat1622float2(v[i]); f[2 * i] = a.x; f[2 * i + 1] = a.y; }
 }
 __device__ __forceinline__ float sigm(float x) { return 1.0f / (1.0f + expf(-x)); }
+constexpr float kLog2e = 1.4426950408889634f;
+// the sink's score of head h, in the scores' base-2 units
+__device__ __forceinline__ float sink_score(const Params& p, int h) { return p.sinks != nullptr ? p.sinks[h] * kLog2e : 0.f; }
+// times the gate of columns c .. c + 3 of head h
+__device__ __forceinline__ float4 gated4(const Params& p, int t, int h, int c, float4 v) {
+  if (p.gate == nullptr) return v;
+  const float* g = p.gate + (size_t)t * p.ld_gate + h * p.gate_cols;
+  if (p.gate_cols == 1) {
+    const float f = sigm(g[0]);
+    return make_float4(v.x * f, v.y * f, v.z * f, v.w * f);
+  }
+  const float4 f = *reinterpret_cast<const float4*>(g + c);
+  return make_float4(v.x * sigm(f.x), v.y * sigm(f.y), v.z * sigm(f.z), v.w * sigm(f.w));
+}
 // channel e of a head whose first 2 * half channels turn
 __device__ __forceinline__ float turned(const float* x, int e, const float* rope, int half) {
   const float a = x[e];
@@ -266,7 +283,7 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
         if (it < items) {
           const int u = it / cols, cc = it % cols, c = u / hg_n;
           const int h0 = c * rep + (u % hg_n) * 4, nh = min(4, rep - (u % hg_n) * 4);
-          const KT* vb = cache + (size_t)G * dp + (size_t)c * dvp + cc * 4;
+          const KT* vb = cache + (size_t)p.v_col0 + (size_t)c * dvp + cc * 4;
           const float* ph[4];
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
@@ -335,9 +352,8 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const Params p) {
           const int h = h0 + i, col = h * dvp + cc * 4;
           const float4 v = make_float4(acc[n][i][0].x, acc[n][i][0].y, acc[n][i][1].x, acc[n][i][1].y);
           if (p.n_splits == 1) {
-            float inv = p.out_scale / (l_s[h] + (p.sink ? exp2f(-m_s[h]) : 0.f));
-            if (p.gate != nullptr) inv *= sigm(p.gate[(size_t)t * p.ld_gate + h]);
-            put4(out + col, make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv));
+            const float inv = p.out_scale / (l_s[h] + (p.sink ? exp2f(sink_score(p, h) - m_s[h]) : 0.f));
+            put4(out + col, gated4(p, t, h, cc * 4, make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv)));
           } else {
             *reinterpret_cast<float4*>(p.part_o + ((size_t)r * p.n_splits + split) * H * dvp + col) = v;
           }
@@ -365,15 +381,15 @@ __global__ void merge_kernel(const Params p) {
     return;
   }
   const float* ml = p.part_ml + (size_t)r * S * p.H * 2 + h * 2;
-  float m = p.sink ? 0.f : -INFINITY;
+  const float sink = p.sink ? sink_score(p, h) : -INFINITY;
+  float m = sink;
   for (int s = 0; s < S; ++s) m = fmaxf(m, ml[(size_t)s * p.H * 2]);
-  float l = p.sink ? exp2f(-m) : 0.f;
+  float l = p.sink ? exp2f(sink - m) : 0.f;
   for (int s = 0; s < S; ++s) {
     const float ms = ml[(size_t)s * p.H * 2];
     if (ms != -INFINITY) l += ml[(size_t)s * p.H * 2 + 1] * exp2f(ms - m);
   }
-  float inv = p.out_scale / l;
-  if (p.gate != nullptr) inv *= sigm(p.gate[(size_t)t * p.ld_gate + h]);
+  const float inv = p.out_scale / l;
   for (int i = threadIdx.x; i < p.dvp / 4; i += blockDim.x) {
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int s = 0; s < S; ++s) {
@@ -383,7 +399,7 @@ __global__ void merge_kernel(const Params p) {
       const float4 v = *reinterpret_cast<const float4*>(p.part_o + ((size_t)r * S + s) * p.H * p.dvp + h * p.dvp + 4 * i);
       a.x += f * v.x; a.y += f * v.y; a.z += f * v.z; a.w += f * v.w;
     }
-    put4(out + 4 * i, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv));
+    put4(out + 4 * i, gated4(p, t, h, 4 * i, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv)));
   }
 }
 
@@ -435,6 +451,7 @@ static int launch_rows(const Params& p, int R, cudaStream_t stream) {
 }  // namespace bg
 
 #include "gqa_rows.cuh"
+#include "latent_rows.cuh"
 
 extern "C" {
 
@@ -442,13 +459,13 @@ extern "C" {
 int bg_talk_rows(int dt, const float* q, int ldq, const float* talk, const void* cache, long long page_stride, int page,
                  int row, const int* block_table, int bt_stride, const int* row_seq, const int* row_ids, const int* lens,
                  void* out, int ldo, float* part_o, float* part_ml, int R, int H, int G, int dp, int dvp, int chunk,
-                 int window, int keep, int sink, float scale, float out_scale, int n_splits, const float* rope, int half, const float* gate, int ld_gate,
-                 cudaStream_t stream) {
+                 int window, int keep, int sink, float scale, float out_scale, int n_splits, const float* rope, int half, const float* gate, int ld_gate, int gate_cols,
+                 const float* sinks, int v_col0, cudaStream_t stream) {
   using namespace bg::talk;
   if (R <= 0) return 0;
-  if (H <= 0 || G <= 0 || H % G || dp <= 0 || dp % 8 || dvp <= 0 || dvp % 8 || row != G * (dp + dvp) || page <= 0 ||
+  if (H <= 0 || G <= 0 || H % G || dp <= 0 || dp % 8 || dvp <= 0 || dvp % 8 || row < G * dp || v_col0 < 0 || v_col0 % 8 || row < v_col0 + G * dvp || row % 8 || page <= 0 ||
       page_stride % 8 || ldq % 4 || ldo % 4 || (rope != nullptr && (half <= 0 || 2 * half > dp)) || n_splits < 1 || n_splits > 65535 || H > 65535 ||
-      window < 0 || keep < 0 ||
+      window < 0 || keep < 0 || (gate != nullptr && gate_cols != 1 && (gate_cols != dvp || ld_gate % 4 || reinterpret_cast<uintptr_t>(gate) % 16)) ||
       (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return -1;
   Params p;
@@ -456,7 +473,8 @@ int bg_talk_rows(int dt, const float* q, int ldq, const float* talk, const void*
   p.block_table = block_table; p.bt_stride = bt_stride; p.row_seq = row_seq; p.row_ids = row_ids; p.lens = lens;
   p.out = out; p.ldo = ldo; p.part_o = part_o; p.part_ml = part_ml; p.H = H; p.G = G; p.dp = dp; p.dvp = dvp;
   p.chunk = chunk; p.window = window; p.keep = keep; p.out_scale = out_scale; p.sink = sink; p.n_splits = n_splits; p.scale_log2 = scale * 1.4426950408889634f;
-  p.rope = rope; p.half = half; p.gate = gate; p.ld_gate = ld_gate;
+  p.rope = rope; p.half = half; p.gate = gate; p.ld_gate = ld_gate; p.gate_cols = gate_cols; p.sinks = sinks;
+  p.v_col0 = v_col0; p.qb = nullptr;
   const int items = G * ((H / G + 3) / 4) * (dvp / 4);
   const int ni = (items + kThreads - 1) / kThreads;
   if (ni > 8 && !(dt == 0 && plain::supported(p))) return -1;

@@ -39,7 +39,7 @@ class ExpertWeights:
     quant: str = "none"
     interleaved: bool = False
     activation: str = "silu"             # silu | swiglu_clamped (GPT-OSS) | silu_limit (DeepSeek-V4: clamp, then SiLU(gate) * up)
-                                         # | swiglu_oai | gelu_tanh | silu (``routed_rows``: fp32 activations of layer-listed models)
+                                         # | swiglu_oai | gelu_tanh | silu | relu2 (``routed_rows``: fp32 activations of layer-listed models)
     act_limit: float = 0.0               # clamp of silu_limit (0 = none)
 
     @property
@@ -292,7 +292,7 @@ def experts_forward(hidden: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.
 
 def routed_rows(x: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.Tensor, ew: ExpertWeights, weight_on_input: bool,
                 num_valid: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
-    """Unquantised routed experts with fp32 pre-activations and outputs.  x [T, Kp] (the experts' input, zero columns past
+    """Unquantised routed experts (gated, or squared ReLU without a gate: w13 [E, F, Kp]) with fp32 pre-activations and outputs.  x [T, Kp] (the experts' input, zero columns past
     the model width) -> (y [rows, N] fp32 grouped by expert, pos [T, k] row of every (token, k) pair, -1 = none).
     ``weight_on_input``: the routing weight scales the expert's input (it is applied to the fp32 gate and up
     pre-activations, the same thing without rounding the product); the caller's sum over k then adds the rows as they are.
@@ -300,7 +300,7 @@ def routed_rows(x: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.Tensor, e
 
     All shapes and row counts stay on the device: the call is graph capturable."""
     E, F2, _ = ew.w13.shape
-    F = F2 // 2
+    F = F2 if ew.activation == "relu2" else F2 // 2
     T, K = topk_idx.shape
     kind = residual.GLU_KINDS[ew.activation]
     if not x.is_cuda:

@@ -1,6 +1,7 @@
 """Paged grouped-query attention for layer-listed models.  Optional parts: heads' scores mixed before the softmax, chunked
-visibility, a sliding window that keeps a sequence's first keys, a zero-score sink, rotary positions on queries and keys, a sigmoid
-gate per head on the output; biases and norms of query and key heads (``prepare_heads``, ``csrc/head_prep.cu``).
+visibility, a sliding window that keeps a sequence's first keys, a sink (score zero, or a learned one per head), rotary positions on
+queries and keys, a sigmoid gate per head or per element on the output; biases and norms of query and key heads (each head alone, or
+all at once; ``prepare_heads``, ``csrc/head_prep.cu``).
 
 Cache rows, and one query row per CTA for decode and short pieces: ``csrc/talking_attn.cu`` (plain bf16 heads on the tensor
 cores, ``csrc/gqa_rows.cuh``); tensor-core flash attention for long pieces of prompts, over mixed queries
@@ -34,10 +35,26 @@ class TalkParams:
     window: int = 0                          # the last so many positions are seen, the query's own among them; 0 = all
     keep: int = 0                            # with a window: so many first positions stay visible
     out_scale: float = 1.0                   # factor of the output
+    sinks: Optional[torch.Tensor] = None     # [heads] fp32: exp of it added to the softmax denominator (``sink`` is set then)
+    gate_all: bool = False                   # the output gate has a column per element, not per head
+    shared_row: bool = False                 # one key head whose first vdim_p channels are the values too (a cached latent)
+
+    def __post_init__(self):
+        if self.sinks is not None:
+            self.sink = True
 
     @property
     def kv_row(self) -> int:
-        return self.kv_heads * (self.dim_p + self.vdim_p)
+        return self.dim_p if self.shared_row else self.kv_heads * (self.dim_p + self.vdim_p)
+
+    @property
+    def v_col0(self) -> int:
+        """First value column of a cached row."""
+        return 0 if self.shared_row else self.kv_heads * self.dim_p
+
+    @property
+    def gate_cols(self) -> int:
+        return self.vdim_p if self.gate_all else 1
 
     def first(self, pos: int) -> int:
         """First position that a query at ``pos`` sees, kept first ones aside."""
@@ -81,8 +98,9 @@ class HeadPrep:
     dim: int                                 # real width of query and key heads
     eps: float = 1e-6
     bias: Optional[torch.Tensor] = None      # [heads * dim_p + kv_row], columns as projected: queries, keys, values
-    q_norm: Optional[torch.Tensor] = None    # [dim_p] gains of the RMS norms of query and key heads
+    q_norm: Optional[torch.Tensor] = None    # [dim_p] gains of the RMS norms of query and key heads, or with ``whole`` [heads * dim_p]
     k_norm: Optional[torch.Tensor] = None
+    whole: bool = False                      # one norm over all query heads of a token, one over all key heads
     interleaved: bool = False                # rotary pairs (2 i, 2 i + 1), else (i, i + dims / 2)
 
 
@@ -98,8 +116,10 @@ def prepare_heads(z: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, p: 
         x = z[:, :n + row] if h.bias is None else z[:, :n + row] + h.bias
 
         def turn(t, heads, w):
+            if w is not None and h.whole:
+                t = t / torch.sqrt((t * t).sum(-1, keepdim=True) / (heads * h.dim) + h.eps) * w
             t = t.reshape(-1, heads, dp)
-            if w is not None:
+            if w is not None and not h.whole:
                 t = t / torch.sqrt((t * t).sum(-1, keepdim=True) / h.dim + h.eps) * w
             return rotate_ref(t, rope, h.interleaved).reshape(-1, heads * dp)
         kv_write(torch.cat([turn(x[:, n:n + G * dp], G, h.k_norm), x[:, n + G * dp:]], 1), slots, cache)
@@ -110,14 +130,16 @@ def prepare_heads(z: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, p: 
     assert cache.stride(1) == row and cache.stride(2) == 1 and slots.dtype == torch.int64 and slots.shape[0] == T
     assert rope is None or (rope.is_contiguous() and rope.shape[0] == T)
     assert h.bias is None or h.bias.shape[0] == H * dp + row
-    assert all(w is None or w.shape[0] == dp for w in (h.q_norm, h.k_norm))
+    assert all(w is None or w.shape[0] == (n * dp if h.whole else dp) for w, n in ((h.q_norm, H), (h.k_norm, G)))
     kc = -(-dp // 64) * 64
     qf = torch.empty(T, H, kc, dtype=torch.bfloat16, device=z.device) if operand else None
     rc = _ext.lib().bg_head_prep(
         _i(_DT[cache.dtype]), _ext.ptr(z), _i(z.stride(0)), _ext.ptr(h.bias), _ext.ptr(h.q_norm), _ext.ptr(h.k_norm),
-        ctypes.c_float(h.eps), _i(h.dim), _ext.ptr(rope), _i(rope.shape[1] // 2 if rope is not None else 0), _i(h.interleaved),
+        _i(h.whole), ctypes.c_float(h.eps), _i(h.dim), _ext.ptr(rope), _i(rope.shape[1] // 2 if rope is not None else 0), _i(h.interleaved),
         _ext.ptr(slots), _ext.ptr(cache), ctypes.c_longlong(cache.stride(0)), _i(page), _i(row), _i(write_q), _ext.ptr(qf), _i(kc),
         ctypes.c_float(p.scale), _i(T), _i(H), _i(G), _i(dp), _i(p.vdim_p), _ext.stream())
+    if rc == -3:
+        raise _ext.KernelError(f"prepare_heads: {H} + {G} heads of {dp} are more than one norm takes (a token's row in shared memory)")
     _ext.check(rc, "bg_head_prep")
     return qf
 
@@ -137,24 +159,25 @@ def _rows_ref(q, p: TalkParams, cache, block_table, lens, out, row_seq, rope, ga
         bt = block_table[int(row_seq[t]) if row_seq is not None else t].long()
         rows = cache[bt[pos // page], pos % page].float()
         k = rows[:, : G * d].view(-1, G, d).repeat_interleave(rep, 1)
-        v = rows[:, G * d:].view(-1, G, dv).repeat_interleave(rep, 1)
+        v = rows[:, p.v_col0:p.v_col0 + G * dv].view(-1, G, dv).repeat_interleave(rep, 1)
         s = torch.einsum("hd,jhd->hj", q[t, : H * d].view(H, d).float(), k) * p.scale
         if p.talk is not None:
             s = p.talk @ s
         m = s.amax(-1, keepdim=True)
+        sink = None if not p.sink else torch.zeros(H, 1) if p.sinks is None else p.sinks.view(H, 1)
         if p.sink:
-            m = m.clamp_min(0)
+            m = torch.maximum(m, sink)
         e = torch.exp(s - m)
-        den = e.sum(-1, keepdim=True) + (torch.exp(-m) if p.sink else 0)
+        den = e.sum(-1, keepdim=True) + (torch.exp(sink - m) if p.sink else 0)
         o = torch.einsum("hj,jhv->hv", e / den, v) * p.out_scale
         if gate is not None:
-            o = o * torch.sigmoid(gate[t, :H].float()).unsqueeze(-1)
+            o = o * torch.sigmoid(gate[t, :H * p.gate_cols].float()).view(H, p.gate_cols)
         out[t, : H * dv] = o.reshape(-1).to(out.dtype)
 
 
 def rows_on_tensor_cores(p: TalkParams, dtype: torch.dtype) -> bool:
     """The row kernel of plain bf16 heads up to 128 wide (``csrc/gqa_rows.cuh``)."""
-    return dtype == torch.bfloat16 and p.talk is None and p.dim_p <= 128 and p.vdim_p <= 128
+    return dtype == torch.bfloat16 and p.talk is None and not p.shared_row and p.dim_p <= 128 and p.vdim_p <= 128
 
 
 def _ranges(ctas: int, keys: int, sms: int) -> int:
@@ -180,8 +203,8 @@ def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table
                 num_splits: int = 0, rope: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """q [T, >= H * dim_p] fp32 -> out [T, >= H * vdim_p] (operand dtype, a column view is fine).  ``lens`` [T] int32 =
     position + 1 of each row (0: no query, zero output); ``row_seq`` [R] block-table row of each query row (None: row i);
-    ``row_ids`` [R] the rows of q to compute (None: all).  ``rope`` [T, dims] turns the queries, ``gate`` [T, >= H] fp32 scales
-    each head's output by its sigmoid.  The keys are in the cache already."""
+    ``row_ids`` [R] the rows of q to compute (None: all).  ``rope`` [T, dims] turns the queries, ``gate`` [T, >= H (* vdim_p)] fp32 scales
+    each head's output, or with ``gate_all`` each element, by its sigmoid.  The keys are in the cache already."""
     if not q.is_cuda:
         if row_ids is not None:
             raise NotImplementedError("row subsets are a device path")
@@ -190,6 +213,8 @@ def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table
     R = q.shape[0] if row_ids is None else row_ids.shape[0]
     assert q.dtype == torch.float32 and q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == cache.dtype
     assert lens.dtype == torch.int32 and block_table.dtype == torch.int32 and row == p.kv_row and cache.stride(1) == row
+    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[1] >= p.heads * p.gate_cols)
+    assert p.sinks is None or (p.sinks.dtype == torch.float32 and p.sinks.shape[0] == p.heads)
     for t in (row_seq, row_ids):
         assert t is None or t.dtype == torch.int32
     H = p.heads
@@ -210,7 +235,8 @@ def attend_rows(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_table
         _ext.ptr(row_seq), _ext.ptr(row_ids), _ext.ptr(lens), _ext.ptr(out), _i(out.stride(0)), _ext.ptr(po),
         _ext.ptr(pml), _i(R), _i(H), _i(p.kv_heads), _i(p.dim_p), _i(p.vdim_p), _i(p.chunk), _i(p.window),
         _i(p.keep), _i(p.sink), ctypes.c_float(p.scale), ctypes.c_float(p.out_scale), _i(num_splits), _ext.ptr(rope), _i(rope.shape[1] // 2 if rope is not None else 0),
-        _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0), _ext.stream())
+        _ext.ptr(gate), _i(gate.stride(0) if gate is not None else 0), _i(p.gate_cols), _ext.ptr(p.sinks), _i(p.v_col0),
+        _ext.stream())
     if rc in (-1, -3):
         raise _ext.KernelError(f"attend_rows: heads {H}/{p.kv_heads}, widths {p.dim_p}/{p.vdim_p} are outside the kernel's "
                                "contract (shared memory of one CTA, 2,048 head-column items)")
@@ -225,7 +251,7 @@ _FOLD_ROWS = 8192            # rows whose mixed queries are held at a time
 def prefill_supported(p: TalkParams, dtype: torch.dtype, page: int) -> bool:
     """The tensor-core kernels read bf16 pages and keep one head's value columns in TMEM (plain heads: its queries in shared
     memory)."""
-    return dtype == torch.bfloat16 and p.vdim_p <= 256 and page >= 16 and (p.talk is not None or p.dim_p <= 256)
+    return dtype == torch.bfloat16 and not p.shared_row and p.vdim_p <= 256 and page >= 16 and (p.talk is not None or p.dim_p <= 256)
 
 
 def prefill_work(cu: Sequence[int], ctx: Sequence[int], chunk: int, min_tokens: int = 1,
@@ -269,8 +295,9 @@ def attend_prefill(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_ta
     P, page, row = cache.shape
     H, G = p.heads, p.kv_heads
     plain = p.talk is None
-    assert plain or (rope is None and gate is None and not p.window and p.out_scale == 1.0), \
-        "mixed heads with rotary queries, windows, output gates or scales are not covered"
+    assert plain or (rope is None and gate is None and not p.window and p.out_scale == 1.0 and p.sinks is None), \
+        "mixed heads with rotary queries, windows, output gates, scales or learned sinks are not covered"
+    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[1] >= H * p.gate_cols)
     kc = -(-(p.dim_p if plain else G * p.dim_p) // 64) * 64
     assert q.dtype == torch.float32 and q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == cache.dtype == torch.bfloat16
     assert row == p.kv_row and cache.stride(1) == row and block_table.dtype == torch.int32
@@ -296,7 +323,8 @@ def attend_prefill(q: torch.Tensor, p: TalkParams, cache: torch.Tensor, block_ta
         status = _ext.ptr(_ext.status_word(q.device))
         if plain:
             rc = L.bg_gqa_prompt(*where, _i(p.window), _i(p.keep), ctypes.c_float(p.out_scale), _ext.ptr(gate),
-                                 _i(gate.stride(0) if gate is not None else 0), status, _ext.stream())
+                                 _i(gate.stride(0) if gate is not None else 0), _i(p.gate_cols), _ext.ptr(p.sinks), status,
+                                 _ext.stream())
         else:
             rc = L.bg_talk_prefill(*where, status, _ext.stream())
         _ext.check(rc, "bg_gqa_prompt" if plain else "bg_talk_prefill")
