@@ -63,7 +63,7 @@ def _run(cmd: List[str], verbose: bool, log: Path) -> None:
 
 
 # kernels of the layer-listed models alone: what a command that serves one of them has to compile in a fresh checkout
-LAYERED_SOURCES = ("residual", "causal_conv", "delta_rule", "channel_delta", "mlstm", "retention", "talking_attn",
+LAYERED_SOURCES = ("residual", "causal_conv", "delta_rule", "channel_delta", "mlstm", "retention", "hgrn2", "latent_attn", "head_gemm", "talking_attn",
                    "talking_prefill", "gqa_prefill", "head_prep", "gemm_f32", "gemm_tcgen05", "moe_route")
 
 

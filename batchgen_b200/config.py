@@ -23,7 +23,7 @@ from typing import Dict, List, Optional, Tuple
 @dataclass(frozen=True)
 class MixerSpec:
     """A token mixer of a layer-listed model."""
-    kind: str                              # "attention" | "general_delta" | "channel_delta" | "mlstm" | "retention"
+    kind: str                              # "attention" | "latent_attention" | "general_delta" | "channel_delta" | "mlstm" | "retention" | "hgrn2"
     heads: int
     dim: int                               # query / key width of a head
     kv_heads: int = 0                      # key / value heads of attention, query / key heads of channel_delta (0 = heads)
@@ -32,11 +32,19 @@ class MixerSpec:
     chunk: int = 0                         # attention: keys are seen inside the query's own chunk of this many positions (0 = all)
     window: int = 0                        # attention: the last so many positions are seen, the query's own among them (0 = all)
     keep_first: int = 0                    # attention with a window: this many first positions of a sequence stay visible
-    bias: bool = False                     # attention: biases on the q, k, v and output projections
+    bias: bool = False                     # attention: biases on the q, k and v projections
+    out_bias: bool = False                 # attention: a bias on the output projection
     qk_norm: bool = False                  # attention: RMS norm of every query and key head, weights shared by the heads
+    qk_norm_all: bool = False              # attention: RMS norm of all query heads (and of all key heads) at once
     talking: bool = False                  # attention: a [heads, heads] matrix mixes the heads' scores before the softmax
     sink: bool = False                     # attention: one is added to the softmax denominator
+    head_sinks: bool = False               # attention: exp of a learned number per head is added to the softmax denominator
     out_gate: bool = False                 # attention: a sigmoid gate per head scales its output
+    out_gate_all: bool = False             # attention: a sigmoid gate per element of the heads' outputs
+    q_rank: int = 0                        # latent_attention: width of the latent that the queries go through
+    kv_rank: int = 0                       # latent_attention: width of the cached latent
+    rot_dim: int = 0                       # latent_attention: rotated query / key dimensions beside the ``dim`` unrotated ones
+    kv_from: int = -1                      # latent_attention: >= 0: the layer whose cached latents this one reads
     rot_dims: int = 0                      # attention, retention: leading head dimensions with rotary positions
     rot_base: float = 10000.0
     rot_interleaved: bool = False          # pairs (2 i, 2 i + 1) turn together; else (i, i + rot_dims / 2)
@@ -50,7 +58,11 @@ class MixerSpec:
 
     @property
     def recurrent(self) -> bool:
-        return self.kind != "attention"
+        return self.kind not in ("attention", "latent_attention")
+
+    @property
+    def latent(self) -> bool:
+        return self.kind == "latent_attention"
 
     @property
     def qk_heads(self) -> int:
@@ -67,8 +79,19 @@ class MixerSpec:
         return -(-self.vdim // 8) * 8
 
     @property
+    def rank_p(self) -> int:
+        """Latent width as stored."""
+        return -(-self.kv_rank // 8) * 8
+
+    @property
+    def rot_p(self) -> int:
+        return -(-self.rot_dim // 8) * 8
+
+    @property
     def kv_row(self) -> int:
-        """Elements of a cached token row: keys of every key head, then values."""
+        """Elements of a cached token row: keys of every key head, then values; the latent, then the shared rotated key part."""
+        if self.latent:
+            return self.rank_p + self.rot_p if self.kv_from < 0 else 0
         return 0 if self.recurrent else self.kv_heads * (self.dim_p + self.vdim_p)
 
     @property
@@ -97,7 +120,10 @@ class MixerSpec:
     def in_columns(self) -> int:
         """fp32 columns a token's projections take (a workspace estimate, padding aside)."""
         qk, v = self.heads * self.dim_p, self.heads * self.vdim_p
-        return {"attention": qk + self.kv_heads * (self.dim_p + self.vdim_p) + self.heads,
+        return {"attention": qk + self.kv_heads * (self.dim_p + self.vdim_p) + (v if self.out_gate_all else self.heads),
+                # projections, queries, then a token's expanded keys and values (16 bits)
+                "latent_attention": 2 * self.q_rank + self.rank_p + 2 * self.heads * (self.dim_p + self.rot_p) + v // 2,
+                "hgrn2": 2 * qk + v,
                 "general_delta": 6 * qk,
                 "channel_delta": 2 * self.conv_channels + 2 * v + qk + self.decay_rank + self.gate_rank + self.heads,
                 "mlstm": 2 * qk + 2 * v + 2 * self.heads, "retention": 2 * qk + 2 * v}[self.kind]
@@ -106,8 +132,14 @@ class MixerSpec:
         qk, v, H = self.heads * self.dim, self.heads * self.vdim, self.heads
         if self.kind == "attention":
             n = width * (H + self.kv_heads) * (self.dim + self.vdim) + (H * H if self.talking else 0)
-            n += (H + self.kv_heads) * self.dim + self.kv_heads * self.vdim + width if self.bias else 0
-            return n + (2 * self.dim if self.qk_norm else 0)
+            n += (H + self.kv_heads) * self.dim + self.kv_heads * self.vdim if self.bias else 0
+            n += (width if self.out_bias else 0) + (width * v if self.out_gate_all else 0)
+            return n + (2 * self.dim if self.qk_norm else 0) + ((H + self.kv_heads) * self.dim if self.qk_norm_all else 0)
+        if self.latent:
+            n = width * (self.q_rank + v) + self.q_rank * H * (self.dim + self.rot_dim) + self.kv_rank * (qk + v)
+            return n + (width * (self.kv_rank + self.rot_dim) if self.kv_from < 0 else 0)
+        if self.kind == "hgrn2":
+            return 2 * width * (qk + v)
         if self.kind == "general_delta":
             return width * (6 * qk + self.decay_rank) + self.decay_rank * qk
         if self.kind == "channel_delta":
@@ -129,7 +161,7 @@ class MlpSpec:
     shared_ff: int = 0                     # shared expert (0 = none), same activation
     shared_limit: float = 0.0
     shared_gate: bool = True               # the shared expert's output is scaled by a sigmoid gate per token
-    scoring: str = "sigmoid"               # router scores: sigmoid | softmax_all (over all experts)
+    scoring: str = "sigmoid"               # router scores: sigmoid | softmax (over the chosen) | softmax_all (over all experts)
     correction: bool = False               # a bias per expert takes part in the choice, not in the weights
     groups: int = 1                        # experts form this many groups, of which the best ``keep_groups`` take part
     keep_groups: int = 1
@@ -154,22 +186,24 @@ class LayerSpec:
     def kv_row(self) -> int:
         return sum(m.kv_row for m in self.mixers)
 
-    def state_parts(self, width: int, canon_taps: int) -> Dict[str, Tuple[int, ...]]:
-        """fp32 state of a sequence in this layer: the mixers' parts (the second mixer's names end in ".1") and, with input
-        convolutions, the last inputs of each sublayer."""
+    def state_parts(self, width: int, canon_taps: int, token_shift: bool = False) -> Dict[str, Tuple[int, ...]]:
+        """fp32 state of a sequence in this layer: the mixers' parts (the second mixer's names end in ".1"), with input
+        convolutions the last inputs of each sublayer, with a token shift the last input of the mixer."""
         parts = {name + (f".{i}" if i else ""): shape for i, m in enumerate(self.mixers) for name, shape in m.state_parts.items()}
         if canon_taps:
             rows = (canon_taps - 1, -(-width // 4) * 4)
             parts["canon1"] = rows
             if self.mlp.kind != "none":
                 parts["canon2"] = rows
+        if token_shift:
+            parts["shift"] = (1, -(-width // 4) * 4)
         return parts
 
 
 @dataclass
 class ModelConfig:
     name: str = "tiny-deepseek-v3"
-    family: str = "deepseek_v3"  # deepseek_v3 | deepseek_v2 | deepseek_v4 | glm5 | kimi_k3 | kimi_k25 | gpt_oss | minimax | mixtral | qwen2_moe | nanurax | pamevik | bolisun
+    family: str = "deepseek_v3"  # deepseek_v3 | deepseek_v2 | deepseek_v4 | glm5 | kimi_k3 | kimi_k25 | gpt_oss | minimax | mixtral | qwen2_moe | nanurax | pamevik | bolisun | pitudra
     vocab_size: int = 1024
     hidden_size: int = 256
     num_layers: int = 2
@@ -242,7 +276,11 @@ class ModelConfig:
     embed_scale: float = 1.0
     sandwich: bool = False                 # False: mixer and feed-forward read one RMS norm and are added together (parallel
                                            # block); True: one after the other, a norm before and after each
+    pre_norm: bool = True                  # sandwich: False: sublayers read the residual itself, only their outputs are normed
     layer_norm: bool = False               # sandwich: norms subtract the mean and have biases (else RMS norms)
+    token_shift: bool = False              # sandwich: a mixer reads h + (h' - h) * shift, h' the previous token's h
+    side_dim: int = 0                      # sandwich: > 0: after the feed-forward a token's own row of a table per layer, so many
+                                           # numbers gated by the residual, is projected, RMS-normed and added
     streams: int = 0                       # > 0: pre-norm blocks (mixer, then feed-forward) around this many residual streams with
                                            # hyper-connections of fixed weights
     canon_taps: int = 0                    # sandwich: every sublayer reads h + conv(h), a causal convolution of this many taps
@@ -277,7 +315,7 @@ class ModelConfig:
     def layered_state_parts(self) -> List[Tuple[Tuple[int, str], Tuple[int, ...]]]:
         """((layer, name), shape) of everything a sequence of a layer-listed model carries outside the paged rows."""
         return [((l, name), shape) for l, s in enumerate(self.layer_specs)
-                for name, shape in s.state_parts(self.hidden_size, self.canon_taps).items()]
+                for name, shape in s.state_parts(self.hidden_size, self.canon_taps, self.token_shift).items()]
 
     def layered_state_floats_per_seq(self) -> int:
         return sum(math.prod(shape) for _, shape in self.layered_state_parts())
@@ -392,7 +430,7 @@ class ModelConfig:
                 f = spec.mlp
                 n += sum(m.param_count(h) for m in spec.mixers)
                 n += (2 if f.activation == "relu2" else 3) * h * f.ff * (f.experts if f.kind == "moe" else 1) + h * f.experts + 3 * h * f.shared_ff
-            return n
+            return n + len(self.layer_specs) * self.side_dim * (self.vocab_size + 2 * h)
         for l in range(self.num_layers):
             if self.layer_is_kda(l):
                 hd = self.kda_num_heads * self.kda_head_dim
@@ -817,7 +855,7 @@ def _bolisun_layer(d: Dict, index: int) -> LayerSpec:
     sc = rot.get("scaling")
     left = MixerSpec(
         "attention", heads=a["heads"], dim=a["dim"], kv_heads=a.get("kv_heads", a["heads"]), vdim=a["vdim"], scale=float(a["scale"]),
-        window=int(mask.get("size", 0)), keep_first=int(mask.get("keep_first", 0)), bias=True, qk_norm=True,
+        window=int(mask.get("size", 0)), keep_first=int(mask.get("keep_first", 0)), bias=True, out_bias=True, qk_norm=True,
         rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)), rot_interleaved=True,
         yarn=tuple(float(sc[k]) for k in ("factor", "original", "fast", "slow")) if sc else (), out_scale=float(m["left_scale"]))
     right = MixerSpec("retention", heads=r["heads"], dim=r["dim"], vdim=r["vdim"], decay=tuple(float(x) for x in r["decay"]),
@@ -881,7 +919,69 @@ def _bolisun_dir(path: str, d: Dict) -> ModelConfig:
     return cfg
 
 
-_ARCHITECTURES = {"Nanurax": _nanurax_dir, "Pamevik": _pamevik_dir, "Bolisun": _bolisun_dir}        # config.json "architecture" -> reader of the model directory
+# ------------------------------------------------------------------ Pitudra: layer-listed config.json
+def _pitudra_layer(d: Dict, index: int, layers: List[Dict]) -> LayerSpec:
+    m, kind, f = d["mixer"], d["type"], d.get("mlp")
+    window = int((m.get("mask") or {}).get("size", 0))
+    if m.get("mask") and window < 1:
+        raise ValueError(f"layer {index}: a window of {window} positions")
+    if kind == "hgrn2":
+        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], vdim=m["vdim"])
+    elif kind == "attention":
+        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], kv_heads=m.get("kv_heads", m["heads"]), vdim=m["vdim"],
+                          scale=float(m["scale"]), window=window, bias=True, qk_norm_all=True, head_sinks=True, out_gate_all=True)
+        if mixer.heads % mixer.kv_heads:
+            raise ValueError(f"layer {index}: {mixer.heads} heads do not divide over {mixer.kv_heads} key/value heads")
+    elif kind == "latent_attention":
+        rot, j = m["rot"], m.get("kv_from")
+        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]), window=window, head_sinks=True,
+                          q_rank=m["q_rank"], kv_rank=m["kv_rank"], rot_dim=m["rot_dim"], rot_dims=int(rot["dims"]),
+                          rot_base=float(rot["base"]), kv_from=-1 if j is None else int(j))
+        if mixer.rot_dims != mixer.rot_dim or mixer.rot_dim % 2:
+            raise ValueError(f"layer {index}: {mixer.rot_dims} rotary dimensions in a rotated part of {mixer.rot_dim}")
+        if j is not None:
+            src = layers[j]["mixer"] if 0 <= j < index and layers[j]["type"] == kind else {"kv_from": j}
+            if src.get("kv_from") is not None:
+                raise ValueError(f"layer {index}: latents of layer {j}, which has none of its own before it")
+            if any(src[k] != m[k] for k in ("kv_rank", "rot_dim", "rot")):
+                raise ValueError(f"layer {index}: latents of another shape or rotation than those of layer {j}")
+    else:
+        raise ValueError(f"layer {index}: unknown mixer type {kind!r}")
+    if not f:
+        return LayerSpec(mixer)
+    if f["kind"] != "moe":
+        raise ValueError(f"layer {index}: unknown feed-forward kind {f['kind']!r}")
+    mlp = MlpSpec("moe", ff=f["expert"]["ff"], activation="relu2", experts=f["router"]["experts"], top=f["router"]["top"], scoring="softmax")
+    if not 0 < mlp.top <= mlp.experts:
+        raise ValueError(f"layer {index}: top {mlp.top} of {mlp.experts} experts")
+    return LayerSpec(mixer, mlp)
+
+
+def pitudra_config(d: Dict, name: str = "pitudra") -> ModelConfig:
+    """A Pitudra config.json (parsed) as a ``ModelConfig``."""
+    layers = tuple(_pitudra_layer(x, i, d["layers"]) for i, x in enumerate(d["layers"]))
+    moe = [s.mlp for s in layers if s.mlp.kind == "moe"]
+    return ModelConfig(
+        name=name, family="pitudra", vocab_size=d["vocab"], hidden_size=d["width"], num_layers=len(layers), layer_specs=layers,
+        rms_eps=float(d["norm"]["eps"]), sandwich=True, pre_norm=False, layer_norm=True, token_shift=True,
+        side_dim=int((d.get("token_side") or {}).get("dim", 0)),
+        # summaries that planners read; the layers themselves are described by ``layer_specs``
+        num_heads=max(s.mixer.heads for s in layers), num_kv_heads=max((s.mixer.kv_heads for s in layers), default=1) or 1,
+        head_dim=max(s.mixer.dim for s in layers), sliding_window=max(s.mixer.window for s in layers), first_k_dense=0,
+        intermediate_size=0, moe_intermediate_size=max((f.ff for f in moe), default=0),
+        n_routed_experts=max((f.experts for f in moe), default=0), num_experts_per_tok=max((f.top for f in moe), default=0),
+        n_shared_experts=0, attention_sinks=any(s.mixer.head_sinks for s in layers), attention_bias=True, scoring_func="softmax",
+        max_position_embeddings=1 << 30, eos_token_id=-1, bos_token_id=-1)
+
+
+def _pitudra_dir(path: str, d: Dict) -> ModelConfig:
+    cfg = pitudra_config(d, os.path.basename(os.path.normpath(path)) or "pitudra")
+    cfg.checkpoint_dir = path
+    return cfg
+
+
+# config.json "architecture" -> reader of the model directory
+_ARCHITECTURES = {"Nanurax": _nanurax_dir, "Pamevik": _pamevik_dir, "Bolisun": _bolisun_dir, "Pitudra": _pitudra_dir}
 
 
 def load_model_dir(path: str) -> ModelConfig:
@@ -980,7 +1080,38 @@ def bolisun_bench() -> ModelConfig:
                           "bolisun-bench")
 
 
+def tiny_pitudra() -> ModelConfig:
+    """One layer of every mixer and one that borrows latents; with and without a feed-forward."""
+    moe = {"kind": "moe", "expert": {"ff": 40}, "router": {"experts": 6, "top": 2}}
+    lat = {"heads": 4, "dim": 24, "rot_dim": 8, "vdim": 16, "q_rank": 40, "kv_rank": 48, "scale": 0.2, "mask": {"size": 50},
+           "rot": {"base": 5000.0, "dims": 8}}
+    return pitudra_config({
+        "vocab": 320, "width": 120, "norm": {"eps": 1e-5}, "token_side": {"dim": 16},
+        "layers": [{"type": "hgrn2", "mixer": {"heads": 3, "dim": 16, "vdim": 24}, "mlp": moe},
+                   {"type": "latent_attention", "mixer": lat, "mlp": moe},
+                   {"type": "attention", "mixer": {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 32, "scale": 0.2, "mask": {"size": 33}},
+                    "mlp": None},
+                   {"type": "latent_attention", "mixer": dict(lat, heads=2, dim=16, vdim=40, kv_from=1, mask={"size": 20}), "mlp": moe}]},
+        "tiny-pitudra")
+
+
+def pitudra_bench() -> ModelConfig:
+    """Layers of a real model's size: two HGRN2 layers, one of windowed attention and one of latent attention, each with 64 experts of
+    which 8 run.  An expert's two matrices hold as many weights as the three of a gated one of width 1024."""
+    moe = {"kind": "moe", "expert": {"ff": 1536}, "router": {"experts": 64, "top": 8}}
+    rec = {"type": "hgrn2", "mlp": moe, "mixer": {"heads": 32, "dim": 128, "vdim": 128}}
+    att = {"type": "attention", "mlp": moe, "mixer": {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                                      "mask": {"size": 1024}}}
+    lat = {"type": "latent_attention", "mlp": moe, "mixer": {
+        "heads": 32, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": 1536, "kv_rank": 512, "scale": 192 ** -0.5,
+        "mask": {"size": 4096}, "rot": {"base": 1e6, "dims": 64}}}
+    return pitudra_config({"vocab": 163840, "width": 2304, "norm": {"eps": 1e-6}, "token_side": {"dim": 128},
+                           "layers": [rec, att, dict(rec), lat]}, "pitudra-bench")
+
+
 _PRESETS = {
+    "tiny-pitudra": tiny_pitudra,
+    "pitudra-bench": pitudra_bench,
     "tiny-bolisun": tiny_bolisun,
     "bolisun-bench": bolisun_bench,
     "tiny-pamevik": tiny_pamevik,
@@ -1040,6 +1171,7 @@ _PATTERNS = [
     (r"nanurax", "nanurax-bench"),
     (r"pamevik", "pamevik-bench"),
     (r"bolisun", "bolisun-bench"),
+    (r"pitudra", "pitudra-bench"),
 ]
 
 

@@ -1,5 +1,5 @@
 """Model families.  ``build_model`` creates a ``Transformer`` (for DeepSeek-V4 a ``DeepSeekV4``, for layer-listed models
-such as Nanurax, Pamevik and Bolisun a ``LayeredDecoder``) for any registered config."""
+such as Nanurax, Pamevik, Bolisun and Pitudra a ``LayeredDecoder``) for any registered config."""
 from __future__ import annotations
 
 from typing import Optional

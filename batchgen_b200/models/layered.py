@@ -3,9 +3,11 @@ fp32 residual stream.  Three block forms:
 
 * parallel (Nanurax): mixer and feed-forward read one RMS norm and their outputs are added together.  Generalised delta-rule
   layers and chunked talking-heads attention layers, dense tanh-GELU or input-weighted clamped-SwiGLU mixture feed-forwards.
-* sandwich (Pamevik, ``ModelConfig.sandwich``): mixer, then feed-forward, each between two norms (``layer_norm``: with mean and
-  bias) and behind an input convolution (``canon_taps``).  mLSTM, gated delta-rule with a decay per channel, and softmax
-  attention beside retention; squared-ReLU feed-forwards.
+* sandwich (Pamevik, Pitudra, ``ModelConfig.sandwich``): mixer, then feed-forward, each between two norms (``layer_norm``: with mean
+  and bias; ``pre_norm`` off: only the output's) and behind an input convolution (``canon_taps``), or the mixer behind a shift towards
+  the previous token (``token_shift``); a gated row of a table per token may follow (``side_dim``).  mLSTM, gated delta-rule with a
+  decay per channel, and softmax attention beside retention, squared-ReLU feed-forwards; or HGRN2, windowed attention with sinks and
+  attention over latents that layers may share, mixtures of squared-ReLU experts.
 * hyper-connected (Bolisun, ``ModelConfig.streams``): mixer, then feed-forward, each behind an RMS norm that reads a weighted sum of
   several residual streams; its output joins all streams, which are mixed with one another.  Windowed attention with normed heads
   beside retention; clamped-SwiGLU feed-forwards and mixtures of experts; layers may share their weights.
@@ -63,14 +65,14 @@ class LayeredLayer:
 @dataclass
 class Sublayer:
     """One half of a sandwich or hyper-connected block: mixer(s) side by side, or a feed-forward."""
-    norm: residual.Norm
+    norm: Optional[residual.Norm]
     post: Optional[residual.Norm]                 # sandwich: norm of the output
     w_in: torch.Tensor                            # [columns, width_p]
     w_out: List[torch.Tensor]                     # per mixer W_o (hyper-connected: one matrix), or [W_down]: [width, operand width
                                                   # padded to K_ALIGN]
     mixers: List[Mixer] = field(default_factory=list)       # empty: feed-forward
     branch_w: Optional[Tuple[torch.Tensor, torch.Tensor]] = None      # weights of two mixers' output norms
-    canon_w: Optional[torch.Tensor] = None        # [taps, width4] fp32 input convolution
+    canon_w: Optional[torch.Tensor] = None        # [taps, width4] fp32 input convolution (a token shift is one of two taps)
     canon_part: str = ""                          # its state part
     ff: int = 0                                   # width of the dense or shared feed-forward (hyper-connected: padded to K_ALIGN)
     hc: Optional[residual.Hyper] = None           # hyper-connected blocks, with what follows
@@ -79,6 +81,7 @@ class Sublayer:
     seg: Dict[str, Tuple[int, int]] = field(default_factory=dict)     # feed-forward part -> (first column of the GEMM output, width)
     correction: Optional[torch.Tensor] = None     # [experts] fp32
     experts: Optional[ExpertWeights] = None
+    side: Optional[torch.Tensor] = None           # [vocab, side dim] (a column view): this sublayer is the token's side input
 
 
 @dataclass
@@ -87,6 +90,7 @@ class LayeredWeights:
     final_norm: torch.Tensor = None               # fp32 gain, or a ``residual.Norm`` (sandwich, hyper-connected)
     lm_head: torch.Tensor = None                  # [vocab, width_p]
     layers: List = field(default_factory=list)    # LayeredLayer, or lists of Sublayers
+    side: Optional[torch.Tensor] = None           # [vocab, layers * side dim]
 
 
 def build_layered_weights(cfg: ModelConfig, layout: ParallelLayout, src: WeightSource, dtype: torch.dtype) -> LayeredWeights:
@@ -100,34 +104,53 @@ def build_layered_weights(cfg: ModelConfig, layout: ParallelLayout, src: WeightS
     w.final_norm = (_norm(src, "final.norm", cfg) if cfg.sandwich or cfg.streams
                     else src.get("final.norm", (D,), "norm").float().contiguous())
     w.lm_head = pad_cols(w.embed if cfg.tie_word_embeddings else src.get("head", (V, D)).to(dtype), Kp).contiguous()
+    if cfg.side_dim:
+        w.side = src.get("side.embed", (V, cfg.num_layers * cfg.side_dim)).to(dtype).contiguous()
     block = _build_hyper if cfg.streams else _build_sandwich if cfg.sandwich else _build_parallel
     own = {i: block(cfg, spec, f"l{i}.", src, dtype) for i, spec in enumerate(cfg.layer_specs) if spec.weights_of < 0}
     w.layers = [own[i if spec.weights_of < 0 else spec.weights_of] for i, spec in enumerate(cfg.layer_specs)]
+    if cfg.side_dim:
+        for i, layer in enumerate(w.layers):
+            layer.append(_build_side(cfg, f"l{i}.", src, dtype, w.side[:, i * cfg.side_dim:(i + 1) * cfg.side_dim]))
     return w
+
+
+def _vec(src: WeightSource, name: str, kind: str, D: int) -> torch.Tensor:
+    return torch.nn.functional.pad(src.get(name, (D,), kind).float(), (0, pad_to(D, 4) - D)).contiguous()
 
 
 def _norm(src: WeightSource, name: str, cfg: ModelConfig) -> residual.Norm:
     D = cfg.hidden_size
+    return residual.Norm(_vec(src, name, "norm", D), _vec(src, name + ".b", "bias", D) if cfg.layer_norm else None, cfg.layer_norm)
 
-    def vec(n, kind):
-        return torch.nn.functional.pad(src.get(n, (D,), kind).float(), (0, pad_to(D, 4) - D)).contiguous()
-    return residual.Norm(vec(name, "norm"), vec(name + ".b", "bias") if cfg.layer_norm else None, cfg.layer_norm)
+
+def _build_side(cfg: ModelConfig, p: str, src: WeightSource, dtype: torch.dtype, table: torch.Tensor) -> Sublayer:
+    D, n = cfg.hidden_size, cfg.side_dim
+    gate = pad_cols(pad_rows(src.get(p + "side.gate", (n, D)).to(dtype), pad_to(n, 8)), pad_to(D, K_ALIGN)).contiguous()
+    proj = pad_cols(src.get(p + "side.proj", (D, n)).to(dtype), pad_to(n, K_ALIGN)).contiguous()
+    return Sublayer(None, residual.Norm(_vec(src, p + "side.norm", "norm", D)), gate, [proj], side=table)
 
 
 def _build_sandwich(cfg: ModelConfig, spec: LayerSpec, p: str, src: WeightSource, dtype: torch.dtype) -> List[Sublayer]:
     D, f = cfg.hidden_size, spec.mlp
     Kp, W4 = pad_to(D, K_ALIGN), pad_to(D, 4)
-    if f.kind not in ("none", "dense") or (f.kind == "dense" and f.activation != "relu2"):
-        raise NotImplementedError("sandwich blocks carry squared-ReLU feed-forwards")
+    if f.kind not in ("none", "dense", "moe") or (f.kind != "none" and f.activation != "relu2") or f.shared_ff or f.correction:
+        raise NotImplementedError("sandwich blocks carry squared-ReLU feed-forwards and mixtures of them without a shared one")
     prefixes = [p + "mix."] if spec.second is None else [p + "mix.left.", p + "mix.right."]
     mixers = [build_mixer(m, q, src, cfg, dtype, i) for i, (m, q) in enumerate(zip(spec.mixers, prefixes))]
     out = []
-    for n in (1, 2) if f.kind == "dense" else (1,):
-        s = Sublayer(_norm(src, f"{p}norm{n}", cfg), _norm(src, f"{p}norm{n}b", cfg), None, [])
+    for n in (1, 2) if f.kind != "none" else (1,):
+        if cfg.pre_norm:
+            s = Sublayer(_norm(src, f"{p}norm{n}", cfg), _norm(src, f"{p}norm{n}b", cfg), None, [])
+        else:
+            s = Sublayer(None, _norm(src, f"{p}norm{n}", cfg), None, [])
         if cfg.canon_taps:
             s.canon_part = f"canon{n}"
             taps = src.get(f"{p}canon{n}", (D, cfg.canon_taps)).float()
             s.canon_w = pad_rows(taps, W4).t().contiguous()
+        elif cfg.token_shift and n == 1:
+            s.canon_part, mu = "shift", _vec(src, p + "shift", "shift", D)
+            s.canon_w = torch.stack([mu, -mu])                      # h + mu h' - mu h
         if n == 1:
             s.mixers = mixers
             s.w_in = stack_parts([(m.seg, name, t) for m in mixers for name, t in m.parts], Kp, dtype)
@@ -137,6 +160,11 @@ def _build_sandwich(cfg: ModelConfig, spec: LayerSpec, p: str, src: WeightSource
             if spec.second is not None:
                 s.branch_w = tuple(torch.nn.functional.pad(src.get(q + "out", (D,), "norm").float(), (0, W4 - D)).contiguous()
                                    for q in prefixes)
+        elif f.kind == "moe":
+            s.mlp = f
+            s.w_in = stack_parts([(s.seg, "router", src.get(p + "mlp.router", (f.experts, D)))], Kp, dtype)
+            s.w_out = []
+            s.experts = _experts(f, p + "mlp.", src, D, dtype)
         else:
             s.ff = f.ff
             s.w_in = pad_cols(pad_rows(src.get(p + "mlp.up", (f.ff, D)).to(dtype), pad_to(f.ff, 8)), Kp).contiguous()
@@ -150,7 +178,7 @@ def _experts(f: MlpSpec, q: str, src: WeightSource, D: int, dtype: torch.dtype) 
     w13, wd = [], []
     for e in range(f.experts):
         ep = f"{q}e{e}."
-        gu = [pad_rows(src.get(ep + x, (f.ff, D)).to(dtype), Fp) for x in ("gate", "up")]
+        gu = [pad_rows(src.get(ep + x, (f.ff, D)).to(dtype), Fp) for x in (("up",) if f.activation == "relu2" else ("gate", "up"))]
         w13.append(pad_cols(torch.cat(gu, 0), Kp))
         wd.append(pad_cols(src.get(ep + "down", (D, f.ff)).to(dtype), Fp))
     return ExpertWeights(w13=torch.stack(w13), w2=torch.stack(wd), activation=f.activation, act_limit=f.limit)
@@ -228,6 +256,7 @@ def layered_tensor_specs(cfg: ModelConfig) -> List[Tuple[str, Tuple[int, ...], s
         return [(name, (D,), "norm", l)] + ([(name + ".b", (D,), "bias", l)] if cfg.layer_norm else [])
     out = [("embed", (V, D), "normal", -1), *norm("final.norm", -1)]
     out += [] if cfg.tie_word_embeddings else [("head", (V, D), "normal", -1)]
+    out += [("side.embed", (V, cfg.num_layers * cfg.side_dim), "normal", -1)] if cfg.side_dim else []
     for i, s in enumerate(cfg.layer_specs):
         if s.weights_of >= 0:
             continue
@@ -235,11 +264,15 @@ def layered_tensor_specs(cfg: ModelConfig) -> List[Tuple[str, Tuple[int, ...], s
         prefixes = [f"l{i}.mix."] if s.second is None else [f"l{i}.mix.left.", f"l{i}.mix.right."]
         if cfg.sandwich:
             for n in ("1", "2") if f.kind != "none" else ("1",):
-                out += norm(f"l{i}.norm{n}", i) + norm(f"l{i}.norm{n}b", i)
+                out += norm(f"l{i}.norm{n}", i) + (norm(f"l{i}.norm{n}b", i) if cfg.pre_norm else [])
                 if cfg.canon_taps:
                     out.append((f"l{i}.canon{n}", (D, cfg.canon_taps), "normal", i))
             if s.second is not None:
                 out += [(q_ + "out", (D,), "norm", i) for q_ in prefixes]
+            out += [(f"l{i}.shift", (D,), "shift", i)] if cfg.token_shift else []
+            if cfg.side_dim:
+                out += [(f"l{i}.side.gate", (cfg.side_dim, D), "normal", i), (f"l{i}.side.proj", (D, cfg.side_dim), "normal", i),
+                        (f"l{i}.side.norm", (D,), "norm", i)]
         elif cfg.streams:
             S = cfg.streams
             for n in ("1", "2") if f.kind != "none" else ("1",):
@@ -259,7 +292,7 @@ def layered_tensor_specs(cfg: ModelConfig) -> List[Tuple[str, Tuple[int, ...], s
             out.append((q + "router", (f.experts, D), "normal", i))
             out += [(q + "correction", (f.experts,), "bias", i)] if f.correction else []
             for e in range(f.experts):
-                out += ff(f"{q}e{e}.", f.ff)
+                out += ff(f"{q}e{e}.", f.ff)[1 if f.activation == "relu2" else 0:]
             if f.shared_ff:
                 out += ff(q + "shared.", f.shared_ff) + ([(q + "shared.sg", (1, D), "normal", i)] if f.shared_gate else [])
     return out
@@ -316,7 +349,9 @@ class LayeredDecoder:
         hist = cache.state.layer(l, s.canon_part)
         if plan.cu is None:
             return residual.sandwich_norm(*args, **pending, canon=residual.Canon(s.canon_w, hist, plan.slots))
-        h = residual.sandwich_norm(*args, **pending, raw=True)
+        h = residual.sandwich_norm(*args, **pending, raw=True) if s.norm is not None else x
+        if s.norm is None:                        # the convolution reads the residual itself
+            residual.sandwich_norm(*args, **pending, emit=False)
         y = torch.empty(x.shape[0], self.width_p, dtype=self.dtype, device=x.device)
         return conv.causal_conv(h, s.canon_w, hist, plan.slots, y, "residual", plan.cu, plan.cu_host, plan.row_seq, plan.has_initial)
 
@@ -334,12 +369,22 @@ class LayeredDecoder:
                     self.layer_hook(l - 1, x[:, :D])
                 with tm.timed("proj_in", l):
                     z = gemm.rows_gemm(y, s.w_in)
+                if s.experts is not None:
+                    f = s.mlp
+                    with tm.timed("moe", l):
+                        idx, rw = moe_ops.router_topk(z[:, :f.experts], None, f.top, scoring=f.scoring, num_valid=meta.num_valid)
+                        routed, pos = moe_ops.routed_rows(y, idx, rw, s.experts, False, meta.num_valid)
+                    pending = dict(routed=routed, pos=pos, route_w=rw, post=s.post)
+                    continue
                 if s.mixers:
                     operands = []
                     with tm.timed("mixer_" + meta.mode, l):
                         for m, wo in zip(s.mixers, s.w_out):
                             operands.append(self._operand(T, m.cols, wo.shape[1]))
                             m.run(l, z, operands[-1][:, :m.cols], plan, meta, cache)
+                elif s.side is not None:
+                    with tm.timed("side", l):
+                        operands = [residual.token_side(z, s.side, ids, s.w_out[0].shape[1], self.dtype)]
                 else:
                     with tm.timed("act", l):
                         operands = [residual.cast_act(z[:, :s.ff], s.w_out[0].shape[1], self.dtype, "relu2")]

@@ -13,7 +13,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..config import MixerSpec, ModelConfig
-from ..ops import conv, delta, gemm, recurrent, residual, talking
+from ..ops import conv, delta, gemm, latent, recurrent, residual, talking
 from ..ops.residual import pad_to
 from .weights import WeightSource
 
@@ -57,6 +57,23 @@ class StepPlan:
             self.tiles[chunk, window] = (blocks, bool(short), rows, seqs)
         return self.tiles[chunk, window]
 
+    def latent_tiles(self, window: int, page: int):
+        """The same for attention over latents in its expanded form: (expansions, rows of short pieces, their block-table rows and
+        lengths), or no rows (None, None, None) when every piece is long."""
+        key = ("latent", window)
+        if key not in self.tiles:
+            cu, least, dev = self.cu_host, talking.PREFILL_MIN_TOKENS, self.lens.device
+            groups = latent.expansions(cu, self.ctx, window, page, dev)
+            short = [t for a, b in zip(cu, cu[1:]) if b - a < least for t in range(a, b)]
+            if not groups:
+                self.tiles[key] = ([], None, self.row_seq, self.lens)
+            elif short:
+                rows = torch.tensor(short, dtype=torch.int32, device=dev)
+                self.tiles[key] = (groups, rows, self.row_seq[rows.long()].contiguous(), self.lens[rows.long()].contiguous())
+            else:
+                self.tiles[key] = (groups, None, None, None)
+        return self.tiles[key]
+
 
 @dataclass
 class Mixer:
@@ -74,6 +91,7 @@ class Mixer:
     prep: Optional[talking.HeadPrep] = None       # attention with biases or norms of its heads
     o_bias: Optional[torch.Tensor] = None         # [width] fp32 bias of the output projection, times the output's scale
     rec: Optional[recurrent.RecurrentParams] = None
+    lat: Optional[latent.LatentParams] = None
 
     def column(self, z: torch.Tensor, name: str) -> torch.Tensor:
         o, n = self.seg[name]
@@ -85,6 +103,9 @@ class Mixer:
     def run(self, l: int, z: torch.Tensor, out: torch.Tensor, plan: StepPlan, meta, cache) -> None:
         if self.talk is not None:
             self._attention(l, z, out, plan, meta, cache)
+            return
+        if self.lat is not None:
+            self._latent(l, z, out, plan, meta, cache)
             return
         if plan.slots is None:
             raise RuntimeError("a model with recurrent layers needs AttnMeta.state_slots")
@@ -104,6 +125,10 @@ class Mixer:
             n = p.heads * p.dim_p
             recurrent.recurrent_forward(p, x[:, :qk], x[:, qk:2 * qk], x[:, 2 * qk:], low[:, n:], state, plan.slots, out,
                                         low=low[:, :n], beta=self.column(z, "b"), **where)
+            return
+        if p.rule == "hgrn2":
+            q, f, v = (self.column(z, x) for x in "qfv")
+            recurrent.recurrent_forward(p, q, f, v, None, state, plan.slots, out, **where)
             return
         q, k, v, g = (self.column(z, x) for x in "qkvg")
         extra = (dict(gate_i=self.column(z, "i"), gate_f=self.column(z, "f")) if p.rule == "mlstm"
@@ -130,6 +155,27 @@ class Mixer:
             talking.attend_prefill(zq, p, kv, meta.block_table, out, blocks, operand=operand, **more)
         if short:
             talking.attend_rows(zq, p, kv, meta.block_table, plan.lens, out, seqs, rows, **more)
+
+    def _latent(self, l: int, z, out, plan: StepPlan, meta, cache) -> None:
+        p, dt = self.lat, out.dtype
+        own = self.spec.kv_from < 0
+        kv, rope = cache.latent(l if own else self.spec.kv_from), plan.rope(self.rot)
+        cols = tuple(self.seg[x][0] if x in self.seg else None for x in ("dq", "c", "r"))
+        q = gemm.rows_gemm(latent.prepare(z, cols, meta.slot_mapping, kv, p, rope, dt), p.w_uq)
+        groups, rows, seqs, lens = [], None, plan.row_seq, plan.lens
+        if plan.cu is not None and z.is_cuda and latent.prompt_supported(p, kv.dtype, kv.shape[1]):
+            groups, rows, seqs, lens = plan.latent_tiles(p.window, kv.shape[1])
+        if groups:
+            latent.attend_prompt(q, p, kv, meta.block_table, rope, out, groups)
+        if lens is None:
+            return
+        o = latent.attend(latent.queries(q, p, rope, rows, dt), p, kv, meta.block_table, lens, seqs)
+        if rows is None:
+            latent.head_product(o, p.w_uv, out.unflatten(1, (p.heads, p.vdim_p)))
+            return
+        short = torch.empty(rows.shape[0], p.heads, p.vdim_p, dtype=dt, device=out.device)
+        latent.head_product(o, p.w_uv, short)
+        out.index_copy_(0, rows.long(), short.view(rows.shape[0], -1))
 
 
 # ---------------------------------------------------------------- weights
@@ -175,17 +221,31 @@ def build_mixer(m: MixerSpec, p: str, src: WeightSource, cfg: ModelConfig, dtype
         mx.parts = [("q", rows("q", H, d, dp)), ("k", rows("k", G, d, dp)), ("v", rows("v", G, dv, dvp))]
         if m.out_gate:
             mx.parts.append(("gate", src.get(p + "g", (H, D))))
+        elif m.out_gate_all:
+            mx.parts.append(("gate", rows("g", H, dv, dvp)))
         talk = src.get(p + "talk", (H, H)).float().contiguous() if m.talking else None
         mx.talk = talking.TalkParams(heads=H, kv_heads=G, dim_p=dp, vdim_p=dvp, scale=m.scale, chunk=m.chunk, sink=m.sink, talk=talk,
-                                     window=m.window, keep=m.keep_first if m.window else 0, out_scale=m.out_scale)
-        if m.bias or m.qk_norm or m.rot_interleaved:
-            mx.prep = talking.HeadPrep(dim=d, eps=cfg.rms_eps, interleaved=m.rot_interleaved)
+                                     window=m.window, keep=m.keep_first if m.window else 0, out_scale=m.out_scale, gate_all=m.out_gate_all,
+                                     sinks=src.get(p + "sink", (H,), "bias").float().contiguous() if m.head_sinks else None)
+        if m.bias or m.qk_norm or m.qk_norm_all or m.rot_interleaved:
+            mx.prep = talking.HeadPrep(dim=d, eps=cfg.rms_eps, interleaved=m.rot_interleaved, whole=m.qk_norm_all)
         if m.bias:
             mx.prep.bias = torch.cat([vector(x + ".b", n, w, wp, "bias") for x, n, w, wp in (("q", H, d, dp), ("k", G, d, dp),
                                                                                         ("v", G, dv, dvp))])
+        if m.out_bias:
             mx.o_bias = src.get(p + "o.b", (D,), "bias").float() * m.out_scale
-        if m.qk_norm:
+        if m.qk_norm_all:
+            mx.prep.q_norm, mx.prep.k_norm = (vector(x + ".norm", n, d, dp, "norm") for x, n in (("q", H), ("k", G)))
+        elif m.qk_norm:
             mx.prep.q_norm, mx.prep.k_norm = (vector(x + ".norm", 1, d, dp, "norm") for x in "qk")
+    elif m.kind == "latent_attention":
+        mx.lat = _build_latent(mx, m, p, src, cfg, dtype)
+    elif m.kind == "hgrn2":
+        mx.parts = [("q", rows("q", H, d, dp)), ("f", rows("f", H, d, dp)), ("v", rows("v", H, dv, dvp))]
+        norm = head_rows(src.get(p + "norm", (dv,), "norm").repeat(H), H, dv, dvp)
+        mx.rec = recurrent.RecurrentParams(rule=m.kind, heads=H, dim_p=dp, vdim=dv, vdim_p=dvp, eps=cfg.rms_eps,
+                                           norm_w=norm.float().contiguous(), f_bias=vector("f.b", H, d, dp, "bias"),
+                                           f_lower=vector("lower", H, d, dp, "lower"))
     elif m.kind == "general_delta":
         mx.parts = [(x, rows(x, H, d, dp)) for x in ("r", "k", "v", "g", "a")]
         mx.parts.append(("low", src.get(p + "w1", (m.decay_rank, D))))
@@ -225,6 +285,40 @@ def build_mixer(m: MixerSpec, p: str, src: WeightSource, cfg: ModelConfig, dtype
     return mx
 
 
+def _build_latent(mx: Mixer, m: MixerSpec, p: str, src: WeightSource, cfg: ModelConfig, dtype: torch.dtype) -> latent.LatentParams:
+    D, H, d, dp, rd, rp, R, Rp, dv, dvp = (cfg.hidden_size, m.heads, m.dim, m.dim_p, m.rot_dim, m.rot_p, m.kv_rank, m.rank_p, m.vdim,
+                                           m.vdim_p)
+    step = K_ALIGN if dtype == torch.bfloat16 else 8
+
+    def gain(name, n):
+        return torch.nn.functional.pad(src.get(p + name, (n,), "norm").float(), (0, pad_to(n, 8) - n)).contiguous()
+    mx.parts = [("dq", src.get(p + "dq", (m.q_rank, D)))]
+    own = m.kv_from < 0
+    if own:
+        dkv = src.get(p + "dkv", (R + rd, D))
+        mx.parts += [("c", dkv[:R]), ("r", dkv[R:])]
+    uq = src.get(p + "uq", (H * (d + rd), m.q_rank)).view(H, d + rd, m.q_rank)
+    heads = uq.new_zeros(H, rp + dp, m.q_rank)                     # [rotated | rest]
+    heads[:, :rd], heads[:, rp:rp + d] = uq[:, d:], uq[:, :d]
+    uk = src.get(p + "uk", (H * d, R)).view(H, d, R)
+    uv = src.get(p + "uv", (H * dv, R)).view(H, dv, R)
+    w_uk = uk.new_zeros(H, Rp, pad_to(dp, step))
+    w_uk[:, :R, :d] = uk.transpose(1, 2)
+    w_uv = uv.new_zeros(H, dvp, pad_to(Rp, step))
+    w_uv[:, :dv, :R] = uv
+    w_up = None
+    if dtype == torch.bfloat16:
+        keys, values = (uk.new_zeros(H, n, pad_to(Rp + rp, step)) for n in (rp + dp, dvp))
+        keys[:, torch.arange(rd), Rp + torch.arange(rd)] = 1.0      # the rotated part passes through, to every head
+        keys[:, rp:rp + d, :R], values[:, :dv, :R] = uk, uv
+        w_up = torch.cat([keys.flatten(0, 1), values.flatten(0, 1)]).to(dtype).contiguous()
+    return latent.LatentParams(
+        heads=H, dim_p=dp, rot_dim=rd, rot_p=rp, rank=R, rank_p=Rp, vdim_p=dvp, q_rank=m.q_rank, scale=m.scale, eps=cfg.rms_eps,
+        window=m.window, sinks=src.get(p + "sink", (H,), "bias").float().contiguous(), q_norm=gain("dq.norm", m.q_rank),
+        c_norm=gain("dkv.norm", R) if own else None, w_uq=pad_cols(heads.flatten(0, 1).to(dtype), pad_to(m.q_rank, K_ALIGN)).contiguous(),
+        w_uk=w_uk.to(dtype).contiguous(), w_uv=w_uv.to(dtype).contiguous(), w_up=w_up)
+
+
 def mixer_tensor_specs(m: MixerSpec, p: str, D: int, layer: int) -> List[Tuple[str, Tuple[int, ...], str, int]]:
     """(name, shape, init kind, layer) of a mixer's checkpoint tensors."""
     qk, kv, n, H = m.heads * m.dim, m.qk_heads * m.dim, m.heads * m.vdim, m.heads
@@ -232,8 +326,20 @@ def mixer_tensor_specs(m: MixerSpec, p: str, D: int, layer: int) -> List[Tuple[s
         out = [("q", (qk, D), "normal"), ("k", (kv, D), "normal"), ("v", (m.kv_heads * m.vdim, D), "normal")]
         out += [("talk", (H, H), "normal")] if m.talking else []
         out += [("g", (H, D), "normal")] if m.out_gate else []
-        out += [("q.b", (qk,), "bias"), ("k.b", (kv,), "bias"), ("v.b", (m.kv_heads * m.vdim,), "bias"), ("o.b", (D,), "bias")] if m.bias else []
+        out += [("g", (n, D), "normal")] if m.out_gate_all else []
+        out += [("q.b", (qk,), "bias"), ("k.b", (kv,), "bias"), ("v.b", (m.kv_heads * m.vdim,), "bias")] if m.bias else []
+        out += [("o.b", (D,), "bias")] if m.out_bias else []
         out += [("q.norm", (m.dim,), "norm"), ("k.norm", (m.dim,), "norm")] if m.qk_norm else []
+        out += [("q.norm", (qk,), "norm"), ("k.norm", (kv,), "norm")] if m.qk_norm_all else []
+        out += [("sink", (H,), "bias")] if m.head_sinks else []
+    elif m.kind == "latent_attention":
+        out = [("dq", (m.q_rank, D), "normal"), ("dq.norm", (m.q_rank,), "norm"), ("uq", (H * (m.dim + m.rot_dim), m.q_rank), "normal"),
+               ("uk", (qk, m.kv_rank), "normal"), ("uv", (n, m.kv_rank), "normal"), ("sink", (H,), "bias")]
+        if m.kv_from < 0:
+            out += [("dkv", (m.kv_rank + m.rot_dim, D), "normal"), ("dkv.norm", (m.kv_rank,), "norm")]
+    elif m.kind == "hgrn2":
+        out = [("q", (qk, D), "normal"), ("f", (qk, D), "normal"), ("f.b", (qk,), "bias"), ("lower", (qk,), "lower"), ("v", (n, D), "normal"),
+               ("norm", (m.vdim,), "norm")]
     elif m.kind == "general_delta":
         out = [(x, (qk, D), "normal") for x in ("r", "k", "v", "g", "a")]
         out += [("w1", (m.decay_rank, D), "normal"), ("w2", (qk, m.decay_rank), "normal"), ("a.b", (qk,), "bias"),

@@ -95,6 +95,8 @@ class WeightSource:
             return 1.0 + 0.1 * t
         if kind == "bias":
             return 0.1 * t
+        if kind in ("lower", "shift"):     # between 0 and 1
+            return torch.sigmoid(t)
         if kind == "mix":             # square, close to the identity
             return torch.eye(shape[0], device=self.device) + 0.1 * t
         return t * self.std

@@ -70,7 +70,7 @@ def weight_bytes_per_rank(cfg: ModelConfig, tp: int, ep: int, sequence_parallel:
     """-> (non-expert bytes, routed-expert bytes resident on the GPU) for one rank."""
     H = cfg.hidden_size
     if cfg.is_layered:
-        experts = sum(3 * H * s.mlp.ff * s.mlp.experts * 2 for s in cfg.layer_specs if s.weights_of < 0)
+        experts = sum((2 if s.mlp.activation == "relu2" else 3) * H * s.mlp.ff * s.mlp.experts * 2 for s in cfg.layer_specs if s.weights_of < 0)
         return int(cfg.param_count() * 2 - experts), int(experts)
     qb = _quant_bytes(cfg)
     lin = 1.0 + 4.0 / (128 * 128) if cfg.quant != "none" else 2.0     # attention / dense linears are FP8 or bf16
