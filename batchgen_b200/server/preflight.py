@@ -156,14 +156,19 @@ def _layered_contract(cfg, world: int, on_gpu: bool) -> List[str]:
         for m in s.mixers:
             if m.recurrent and m.dim > 512:
                 bad.append(f"layer {i}: {m.kind} head width {m.dim} exceeds 512")
-            if not m.recurrent and m.kv_heads * -(-(m.heads // m.kv_heads) // 4) * (m.vdim_p // 4) > 2048:
+            if m.kind == "attention" and m.kv_heads * -(-(m.heads // m.kv_heads) // 4) * (m.vdim_p // 4) > 2048:
                 bad.append(f"layer {i}: {m.heads} heads x {m.vdim} value channels exceed the decode attention kernel")
         if f.kind == "moe" and (f.top > 16 or f.experts > 1024 or f.top > f.experts):
             bad.append(f"layer {i}: top {f.top} of {f.experts} experts (the router takes up to 16 of 1,024)")
         if f.kind == "moe" and f.groups > 32:
             bad.append(f"layer {i}: {f.groups} groups of experts (the router takes up to 32)")
-        if any(not m.recurrent and (m.bias or m.qk_norm or m.rot_interleaved) and max(m.dim_p, m.vdim_p) > 1024 for m in s.mixers):
+        if any(m.kind == "attention" and (m.bias or m.qk_norm or m.rot_interleaved) and max(m.dim_p, m.vdim_p) > 1024 for m in s.mixers):
             bad.append(f"layer {i}: attention head widths {s.mixer.dim}, {s.mixer.vdim} exceed 1024")
+        for m in s.mixers:
+            if m.latent and m.rank_p + m.rot_p > 1536:
+                bad.append(f"layer {i}: latent rows of {m.rank_p + m.rot_p} numbers exceed the decode attention kernel's 1536")
+            if m.qk_norm_all and m.heads * m.dim_p + m.kv_row > 32768:
+                bad.append(f"layer {i}: {m.heads} heads of {m.dim} exceed one norm over all of them (32,768 columns of a token)")
     if bad:
         raise PreflightError("model contract: " + "; ".join(bad))
     if not on_gpu:
