@@ -100,8 +100,8 @@ class HeadPrep:
     bias: Optional[torch.Tensor] = None      # [heads * dim_p + kv_row], columns as projected: queries, keys, values
     q_norm: Optional[torch.Tensor] = None    # [dim_p] gains of the RMS norms of query and key heads, or with ``whole`` [heads * dim_p]
     k_norm: Optional[torch.Tensor] = None
-    whole: bool = False                      # one norm over all query heads of a token, one over all key heads
     interleaved: bool = False                # rotary pairs (2 i, 2 i + 1), else (i, i + dims / 2)
+    whole: bool = False                      # one norm over all query heads of a token, one over all key heads
 
 
 def prepare_heads(z: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, p: TalkParams, h: HeadPrep,

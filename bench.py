@@ -402,8 +402,8 @@ def main() -> int:
     ap.add_argument("--bct", action="store_true", help="also run the 512-request workload through the batch API")
     ap.add_argument("--bct-requests", type=int, default=512)
     ap.add_argument("--bct-tokens", type=int, default=1024)
-    ap.add_argument("--workload", default="decode", choices=["decode", "distinct64k", "grouped64k", "streamed", "nanurax", "pamevik", "bolisun"],
-                    help="decode: the headline decode-step benchmark; nanurax, pamevik, bolisun: a layer-listed design beside its "
+    ap.add_argument("--workload", default="decode", choices=["decode", "distinct64k", "grouped64k", "streamed", "nanurax", "pamevik", "bolisun", "pitudra"],
+                    help="decode: the headline decode-step benchmark; nanurax, pamevik, bolisun, pitudra: a layer-listed design beside its "
                          "closest existing model (benchmarks/design_bench.py); the others: long-context DSA workloads "
                          "(use with --model glm-5.3-fp8)")
     ap.add_argument("--requests", type=int, default=2, help="requests of a long-context workload")
@@ -417,7 +417,7 @@ def main() -> int:
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
-    if args.workload in ("nanurax", "pamevik", "bolisun"):
+    if args.workload in ("nanurax", "pamevik", "bolisun", "pitudra"):
         from benchmarks import design_bench
         return design_bench.run(args, ROOT, args.workload)
     if args.workload == "streamed":

@@ -1,18 +1,18 @@
-"""Layer-listed models (Nanurax, Pamevik, Bolisun) beside the framework's closest existing model at equal size.
+"""Layer-listed models (Nanurax, Pamevik, Bolisun, Pitudra) beside the framework's closest existing model at equal size.
 
-``bench.py --workload nanurax | pamevik | bolisun``: both models have four layers of a real model's size (width 2304, 32 heads of 128,
+``bench.py --workload nanurax | pamevik | bolisun | pitudra``: both models have four layers of a real model's size (width 2304, 32 heads of 128,
 bf16), three recurrent layers to one attention layer.  Nanurax runs the generalised delta rule and chunked talking-heads
 attention with one dense and three mixture feed-forwards (64 experts of which 8 run); Pamevik runs two channel-delta layers, an
 mLSTM layer and attention beside retention, with dense feed-forwards.  The other one is a Kimi-Linear cut with KDA and MLA
 layers and the same kinds of feed-forwards.  Bolisun runs four layers of windowed attention beside retention, with one dense and
 three mixture feed-forwards; next to the Kimi-Linear cut (mixtures of the same size) it has Pamevik with four layers of attention
-beside retention, whose dense feed-forwards hold as many weights as a token's experts.  Prefill is one packed forward over fresh prompts, decode is a captured step over
+beside retention, whose dense feed-forwards hold as many weights as a token's experts.  Pitudra runs two HGRN2 layers, one of windowed
+and one of latent attention, with four mixtures, next to a Kimi-Linear cut with four mixtures of as many weights.  Prefill is one packed forward over fresh prompts, decode is a captured step over
 sequences with cached context; random weights, CUDA events, medians, the L2 flushed before every timed call.
 
 ``kernels`` of the result times the new kernels beside their likes (recurrences against KDA, decode attention against the
-paged GQA kernel, prompt attention against the expanded MLA kernel, norms against the fused residual norm; Bolisun's against
-Pamevik's and Nanurax's) with the share of
-the measured roofline each reaches.
+paged GQA kernel, prompt attention against the expanded MLA kernel, norms against the fused residual norm, latent attention against the MLA kernels; Bolisun's and Pitudra's others against
+those of the designs before them) with the share of the measured roofline each reaches.
 """
 from __future__ import annotations
 
@@ -61,6 +61,8 @@ def _closest(design: str):
     import dataclasses
     from batchgen_b200.config import get_model_config
     mlp = dict(first_k_dense=4) if design == "pamevik" else dict(n_routed_experts=64, num_experts_per_tok=8)
+    if design == "pitudra":
+        mlp.update(first_k_dense=0, n_shared_experts=0)
     out = [get_model_config("kimi-linear-48b", num_layers=4, kda_layers=(0, 1, 2), **mlp)]
     if design == "bolisun":
         cfg = get_model_config("pamevik-bench")
@@ -367,6 +369,140 @@ def _bolisun_kernels(dev, timer: _Timer, peaks) -> List[Dict[str, object]]:
     return add.rows
 
 
+def _pitudra_kernels(dev, timer: _Timer, peaks) -> List[Dict[str, object]]:
+    import torch
+    from batchgen_b200.config import get_model_config
+    from batchgen_b200.models import mixers
+    from batchgen_b200.models.weights import WeightSource
+    from batchgen_b200.ops import attention, conv, gemm, latent, moe, recurrent, residual, talking
+    bf, add = torch.bfloat16, _Rows(peaks)
+    cfg = get_model_config("pitudra-bench")
+    att, W, E, K, side = cfg.layer_specs[1].mixer, 2304, 64, 8, cfg.side_dim
+    row, win = att.kv_row, att.window
+    near = talking.TalkParams(H, G, D, D, D ** -0.5, window=win, sinks=torch.zeros(H, device=dev), gate_all=True)
+    plain = talking.TalkParams(H, G, D, D, D ** -0.5, window=win)
+    whole = talking.HeadPrep(D, 1e-6, torch.zeros(HD + row, device=dev), torch.ones(HD, device=dev), torch.ones(G * D, device=dev), whole=True)
+    single = talking.HeadPrep(D, 1e-6, torch.zeros(HD + row, device=dev), torch.ones(D, device=dev), torch.ones(D, device=dev), True)
+    mx = mixers.build_mixer(cfg.layer_specs[3].mixer, "mix.", WeightSource(seed=1, device=dev, gen_device=dev), cfg, bf)
+    lat = mx.lat
+    gains = residual.Norm(torch.ones(W, device=dev), torch.zeros(W, device=dev), True)
+    for B, T in STATE_CASES:
+        R, size, slots, cu, init = _state_case(dev, B, T)
+        prompt = T > 1
+        row_seq = torch.arange(B, dtype=torch.int32, device=dev).repeat_interleave(T) if prompt else None
+        z, out = torch.randn(R, 4 * HD, device=dev), torch.empty(R, HD, dtype=bf, device=dev)
+        S = torch.zeros(B + 1, HD * D, device=dev)
+        q, k, v, g = (z[:, i * HD:(i + 1) * HD] for i in range(4))
+        base = dict(heads=H, dim_p=D, vdim=D, vdim_p=D, norm_w=torch.ones(HD, device=dev), eps=1e-6)
+        p = recurrent.RecurrentParams("hgrn2", **base, f_bias=torch.zeros(HD, device=dev), f_lower=torch.full((HD,), 0.5, device=dev))
+        ms = timer(lambda: recurrent.recurrent_forward(p, q, k, v, None, {"S": S}, slots, out, cu, None, init))
+        add("HGRN2", size, ms, (R * HD * 14 + B * HD * D * 8) / 1e9)
+        p = recurrent.RecurrentParams("retention", **base, gate="silu", decay=torch.full((H,), 0.99, device=dev))
+        ms = timer(lambda: recurrent.recurrent_forward(p, q, k, v, g, {"S": S}, slots, out, cu, None, init))
+        add("  retention", size, ms, (R * HD * 18 + B * HD * D * 8) / 1e9)
+        _kda_row(dev, timer, add, B, T)
+        n = -(-R // PAGE)
+        cache, at = torch.zeros(n, PAGE, row, dtype=bf, device=dev), torch.arange(R, device=dev)
+        tab = conv.Rotary.make(D, 1e6, dev).table(torch.arange(1, R + 1, dtype=torch.int32, device=dev))
+        gb = R * (HD + row) * 4 / 1e9 + R * (row * 2 + HD * (2 if prompt else 4)) / 1e9
+        add("heads: bias, norm over all, cache", size, timer(lambda: talking.prepare_heads(z, at, cache, near, whole, None, not prompt, prompt)), gb)
+        ms = timer(lambda: talking.prepare_heads(z, at, cache, plain, single, tab, not prompt, prompt))
+        add("  heads: bias, norm each, rotation, cache", size, ms, gb + R * D * 4 / 1e9)
+        rope, rows = mixers.conv.Rotary.make(64, 1e6, dev).table(torch.arange(1, R + 1, dtype=torch.int32, device=dev)), torch.zeros(n, PAGE, 576, dtype=bf, device=dev)
+        ms = timer(lambda: latent.prepare(z, (0, 1536, 2048), at, rows, lat, rope, bf))
+        add("latents: norms, rotation, cache", size, ms, R * 2112 * 6 / 1e9)
+        x, a = torch.randn(R, W, device=dev), torch.randn(R, W, device=dev)
+        w2 = torch.rand(2, W, device=dev)
+        hist, y = torch.zeros(B + 1, W, device=dev), torch.empty(R, W, dtype=bf, device=dev)
+
+        def shift():
+            if not prompt:
+                return residual.sandwich_norm(x, None, 1e-6, W, W, bf, add=a, post=gains, canon=residual.Canon(w2, hist, slots))
+            residual.sandwich_norm(x, None, 1e-6, W, W, bf, add=a, post=gains, emit=False)
+            return conv.causal_conv(x, w2, hist, slots, y, "residual", cu, None, row_seq, init)
+        add("norm of the output + token shift", size, timer(shift), (R * W * (4 * 3 + 2) + B * W * 8) / 1e9)
+        add("norm of the output", size, timer(lambda: residual.sandwich_norm(x, None, 1e-6, W, W, bf, add=a, post=gains)), R * W * 14 / 1e9)
+        routed = torch.randn(R * K, W, device=dev)
+        pos = torch.randperm(R * K, device=dev).to(torch.int32).view(R, K).contiguous()
+        rw = torch.rand(R, K, device=dev)
+        ms = timer(lambda: residual.sandwich_norm(x, None, 1e-6, W, W, bf, routed=routed, pos=pos, route_w=rw, post=gains))
+        add("norm of the experts' sum", size, ms, R * W * (4 * (2 + K) + 2) / 1e9)
+        ms = timer(lambda: residual.sandwich_norm(x, gains, 1e-6, W, W, bf, add=a, post=gains))
+        add("  norms of a sandwich block", size, ms, R * W * (4 * 3 + 2) / 1e9)
+        ms = timer(lambda: residual.residual_norm(x, gains.w, 1e-6, W, W, bf, add=a, routed=routed, pos=pos))
+        add("  residual + norm + experts' rows", size, ms, R * W * (4 * (3 + K) + 2) / 1e9)
+        zs, table, ids = torch.randn(R, side, device=dev), torch.randn(9999, 4 * side, device=dev, dtype=bf), torch.randint(0, 9999, (R,), device=dev).to(torch.int32)
+        add("token side input", size, timer(lambda: residual.token_side(zs, table[:, side:2 * side], ids, side, bf)), R * side * 8 / 1e9)
+        logits = torch.randn(R, E, device=dev)
+        idx, rw = moe.router_topk(logits, None, K, scoring="softmax")
+        h = torch.randn(R, W, device=dev).to(bf)
+        for name, kind, ff in (("experts", "relu2", 1536), ("  experts, gated", "silu", 1024)):
+            w13 = torch.randn(E, ff if kind == "relu2" else 2 * ff, W, device=dev, dtype=bf) * 0.02
+            ew = moe.ExpertWeights(w13, torch.randn(E, W, ff, device=dev, dtype=bf) * 0.02, activation=kind)
+            flops = 2 * W * ff * (2 if kind == "relu2" else 3)
+            add(name, size, timer(lambda: moe.routed_rows(h, idx, rw, ew, False)), E * flops / 1e9 + R * K * W * 4 / 1e9, R * K * flops / 1e12)
+            del w13, ew
+        del x, a, routed, z
+    for B, ctx in ((16, 4096), (64, 4096), (256, 4096)):
+        n = B * ctx // PAGE
+        cache = torch.randn(n, PAGE, row, device=dev).bfloat16()
+        bt = torch.randperm(n, device=dev).to(torch.int32).view(B, -1).contiguous()
+        lens = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+        q, gate, out = torch.randn(B, HD, device=dev), torch.randn(B, HD, device=dev), torch.empty(B, HD, dtype=bf, device=dev)
+        for name, p, more in (("attention, decode, window, sinks, gates", near, dict(gate=gate)), ("  attention, decode, window", plain, {})):
+            add(name, f"{B} x {win} of {ctx} keys", timer(lambda: talking.attend_rows(q, p, cache, bt, lens, out, **more)), B * win * row * 2 / 1e9)
+        del cache
+    for B, ctx in ((16, 2048), (64, 2048), (256, 2048), (16, 4096), (64, 4096)):
+        n = B * ctx // PAGE
+        cache = torch.randn(n, PAGE, 576, device=dev).bfloat16()
+        bt = torch.randperm(n, device=dev).to(torch.int32).view(B, -1).contiguous()
+        lens = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+        qa = torch.randn(B, H, 576, device=dev).bfloat16()
+        gb, tf = B * ctx * 576 * 2 / 1e9, B * ctx * H * 1088 * 2 / 1e12
+        add("latent attention, decode", f"{B} x {ctx} keys", timer(lambda: latent.attend(qa, lat, cache, bt, lens)), gb, tf)
+        ms = timer(lambda: attention.mla_decode(qa[..., :512], qa[..., 512:], cache, bt, lens, lat.scale, 512))
+        add("  MLA decode", f"{B} x {ctx} keys", ms, gb, tf)
+        del cache
+    for B in (16, 64, 256):
+        q = torch.randn(B, H * 192, device=dev)
+        rope = mx.rot.table(torch.arange(1, B + 1, dtype=torch.int32, device=dev))
+        add("latent queries", f"{B} tokens", timer(lambda: latent.queries(q, lat, rope, None, bf)), (B * H * (192 * 4 + 576 * 2) + H * 128 * 512 * 2) / 1e9)
+    for B, T in ((1, 4096), (8, 1024), (1, 16384)):
+        n, R = T // PAGE, B * T
+        cu = list(range(0, R + 1, T))
+        cache = torch.randn(B * n, PAGE, row, device=dev).bfloat16()
+        bt = torch.arange(B * n, device=dev, dtype=torch.int32).view(B, n).contiguous()
+        qf = torch.randn(R, H, D, device=dev).bfloat16()
+        q, gate, out = torch.randn(R, HD, device=dev), torch.randn(R, HD, device=dev), torch.empty(R, HD, dtype=bf, device=dev)
+        blocks = talking.work_blocks(talking.prefill_work(cu, [0] * B, 0, 1, win), R, dev)
+        tf = B * sum(near.most_keys(t) for t in range(1, T + 1)) * 4 * H * D / 1e12
+        for name, p, more in (("attention, prompt, window, sinks, gates", near, dict(gate=gate)), ("  attention, prompt, window", plain, {})):
+            add(name, f"{B} x {T} tokens", timer(lambda: talking.attend_prefill(q, p, cache, bt, out, blocks, operand=qf, **more)), 0, tf)
+        # whole latents' prompt path; then its attention alone, and the expanded MLA kernel on the same keys and values
+        cache = torch.randn(B * n, PAGE, 576, device=dev).bfloat16()
+        ql = torch.randn(R, H * 192, device=dev)
+        rope = mx.rot.table(torch.arange(1, T + 1, dtype=torch.int32, device=dev).repeat(B))
+        groups = latent.expansions(cu, [0] * B, lat.window, PAGE, dev)
+        seen = B * sum(min(t, lat.window) for t in range(1, T + 1))
+        add("latents: expansion and attention, prompt", f"{B} x {T} tokens", timer(lambda: latent.attend_prompt(ql, lat, cache, bt, rope, out, groups)), 0,
+            (seen * 2 * H * 320 + R * 2 * 512 * H * 256) / 1e12)
+        e = lat.expanded
+        up = torch.randn(B * n, PAGE, e.kv_row, device=dev).bfloat16()
+        add("latents: attention, prompt", f"{B} x {T} tokens",
+            timer(lambda: [talking.attend_prefill(ql, e, up, x.table, out, x.blocks, rope=rope) for x in groups]), 0, seen * 2 * H * 320 / 1e12)
+        q3, kv = torch.randn(R, H, 192, device=dev).bfloat16(), torch.randn(R, H, 256, device=dev).bfloat16()
+        kpe = torch.randn(R, 64, device=dev).bfloat16()
+        work = attention.mha_prefill_work(cu, [0] * B, cu[:-1]).to(dev)
+        add("  expanded MLA prompt", f"{B} x {T} tokens", timer(lambda: attention.mha_prefill(q3, kv, kpe, work, 0.07)), 0,
+            B * T * (T + 1) / 2 * 2 * H * 320 / 1e12)
+        c, wk = torch.randn(R, 512, device=dev).bfloat16(), torch.randn(H * 256, 512, device=dev).bfloat16()
+        cw = torch.randn(R, 576, device=dev).bfloat16()
+        add("latents: expansion product", f"{R} rows", timer(lambda: gemm.bf16_gemm(cw, lat.w_up)), 0, R * 2 * 512 * H * 256 / 1e12)
+        add("  MLA expansion product", f"{R} rows", timer(lambda: gemm.bf16_gemm(c, wk)), 0, R * 2 * 512 * H * 256 / 1e12)
+        del cache, q, qf, up, ql
+    return add.rows
+
+
 def run(args, root: str, design: str) -> int:
     import torch
     from batchgen_b200.config import get_model_config
@@ -383,7 +519,7 @@ def run(args, root: str, design: str) -> int:
     models = {}
     for cfg in (get_model_config(f"{design}-bench"), *_closest(design)):
         models[cfg.name] = _model_rates(cfg, dev, timer)
-    kernels = {"nanurax": _nanurax_kernels, "pamevik": _pamevik_kernels, "bolisun": _bolisun_kernels}[design](dev, timer, peaks)
+    kernels = {"nanurax": _nanurax_kernels, "pamevik": _pamevik_kernels, "bolisun": _bolisun_kernels, "pitudra": _pitudra_kernels}[design](dev, timer, peaks)
     _ext.check_status()
     step = models[f"{design}-bench"]["decode"][1]
     print(json.dumps({
