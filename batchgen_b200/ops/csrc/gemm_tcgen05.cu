@@ -37,6 +37,7 @@ constexpr int KIND_FP8 = 0;
 constexpr int KIND_BF16 = 1;
 constexpr int EPI_STORE = 0;
 constexpr int EPI_SILU_MUL = 1;  // B rows interleaved (32 gate, 32 up): out = silu(gate) * up
+constexpr int EPI_RELU2 = 3;      // square of the positive part, stored like EPI_STORE
 constexpr int EPI_STORE_F32 = 2;  // fp32 output (router logits): D is float*, ldd in floats
 
 struct GemmParams {
@@ -454,6 +455,13 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
             }
           }
         } else if (p.peer_out[0] == nullptr) {
+          if (EPI == EPI_RELU2) {
+#pragma unroll
+            for (int j = 0; j < 64; ++j) {
+              const float a = fmaxf(r[j], 0.f);
+              r[j] = a * a;
+            }
+          }
           const int col0 = t.nt * BN + half * 64;
           __nv_bfloat16* dst = out_base + out_row * p.ldd + col0;
 #pragma unroll
@@ -677,7 +685,7 @@ int bg_gemm_set_splitk_ws(float* ws, long long max_items, int* counters, int max
 void bg_gemm_set_counts(const int* counts) { g_counts = counts; }
 
 // Dense or grouped GEMM.  kind: 0 = e4m3 block scaled, 1 = bf16.  epi: 0 = store, 1 = silu-mul
-// (weight rows interleaved in 32-row gate/up blocks; output has N/2 columns).
+// (weight rows interleaved in 32-row gate/up blocks; output has N/2 columns), 2 = fp32 store, 3 = squared ReLU (bf16 operands).
 // offsets == nullptr -> dense [M, K] x [N, K]^T.  Otherwise A holds `groups` row segments
 // (128-aligned starts, offsets[groups] <= M) and B is [groups * N, K].
 // K must be a multiple of 128 elements (fp8) / 64 (bf16).  Returns 0 on a successful launch.
@@ -714,6 +722,7 @@ int bg_gemm(int kind, int epi, const void* A, const float* sA, int sa_stride, co
   if (kind == KIND_FP8 && epi == EPI_SILU_MUL) return launch_gemm<KIND_FP8, EPI_SILU_MUL>(A, B, p, M, b_rows, num_sms, stream);
   if (kind == KIND_BF16 && epi == EPI_STORE) return launch_gemm<KIND_BF16, EPI_STORE>(A, B, p, M, b_rows, num_sms, stream);
   if (kind == KIND_BF16 && epi == EPI_SILU_MUL) return launch_gemm<KIND_BF16, EPI_SILU_MUL>(A, B, p, M, b_rows, num_sms, stream);
+  if (kind == KIND_BF16 && epi == EPI_RELU2) return launch_gemm<KIND_BF16, EPI_RELU2>(A, B, p, M, b_rows, num_sms, stream);
   if (kind == KIND_BF16 && epi == EPI_STORE_F32) return launch_gemm<KIND_BF16, EPI_STORE_F32>(A, B, p, M, b_rows, num_sms, stream);
   return -2;
 }

@@ -51,6 +51,7 @@ struct Params {
   const float* gate;             // [T, ld_gate] or null: out[h] *= sigmoid(gate[h]), or per element
   int ld_gate, gate_cols;        // columns of a head: 1 or dvp
   const float* sinks;            // [H] scores of the sink, or null: zero
+  int staged;                    // gates per element: rows leave through shared memory, a warp a row at a time
   int row_shift;                 // rows of Q = rows of out - row_shift
   int smem_bytes;
   int* status;
@@ -343,8 +344,43 @@ attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CU
       const bool each = gate != nullptr && p.gate_cols > 1;
       if (gate != nullptr && !each && live) inv *= 1.0f / (1.0f + expf(-gate[0]));
       __nv_bfloat16* orow = p.out + (size_t)(w.q_row0 + r) * p.ldo + h * p.dvp;
+      if (p.staged) {                                          // the tiles are done with: their memory takes fp32 rows of this warp
+        const int W = p.VB * 64;                               // row r: 16-byte chunks c at c ^ (r & 7)
+        float* stage = reinterpret_cast<float*>(smem);
 #pragma unroll 1
-      for (int c = 0; c < p.VB * 2; ++c) {
+        for (int c = 0; c < p.VB * 2; ++c) {
+          uint32_t ov[32];
+          tmem_ld_32x32(tm_o + c * 32, ov);
+          tmem_ld_wait();
+#pragma unroll
+          for (int j = 0; j < 8; ++j)
+            *reinterpret_cast<float4*>(stage + r * W + (((c * 8 + j) ^ (r & 7)) << 2)) =
+                make_float4(__uint_as_float(ov[4 * j]) * inv, __uint_as_float(ov[4 * j + 1]) * inv, __uint_as_float(ov[4 * j + 2]) * inv,
+                            __uint_as_float(ov[4 * j + 3]) * inv);
+        }
+        __syncwarp();
+        const int rows = min(32, w.n_q - quad * 32), c4 = p.dvp / 4;
+        const size_t row0 = (size_t)w.q_row0 + quad * 32;
+        for (int ch = lane; ch < c4; ch += 32) {
+          for (int i0 = 0; i0 < rows; i0 += 8) {               // eight rows' gates in flight
+            float4 g[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+              g[i] = *reinterpret_cast<const float4*>(p.gate + (row0 + min(i0 + i, rows - 1)) * p.ld_gate + h * p.dvp + ch * 4);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+              if (i0 + i >= rows) break;
+              const int sr = quad * 32 + i0 + i;
+              const float4 o = *reinterpret_cast<const float4*>(stage + sr * W + ((ch ^ (sr & 7)) << 2));
+              __align__(8) __nv_bfloat162 y[2] = {__floats2bfloat162_rn(o.x / (1.0f + expf(-g[i].x)), o.y / (1.0f + expf(-g[i].y))),
+                                                  __floats2bfloat162_rn(o.z / (1.0f + expf(-g[i].z)), o.w / (1.0f + expf(-g[i].w)))};
+              *reinterpret_cast<uint2*>(p.out + (row0 + i0 + i) * p.ldo + h * p.dvp + ch * 4) = *reinterpret_cast<const uint2*>(y);
+            }
+          }
+        }
+      }
+#pragma unroll 1
+      for (int c = 0; c < (p.staged ? 0 : p.VB * 2); ++c) {
         uint32_t ov[32];
         tmem_ld_32x32(tm_o + c * 32, ov);
         tmem_ld_wait();
@@ -494,6 +530,7 @@ int bg_gqa_prompt(const void* qf, const void* cache, long long page_stride, int 
   const int room = (two ? kSmemTwo : 226 * 1024) - (int)sizeof(Shared);
   p.stages = 2;
   while (p.stages < kMaxStages && tile_bytes(p.KB, p.VB, p.stages + 1) <= room) ++p.stages;
+  p.staged = gate != nullptr && gate_cols > 1 && tile_bytes(p.KB, p.VB, p.stages) >= BM * p.VB * 256;
   p.tmem_cols = two ? 256 : 512;
   p.smem_bytes = two ? kSmemTwo : 227 * 1024;
   static bg::DeviceOnce once;

@@ -4,34 +4,43 @@
 //
 //   s[h, j] = scale * qb[h, :] . row_j      o[h] = sum_j softmax(s)[h, j] row_j[0 : dvp]
 //
-// Tiles of 32 keys come through a cp.async ring.  Eight warps share a tile: for the scores a warp takes a quarter of the channels
-// and half of the keys (its queries stay in registers, every key byte is read from shared memory once per 16 heads' products), the
-// quarters meet in shared memory, eight threads a head take the online softmax, and for the values a warp owns an eighth of the
-// columns.  The scores of tile t + 1 and the values of tile t are multiplied between the same two barriers.  A handful of heads
-// per row would leave most of a 128-row tcgen05 shape idle, so the products are mma m16n8k16.
+// Tiles of 32 keys come through a ring of bulk copies, a cached row each (rows lie 16 bytes further apart in shared memory, so that
+// fragments hit different banks).  Sixteen warps share a tile: for the scores a warp takes an eighth of the channels and half of the
+// keys (its queries stay in registers, every key byte is read from shared memory once for all heads), the eighths meet in shared
+// memory, sixteen threads a head take the online softmax, and for the values a warp owns a sixteenth of the columns.  The scores of
+// tile t + 1 and the values of tile t are multiplied between the same two barriers.  A few dozen heads would leave most of a 128-row
+// tcgen05 shape idle, so the products are mma m16n8k16.
 #pragma once
 
 namespace bg {
 namespace talk {
 namespace latent {
 
-constexpr int kWarpsL = 8, kTileL = 32, kStagesL = 4;
+constexpr int kWarpsL = 16, kTileL = 32, kStagesL = 4;
+constexpr int kParts = kWarpsL / 2;             // shares of the channels
 constexpr int kPartRow = kTileL + 8;            // floats of a head's partial scores: rows of a fragment hit different banks
 constexpr int kProbBytes = kTileL * 2 + 16;     // bytes of a head's probabilities
 
 __host__ __device__ inline int row_bytes(int row) { return (row + 15) / 16 * 32 + 16; }
 __host__ __device__ inline int ring_bytes(int row) { return kStagesL * kTileL * row_bytes(row); }
 __host__ __device__ inline int shared_bytes(int row, int mt) {
-  return ring_bytes(row) + 16 * mt * (4 * kPartRow * 4 + kProbBytes + 4 + 8);
+  return ring_bytes(row) + 16 * mt * (kParts * kPartRow * 4 + kProbBytes + 4 + 8);
 }
 
-// MT: 16-head tiles; KQ: upper bound of the 16-wide steps in a quarter of the channels; NV: 8-wide value tiles of a warp (even)
+__device__ __forceinline__ void bulk_row(uint32_t dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes),
+               "r"(smem_u32(bar))
+               : "memory");
+}
+
+// MT: 16-head tiles; KQ: upper bound of the 16-wide steps in a share of the channels; NV: 8-wide value tiles of a warp (even)
 template <int MT, int KQ, int NV>
 __global__ void __launch_bounds__(kWarpsL * 32, 1) latent_rows_kernel(const Params p) {
   bg::pdl_prologue((BG_FILE_TAG << 16) | __LINE__);
   extern __shared__ __align__(16) char sm_raw[];
-  using plain::cp16_or_zero;
-  using plain::cp_wait;
+  __shared__ uint64_t full[kStagesL];
+  __shared__ int abort_s;
+  volatile int* abort_flag = &abort_s;
   using plain::ldsm4;
   using plain::ldsm4t;
   using plain::mma16816;
@@ -46,8 +55,8 @@ __global__ void __launch_bounds__(kWarpsL * 32, 1) latent_rows_kernel(const Para
     return;                                                        // (a split row without a query is zeroed by the merge)
   }
   char* ring = sm_raw;
-  float* part = reinterpret_cast<float*>(sm_raw + ring_bytes(row));                    // [4][16 MT][kPartRow]
-  char* prob = reinterpret_cast<char*>(part + 4 * 16 * MT * kPartRow);                 // [16 MT] rows of kProbBytes
+  float* part = reinterpret_cast<float*>(sm_raw + ring_bytes(row));                    // [kParts][16 MT][kPartRow]
+  char* prob = reinterpret_cast<char*>(part + kParts * 16 * MT * kPartRow);                 // [16 MT] rows of kProbBytes
   float* alpha = reinterpret_cast<float*>(prob + 16 * MT * kProbBytes);                // [16 MT]
   float2* ml = reinterpret_cast<float2*>(alpha + 16 * MT);                             // [16 MT] maximum, sum
   const uint32_t ring_u = smem_u32(ring), prob_u = smem_u32(prob);
@@ -58,29 +67,32 @@ __global__ void __launch_bounds__(kWarpsL * 32, 1) latent_rows_kernel(const Para
   const int n = my_hi - my_lo;
   const int* bt = p.block_table + (size_t)(p.row_seq != nullptr ? p.row_seq[r] : r) * p.bt_stride;
   const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(p.cache);
-  // a warp copies rows 4 warp .. 4 warp + 3 of a tile; a lane looks up row 4 warp + lane % 4; < 0: not seen
-  auto key_offset = [&](int i) -> long long {
-    const int pos = (my_lo + i) * kTileL + warp * 4 + (lane & 3);
-    if (i >= n || pos < first || pos >= L) return -1;
-    return (long long)bt[pos / p.page] * p.page_stride + (long long)(pos % p.page) * row;
+  // warp 0 copies: a lane a key.  Keys that are not seen are another copy of a seen one, with a score of minus infinity
+  auto key_row = [&](int i) {
+    const int pos = max(first, min((my_lo + i) * kTileL + lane, L - 1));
+    return cache + (long long)bt[pos / p.page] * p.page_stride + (long long)(pos % p.page) * row;
   };
-  auto fetch = [&](int i, long long off) {
-    const uint32_t dst = ring_u + ((i % kStagesL) * kTileL + warp * 4) * rb;
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      const long long o = __shfl_sync(0xffffffffu, off, k);
-      if (i < n)
-        for (int c = lane; c < row / 8; c += 32) cp16_or_zero(dst + k * rb + c * 16, cache + (o >= 0 ? o + c * 8 : 0), o >= 0);
-    }
-    cp_commit();                                                   // an empty group keeps the count of groups in step
+  auto fetch = [&](int i, const __nv_bfloat16* src) {
+    uint64_t* bar = &full[i % kStagesL];
+    if (lane == 0) mbar_expect_tx(bar, kTileL * row * 2);
+    __syncwarp();
+    bulk_row(ring_u + ((i % kStagesL) * kTileL + lane) * rb, src, row * 2, bar);
   };
-#pragma unroll
-  for (int s = 0; s < kStagesL - 1; ++s) fetch(s, key_offset(s));
-  long long off = key_offset(kStagesL - 1);
+  if (tid == 0) {
+    for (int k = 0; k < kStagesL; ++k) mbar_init(&full[k], 1);
+    abort_s = 0;
+    mbar_fence_init();
+  }
+  __syncthreads();
+  const __nv_bfloat16* ahead = cache;
+  if (warp == 0) {
+    for (int k = 0; k < kStagesL - 1 && k < n; ++k) fetch(k, key_row(k));
+    ahead = key_row(kStagesL - 1);
+  }
   if (row % 16)                                                    // the last 8 channels of a step past the row meet zero queries
     for (int i = tid; i < kStagesL * kTileL; i += kWarpsL * 32) *reinterpret_cast<uint4*>(ring + (size_t)i * rb + row * 2) = make_uint4(0, 0, 0, 0);
-  // queries of this warp's quarter of the channels
-  const int ksteps = (row + 15) / 16, per = (ksteps + 3) / 4, kq = warp & 3, khalf = warp >> 2;
+  // queries of this warp's share of the channels
+  const int ksteps = (row + 15) / 16, per = (ksteps + kParts - 1) / kParts, kq = warp & (kParts - 1), khalf = warp / kParts;
   const int k_lo = kq * per, k_n = max(0, min(per, ksteps - k_lo));
   uint32_t qa[MT][KQ][4];
 #pragma unroll
@@ -99,12 +111,12 @@ __global__ void __launch_bounds__(kWarpsL * 32, 1) latent_rows_kernel(const Para
 #pragma unroll
     for (int v = 0; v < NV; ++v) o[m][v][0] = o[m][v][1] = o[m][v][2] = o[m][v][3] = 0.f;
   const int v0 = warp * NV * 8;                                    // first value column of the warp
-  const int sh = tid >> 3, sj = (tid & 7) * 4;                     // softmax: head, first of 4 keys
+  const int sh = tid >> 4, sj = (tid & 15) * 2;                    // softmax: head, first of 2 keys
   float run_m = -INFINITY, run_l = 0.f;                            // of head sh; run_l: this thread's keys only
-  cp_wait<kStagesL - 2>();
-  __syncthreads();
+  if (row % 16) __syncthreads();
   for (int i = 0; i <= n; ++i) {
     if (i < n) {                                                   // partial scores of tile i
+      mbar_wait(&full[i % kStagesL], (i / kStagesL) & 1, abort_flag, kTimeoutMma);      // (after a time-out the loop runs out without waiting)
       float s[MT][2][4] = {};
       const uint32_t ka = ring_u + ((i % kStagesL) * kTileL + khalf * 16 + (lane >> 4) * 8 + (lane & 7)) * rb + ((lane >> 3) & 1) * 16 + k_lo * 32;
 #pragma unroll
@@ -155,39 +167,40 @@ __global__ void __launch_bounds__(kWarpsL * 32, 1) latent_rows_kernel(const Para
           }
     }
     __syncthreads();                                               // scores are there; tile i - 1 and its probabilities are done with
-    fetch(i + kStagesL - 1, off);
-    off = key_offset(i + kStagesL);
+    if (warp == 0 && i + kStagesL - 1 < n) {
+      if (!__any_sync(0xffffffffu, abort_s != 0)) fetch(i + kStagesL - 1, ahead);
+      ahead = key_row(i + kStagesL);
+    }
     if (i < n && sh < 16 * MT) {
-      float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+      float2 s = make_float2(0.f, 0.f);
 #pragma unroll
-      for (int q = 0; q < 4; ++q) {
-        const float4 x = *reinterpret_cast<const float4*>(part + ((size_t)q * 16 * MT + sh) * kPartRow + sj);
-        s.x += x.x; s.y += x.y; s.z += x.z; s.w += x.w;
+      for (int q = 0; q < kParts; ++q) {
+        const float2 x = *reinterpret_cast<const float2*>(part + ((size_t)q * 16 * MT + sh) * kPartRow + sj);
+        s.x += x.x; s.y += x.y;
       }
       const int pos = (my_lo + i) * kTileL + sj;
       s.x = pos >= first && pos < L ? s.x * p.scale_log2 : -INFINITY;
       s.y = pos + 1 >= first && pos + 1 < L ? s.y * p.scale_log2 : -INFINITY;
-      s.z = pos + 2 >= first && pos + 2 < L ? s.z * p.scale_log2 : -INFINITY;
-      s.w = pos + 3 >= first && pos + 3 < L ? s.w * p.scale_log2 : -INFINITY;
-      float mt = fmaxf(fmaxf(s.x, s.y), fmaxf(s.z, s.w));
+      float mt = fmaxf(s.x, s.y);
 #pragma unroll
-      for (int b = 1; b < 8; b <<= 1) mt = fmaxf(mt, __shfl_xor_sync(0xffffffffu, mt, b));
+      for (int b = 1; b < 16; b <<= 1) mt = fmaxf(mt, __shfl_xor_sync(0xffffffffu, mt, b));
       const float mn = fmaxf(run_m, mt), sub = mn == -INFINITY ? 0.f : mn, al = exp2f(run_m - sub);
       run_m = mn;
-      __align__(8) __nv_bfloat162 e[2] = {__floats2bfloat162_rn(exp2f(s.x - sub), exp2f(s.y - sub)),
-                                          __floats2bfloat162_rn(exp2f(s.z - sub), exp2f(s.w - sub))};
-      run_l = run_l * al + (__low2float(e[0]) + __high2float(e[0])) + (__low2float(e[1]) + __high2float(e[1]));
-      *reinterpret_cast<uint2*>(prob + sh * kProbBytes + sj * 2) = *reinterpret_cast<const uint2*>(e);
-      if ((tid & 7) == 0) alpha[sh] = al;
+      const __nv_bfloat162 e = __floats2bfloat162_rn(exp2f(s.x - sub), exp2f(s.y - sub));
+      run_l = run_l * al + (__low2float(e) + __high2float(e));
+      *reinterpret_cast<__nv_bfloat162*>(prob + sh * kProbBytes + sj * 2) = e;
+      if ((tid & 15) == 0) alpha[sh] = al;
     }
-    cp_wait<kStagesL - 2>();
-    __syncthreads();                                               // probabilities and tile i + 1 are there
+    __syncthreads();                                               // the probabilities are there
   }
-  cp_wait<0>();
+  if (tid == 0 && abort_s != 0) {
+    for (uint32_t k = 0; k < (1u << 16); ++k) __nanosleep(20);     // bounded grace period for copies in flight
+    if (p.status != nullptr) atomicMax(p.status, abort_s);
+  }
   if (sh < 16 * MT) {
 #pragma unroll
-    for (int b = 1; b < 8; b <<= 1) run_l += __shfl_xor_sync(0xffffffffu, run_l, b);
-    if ((tid & 7) == 0) ml[sh] = make_float2(run_m, run_l);
+    for (int b = 1; b < 16; b <<= 1) run_l += __shfl_xor_sync(0xffffffffu, run_l, b);
+    if ((tid & 15) == 0) ml[sh] = make_float2(run_m, run_l);
   }
   __syncthreads();
 #pragma unroll
@@ -216,7 +229,7 @@ template <int MT, int KQ, int NV>
 static int launch_as(const Params& p, int R, cudaStream_t stream) {
   static DeviceOnce once;
   auto kern = latent_rows_kernel<MT, KQ, NV>;
-  if (!ensure_dynamic_smem(kern, shared_bytes(64 * KQ, MT), once)) return -4;
+  if (!ensure_dynamic_smem(kern, shared_bytes(16 * kParts * KQ, MT), once)) return -4;
   bg::launch_pdl(kern, dim3(R, (p.H + 16 * MT - 1) / (16 * MT), p.n_splits), dim3(kWarpsL * 32), shared_bytes(p.row, MT), stream, p);
   if (p.n_splits > 1) bg::launch_pdl(merge_kernel<__nv_bfloat16>, dim3(R, p.H), dim3(64), 0, stream, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
@@ -236,10 +249,10 @@ extern "C" {
 // [R, ldo] bf16, heads of dvp.  row <= 640, dvp <= 512, both multiples of 8.
 int bg_latent_rows(const void* qb, const void* cache, long long page_stride, int page, int row, const int* block_table, int bt_stride,
                    const int* row_seq, const int* lens, void* out, int ldo, float* part_o, float* part_ml, int R, int H, int dvp, int window,
-                   const float* sinks, float scale, int n_splits, cudaStream_t stream) {
+                   const float* sinks, float scale, int n_splits, int* status, cudaStream_t stream) {
   using namespace bg::talk;
   if (R <= 0) return 0;
-  if (H <= 0 || H > 65535 || row <= 0 || row % 8 || row > 640 || dvp <= 0 || dvp % 8 || dvp > 512 || dvp > row || page <= 0 || page_stride % 8 ||
+  if (H <= 0 || H > 65535 || row <= 0 || row % 8 || row > 640 || dvp <= 0 || dvp % 8 || dvp > 512 || dvp > row || page <= 0 || page_stride % 8 || reinterpret_cast<uintptr_t>(cache) % 16 ||
       ldo % 8 || ldo < H * dvp || window < 0 || n_splits < 1 || n_splits > 65535 || (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return -1;
   Params p = {};
@@ -247,9 +260,9 @@ int bg_latent_rows(const void* qb, const void* cache, long long page_stride, int
   p.block_table = block_table; p.bt_stride = bt_stride; p.row_seq = row_seq; p.lens = lens; p.out = out; p.ldo = ldo; p.part_o = part_o;
   p.part_ml = part_ml; p.H = H; p.G = 1; p.dp = row; p.dvp = dvp; p.window = window; p.sink = sinks != nullptr; p.sinks = sinks;
   p.n_splits = n_splits; p.scale_log2 = scale * kLog2e; p.out_scale = 1.0f; p.gate_cols = 1;
-  if (row <= 192 && dvp <= 128) return latent::launch_heads<3, 2>(p, R, stream);
-  if (row <= 384 && dvp <= 256) return latent::launch_heads<6, 4>(p, R, stream);
-  return latent::launch_heads<10, 8>(p, R, stream);
+  p.status = status;
+  if (row <= 384 && dvp <= 256) return latent::launch_heads<3, 2>(p, R, stream);
+  return latent::launch_heads<5, 4>(p, R, stream);
 }
 
 }  // extern "C"

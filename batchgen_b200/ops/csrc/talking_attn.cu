@@ -53,6 +53,7 @@ struct Params {
   const float* sinks;           // [H] or null: all zero
   int v_col0;                   // first value column of a cache row
   const __nv_bfloat16* qb;      // latent_rows.cuh: [R, H, row] queries
+  int* status;
 };
 
 template <typename T> __device__ __forceinline__ float to_f(T v);
@@ -474,7 +475,7 @@ int bg_talk_rows(int dt, const float* q, int ldq, const float* talk, const void*
   p.out = out; p.ldo = ldo; p.part_o = part_o; p.part_ml = part_ml; p.H = H; p.G = G; p.dp = dp; p.dvp = dvp;
   p.chunk = chunk; p.window = window; p.keep = keep; p.out_scale = out_scale; p.sink = sink; p.n_splits = n_splits; p.scale_log2 = scale * 1.4426950408889634f;
   p.rope = rope; p.half = half; p.gate = gate; p.ld_gate = ld_gate; p.gate_cols = gate_cols; p.sinks = sinks;
-  p.v_col0 = v_col0; p.qb = nullptr;
+  p.v_col0 = v_col0; p.qb = nullptr; p.status = nullptr;
   const int items = G * ((H / G + 3) / 4) * (dvp / 4);
   const int ni = (items + kThreads - 1) / kThreads;
   if (ni > 8 && !(dt == 0 && plain::supported(p))) return -1;

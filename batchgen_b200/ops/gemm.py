@@ -16,7 +16,7 @@ import torch
 from . import _ext, ref
 
 KIND_FP8, KIND_BF16 = 0, 1
-EPI_STORE, EPI_SILU_MUL, EPI_STORE_F32 = 0, 1, 2
+EPI_STORE, EPI_SILU_MUL, EPI_STORE_F32, EPI_RELU2 = 0, 1, 2, 3
 
 
 def interleave_gate_up_rows(n_rows: int, device=None) -> torch.Tensor:
@@ -217,13 +217,13 @@ def bf16_gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = No
     return out
 
 
-def grouped_bf16_gemm(x: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, counts: torch.Tensor) -> torch.Tensor:
-    """Ragged grouped bf16 GEMM on the GPU: x [R, K] rows grouped by expert, w [E, N, K] -> [R, N] bf16; ``counts`` rows of
-    each segment are present, the others stay undefined."""
+def grouped_bf16_gemm(x: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, counts: torch.Tensor, relu2: bool = False) -> torch.Tensor:
+    """Ragged grouped bf16 GEMM on the GPU: x [R, K] rows grouped by expert, w [E, N, K] -> [R, N] bf16 (``relu2``: the squared
+    positive part of the products); ``counts`` rows of each segment are present, the others stay undefined."""
     E, N, K = w.shape
     out = torch.empty(x.shape[0], N, dtype=torch.bfloat16, device=x.device)
     if x.shape[0]:
-        _launch(KIND_BF16, EPI_STORE, x.contiguous(), None, 0, w.view(E * N, K), None, out, offsets, E, x.shape[0], N, K,
+        _launch(KIND_BF16, EPI_RELU2 if relu2 else EPI_STORE, x.contiguous(), None, 0, w.view(E * N, K), None, out, offsets, E, x.shape[0], N, K,
                 counts=counts)
     return out
 

@@ -172,7 +172,8 @@ def attend(qa: torch.Tensor, p: LatentParams, cache: torch.Tensor, block_table: 
         rc = _ext.lib().bg_latent_rows(
             _ext.ptr(qa), _ext.ptr(cache), ctypes.c_longlong(cache.stride(0)), _i(cache.shape[1]), _i(row), _ext.ptr(block_table),
             _i(block_table.stride(0)), _ext.ptr(row_seq), _ext.ptr(lens), _ext.ptr(out), _i(flat.stride(0)), _ext.ptr(po), _ext.ptr(pml),
-            _i(R), _i(H), _i(p.rank_p), _i(p.window), _ext.ptr(p.sinks), ctypes.c_float(p.scale), _i(num_splits), _ext.stream())
+            _i(R), _i(H), _i(p.rank_p), _i(p.window), _ext.ptr(p.sinks), ctypes.c_float(p.scale), _i(num_splits),
+            _ext.ptr(_ext.status_word(qa.device)), _ext.stream())
         _ext.check(rc, "bg_latent_rows", kernels=2 if num_splits > 1 else 1)
         return out
     q = qa.view(R, H * row).float()

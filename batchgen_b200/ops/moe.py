@@ -320,6 +320,9 @@ def routed_rows(x: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.Tensor, e
     counts = offsets.real_counts
     cap = src.shape[0]
     xs, ws = residual.moe_gather(x, pos, topk_w, cap)
+    if ew.activation == "relu2" and not weight_on_input and x.dtype == torch.bfloat16:      # the activation is the product's epilogue
+        act = gemm.grouped_bf16_gemm(xs, ew.w13, offsets, counts, relu2=True)
+        return gemm.grouped_rows_gemm(act, ew.w2, offsets, counts, max_rows=T), pos
     z = gemm.grouped_rows_gemm(xs, ew.w13, offsets, counts, max_rows=T)
     act = residual.glu(z, F, ew.activation, ew.act_limit, row_scale=ws if weight_on_input else None, total_rows=offsets[-1:],
                        dtype=x.dtype)

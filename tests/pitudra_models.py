@@ -14,13 +14,18 @@ def hgrn2(heads, dim, vdim, mlp=None):
     return {"type": "hgrn2", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "vdim": vdim}}
 
 
+def _mask(window):
+    """No window: every earlier token is seen."""
+    return {"mask": {"size": window}} if window else {}
+
+
 def attention(heads, kv_heads, dim, vdim, window, mlp=None, scale=None):
-    return {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim,
-                                                       "scale": scale or 1.3 * dim ** -0.5, "mask": {"size": window}}}
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale or 1.3 * dim ** -0.5}
+    return {"type": "attention", "mlp": mlp, "mixer": {**m, **_mask(window)}}
 
 
 def latent(heads, dim, rot, vdim, q_rank, kv_rank, window, mlp=None, base=700.0, kv_from=None, scale=None):
-    m = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "mask": {"size": window},
+    m = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, **_mask(window),
          "scale": scale or 1.3 * (dim + rot) ** -0.5, "rot": {"base": base, "dims": rot}}
     if kv_from is not None:
         m["kv_from"] = kv_from
@@ -44,11 +49,11 @@ CONFIGS = {
                             hgrn2(1, 8, 8, moe(16, 4, 1))]),
     # whole tiles everywhere, windows on page borders
     "whole": config(160, 128, [hgrn2(2, 128, 128, moe(128, 8, 2)), attention(8, 1, 64, 64, 64, moe(64, 4, 2)),
-                               latent(4, 64, 64, 64, 128, 128, 128, moe(64, 4, 2), 1e6), attention(2, 2, 128, 128, 128)], 64),
+                               latent(4, 64, 64, 64, 128, 128, 128, moe(64, 4, 2), 1e6), attention(2, 2, 128, 128, 0)], 64),
     # heads and latents wider than the tensor-core kernels take, wider states than the decode ring takes, more than 32 heads
     "wide": config(120, 72, [latent(2, 200, 72, 264, 40, 584, 40, moe(40, 5, 2)), hgrn2(1, 152, 136, moe(48, 3, 1)),
                              attention(3, 1, 264, 72, 90), latent(35, 8, 72, 16, 24, 584, 300, kv_from=0),
-                             latent(33, 24, 8, 16, 40, 520, 70)], 136),
+                             latent(33, 24, 8, 16, 40, 520, 0)], 136),
     # latent layers alone, several widths of the score kernel
     "latents": config(140, 80, [latent(16, 16, 16, 24, 32, 200, 100, moe(32, 12, 5)), latent(4, 24, 8, 16, 24, 96, 33),
                                 latent(24, 16, 16, 32, 40, 200, 64, moe(24, 4, 2), kv_from=0), latent(20, 32, 32, 32, 64, 400, 200)], 24),
