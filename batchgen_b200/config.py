@@ -926,15 +926,15 @@ def _pitudra_layer(d: Dict, index: int, layers: List[Dict]) -> LayerSpec:
     if m.get("mask") and window < 1:
         raise ValueError(f"layer {index}: a window of {window} positions")
     if kind == "hgrn2":
-        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], vdim=m["vdim"])
+        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], vdim=m.get("vdim", m["dim"]))
     elif kind == "attention":
-        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], kv_heads=m.get("kv_heads", m["heads"]), vdim=m["vdim"],
+        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], kv_heads=m.get("kv_heads", m["heads"]), vdim=m.get("vdim", m["dim"]),
                           scale=float(m["scale"]), window=window, bias=True, qk_norm_all=True, head_sinks=True, out_gate_all=True)
         if mixer.heads % mixer.kv_heads:
             raise ValueError(f"layer {index}: {mixer.heads} heads do not divide over {mixer.kv_heads} key/value heads")
     elif kind == "latent_attention":
         rot, j = m["rot"], m.get("kv_from")
-        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]), window=window, head_sinks=True,
+        mixer = MixerSpec(kind, heads=m["heads"], dim=m["dim"], vdim=m.get("vdim", m["dim"]), scale=float(m["scale"]), window=window, head_sinks=True,
                           q_rank=m["q_rank"], kv_rank=m["kv_rank"], rot_dim=m["rot_dim"], rot_dims=int(rot["dims"]),
                           rot_base=float(rot["base"]), kv_from=-1 if j is None else int(j))
         if mixer.rot_dims != mixer.rot_dim or mixer.rot_dim % 2:

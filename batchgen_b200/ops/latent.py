@@ -139,8 +139,8 @@ def _key_ranges(ctas: int, keys: int, sms: int) -> int:
     return min(range(1, max(1, min(16, keys // 64)) + 1), key=lambda s: math.ceil(ctas * s / sms) * (keys / s + 128) + 4 * s)
 
 
-def on_tensor_cores(p: LatentParams, dtype: torch.dtype) -> bool:
-    return dtype == torch.bfloat16 and p.row <= 640 and p.rank_p <= 512
+def on_tensor_cores(p: LatentParams, dtype: torch.dtype, page: int) -> bool:
+    return dtype == torch.bfloat16 and p.row <= 640 and p.rank_p <= 512 and page >= 16
 
 
 def _heads_at_a_time(p: LatentParams, esize: int) -> int:
@@ -158,7 +158,7 @@ def attend(qa: torch.Tensor, p: LatentParams, cache: torch.Tensor, block_table: 
     R, H, row = qa.shape
     out = torch.empty(R, H, p.rank_p, dtype=qa.dtype, device=qa.device)
     flat = out.view(R, H * p.rank_p)
-    if qa.is_cuda and on_tensor_cores(p, qa.dtype):
+    if qa.is_cuda and on_tensor_cores(p, qa.dtype, cache.shape[1]):
         assert qa.is_contiguous() and row == p.row == cache.shape[2] == cache.stride(1) and cache.dtype == qa.dtype
         assert lens.dtype == torch.int32 and lens.shape[0] == R and block_table.dtype == torch.int32
         assert row_seq is None or (row_seq.dtype == torch.int32 and row_seq.shape[0] == R)
@@ -170,8 +170,8 @@ def attend(qa: torch.Tensor, p: LatentParams, cache: torch.Tensor, block_table: 
             po = torch.empty(R * num_splits * H * p.rank_p, dtype=torch.float32, device=qa.device)
             pml = torch.empty(R * num_splits * H * 2, dtype=torch.float32, device=qa.device)
         rc = _ext.lib().bg_latent_rows(
-            _ext.ptr(qa), _ext.ptr(cache), ctypes.c_longlong(cache.stride(0)), _i(cache.shape[1]), _i(row), _ext.ptr(block_table),
-            _i(block_table.stride(0)), _ext.ptr(row_seq), _ext.ptr(lens), _ext.ptr(out), _i(flat.stride(0)), _ext.ptr(po), _ext.ptr(pml),
+            _ext.ptr(qa), _ext.ptr(cache), ctypes.c_longlong(cache.stride(0)), _i(cache.shape[0]), _i(cache.shape[1]), _i(row),
+            _ext.ptr(block_table), _i(block_table.stride(0)), _ext.ptr(row_seq), _ext.ptr(lens), _ext.ptr(out), _i(flat.stride(0)), _ext.ptr(po), _ext.ptr(pml),
             _i(R), _i(H), _i(p.rank_p), _i(p.window), _ext.ptr(p.sinks), ctypes.c_float(p.scale), _i(num_splits),
             _ext.ptr(_ext.status_word(qa.device)), _ext.stream())
         _ext.check(rc, "bg_latent_rows", kernels=2 if num_splits > 1 else 1)
