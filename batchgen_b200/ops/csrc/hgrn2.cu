@@ -1,4 +1,4 @@
-// HGRN2: linear attention whose forget gate also decides what is written.  Per head and key channel
+// HGRN2: every row of a head's state keeps the share f of itself and takes the rest from the token's value.  Per head and key channel
 //
 //   f  = l + (1 - l) * sigmoid(z + bias), l the channel's lower bound
 //   S' = diag(f) S + (1 - f) v^T,  o = S'^T silu(q)

@@ -180,6 +180,7 @@ def sandwich_norm(x: torch.Tensor, norm: Optional[Norm], eps: float, width: int,
             cur = cur + post.ref(s, eps, width)
         if keep:
             x[r, :width] = cur
+            x[r, width:W4] = 0                    # (an input convolution reads whole vectors of 4)
         if not emit:
             return None
         h = torch.nn.functional.pad(cur if norm is None else norm.ref(cur, eps, width), (0, W4 - width))

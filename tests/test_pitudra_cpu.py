@@ -71,6 +71,7 @@ def test_routed_rows_join_behind_their_norm_and_the_next_sublayer_reads_the_resi
     r = lambda *s: torch.randn(*s, generator=g)      # noqa: E731
     x, routed = torch.zeros(T, 12), torch.zeros(9, 12)
     x[:, :D], routed[:, :D] = r(T, D), r(9, D)
+    x[:, D:] = float("nan")                          # what memory held before
     pos = torch.randint(-1, 9, (T, 4), generator=g).to(torch.int32)
     rw, w, b = torch.rand(T, 4, generator=g), torch.zeros(12), torch.zeros(12)
     w[:D], b[:D] = 1 + 0.2 * r(D), r(D)
@@ -78,6 +79,7 @@ def test_routed_rows_join_behind_their_norm_and_the_next_sublayer_reads_the_resi
     want = x[:, :D] + oracle.layer_norm(y, w[:D], b[:D], 1e-5)
     h = residual.sandwich_norm(x, None, 1e-5, D, 64, torch.float32, routed=routed, pos=pos, route_w=rw, post=residual.Norm(w, b, True))
     assert torch.allclose(x[:, :D], want, atol=1e-5) and torch.allclose(h[:, :D], want, atol=1e-5) and float(h[:, D:].abs().sum()) == 0
+    assert float(x[:, D:].abs().sum()) == 0
     before = x.clone()
     assert residual.sandwich_norm(x, None, 1e-5, D, 64, torch.float32, add=y, post=residual.Norm(w), emit=False) is None
     assert torch.allclose(x[:, :D], before[:, :D] + oracle.rms(y, 1e-5) * w[:D], atol=1e-5)
